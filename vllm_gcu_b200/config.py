@@ -26,6 +26,24 @@ def to_dtype(x: Any) -> torch.dtype:
     return _DTYPES[str(x).replace("torch.", "")]
 
 
+@dataclass(frozen=True)
+class LayerSpec:
+    """One layer of a design whose layers differ: mixer type and sizes, feed-forward sizes."""
+    mixer: str                             # "latent_attention"
+    num_heads: int
+    head_dim: int                          # query / key dimensions per head
+    v_head_dim: int
+    kv_lora_rank: int                      # latent width
+    scale: float                           # score scale
+    num_experts: int = 0                   # 0: no feed-forward
+    num_experts_per_tok: int = 0
+    moe_intermediate_size: int = 0
+
+    @property
+    def has_mlp(self) -> bool:
+        return self.num_experts > 0
+
+
 @dataclass
 class ModelConfig:
     architecture: str = "LlamaForCausalLM"
@@ -75,6 +93,9 @@ class ModelConfig:
     quantization: Optional[str] = None
     quant_config: Optional[dict] = None
     kv_cache_dtype: str = "auto"
+    # designs described layer by layer (None: every layer has the sizes above)
+    layer_specs: Optional[tuple[LayerSpec, ...]] = None
+    residual_alpha: float = 1.0            # norm after the sum: norm(alpha * x + sublayer(x))
     extra: dict = field(default_factory=dict)
 
     def __post_init__(self) -> None:
@@ -109,6 +130,8 @@ class ModelConfig:
     def kv_bytes_per_token(self, tp_size: int = 1) -> int:
         es = 1 if self.kv_cache_dtype.startswith("fp8") or self.kv_cache_dtype == "int8" else \
             torch.empty((), dtype=self.dtype).element_size()
+        if self.layer_specs is not None:
+            return sum(s.kv_lora_rank for s in self.layer_specs) * es
         if self.is_mla:
             return self.num_hidden_layers * (self.kv_lora_rank + self.qk_rope_head_dim) * es
         kvh = max(1, self.num_key_value_heads // tp_size)
@@ -151,6 +174,9 @@ class ModelConfig:
     # -- construction ----------------------------------------------------
     @classmethod
     def from_hf_dict(cls, d: dict, **overrides) -> "ModelConfig":
+        if d.get("architecture") == "Sapapel" or "SapapelForCausalLM" in (
+                d.get("architectures") or ()):
+            return cls._from_layer_list(d, **overrides)
         archs = d.get("architectures") or ["LlamaForCausalLM"]
         for nested in ("text_config", "language_config", "llm_config"):
             if isinstance(d.get(nested), dict):
@@ -236,6 +262,51 @@ class ModelConfig:
         return cls(**kw)
 
     @classmethod
+    def _from_layer_list(cls, d: dict, **overrides) -> "ModelConfig":
+        """Sapapel's ``config.json``: ``vocab``, ``width``, ``norm.eps``, ``postln_alpha`` and one
+        entry of ``layers`` per layer with its mixer's and its feed-forward's sizes."""
+        specs = []
+        for i, layer in enumerate(d["layers"]):
+            if layer["type"] != "latent_attention":
+                raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+            m, f = layer["mixer"], layer.get("mlp")
+            moe = {}
+            if f is not None:
+                if f.get("kind", "moe") != "moe":
+                    raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
+                moe = dict(num_experts=int(f["router"]["experts"]),
+                           num_experts_per_tok=int(f["router"]["top"]),
+                           moe_intermediate_size=int(f["expert"]["ff"]))
+                if not 0 < moe["num_experts_per_tok"] <= moe["num_experts"]:
+                    raise ValueError(f"layer {i}: {moe['num_experts_per_tok']} of "
+                                     f"{moe['num_experts']} experts per token")
+            specs.append(LayerSpec("latent_attention", int(m["heads"]), int(m["dim"]),
+                                   int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]), **moe))
+        if not specs:
+            raise ValueError("the configuration lists no layers")
+        kw: dict[str, Any] = dict(
+            architecture="SapapelForCausalLM", vocab_size=int(d["vocab"]),
+            hidden_size=int(d["width"]), num_hidden_layers=len(specs),
+            rms_norm_eps=float(d["norm"]["eps"]), residual_alpha=float(d["postln_alpha"]),
+            layer_specs=tuple(specs),
+            # the largest layer stands for the model where one number is asked for
+            num_attention_heads=max(s.num_heads for s in specs), num_key_value_heads=1,
+            head_dim=max(s.head_dim for s in specs),
+            v_head_dim=max(s.v_head_dim for s in specs),
+            kv_lora_rank=max(s.kv_lora_rank for s in specs),
+            num_experts=max(s.num_experts for s in specs),
+            num_experts_per_tok=max(s.num_experts_per_tok for s in specs),
+            moe_intermediate_size=max(s.moe_intermediate_size for s in specs),
+            scoring_func="sigmoid", norm_topk_prob=False,
+            # no positions in the design, so no limit of its own: bounds the block tables only
+            max_position_embeddings=int(d.get("max_position_embeddings", 131072)),
+            extra={k: v for k, v in d.items() if k not in (
+                "layers", "vocab", "width", "norm", "postln_alpha", "architecture",
+                "architectures", "max_position_embeddings")})
+        kw.update(overrides)
+        return cls(**kw)
+
+    @classmethod
     def from_pretrained(cls, path: str, **overrides) -> "ModelConfig":
         p = Path(path)
         d = json.loads((p / "config.json").read_text())
@@ -309,9 +380,34 @@ def preset(name: str, **overrides) -> ModelConfig:
                               routed_scaling_factor=2.5, num_nextn_predict_layers=1,
                               rope_is_neox=False, dtype="float32"),
     }
+    if name in _LAYER_LIST_PRESETS:
+        n = overrides.pop("num_hidden_layers", None)
+        d = _LAYER_LIST_PRESETS[name]
+        layers = d["layers"] if n is None else (d["layers"] * n)[:n]
+        return ModelConfig.from_hf_dict({**d, "layers": layers}, **overrides)
     kw = dict(presets[name])
     kw.update(overrides)
     return ModelConfig(**kw)
+
+
+def _sapapel_preset(layers: int, vocab: int, width: int, heads: int, dim: int, vdim: int,
+                    kv_rank: int, experts: int, top: int, ff: int) -> dict:
+    layer = {"type": "latent_attention",
+             "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": kv_rank,
+                       "scale": dim ** -0.5},
+             "mlp": {"kind": "moe", "router": {"experts": experts, "top": top},
+                     "expert": {"ff": ff}}}
+    return {"architecture": "Sapapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "postln_alpha": (2.0 * layers) ** 0.25, "layers": [layer] * layers}
+
+
+#: configurations of designs that are described layer by layer (``num_hidden_layers`` repeats or
+#: truncates the list)
+_LAYER_LIST_PRESETS: dict[str, dict] = {
+    "tiny-sapapel": _sapapel_preset(3, 1024, 128, 4, 24, 40, 48, 6, 2, 48),
+    # layers of the size of DeepSeek-V2-Lite's
+    "sapapel-16b": _sapapel_preset(27, 102400, 2048, 16, 128, 128, 512, 64, 6, 1408),
+}
 
 
 @dataclass

@@ -93,17 +93,45 @@ def _compile_one(src: Path, force: bool, verbose: bool, sanitize: str | None = N
     return obj
 
 
+def partial_lib_path(sources) -> Path:
+    """Library that holds only the kernels of ``sources`` (file stems), named by their digest."""
+    return PKG / f"_b200_{hashlib.sha256(','.join(sorted(sources)).encode()).hexdigest()[:10]}.so"
+
+
+def up_to_date() -> bool:
+    """True when the full library exists and was built from the sources as they are."""
+    if not LIB_PATH.exists():
+        return False
+    flags = " ".join(NVCC_FLAGS)
+    for src in CSRC.glob("*.cu"):
+        stamp = OBJ_DIR / (src.stem + ".sha")
+        if not stamp.exists() or stamp.read_text() != _digest(src, flags):
+            return False
+    return True
+
+
+def ensure(sources) -> tuple[Path, bool]:
+    """A library with (at least) the kernels of ``sources``: the full one when it is current,
+    else a partial one, compiling what is missing.  Returns (path, is partial)."""
+    if up_to_date():
+        return LIB_PATH, False
+    return build(sources=sources), True
+
+
 def build(force: bool = False, verbose: bool = False, jobs: int | None = None,
-          sanitize: str | None = None) -> Path:
-    """Compiles what changed and links the library.  Returns its path."""
+          sanitize: str | None = None, sources=None) -> Path:
+    """Compiles what changed and links the library.  Returns its path.  ``sources`` (file
+    stems) restricts the build to those files and writes a partial library of its own."""
     srcs = sorted(CSRC.glob("*.cu"))
+    if sources is not None:
+        srcs = [s for s in srcs if s.stem in sources]
     if not srcs:
         raise RuntimeError("no CUDA sources found")
     jobs = jobs or min(len(srcs), os.cpu_count() or 4)
     with cf.ThreadPoolExecutor(max_workers=jobs) as ex:
         objs = list(ex.map(lambda s: _compile_one(s, force, verbose, sanitize), srcs))
     newest = max(o.stat().st_mtime for o in objs)
-    out = lib_path_for(sanitize)
+    out = lib_path_for(sanitize) if sources is None else partial_lib_path(sources)
     if force or not out.exists() or out.stat().st_mtime < newest:
         cmd = [nvcc_path(), "-shared", "-o", str(out), *map(str, objs),
                "-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"]

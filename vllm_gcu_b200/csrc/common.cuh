@@ -433,6 +433,32 @@ template <typename T>
 __device__ __forceinline__ float round_like(float v) {
   return to_f32<T>(from_f32<T>(v));
 }
+// Which request a token of a step belongs to.  A step holds `nd` single-token requests followed
+// by the tokens of `np` requests whose offsets (relative to token nd) are in cu_q.
+struct TokenPlace {
+  int req;      // request of the step, -1 for a row behind the last one
+  bool first;   // first token that the step brings for the request
+  bool last;    // last one
+};
+__device__ __forceinline__ TokenPlace token_place(int t, int nd, int np, const int* cu_q) {
+  TokenPlace p{t, true, true};
+  if (t < nd) return p;
+  if (cu_q == nullptr || np <= 0 || t - nd >= cu_q[np]) {
+    p.req = -1;
+    return p;
+  }
+  const int r = t - nd;
+  int lo = 0, hi = np;           // last i with cu_q[i] <= r
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (cu_q[mid] <= r) lo = mid; else hi = mid;
+  }
+  p.req = nd + lo;
+  p.first = cu_q[lo] == r;
+  p.last = cu_q[lo + 1] == r + 1;
+  return p;
+}
+
 __device__ __forceinline__ uint8_t f32_to_e4m3(float v) {
   return static_cast<uint8_t>(__nv_cvt_float_to_fp8(v, __NV_SATFINITE, __NV_E4M3));
 }

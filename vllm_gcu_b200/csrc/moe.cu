@@ -8,6 +8,9 @@
 //                     the expert of every tile, the padded row count and the inverse map
 //   moe_permute       gathers activation rows into expert-sorted order (the A operand of
 //                     the grouped tcgen05 GEMM in gemm_bf16.cu)
+//   moe_permute_weighted  the same from an fp32 stream, every row scaled by its routing weight
+//                     (designs whose weight multiplies the expert's input)
+//   grouped_gemm_f32  the expert products of models that run in 32-bit
 //   moe_unpermute_sum out[t] = sum_slots y[pos(t, slot)] (+ shared-expert output); the top-k
 //                     weights were already applied by the second GEMM's epilogue
 //   get_ep_indices    per destination rank, the tokens that have an expert there
@@ -67,7 +70,7 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const TopkArgs a) {
   }
   mx = warp_max(mx);
   if (a.sigmoid) {
-    for (int e = lane; e < a.E; e += 32) sc[e] = 1.0f / (1.0f + __expf(-sc[e]));
+    for (int e = lane; e < a.E; e += 32) sc[e] = 1.0f / (1.0f + expf(-sc[e]));
   } else {
     float sum = 0.0f;
     for (int e = lane; e < a.E; e += 32) {
@@ -243,6 +246,99 @@ __global__ void __launch_bounds__(256)
   for (int v = threadIdx.x; v < nvec; v += blockDim.x) dst[v] = src[v];
 }
 
+// A_sorted[pos] = weight(pair) * x[pair / k] from an fp32 stream: routing that weights the
+// expert's input.  One rounding, to the type of the expert GEMM's operand.
+template <typename T>
+__global__ void __launch_bounds__(256)
+    moe_permute_weighted_kernel(const float* x, long long ldx, const float* topk_w, T* out,
+                                long long ldo, const int* sorted_ids, const int* num_post_pad,
+                                int numel, int k, int H, int Ho) {
+  const int pos = blockIdx.x;
+  if (pos >= *num_post_pad) return;
+  const int pair = sorted_ids[pos];
+  T* dst = out + static_cast<long long>(pos) * ldo;
+  const bool pad = pair >= numel;
+  const float w = pad ? 0.0f : topk_w[pair];
+  const float* src = x + static_cast<long long>(pad ? 0 : pair / k) * ldx;
+  const bool vec = (H % 4) == 0 && (ldx % 4) == 0;
+  for (int c = threadIdx.x * 4; c < Ho; c += blockDim.x * 4) {
+    float4 f = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (!pad && vec && c < H) {
+      f = *reinterpret_cast<const float4*>(src + c);
+    } else if (!pad) {
+      if (c < H) f.x = src[c];
+      if (c + 1 < H) f.y = src[c + 1];
+      if (c + 2 < H) f.z = src[c + 2];
+      if (c + 3 < H) f.w = src[c + 3];
+    }
+    if constexpr (sizeof(T) == 2) {
+      *reinterpret_cast<uint2*>(dst + c) =
+          make_uint2(pack_bf16x2(w * f.x, w * f.y), pack_bf16x2(w * f.z, w * f.w));
+    } else {
+      *reinterpret_cast<float4*>(dst + c) = make_float4(w * f.x, w * f.y, w * f.z, w * f.w);
+    }
+  }
+}
+
+// Grouped GEMM in fp32 arithmetic (no reduced-precision tensor mode), for models that run in
+// 32-bit: C[r, n] = sum_k A[r, k] * B_e[n, k] over rows sorted by expert in tiles of 128, e the
+// tile's expert.  64 x 64 output tile per CTA, 4 x 4 per thread.
+constexpr int kF32Tile = 64, kF32K = 16;
+__global__ void __launch_bounds__(256)
+    grouped_gemm_f32_kernel(const float* A, long long lda, const float* B, float* C, long long ldc,
+                            int N, int K, int E, const int* expert_ids, const int* num_valid_rows) {
+  __shared__ float as[kF32K][kF32Tile + 4];
+  __shared__ float bs[kF32K][kF32Tile + 4];
+  const int m0 = blockIdx.y * kF32Tile, n0 = blockIdx.x * kF32Tile;
+  if (m0 >= *num_valid_rows) return;
+  const int e = expert_ids[m0 / kTileM];
+  if (e < 0 || e >= E) return;
+  const float* Be = B + static_cast<long long>(e) * N * K;
+  const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kF32K) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int kk = k0 + lk + i;
+      as[lk + i][lr] = kk < K ? A[static_cast<long long>(m0 + lr) * lda + kk] : 0.0f;
+      bs[lk + i][lr] = (kk < K && n0 + lr < N) ? Be[static_cast<long long>(n0 + lr) * K + kk] : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < kF32K; ++kk) {
+      float av[4], bv[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        av[i] = as[kk][ty * 4 + i];
+        bv[i] = bs[kk][tx * 4 + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += av[i] * bv[j];
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n < N) C[static_cast<long long>(m0 + ty * 4 + i) * ldc + n] = acc[i][j];
+    }
+}
+
+// h[r, i] = silu(u[r, i]) * u[r, I + i] of the rows in use
+__global__ void __launch_bounds__(256)
+    silu_mul_rows_f32_kernel(const float* u, float* h, int I, const int* num_valid_rows) {
+  const int r = blockIdx.x;
+  if (r >= *num_valid_rows) return;
+  const float* g = u + static_cast<long long>(r) * 2 * I;
+  for (int c = threadIdx.x; c < I; c += blockDim.x)
+    h[static_cast<long long>(r) * I + c] = g[c] / (1.0f + expf(-g[c])) * g[I + c];
+}
+
 // out[t] = (add ? add[t] : 0) + alpha * sum_s y[pos_of[t * k + s]]   (fp32 accumulation)
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -383,6 +479,47 @@ B200_API int b200_moe_permute(const void* x, long long ldx, void* out, long long
                                                    num_post_pad, numel, k, H);
   else
     return -8;
+  return static_cast<int>(cudaGetLastError());
+}
+
+// x fp32 [T, ldx], H columns; out bf16 (dtype 0) or fp32 (2) rows [cap, ldo] of Ho >= H columns
+// (zeros behind H); Ho and ldo are multiples of 4.
+B200_API int b200_moe_permute_weighted(const float* x, long long ldx, const float* topk_w,
+                                       void* out, long long ldo, const int* sorted_ids,
+                                       const int* num_post_pad, int numel, int k, int H, int Ho,
+                                       int cap, int dtype, void* stream) {
+  if (cap <= 0) return 0;
+  if ((Ho % 4) != 0 || (ldo % 4) != 0 || Ho < H || ldo < Ho || k <= 0) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 0)
+    moe_permute_weighted_kernel<__nv_bfloat16><<<cap, 256, 0, s>>>(
+        x, ldx, topk_w, static_cast<__nv_bfloat16*>(out), ldo, sorted_ids, num_post_pad, numel, k,
+        H, Ho);
+  else if (dtype == 2)
+    moe_permute_weighted_kernel<float><<<cap, 256, 0, s>>>(
+        x, ldx, topk_w, static_cast<float*>(out), ldo, sorted_ids, num_post_pad, numel, k, H, Ho);
+  else
+    return -8;
+  return static_cast<int>(cudaGetLastError());
+}
+
+// A [M_cap, K] expert-sorted rows (M_cap a multiple of 128), B [E, N, K], C [M_cap, N].
+B200_API int b200_grouped_gemm_f32(const float* A, long long lda, const float* B, float* C,
+                                   long long ldc, int M_cap, int N, int K, int E,
+                                   const int* expert_ids, const int* num_valid_rows, void* stream) {
+  if (M_cap <= 0 || N <= 0) return 0;
+  if ((M_cap % kTileM) != 0 || K <= 0 || E <= 0) return -2;
+  dim3 grid((N + kF32Tile - 1) / kF32Tile, M_cap / kF32Tile);
+  grouped_gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      A, lda, B, C, ldc, N, K, E, expert_ids, num_valid_rows);
+  return static_cast<int>(cudaGetLastError());
+}
+
+B200_API int b200_silu_mul_rows_f32(const float* u, float* h, int rows, int I,
+                                    const int* num_valid_rows, void* stream) {
+  if (rows <= 0 || I <= 0) return 0;
+  silu_mul_rows_f32_kernel<<<rows, 256, 0, static_cast<cudaStream_t>(stream)>>>(u, h, I,
+                                                                             num_valid_rows);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -1,0 +1,347 @@
+// Kernels around a 32-bit residual stream whose norms come after the sums (sm_100a).
+//
+//   token_shift     h[t] = x[t] + (x[t - 1] - x[t]) * mu, per coordinate; the row before the
+//                   first row of a request's portion comes from the state that earlier steps
+//                   left with the request's cache blocks (zero in front of position 0)
+//   post_norm       r = rms(alpha * x + y) * g with one gain g per norm, where y is a dense row
+//                   or the sum of a token's routed-expert rows; optionally followed in the same
+//                   pass by the depth-weighted average x' = sum_j w[j] * X_j + w[n] * r over the
+//                   results X_j of the layers so far, and by the final norm of that row
+//   sigmoid_gate    o = o * sigmoid(z), z a strided view of a wider projection
+//
+// The residual stream, the statistics and the averages are fp32; LO is the type of the rows that
+// feed matrix products (bf16, or fp32 when the whole model runs in 32-bit).  One CTA per row,
+// vectors of V elements (4 where every row is 4-aligned, else 1).
+#include "common.cuh"
+
+namespace b200 {
+namespace residual {
+
+template <int V>
+__device__ __forceinline__ void ldv(const float* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
+  } else {
+    f[0] = p[0];
+  }
+}
+template <int V>
+__device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else {
+    f[0] = __bfloat162float(p[0]);
+  }
+}
+template <int V>
+__device__ __forceinline__ void stv(float* p, const float (&f)[V]) {
+  if constexpr (V == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    p[0] = f[0];
+  }
+}
+template <int V>
+__device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&f)[V]) {
+  if constexpr (V == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+  } else {
+    p[0] = __float2bfloat16(f[0]);
+  }
+}
+
+// ---------------------------------------------------------------------------
+struct ShiftArgs {
+  const float* x;          // [T, H]
+  const float* mu;         // [H]
+  const float* state;      // [num_blocks, H] last row written into every cache block, or null
+  const int* block_tables; // [B, max_blocks]
+  const long long* positions;
+  const int* cu_q;         // [num_prefills + 1] relative to token num_decodes, or null
+  void* out;               // [T, H]
+  int T, H, num_decodes, num_prefills, max_blocks, block_size, num_blocks;
+};
+
+template <typename LO, int V>
+__global__ void __launch_bounds__(256) token_shift_kernel(const ShiftArgs a) {
+  const int t = blockIdx.x;
+  const float* prev = nullptr;             // null: zeros
+  const TokenPlace pl = token_place(t, a.num_decodes, a.num_prefills, a.cu_q);
+  if (!pl.first) {
+    prev = a.x + static_cast<long long>(t - 1) * a.H;
+  } else if (a.state != nullptr && pl.req >= 0) {
+    const long long pos = a.positions[t];
+    if (pos > 0) {
+      const long long bi = (pos - 1) / a.block_size;
+      if (bi < a.max_blocks) {
+        const int blk = a.block_tables[static_cast<long long>(pl.req) * a.max_blocks + bi];
+        if (blk >= 0 && blk < a.num_blocks) prev = a.state + static_cast<long long>(blk) * a.H;
+      }
+    }
+  }
+  const float* x = a.x + static_cast<long long>(t) * a.H;
+  LO* out = static_cast<LO*>(a.out) + static_cast<long long>(t) * a.H;
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
+    float xv[V], m[V], pv[V], o[V];
+    ldv<V>(x + c, xv);
+    ldv<V>(a.mu + c, m);
+    if (prev != nullptr) {
+      ldv<V>(prev + c, pv);
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) pv[i] = 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) o[i] = xv[i] + (pv[i] - xv[i]) * m[i];
+    stv<V>(out + c, o);
+  }
+}
+
+// ---------------------------------------------------------------------------
+struct PostNormArgs {
+  const float* x;        // [T, H] residual stream
+  const void* y;         // dense: [T, ldy]; routed: expert-sorted rows [cap, ldy]
+  const int* pos_of;     // routed: [T, k] row of every (token, slot) pair (-1: none), else null
+  const float* gain;     // scalar
+  const float* hist;     // results of earlier layers: [n][T, H], hist_stride apart, or null
+  const float* w;        // [n + 1] average weights (with hist)
+  const float* fgain;    // final norm's scalar gain, or null
+  float* res;            // [T, H] the norm's result, or null
+  float* xo;             // [T, H] the average (with hist), or null
+  void* lo;              // [T, H] LO copy: final-normed average, else the last fp32 result
+  long long ldy, hist_stride;
+  int T, H, k, n;
+  float alpha, eps;
+};
+
+template <typename Y, typename LO, int V>
+__global__ void __launch_bounds__(512) post_norm_kernel(const PostNormArgs a) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  float* z = sm;                 // [H]
+  float* acc = sm + a.H;         // [H] partial average (with hist)
+  const int t = blockIdx.x;
+  const long long row = static_cast<long long>(t) * a.H;
+  const Y* y = static_cast<const Y*>(a.y);
+  float ss = 0.0f;
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
+    float xv[V], yv[V];
+    ldv<V>(a.x + row + c, xv);
+    if (a.pos_of == nullptr) {
+      ldv<V>(y + static_cast<long long>(t) * a.ldy + c, yv);
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) yv[i] = 0.0f;
+      for (int s = 0; s < a.k; ++s) {
+        const int p = a.pos_of[static_cast<long long>(t) * a.k + s];
+        if (p < 0) continue;
+        float f[V];
+        ldv<V>(y + static_cast<long long>(p) * a.ldy + c, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) yv[i] += f[i];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      xv[i] = a.alpha * xv[i] + yv[i];
+      ss += xv[i] * xv[i];
+    }
+    stv<V>(z + c, xv);
+    if (a.hist != nullptr) {
+      // the earlier results do not depend on this norm: read them while the row is in flight
+      float s[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) s[i] = 0.0f;
+      const float* hp = a.hist + row + c;
+      int j = 0;
+      for (; j + 4 <= a.n; j += 4) {
+        float f0[V], f1[V], f2[V], f3[V];
+        ldv<V>(hp + (j + 0) * a.hist_stride, f0);
+        ldv<V>(hp + (j + 1) * a.hist_stride, f1);
+        ldv<V>(hp + (j + 2) * a.hist_stride, f2);
+        ldv<V>(hp + (j + 3) * a.hist_stride, f3);
+        const float w0 = a.w[j], w1 = a.w[j + 1], w2 = a.w[j + 2], w3 = a.w[j + 3];
+#pragma unroll
+        for (int i = 0; i < V; ++i) s[i] += w0 * f0[i] + w1 * f1[i] + w2 * f2[i] + w3 * f3[i];
+      }
+      for (; j < a.n; ++j) {
+        float f[V];
+        ldv<V>(hp + j * a.hist_stride, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) s[i] += a.w[j] * f[i];
+      }
+      stv<V>(acc + c, s);
+    }
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.H) + a.eps) * a.gain[0];
+  LO* lo = static_cast<LO*>(a.lo);
+  float ss2 = 0.0f;
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
+    float r[V];
+    ldv<V>(z + c, r);
+#pragma unroll
+    for (int i = 0; i < V; ++i) r[i] *= inv;
+    if (a.res != nullptr) stv<V>(a.res + row + c, r);
+    if (a.hist != nullptr) {
+      float s[V];
+      ldv<V>(acc + c, s);
+      const float wn = a.w[a.n];
+#pragma unroll
+      for (int i = 0; i < V; ++i) r[i] = s[i] + wn * r[i];
+      if (a.xo != nullptr) stv<V>(a.xo + row + c, r);
+    }
+    if (lo != nullptr) {
+      if (a.fgain == nullptr) {
+        stv<V>(lo + row + c, r);
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss2 += r[i] * r[i];
+        stv<V>(z + c, r);
+      }
+    }
+  }
+  if (lo == nullptr || a.fgain == nullptr) return;
+  ss2 = block_sum(ss2, red);
+  const float inv2 = 1.0f / sqrtf(ss2 / static_cast<float>(a.H) + a.eps) * a.fgain[0];
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
+    float r[V];
+    ldv<V>(z + c, r);
+#pragma unroll
+    for (int i = 0; i < V; ++i) r[i] *= inv2;
+    stv<V>(lo + row + c, r);
+  }
+}
+
+// out[t, c] = o[t, c] * sigmoid(z[t, c])
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+    sigmoid_gate_kernel(const T* o, long long ldo, const T* z, long long ldz, T* out,
+                        long long ldout, long long rows, int D) {
+  const int nv = D / V;
+  const long long n = rows * nv;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / nv;
+    const int c = static_cast<int>(i - t * nv) * V;
+    float a[V], g[V];
+    ldv<V>(o + t * ldo + c, a);
+    ldv<V>(z + t * ldz + c, g);
+#pragma unroll
+    for (int k = 0; k < V; ++k) a[k] = a[k] / (1.0f + expf(-g[k]));
+    stv<V>(out + t * ldout + c, a);
+  }
+}
+
+static int row_threads(int H, int V, int most) {
+  int n = (H / V + 31) / 32 * 32;
+  return n < 32 ? 32 : (n > most ? most : n);
+}
+
+template <typename Y, typename LO, int V>
+static int launch_post_norm(const PostNormArgs& a, cudaStream_t s) {
+  const size_t smem = static_cast<size_t>(a.hist != nullptr ? 2 : 1) * a.H * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(post_norm_kernel<Y, LO, V>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  // few rows: more threads per row, so that a row's loads are in flight together
+  const int threads = row_threads(a.H, V, a.T < 2 * sm_count() ? 512 : 256);
+  post_norm_kernel<Y, LO, V><<<a.T, threads, smem, s>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+static bool aligned(const void* p, int bytes) {
+  return (reinterpret_cast<uintptr_t>(p) % bytes) == 0;
+}
+
+}  // namespace residual
+}  // namespace b200
+
+using namespace b200;
+using namespace b200::residual;
+
+// out_dtype: 0 bf16, 2 fp32.  state / block_tables null: every portion starts from zeros.
+B200_API int b200_token_shift(const float* x, const float* mu, const float* state,
+                              const int* block_tables, const long long* positions, const int* cu_q,
+                              void* out, int T, int H, int num_decodes, int num_prefills,
+                              int max_blocks, int block_size, int num_blocks, int out_dtype,
+                              void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || block_size <= 0 || (out_dtype != 0 && out_dtype != 2)) return -2;
+  ShiftArgs a;
+  a.x = x; a.mu = mu; a.state = block_tables ? state : nullptr; a.block_tables = block_tables;
+  a.positions = positions; a.cu_q = cu_q; a.out = out; a.T = T; a.H = H;
+  a.num_decodes = num_decodes; a.num_prefills = num_prefills; a.max_blocks = max_blocks;
+  a.block_size = block_size; a.num_blocks = num_blocks;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (H % 4) == 0 && aligned(x, 16) && aligned(mu, 16) && aligned(state, 16) &&
+                  aligned(out, 16);
+  const int th = row_threads(H, v4 ? 4 : 1, 256);
+  if (out_dtype == 0) {
+    if (v4) token_shift_kernel<__nv_bfloat16, 4><<<T, th, 0, s>>>(a);
+    else token_shift_kernel<__nv_bfloat16, 1><<<T, th, 0, s>>>(a);
+  } else {
+    if (v4) token_shift_kernel<float, 4><<<T, th, 0, s>>>(a);
+    else token_shift_kernel<float, 1><<<T, th, 0, s>>>(a);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+// dtype (of y and lo): 0 bf16, 2 fp32.  pos_of non-null: y holds expert-sorted rows, k per token.
+// hist non-null: depth average over n earlier results.  The rows of res, xo and hist are H wide.
+B200_API int b200_post_norm(const float* x, const void* y, long long ldy, const int* pos_of, int k,
+                            const float* gain, float alpha, float eps, float* res,
+                            const float* hist, long long hist_stride, int n, const float* w,
+                            float* xo, const float* fgain, void* lo, int T, int H, int dtype,
+                            void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || (dtype != 0 && dtype != 2) || (hist != nullptr && (w == nullptr || n < 0)))
+    return -2;
+  PostNormArgs a;
+  a.x = x; a.y = y; a.ldy = ldy; a.pos_of = pos_of; a.k = k; a.gain = gain; a.alpha = alpha;
+  a.eps = eps; a.res = res; a.hist = hist; a.hist_stride = hist_stride; a.n = n; a.w = w;
+  a.xo = xo; a.fgain = fgain; a.lo = lo; a.T = T; a.H = H;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (H % 4) == 0 && (ldy % 4) == 0 && (hist_stride % 4) == 0 && aligned(x, 16) &&
+                  aligned(y, 16) && aligned(res, 16) && aligned(hist, 16) && aligned(xo, 16) &&
+                  aligned(lo, 16);
+  if (dtype == 0)
+    return v4 ? launch_post_norm<__nv_bfloat16, __nv_bfloat16, 4>(a, s)
+              : launch_post_norm<__nv_bfloat16, __nv_bfloat16, 1>(a, s);
+  return v4 ? launch_post_norm<float, float, 4>(a, s) : launch_post_norm<float, float, 1>(a, s);
+}
+
+B200_API int b200_sigmoid_gate(const void* o, long long ldo, const void* z, long long ldz,
+                               void* out, long long ldout, int T, int D, int dtype, void* stream) {
+  if (T <= 0 || D <= 0) return 0;
+  if (dtype != 0 && dtype != 2) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (D % 4) == 0 && (ldo % 4) == 0 && (ldz % 4) == 0 && (ldout % 4) == 0 &&
+                  aligned(o, 16) && aligned(z, dtype == 0 ? 8 : 16) && aligned(out, 16);
+  const long long items = static_cast<long long>(T) * (v4 ? D / 4 : D);
+  long long blocks = (items + 255) / 256;
+  const long long cap = static_cast<long long>(sm_count()) * 16;
+  if (blocks > cap) blocks = cap;
+  const int g = static_cast<int>(blocks);
+  if (dtype == 0) {
+    const __nv_bfloat16* po = static_cast<const __nv_bfloat16*>(o);
+    const __nv_bfloat16* pz = static_cast<const __nv_bfloat16*>(z);
+    __nv_bfloat16* pq = static_cast<__nv_bfloat16*>(out);
+    if (v4) sigmoid_gate_kernel<__nv_bfloat16, 4><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
+    else sigmoid_gate_kernel<__nv_bfloat16, 1><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
+  } else {
+    const float* po = static_cast<const float*>(o);
+    const float* pz = static_cast<const float*>(z);
+    float* pq = static_cast<float*>(out);
+    if (v4) sigmoid_gate_kernel<float, 4><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
+    else sigmoid_gate_kernel<float, 1><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
+  }
+  return static_cast<int>(cudaGetLastError());
+}

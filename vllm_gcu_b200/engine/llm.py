@@ -82,6 +82,9 @@ class LLMEngine:
         self.proposer = None
         self.spec_metrics = None
         sp = cfg.speculative
+        if sp.method and getattr(self.model, "has_block_state", False):
+            raise ValueError(f"{cfg.model.architecture} keeps recurrent state with its cache "
+                             "blocks: draft tokens cannot be taken back")
         if sp.method:
             from ..spec import NgramProposer, SpecMetrics
             self.spec_metrics = SpecMetrics()
@@ -276,6 +279,9 @@ class LLMEngine:
         """Disaggregated prefill: requests with ``kv_transfer_params`` send their KV to /
         take their KV from the peer instance through ``connector`` (engine/kv_disagg.py)."""
         from .kv_disagg import DisaggCoordinator
+        if getattr(self.model, "has_block_state", False):
+            raise ValueError(f"{self.cfg.model.architecture} keeps recurrent state with its cache "
+                             "blocks, which the connector does not ship")
         self.disagg = DisaggCoordinator(self, connector, recv_timeout_s)
         self.scheduler.on_free = self.disagg.before_free
         return self.disagg

@@ -98,6 +98,7 @@ class ModelRunner:
         self.max_tokens = max(sc.max_num_batched_tokens, sc.max_num_seqs)
         self.max_blocks = -(-sc.max_model_len // self.block_size) + 1
         self.kv_caches: list[torch.Tensor] = []
+        self.block_state: list[torch.Tensor] = []
         self.num_blocks = 0
         tp = cfg.parallel.tensor_parallel_size
         # under tensor parallelism every rank samples its slice of the batch rows and the ids
@@ -128,6 +129,11 @@ class ModelRunner:
         self.keep_hidden = False                   # a pooling request samples in this step:
         self._last_hidden = None                   # keep the sampled rows' final hidden states
         self._features = None                      # per-step sampling extras (penalties, logprobs)
+        self._logit_rows = None                    # rows whose logits the caller wants back
+        self._logits_out = None
+        # decode graphs keep their logits readable after a replay (teacher-forced replays)
+        self.keep_graph_logits = bool((cfg.additional_config or {}).get("keep_graph_logits"))
+        self.graph_logits: dict = {}
         self._mm_inputs = None                     # (inputs_embeds, mrope positions) of a step
         from .. import envs
         self.nvtx = bool(envs.NVTX) and self.is_cuda
@@ -207,10 +213,16 @@ class ModelRunner:
         cc = self.cfg.cache
         if cc.num_gpu_blocks is not None:
             return cc.num_gpu_blocks
-        bytes_per_block = self.cfg.model.kv_bytes_per_token(
-            self.cfg.parallel.tensor_parallel_size) * self.block_size
-        bytes_per_block = bytes_per_block * self.model.num_local_layers \
-            // max(1, self.cfg.model.num_hidden_layers)
+        spec = self.model.kv_cache_spec()
+        if "widths" in spec:
+            bytes_per_block = self.block_size * sum(spec["widths"]) \
+                * torch.empty((), dtype=self.cfg.model.dtype).element_size() \
+                + 4 * sum(spec.get("block_state", ()))
+        else:
+            bytes_per_block = self.cfg.model.kv_bytes_per_token(
+                self.cfg.parallel.tensor_parallel_size) * self.block_size
+            bytes_per_block = bytes_per_block * self.model.num_local_layers \
+                // max(1, self.cfg.model.num_hidden_layers)
         if not self.is_cuda:
             return max(64, min(4096, (1 << 28) // max(1, bytes_per_block)))
         torch.cuda.synchronize()
@@ -253,12 +265,16 @@ class ModelRunner:
             elif kvd == "int8":
                 dt = torch.int8
         if spec["type"] == "mla":
-            self.kv_caches = [torch.zeros(num_blocks, self.block_size, spec["width"], dtype=dt,
-                                          device=self.device) for _ in range(spec["layers"])]
+            widths = spec.get("widths") or [spec["width"]] * spec["layers"]
+            self.kv_caches = [torch.zeros(num_blocks, self.block_size, w, dtype=dt,
+                                          device=self.device) for w in widths]
         else:
             self.kv_caches = [torch.zeros(2, num_blocks, self.block_size, spec["kv_heads"],
                                           spec["head_dim"], dtype=dt, device=self.device)
                               for _ in range(spec["layers"])]
+        # recurrent rows that live with the cache blocks (token shift): one per block and layer
+        self.block_state = [torch.zeros(num_blocks, w, dtype=torch.float32, device=self.device)
+                            for w in spec.get("block_state", ())]
         self.num_blocks = num_blocks
         if self.drafter is not None:
             ds = self.drafter.kv_cache_spec()
@@ -343,17 +359,17 @@ class ModelRunner:
         if getattr(self, "cpu_caches", None) is None:
             pin = self.is_cuda
             self.cpu_caches = []
-            for c in self.kv_caches:
+            for c in self.kv_caches + self.block_state:
                 shape = list(c.shape)
-                shape[0 if c.dim() == 3 else 1] = n_cpu
+                shape[0 if c.dim() <= 3 else 1] = n_cpu
                 self.cpu_caches.append(torch.zeros(shape, dtype=c.dtype, device="cpu",
                                                    pin_memory=pin))
         from ..ops import cuda as C, ref
         swap = C.swap_blocks if self.is_cuda else ref.swap_blocks
         m_in = torch.tensor(so.swap_in, dtype=torch.int64).view(-1, 2)
         m_out = torch.tensor(so.swap_out, dtype=torch.int64).view(-1, 2)
-        for dev_c, cpu_c in zip(self.kv_caches, self.cpu_caches):
-            planes = [(dev_c, cpu_c)] if dev_c.dim() == 3 else [(dev_c[0], cpu_c[0]),
+        for dev_c, cpu_c in zip(self.kv_caches + self.block_state, self.cpu_caches):
+            planes = [(dev_c, cpu_c)] if dev_c.dim() <= 3 else [(dev_c[0], cpu_c[0]),
                                                                 (dev_c[1], cpu_c[1])]
             for d, h in planes:
                 if len(so.swap_in):
@@ -395,7 +411,8 @@ class ModelRunner:
         use_graph = (self.is_cuda and npf == 0 and bool(self.graphs)
                      and nd_graph <= self.graph_sizes[-1]
                      and self.drafter is None and self.head_drafter is None
-                     and not batch_has_lora and not feat and not self.keep_hidden)
+                     and not batch_has_lora and not feat and not self.keep_hidden
+                     and (self.keep_graph_logits or not any(s.logit_rows for s in sched)))
         B_pad = _pad_batch(nd_graph, self.graph_sizes) if use_graph else B
         T = T_real + (B_pad - B)
 
@@ -609,11 +626,14 @@ class ModelRunner:
             decode_workspace=self.decode_ws,
             sample_indices=self.sample_indices[:max(ns * width, 1)],
             q_lens_cpu=[int(x) for x in ntok], seq_lens_cpu=[int(x) for x in seq_after],
-            common_prefix_len=common_prefix,
+            common_prefix_len=common_prefix, block_state=self.block_state,
             cu_q_all=torch.tensor(tok_off, dtype=torch.int32, device=self.device)
             if common_prefix else None)
 
         self._features = self._build_features(order, samplers, tok_off) if feat else None
+        rows_wanted = [int(tok_off[j]) + o for j, s in enumerate(order) for o in s.logit_rows]
+        self._logit_rows = torch.tensor(rows_wanted, device=self.device) if rows_wanted else None
+        self._logits_out = None
         self._mm_inputs = self._build_mm_inputs(mm_chunks, T) if mm_chunks else None
         if self._mm_inputs is not None:
             md.mrope_positions = self._mm_inputs[1]
@@ -623,6 +643,8 @@ class ModelRunner:
         if use_graph:
             key = (B_pad, cur, all_greedy)
             self.graphs[key].replay()
+            if self._logit_rows is not None:     # decode-only: row i is token i
+                self._logits_out = self.graph_logits[key].index_select(0, self._logit_rows).float()
             self.graph_launches += self.graph_kernel_counts.get(key, 0)
         else:
             with torch.inference_mode():
@@ -652,6 +674,14 @@ class ModelRunner:
         self.step_counter += 1
         extra = {"num_draft": nspec,
                  "draft_width": self.head_drafter.k if self.head_drafter is not None else 1}
+        if self._logits_out is not None:
+            # caller's order of requests and, inside a request, of its wanted offsets
+            by_req, at = {}, 0
+            for s in order:
+                by_req[s.req.request_id] = self._logits_out[at:at + len(s.logit_rows)]
+                at += len(s.logit_rows)
+            extra["logits"] = by_req
+            self._logits_out = None
         if self.keep_hidden and ns and self._last_hidden is not None:
             extra["hidden"] = self._last_hidden[:ns * width:width]     # row i = i-th sampler
             self._last_hidden = None
@@ -813,6 +843,9 @@ class ModelRunner:
                     dist.broadcast(out_ids[:ns * width], last, group=pp.device_group)
                 return
         feats = getattr(self, "_features", None)
+        if self._logit_rows is not None:
+            self._logits_out = self.model.compute_logits(
+                hidden.index_select(0, self._logit_rows)).float()
         if ns == 0:
             if feats is not None and "prompt_logprobs" in feats and self.model.is_last_stage:
                 self._apply_features(hidden, hidden, 0, out_ids, before_sampling=False)
@@ -836,6 +869,8 @@ class ModelRunner:
         logits = self.model.compute_logits(rows)
         if self.keep_logits:
             self.last_logits = logits.float().cpu()
+        if self.keep_graph_logits:
+            self._step_logits = logits
         if feats is not None:
             logits = self._apply_features(hidden, logits, ns, out_ids, before_sampling=True,
                                           width=width)
@@ -1009,7 +1044,8 @@ class ModelRunner:
                             max_seq_len=self.cfg.scheduler.max_model_len,
                             decode_splits=self._decode_splits(Bp, self.cfg.scheduler.max_model_len),
                             decode_workspace=self.decode_ws,
-                            sample_indices=self.sample_indices[:Bp])
+                            sample_indices=self.sample_indices[:Bp],
+                            block_state=self.block_state)
                         # warm-up outside the graph (lazy initialisation, autotuning)
                         self._forward_and_sample(md, Bp, Bp, self.sampled[cur], greedy)
                         stream.synchronize()
@@ -1021,5 +1057,7 @@ class ModelRunner:
                         if self.graph_pool is None:
                             self.graph_pool = g.pool()
                         self.graphs[(Bp, cur, greedy)] = g
+                        if self.keep_graph_logits:
+                            self.graph_logits[(Bp, cur, greedy)] = self._step_logits
         torch.cuda.synchronize()
         _native.check_status()

@@ -36,6 +36,8 @@ class ScheduledRequest:
     will_sample: bool = False  # this step produces the next token(s) of the request
     epoch: int = 0             # the request's preemption count when this step was planned
     sample_index: int = 0      # index of the first output token this step produces
+    # offsets among this step's tokens whose logits go back to the caller
+    logit_rows: list[int] = field(default_factory=list)
 
 
 @dataclass
@@ -326,6 +328,38 @@ class Scheduler:
 
         out.total_tokens = sum(s.num_tokens for s in out.scheduled)
         self._update_after_schedule(out)
+        return out
+
+    def schedule_portions(self, portions: Sequence[tuple[Request, int, Sequence[int]]]
+                          ) -> SchedulerOutput:
+        """A step with exactly the given portions, as one batch: ``(request, number of its next
+        known tokens, offsets among them whose logits are wanted)``.  For callers that decide
+        themselves what runs when (replay of a trace); blocks, state and batch layout are those of
+        :meth:`schedule`.  A request is admitted with its first portion and ends with
+        :meth:`abort_request`.  A portion of one token runs as a decode, like a generated token."""
+        out = SchedulerOutput(step_id=self.step_id)
+        self.step_id += 1
+        out.finished_req_ids, self.finished_since_last = self.finished_since_last, set()
+        for req, n, rows in portions:
+            if n <= 0 or req.num_computed_tokens + n > req.num_tokens:
+                raise ValueError(f"{req.request_id}: a portion of {n} tokens, "
+                                 f"{req.num_tokens - req.num_computed_tokens} known")
+            is_new = req.request_id not in self.requests
+            if is_new:
+                if len(self.running) >= self.cfg.max_num_seqs:
+                    raise RuntimeError(f"more than {self.cfg.max_num_seqs} live requests")
+                self.requests[req.request_id] = req
+                self.running.append(req)
+                req.status = RequestStatus.RUNNING
+            blocks = self.kv.allocate_slots(req, n)
+            if blocks is None:
+                raise RuntimeError("the cache pool has no free block left")
+            out.scheduled.append(ScheduledRequest(req, req.num_computed_tokens, n, blocks, is_new,
+                                                  logit_rows=list(rows)))
+        out.total_tokens = sum(s.num_tokens for s in out.scheduled)
+        self._update_after_schedule(out)
+        for s in out.scheduled:
+            s.will_sample = s.num_tokens == 1
         return out
 
     def _preempt_for(self, newcomer: Request, out: SchedulerOutput, placed: set[str]) -> bool:

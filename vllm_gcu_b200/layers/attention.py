@@ -56,6 +56,9 @@ class AttentionMetadata:
     # ``common_prefix_len`` cached tokens (a multiple of the block size; 0 = off) and
     # ``cu_q_all`` holds the query offsets of all requests, decodes included
     common_prefix_len: int = 0
+    # per layer [num_blocks, width] fp32: state rows that models with ``has_block_state`` keep
+    # with every cache block
+    block_state: Optional[list] = None
     cu_q_all: Optional[torch.Tensor] = None
 
 

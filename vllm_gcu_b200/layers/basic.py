@@ -55,6 +55,19 @@ class RMSNorm(nn.Module):
         self.weight.data.copy_(full)
 
 
+class ScalarGain(nn.Module):
+    """Gain of an RMS norm with one number for all coordinates (fp32; the norm itself is fused
+    with the residual sum in ``ops.cuda.post_norm``)."""
+
+    def __init__(self, device=None):
+        super().__init__()
+        self.gain = nn.Parameter(torch.ones((), dtype=torch.float32, device=device),
+                                 requires_grad=False)
+
+    def load_weight(self, name: str, full: torch.Tensor, shard_id=None) -> None:
+        self.gain.data.copy_(full.reshape(()))
+
+
 def _yarn_find_correction_dim(num_rot, dim, base, max_pos):
     return (dim * math.log(max_pos / (num_rot * 2 * math.pi))) / (2 * math.log(base))
 

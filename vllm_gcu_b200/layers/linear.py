@@ -7,6 +7,7 @@ Parallel flavours (names follow the checkpoint conventions the reference loads,
 vllm_gcu/models/deepseek_v3/deepseek_v3.py:1037-1173):
 
 * ``ColumnParallelLinear``        – output sharded over TP
+* ``MixedParallelLinear``         – sharded and replicated projections of one input in one GEMM
 * ``MergedColumnParallelLinear``  – several column-parallel matrices stacked
   (``gate_up_proj``); with ``fuse_silu`` the gate/up rows are interleaved in blocks
   of 128 at load time and SiLU(gate)*up runs in the GEMM epilogue
@@ -190,6 +191,28 @@ class ColumnParallelLinear(LinearBase):
         if self.gather_output and tp_size() > 1:
             y = get_comm("tp").all_gather(y, dim=-1)
         return y
+
+
+class MixedParallelLinear(LinearBase):
+    """Projections of one input stacked along the output dim, each either sharded over TP
+    (``sharded[i]``) or replicated; ``split(y)`` gives the views of an output row."""
+
+    def __init__(self, in_features, output_sizes: Sequence[int], sharded: Sequence[bool],
+                 dtype=torch.bfloat16, device=None, quant_method=None, prefix=""):
+        tp = tp_size()
+        assert all(n % tp == 0 for n, s in zip(output_sizes, sharded) if s)
+        self.sharded = list(sharded)
+        self.local_sizes = [n // tp if s else n for n, s in zip(output_sizes, sharded)]
+        super().__init__(in_features, sum(output_sizes), in_features, sum(self.local_sizes), False,
+                         dtype, device, quant_method, prefix)
+
+    def shard_spec(self, shard_id=None):
+        n = self.local_sizes[shard_id]
+        src = tp_rank() * n if self.sharded[shard_id] else 0
+        return [(src, n, sum(self.local_sizes[:shard_id]))], None
+
+    def split(self, y: torch.Tensor):
+        return y.split(self.local_sizes, dim=-1)
 
 
 class MergedColumnParallelLinear(LinearBase):

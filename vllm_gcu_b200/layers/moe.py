@@ -390,6 +390,61 @@ class FusedMoE(nn.Module):
         return y if add is None else y + add
 
 
+class InputWeightedMoE(FusedMoE):
+    """Routed experts whose routing weight multiplies the expert's input:
+    ``sum_e down_e(silu(gate_e(w h)) * up_e(w h))``.
+
+    ``forward`` takes the fp32 stream and returns what the norm after the residual sum takes:
+    the experts' output rows in sorted order and the row of every (token, slot) pair (this
+    rank's slice of the intermediate dimension under TP).  On the GPU the stacked weights are
+    padded with zeros to the tile sizes of the grouped GEMM (64 columns of the hidden, 128 of the
+    intermediate dimension), which leaves the result as it is."""
+
+    def __init__(self, num_experts: int, hidden: int, inter: int, dtype, device, prefix: str = ""):
+        tp = tp_size()
+        assert inter % tp == 0
+        self.hidden_full = hidden
+        self.inter_real = inter // tp
+        native = torch.device(device).type == "cuda" if device is not None else False
+        hm, im = (64, 128) if native and dtype == torch.bfloat16 else ((4, 1) if native else (1, 1))
+        up = lambda n, m: -(-n // m) * m  # noqa: E731
+        super().__init__(num_experts, up(hidden, hm), up(self.inter_real, im) * tp, dtype, device,
+                         False, prefix)
+        self.w13.data.zero_()
+        self.w2.data.zero_()
+
+    def _load_one(self, expert_id: int, which: str, full: torch.Tensor) -> bool:
+        I, H = self.inter_real, self.hidden_full
+        lo = self.shard_index * I
+        if which == "gate":
+            self.w13.data[expert_id, :I, :H].copy_(full[lo:lo + I])
+        elif which == "up":
+            self.w13.data[expert_id, self.inter:self.inter + I, :H].copy_(full[lo:lo + I])
+        elif which == "down":
+            self.w2.data[expert_id, :H, :I].copy_(full[:, lo:lo + I])
+        else:
+            raise ValueError(which)
+        return True
+
+    def zero_padding(self) -> None:
+        """Clears the padding (after a random initialisation of the whole parameters)."""
+        I, H = self.inter_real, self.hidden_full
+        for w in (self.w13.data[:, :self.inter], self.w13.data[:, self.inter:],
+                  self.w2.data.transpose(1, 2)):
+            w[:, I:] = 0
+            w[:, :, H:] = 0
+
+    def finalize(self) -> None:
+        if not self._interleaved:
+            self.zero_padding()
+        super().finalize()
+
+    def forward(self, x: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor
+                ) -> tuple[torch.Tensor, torch.Tensor]:
+        op = C.input_weighted_experts if ops.use_native(x) else ref.input_weighted_experts
+        return op(x, self.w13, self.w2, topk_w, topk_ids)
+
+
 class EplbState:
     """Logical -> physical expert mapping with redundant replicas and a load histogram
     (``enable_eplb`` / ``num_redundant_experts`` of the reference's ``additional_config``,

@@ -50,6 +50,7 @@ _REGISTRY: dict[str, str] = {
     "DeepseekV2ForCausalLM": "vllm_gcu_b200.models.deepseek:DeepseekV3ForCausalLM",
     "DeepseekV3ForCausalLM": "vllm_gcu_b200.models.deepseek:DeepseekV3ForCausalLM",
     "DeepseekVLV2ForCausalLM": "vllm_gcu_b200.models.deepseek_vl2:DeepseekVLV2ForCausalLM",
+    "SapapelForCausalLM": "vllm_gcu_b200.models.sapapel:SapapelForCausalLM",
     "DeepSeekMTPModel": "vllm_gcu_b200.models.deepseek_mtp:DeepSeekMTP",
     # pooling models (no KV cache; built by build_pooling_model)
     "XLMRobertaForSequenceClassification":

@@ -13,8 +13,8 @@ vllm_gcu/models/deepseek_v3/deepseek_v3_fusion.py:105-258):
 3. ``q_nope x W_UK`` -> latent query; attention over the cached latents; ``x W_UV``; ``o_proj``.
 
 The attention core runs in the tcgen05 latent attention kernel (csrc/attention_mla.cu:
-decode, multi-token verification and prefill chunks in one kernel) for bf16 caches and a
-power-of-two head count up to 128; other layouts fall back to batched matrix products over
+decode, multi-token verification and prefill chunks in one kernel) for bf16 caches and
+up to 128 heads; other layouts fall back to batched matrix products over
 gathered latent rows (decode: one padded batch; prefill: per sequence).
 """
 from __future__ import annotations
@@ -40,31 +40,7 @@ from .moe_models import MoeDecoderLM
 USE_MLA_KERNEL = True     # tcgen05 latent attention (csrc/attention_mla.cu) where the layout allows
 
 
-def mla_attention_ref(q_full: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
-                      q_lens: list[int], seq_lens: list[int], scale: float, L: int
-                      ) -> torch.Tensor:
-    """q_full ``[T, N, L + R]`` (latent query | rotated rope part); cache ``[blocks, bs, L + R]``.
-    Returns the latent-space output ``[T, N, L]``.  Causal inside each request."""
-    T, N, W = q_full.shape
-    nb, bs, _ = cache.shape
-    flat = cache.view(nb * bs, W)
-    out = torch.zeros(T, N, L, dtype=q_full.dtype, device=q_full.device)
-    t0 = 0
-    for b, (ql, n) in enumerate(zip(q_lens, seq_lens)):
-        if ql == 0 or n == 0:
-            t0 += ql
-            continue
-        pos = torch.arange(n, device=cache.device)
-        slots = block_tables[b, (pos // bs).long()].long() * bs + pos % bs
-        kv = flat[slots].float()                               # [n, W]
-        q = q_full[t0:t0 + ql].float()                         # [ql, N, W]
-        s = torch.einsum("qhw,nw->hqn", q, kv) * scale
-        qpos = torch.arange(n - ql, n, device=cache.device)[:, None]
-        s = s.masked_fill((pos[None, :] > qpos)[None], float("-inf"))
-        p = torch.softmax(s, dim=-1)
-        out[t0:t0 + ql] = torch.einsum("hqn,nl->qhl", p, kv[:, :L]).to(out.dtype)
-        t0 += ql
-    return out
+mla_attention_ref = ref.latent_attention
 
 
 def mla_decode_batched(q_full: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
@@ -185,14 +161,14 @@ class MLAAttention(nn.Module):
             max_len = max(md.max_seq_len, 1)
             if nd > 0:
                 C.mla_attention(q_full[:nd], kv_cache, md.block_tables[:nd], md.seq_lens[:nd],
-                                None, nd, max_len, self.scale, out=o_lat[:nd])
+                                None, nd, max_len, self.scale, out=o_lat[:nd], L=L)
             if md.num_prefills > 0:
                 tq = 128 // N
                 n_pf = sum(md.q_lens_cpu[md.num_decodes:B])
                 tiles = sum(-(-q // tq) for q in md.q_lens_cpu[md.num_decodes:B])
                 C.mla_attention(q_full[nd:nd + n_pf], kv_cache, md.block_tables[md.num_decodes:B],
                                 md.seq_lens[md.num_decodes:B], md.cu_q_prefill, tiles, max_len,
-                                self.scale, out=o_lat[nd:nd + n_pf])
+                                self.scale, out=o_lat[nd:nd + n_pf], L=L)
                 if nd + n_pf < T:
                     o_lat[nd + n_pf:] = 0
             elif nd < T:

@@ -22,6 +22,7 @@ _LIB_PATH = Path(os.environ["VLLM_B200_NATIVE_LIB"]) if os.environ.get("VLLM_B20
 _lock = threading.Lock()
 _lib: Optional[ctypes.CDLL] = None
 _tried = False
+_partial = False
 
 #: number of kernel launches issued through this module (bench.py reports it)
 launch_count = 0
@@ -37,6 +38,16 @@ class KernelTimeoutError(RuntimeError):
 
 def lib_path() -> Path:
     return _LIB_PATH
+
+
+def use_partial_library(path) -> None:
+    """Selects a library that holds only the kernels of one model family
+    (``csrc.build.build(sources=...)``); entry points it lacks raise when they are called.  Must
+    come before the first use of the library."""
+    global _LIB_PATH, _partial
+    if _tried and Path(path) != _LIB_PATH:
+        raise NativeError("the native library is already loaded")
+    _LIB_PATH, _partial = Path(path), True
 
 
 def lib() -> Optional[ctypes.CDLL]:
@@ -61,6 +72,8 @@ def lib() -> Optional[ctypes.CDLL]:
         for name in dir(_Sigs):
             if name.startswith("b200_"):
                 fn = getattr(_lib, name, None)
+                if fn is None and _partial:
+                    continue
                 if fn is None:
                     raise NativeError(f"symbol {name} missing from {_LIB_PATH}; rebuild")
                 fn.restype = ctypes.c_int
@@ -110,7 +123,12 @@ class _Sigs:
     b200_fmha_prefill = [P, L, P, L, P, P, P, P, P, L, L, L, P, I, I, I, I, I, I, I, I, F,
                          I, I, I, P]
     b200_merge_attn_states = [P, P, P, P, P, P, I, I, I, I, P]
-    b200_mla_attention = [P, P, P, L, P, P, P, I, I, I, I, I, I, I, P, F, P]
+    b200_mla_attention = [P, P, P, L, P, P, P, I, I, I, I, I, I, I, I, I, P, F, P]
+    b200_latent_cache = [P, L, P, F, P, L, I, P, P, P, P, I, I, I, I, I, I, I, P]
+    b200_latent_attention = [P, P, L, P, P, I, I, P, P, I, I, I, I, I, F, I, P]
+    b200_token_shift = [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P]
+    b200_post_norm = [P, P, L, P, I, P, F, F, P, P, L, I, P, P, P, P, I, I, I, P]
+    b200_sigmoid_gate = [P, L, P, L, P, L, I, I, I, P]
     b200_gemm_wna16 = [P, L, P, P, P, P, P, L, I, I, I, I, I, P, P]
     b200_gemm_wna16_workspace = [I, I, I]
     b200_gemm_wna16_grouped = [P, L, P, P, P, P, L, I, I, I, I, I, I, P, P, P, P]
@@ -121,6 +139,9 @@ class _Sigs:
     b200_moe_topk = [P, L, P, P, P, I, I, I, I, I, I, I, F, P, I, P, P, I, P]
     b200_moe_align = [P, P, P, P, P, P, P, I, I, I, I, P]
     b200_moe_permute = [P, L, P, L, P, P, I, I, I, I, I, P]
+    b200_moe_permute_weighted = [P, L, P, P, L, P, P, I, I, I, I, I, I, P]
+    b200_grouped_gemm_f32 = [P, L, P, P, L, I, I, I, I, P, P, P]
+    b200_silu_mul_rows_f32 = [P, P, I, I, P, P]
     b200_moe_row_weights = [P, P, P, P, I, I, P]
     b200_moe_unpermute_sum = [P, L, P, P, L, P, L, P, I, I, I, F, I, P]
     b200_get_ep_indices = [P, I, I, I, I, P, P, P, P]
@@ -165,7 +186,11 @@ def call(name: str, *args) -> None:
     l = lib()
     if l is None:
         raise NativeError("native library not loaded")
-    rc = getattr(l, name)(*args)
+    fn = getattr(l, name, None)
+    if fn is None:
+        raise NativeError(f"{name} is not part of {_LIB_PATH}; run "
+                          "`python -m vllm_gcu_b200.csrc.build`")
+    rc = fn(*args)
     launch_count += 1
     if rc != 0:
         raise NativeError(f"{name} failed with code {rc}")

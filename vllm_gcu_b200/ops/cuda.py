@@ -619,44 +619,125 @@ def gemm_wna16(x: torch.Tensor, qw: torch.Tensor, scales: torch.Tensor, zs: torc
 
 
 def mla_attention_supported(q: torch.Tensor, cache: torch.Tensor, L: int) -> bool:
-    """Layouts the tcgen05 MLA kernel covers: bf16, 512 + 64 wide latent rows, a power-of-two
-    number of heads up to 128, cache blocks that are a multiple of 16 tokens."""
-    Nh = q.shape[1]
+    """Layouts the tcgen05 MLA kernel covers: bf16, latent and row widths that are multiples of
+    64 (at most 512 and 576), up to 128 heads, cache blocks that are a multiple of 16 tokens."""
+    Nh, W = q.shape[1], q.shape[2]
     return (q.is_cuda and q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16
-            and L == 512 and q.shape[2] == 576 and cache.shape[-1] == 576
-            and 0 < Nh <= 128 and (Nh & (Nh - 1)) == 0 and cache.shape[-2] % 16 == 0)
+            and 0 < L <= 512 and L % 64 == 0 and L <= W <= 576 and W % 64 == 0
+            and cache.shape[-1] == W and 0 < Nh <= 128 and cache.shape[-2] % 16 == 0)
 
 
 def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
                   seq_lens: torch.Tensor, cu_q: Optional[torch.Tensor], num_tiles: int,
                   max_seq_len: int, scale: float, out: Optional[torch.Tensor] = None,
-                  splits: Optional[int] = None) -> torch.Tensor:
-    """Latent-absorbed multi-head latent attention (attention_mla.cu).  q ``[T, N, 576]``,
-    cache ``[blocks, block_size, 576]``, returns ``[T, N, 512]``.  ``cu_q`` None: one query
-    token per request (decode).  ``num_tiles`` >= sum over requests of
-    ceil(q_len / (128 // N)).  Causal inside each request over absolute positions."""
+                  splits: Optional[int] = None, L: int = 512) -> torch.Tensor:
+    """Latent-absorbed multi-head latent attention (attention_mla.cu).  q ``[T, N, W]``,
+    cache ``[blocks, block_size, W]`` whose first ``L`` columns are the value, returns
+    ``[T, N, L]``.  ``cu_q`` None: one query token per request (decode).  ``num_tiles`` >= sum
+    over requests of ceil(q_len / (128 // N)).  Causal inside each request over absolute
+    positions."""
     T, Nh, W = q.shape
     assert q.is_contiguous() and cache.is_contiguous()
     nb, bs, _ = cache.shape
     if out is None:
-        out = torch.empty((T, Nh, 512), dtype=q.dtype, device=q.device)
+        out = torch.empty((T, Nh, L), dtype=q.dtype, device=q.device)
     B = block_tables.shape[0]
     if splits is None:
-        ctas = max(num_tiles, 1) * 2
+        ctas = max(num_tiles, 1) * (2 if L > 256 else 1)
         global _SM_COUNT
         if _SM_COUNT == 0:
             _SM_COUNT = max(1, int(N.lib().b200_sm_count()))
         splits = max(1, min(_SM_COUNT // ctas, (max_seq_len + 255) // 256, 16))
     ws = None
     if splits > 1:
-        ws = torch.empty(splits * T * Nh * 513, dtype=torch.float32, device=q.device)
+        ws = torch.empty(splits * T * Nh * (L + 1), dtype=torch.float32, device=q.device)
     rc = N.lib().b200_mla_attention(
         ptr(q), ptr(out), ptr(cache), nb * bs, ptr(cu_q), ptr(seq_lens), ptr(block_tables),
-        block_tables.stride(0), bs, B, T, Nh, int(num_tiles), int(splits), ptr(ws), float(scale),
-        stream_ptr())
+        block_tables.stride(0), bs, B, T, Nh, W, L, int(num_tiles), int(splits), ptr(ws),
+        float(scale), stream_ptr())
     N.launch_count += 1
     if rc != 0:
         raise N.NativeError(f"b200_mla_attention failed with code {rc}")
+    return out
+
+
+def latent_cache(kv: torch.Tensor, weight: torch.Tensor, eps: float, cache: torch.Tensor,
+                 slot_mapping: torch.Tensor, x: Optional[torch.Tensor] = None,
+                 state: Optional[torch.Tensor] = None, num_decodes: int = 0,
+                 cu_q: Optional[torch.Tensor] = None) -> None:
+    """RMSNorm of the latent projection ``kv [T, L]`` (a row-strided view) into the rows of
+    ``cache [blocks, block_size, W >= L]`` (zeros behind L).  With ``state [blocks, H]`` fp32 the
+    row of ``x [T, H]`` fp32 of the last token that the step writes into a block is kept there."""
+    T, L = kv.shape
+    nb, bs, W = cache.shape
+    assert kv.stride(1) == 1 and cache.is_contiguous() and cache.dtype == kv.dtype
+    call("b200_latent_cache", ptr(kv), kv.stride(0), ptr(weight), float(eps), ptr(cache), nb * bs,
+         W, ptr(slot_mapping), ptr(x), ptr(state), ptr(cu_q), T, L,
+         x.shape[1] if x is not None else 0, num_decodes,
+         cu_q.shape[0] - 1 if cu_q is not None else 0, bs, DTYPE_CODE[kv.dtype], stream_ptr())
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
+                     seq_lens: torch.Tensor, num_decodes: int, cu_q: Optional[torch.Tensor],
+                     scale: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Latent attention for any width and head count, fp32 or bf16 (csrc/latent.cu): q
+    ``[T, N, W]``, the first ``num_decodes`` tokens one per request, the rest by ``cu_q``."""
+    T, Nh, W = q.shape
+    nb, bs, _ = cache.shape
+    assert q.is_contiguous() and cache.is_contiguous() and cache.dtype == q.dtype
+    if out is None:
+        out = torch.empty_like(q)
+    call("b200_latent_attention", ptr(q), ptr(cache), nb * bs, ptr(out), ptr(block_tables),
+         block_tables.stride(0), bs, ptr(seq_lens), ptr(cu_q), T, Nh, W, num_decodes,
+         cu_q.shape[0] - 1 if cu_q is not None else 0, float(scale), DTYPE_CODE[q.dtype],
+         stream_ptr())
+    return out
+
+
+# ---------------------------------------------------------------------------
+# fp32 residual stream: token shift, post-norm, depth average, output gate (csrc/residual.cu)
+# ---------------------------------------------------------------------------
+def token_shift(x: torch.Tensor, mu: torch.Tensor, dtype: torch.dtype,
+                state: Optional[torch.Tensor] = None,
+                block_tables: Optional[torch.Tensor] = None,
+                positions: Optional[torch.Tensor] = None, num_decodes: int = 0,
+                cu_q: Optional[torch.Tensor] = None, block_size: int = 1) -> torch.Tensor:
+    """``x + (x_prev - x) * mu`` on fp32 rows ``[T, H]``; rows in front of a portion come from
+    ``state [blocks, H]`` (see :func:`latent_cache`).  Result in ``dtype``."""
+    T, H = x.shape
+    out = torch.empty((T, H), dtype=dtype, device=x.device)
+    use = state is not None
+    call("b200_token_shift", ptr(x), ptr(mu), ptr(state), ptr(block_tables) if use else None,
+         ptr(positions), ptr(cu_q), ptr(out), T, H, num_decodes,
+         cu_q.shape[0] - 1 if cu_q is not None else 0,
+         block_tables.stride(0) if use else 0, block_size, state.shape[0] if use else 0,
+         DTYPE_CODE[dtype], stream_ptr())
+    return out
+
+
+def post_norm(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, alpha: float, eps: float,
+              pos_of: Optional[torch.Tensor] = None, k: int = 0,
+              res: Optional[torch.Tensor] = None, hist: Optional[torch.Tensor] = None, n: int = 0,
+              weights: Optional[torch.Tensor] = None, avg: Optional[torch.Tensor] = None,
+              final_gain: Optional[torch.Tensor] = None, lo: Optional[torch.Tensor] = None) -> None:
+    """``r = rms(alpha * x + y) * gain`` over fp32 rows ``x [T, H]``; ``y`` a dense row, or with
+    ``pos_of [T * k]`` the sum of the token's expert-sorted rows.  ``res`` takes r.  With ``hist
+    [>= n, T, H]``: ``avg = sum_j weights[j] * hist[j] + weights[n] * r``.  ``lo`` takes the last
+    result in ``y``'s type, through the final norm if ``final_gain`` is given."""
+    T, H = x.shape
+    call("b200_post_norm", ptr(x), ptr(y), y.stride(0), ptr(pos_of), k, ptr(gain), float(alpha),
+         float(eps), ptr(res), ptr(hist), hist.stride(0) if hist is not None else 0, n,
+         ptr(weights), ptr(avg), ptr(final_gain), ptr(lo), T, H, DTYPE_CODE[y.dtype], stream_ptr())
+
+
+def sigmoid_gate(o: torch.Tensor, z: torch.Tensor, out: Optional[torch.Tensor] = None
+                 ) -> torch.Tensor:
+    """``o * sigmoid(z)``; both ``[T, D]``, row-strided views are fine."""
+    T, D = o.shape
+    if out is None:
+        out = torch.empty((T, D), dtype=o.dtype, device=o.device)
+    call("b200_sigmoid_gate", ptr(o), o.stride(0), ptr(z), z.stride(0), ptr(out), out.stride(0), T,
+         D, DTYPE_CODE[o.dtype], stream_ptr())
     return out
 
 
@@ -792,6 +873,38 @@ def fused_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: 
          add.stride(0) if add is not None else 0, ptr(out), H, ptr(valid_tokens), T, k, H,
          float(alpha), DTYPE_CODE[x.dtype], stream_ptr())
     return out
+
+
+def input_weighted_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor,
+                           topk_w: torch.Tensor, topk_ids: torch.Tensor
+                           ) -> tuple[torch.Tensor, torch.Tensor]:
+    """Routed experts whose weight multiplies their input: align -> permute fp32 rows ``x [T, H]``
+    times the weight -> grouped GEMM1 (SiLU-mul) -> grouped GEMM2.  Returns the expert-sorted
+    outputs ``[cap, Hp]`` and ``pos_of [T * k]``, the row of every (token, slot) pair; the caller's
+    norm kernel sums them.  bf16 experts: ``w13 [E, 2I, Hp]`` interleaved in blocks of
+    ``ref.GATE_UP_BLOCK`` rows; fp32 experts: gate rows first, plain fp32 arithmetic."""
+    T, H = x.shape
+    k = topk_ids.shape[1]
+    E, I2, Hp = w13.shape
+    numel = T * k
+    cap = moe_align_cap(numel, E)
+    sorted_ids, expert_ids, npp, pos_of = moe_align(topk_ids, E, cap)
+    a_sorted = torch.empty((cap, Hp), device=x.device, dtype=w13.dtype)
+    call("b200_moe_permute_weighted", ptr(x), x.stride(0), ptr(topk_w), ptr(a_sorted), Hp,
+         ptr(sorted_ids), ptr(npp), numel, k, H, Hp, cap, DTYPE_CODE[w13.dtype], stream_ptr())
+    if w13.dtype == torch.bfloat16:
+        h = gemm_bf16_grouped(a_sorted, w13, expert_ids, npp, silu_mul=True)
+        return gemm_bf16_grouped(h, w2, expert_ids, npp), pos_of
+    I = I2 // 2
+    u = torch.empty((cap, I2), device=x.device, dtype=torch.float32)
+    call("b200_grouped_gemm_f32", ptr(a_sorted), Hp, ptr(w13), ptr(u), I2, cap, I2, Hp, E,
+         ptr(expert_ids), ptr(npp), stream_ptr())
+    h = torch.empty((cap, I), device=x.device, dtype=torch.float32)
+    call("b200_silu_mul_rows_f32", ptr(u), ptr(h), cap, I, ptr(npp), stream_ptr())
+    y = torch.empty((cap, Hp), device=x.device, dtype=torch.float32)
+    call("b200_grouped_gemm_f32", ptr(h), I, ptr(w2), ptr(y), Hp, cap, Hp, I, E, ptr(expert_ids),
+         ptr(npp), stream_ptr())
+    return y, pos_of
 
 
 def gemm_q8_grouped(a: torch.Tensor, a_scale: torch.Tensor, w: torch.Tensor,

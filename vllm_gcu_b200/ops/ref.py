@@ -576,6 +576,125 @@ def advance_step(num_seqs: int, num_queries: int, block_size: int, input_tokens:
 
 
 # ---------------------------------------------------------------------------
+# latent attention, fp32 residual stream
+# ---------------------------------------------------------------------------
+def latent_attention(q_full: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
+                     q_lens: list[int], seq_lens: list[int], scale: float, L: int
+                     ) -> torch.Tensor:
+    """q_full ``[T, N, W]`` (latent query, then the rotated rope part if there is one); cache
+    ``[blocks, bs, W]``.  Returns the latent-space output ``[T, N, L]``.  Causal inside each
+    request."""
+    T, N, W = q_full.shape
+    nb, bs, _ = cache.shape
+    flat = cache.view(nb * bs, W)
+    out = torch.zeros(T, N, L, dtype=q_full.dtype, device=q_full.device)
+    t0 = 0
+    for b, (ql, n) in enumerate(zip(q_lens, seq_lens)):
+        if ql == 0 or n == 0:
+            t0 += ql
+            continue
+        pos = torch.arange(n, device=cache.device)
+        slots = block_tables[b, (pos // bs).long()].long() * bs + pos % bs
+        kv = flat[slots].float()                               # [n, W]
+        q = q_full[t0:t0 + ql].float()                         # [ql, N, W]
+        s = torch.einsum("qhw,nw->hqn", q, kv) * scale
+        qpos = torch.arange(n - ql, n, device=cache.device)[:, None]
+        s = s.masked_fill((pos[None, :] > qpos)[None], float("-inf"))
+        p = torch.softmax(s, dim=-1)
+        out[t0:t0 + ql] = torch.einsum("hqn,nl->qhl", p, kv[:, :L]).to(out.dtype)
+        t0 += ql
+    return out
+
+
+def _portions(T: int, num_decodes: int, cu_q: Optional[torch.Tensor]) -> list[tuple[int, int]]:
+    """(first, end) token of every request of a step, in order."""
+    out = [(t, t + 1) for t in range(num_decodes)]
+    if cu_q is not None:
+        c = [int(v) + num_decodes for v in cu_q]
+        out += list(zip(c[:-1], c[1:]))
+    return out
+
+
+def latent_cache(kv, weight, eps, cache, slot_mapping, x=None, state=None, num_decodes=0,
+                 cu_q=None) -> None:
+    """See ``ops.cuda.latent_cache``."""
+    L = kv.shape[1]
+    nb, bs, W = cache.shape
+    c = rms_norm(kv, weight, eps)
+    ok = slot_mapping >= 0
+    rows = torch.zeros(int(ok.sum()), W, dtype=cache.dtype, device=cache.device)
+    rows[:, :L] = c[ok].to(cache.dtype)
+    cache.view(nb * bs, W)[slot_mapping[ok].long()] = rows
+    if state is None:
+        return
+    for lo, hi in _portions(kv.shape[0], num_decodes, cu_q):
+        for t in range(lo, hi):
+            slot = int(slot_mapping[t])
+            if slot >= 0 and (t == hi - 1 or (slot + 1) % bs == 0):
+                state[slot // bs] = x[t]
+
+
+def token_shift(x, mu, dtype, state=None, block_tables=None, positions=None, num_decodes=0,
+                cu_q=None, block_size=1) -> torch.Tensor:
+    """See ``ops.cuda.token_shift``."""
+    prev = torch.zeros_like(x)
+    prev[1:] = x[:-1]
+    for r, (lo, hi) in enumerate(_portions(x.shape[0], num_decodes, cu_q)):
+        if hi == lo:
+            continue
+        pos = int(positions[lo])
+        prev[lo] = 0.0 if state is None or pos == 0 else \
+            state[int(block_tables[r, (pos - 1) // block_size])]
+    return (x + (prev - x) * mu).to(dtype)
+
+
+def scalar_rms_norm(x: torch.Tensor, gain: torch.Tensor, eps: float) -> torch.Tensor:
+    """RMS norm with one gain for all coordinates, fp32."""
+    x = x.float()
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * gain.float()
+
+
+def post_norm(x, y, gain, alpha, eps, pos_of=None, k=0, res=None, hist=None, n=0, weights=None,
+              avg=None, final_gain=None, lo=None) -> None:
+    """See ``ops.cuda.post_norm``."""
+    T, H = x.shape
+    if pos_of is not None:
+        p = pos_of[:T * k].view(T, k).long()
+        y = (y[p.clamp(min=0)].float() * (p >= 0).unsqueeze(-1)).sum(1)[:, :H]
+    r = scalar_rms_norm(alpha * x + y.float(), gain, eps)
+    if res is not None:
+        res.copy_(r)
+    if hist is not None:
+        r = (weights[:n, None, None] * hist[:n]).sum(0) + weights[n] * r
+        if avg is not None:
+            avg.copy_(r)
+    if lo is not None:
+        lo.copy_(r if final_gain is None else scalar_rms_norm(r, final_gain, eps))
+
+
+def sigmoid_gate(o: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
+    return (o.float() * torch.sigmoid(z.float())).to(o.dtype)
+
+
+def input_weighted_experts(x, w13, w2, topk_w, topk_ids) -> tuple[torch.Tensor, torch.Tensor]:
+    """See ``ops.cuda.input_weighted_experts`` (gate rows first in ``w13``); one output row per
+    (token, slot) pair, so ``pos_of`` is the identity."""
+    T, H = x.shape
+    k = topk_ids.shape[1]
+    Hp = w13.shape[2]
+    y = torch.zeros(T * k, Hp, dtype=w13.dtype, device=x.device)
+    xi = torch.nn.functional.pad(x, (0, Hp - H))
+    a = (topk_w.unsqueeze(-1) * xi.unsqueeze(1)).reshape(T * k, Hp).to(w13.dtype)
+    flat = topk_ids.reshape(-1)
+    for e in range(w13.shape[0]):
+        rows = (flat == e).nonzero(as_tuple=True)[0]
+        if rows.numel():
+            h = silu_and_mul(a[rows] @ w13[e].t())
+            y[rows] = h @ w2[e].t()
+    return y, torch.arange(T * k, dtype=torch.int32, device=x.device)
+
+
+# ---------------------------------------------------------------------------
 # mixture of experts
 # ---------------------------------------------------------------------------
 def topk_softmax(gating: torch.Tensor, k: int, renormalize: bool
