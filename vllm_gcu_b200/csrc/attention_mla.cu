@@ -97,8 +97,10 @@ struct Args {
   unsigned int* status;
 };
 
-template <int QROWS, int kStages>
-__global__ void __launch_bounds__(kThreads, 1)
+// kResident CTAs share an SM: two where shared and tensor memory allow it (narrow latents, whose
+// tiles are too small to hide the latency of the chain loads -> scores -> softmax -> output)
+template <int QROWS, int kStages, int kResident>
+__global__ void __launch_bounds__(kThreads, kResident)
     mla_attn_kernel(const __grid_constant__ CUtensorMap tmQ,
                     const __grid_constant__ CUtensorMap tmK, const Args a) {
   extern __shared__ uint8_t smem_raw[];
@@ -559,19 +561,19 @@ static int get_map(const void* base, unsigned long long rows, int W, int box_row
 namespace b200 {
 namespace mla {
 
-template <int QROWS, int STAGES>
+template <int QROWS, int STAGES, int RESIDENT>
 static int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const Args& a, dim3 grid,
                   int smem, cudaStream_t s) {
   static int configured[64] = {0};       // largest size allowed so far, per device
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && configured[dev] < smem) {
-    cudaError_t e = cudaFuncSetAttribute(mla_attn_kernel<QROWS, STAGES>,
+    cudaError_t e = cudaFuncSetAttribute(mla_attn_kernel<QROWS, STAGES, RESIDENT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev] = smem;
   }
-  mla_attn_kernel<QROWS, STAGES><<<grid, kThreads, smem, s>>>(tmQ, tmK, a);
+  mla_attn_kernel<QROWS, STAGES, RESIDENT><<<grid, kThreads, smem, s>>>(tmQ, tmK, a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -633,10 +635,13 @@ B200_API int b200_mla_attention(const void* q, void* out, const void* cache, lon
   a.status = status_ptr();
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   dim3 grid(num_tiles * a.halves, splits);
+  const bool pair = stages == 2 && a.tmem_cols == 256 && lay.bytes <= kMaxSmem / 2 - 1024;
   int e;
-  if (small) e = launch<32, 2>(tmQ, tmK, a, grid, lay.bytes, s);
-  else if (stages == 2) e = launch<BQ, 2>(tmQ, tmK, a, grid, lay.bytes, s);
-  else e = launch<BQ, 1>(tmQ, tmK, a, grid, lay.bytes, s);
+  if (small) e = pair ? launch<32, 2, 2>(tmQ, tmK, a, grid, lay.bytes, s)
+                      : launch<32, 2, 1>(tmQ, tmK, a, grid, lay.bytes, s);
+  else if (stages == 2) e = pair ? launch<BQ, 2, 2>(tmQ, tmK, a, grid, lay.bytes, s)
+                                 : launch<BQ, 2, 1>(tmQ, tmK, a, grid, lay.bytes, s);
+  else e = launch<BQ, 1, 1>(tmQ, tmK, a, grid, lay.bytes, s);
   if (e != 0 || splits == 1) return e;
   mla_combine_kernel<<<static_cast<unsigned>(rows_total), L / 4, 0, s>>>(
       a.ws_o, a.ws_lse, a.out, rows_total, splits, L);

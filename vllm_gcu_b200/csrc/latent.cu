@@ -42,28 +42,45 @@ __global__ void __launch_bounds__(128) latent_cache_kernel(const CacheArgs a) {
     return;
   }
   const T* kv = static_cast<const T*>(a.kv) + static_cast<long long>(t) * a.ldkv;
+  // the state row first: its loads and stores overlap the latency of the norm
+  if (a.x != nullptr) {
+    const TokenPlace pl = token_place(t, a.num_decodes, a.num_prefills, a.cu_q);
+    if (pl.last || (slot + 1) % a.block_size == 0) {
+      const float* x = a.x + static_cast<long long>(t) * a.H;
+      float* st = a.state + slot / a.block_size * a.H;
+      if ((a.H % 4) == 0) {
+#pragma unroll 4
+        for (int c = threadIdx.x; c < a.H / 4; c += blockDim.x)
+          reinterpret_cast<float4*>(st)[c] = reinterpret_cast<const float4*>(x)[c];
+      } else {
+        for (int c = threadIdx.x; c < a.H; c += blockDim.x) st[c] = x[c];
+      }
+    }
+  }
+  const T* w = static_cast<const T*>(a.weight);
+  T* dst = static_cast<T*>(a.cache) + slot * a.W;
+  constexpr int kKeep = 8;                 // columns per thread that stay in registers
+  float v[kKeep];
   float ss = 0.0f;
-  for (int c = threadIdx.x; c < a.L; c += blockDim.x) {
-    const float v = to_f32<T>(kv[c]);
-    ss += v * v;
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    v[i] = c < a.L ? to_f32<T>(kv[c]) : 0.0f;
+    ss += v[i] * v[i];
+  }
+  for (int c = threadIdx.x + kKeep * blockDim.x; c < a.L; c += blockDim.x) {
+    const float u = to_f32<T>(kv[c]);
+    ss += u * u;
   }
   ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.L) + a.eps);
-  const T* w = static_cast<const T*>(a.weight);
-  T* dst = static_cast<T*>(a.cache) + slot * a.W;
-  for (int c = threadIdx.x; c < a.W; c += blockDim.x)
-    dst[c] = c < a.L ? from_f32<T>(to_f32<T>(kv[c]) * inv * to_f32<T>(w[c])) : from_f32<T>(0.0f);
-  if (a.x == nullptr) return;
-  const TokenPlace pl = token_place(t, a.num_decodes, a.num_prefills, a.cu_q);
-  if (!pl.last && (slot + 1) % a.block_size != 0) return;
-  const float* x = a.x + static_cast<long long>(t) * a.H;
-  float* st = a.state + slot / a.block_size * a.H;
-  if ((a.H % 4) == 0) {
-    for (int c = threadIdx.x; c < a.H / 4; c += blockDim.x)
-      reinterpret_cast<float4*>(st)[c] = reinterpret_cast<const float4*>(x)[c];
-  } else {
-    for (int c = threadIdx.x; c < a.H; c += blockDim.x) st[c] = x[c];
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < a.W) dst[c] = from_f32<T>(c < a.L ? v[i] * inv * to_f32<T>(w[c]) : 0.0f);
   }
+  for (int c = threadIdx.x + kKeep * blockDim.x; c < a.W; c += blockDim.x)
+    dst[c] = from_f32<T>(c < a.L ? to_f32<T>(kv[c]) * inv * to_f32<T>(w[c]) : 0.0f);
 }
 
 // ---------------------------------------------------------------------------

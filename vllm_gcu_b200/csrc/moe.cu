@@ -261,6 +261,22 @@ __global__ void __launch_bounds__(256)
   const float w = pad ? 0.0f : topk_w[pair];
   const float* src = x + static_cast<long long>(pad ? 0 : pair / k) * ldx;
   const bool vec = (H % 4) == 0 && (ldx % 4) == 0;
+  if constexpr (sizeof(T) == 2) {
+    if ((H % 8) == 0 && (ldx % 4) == 0 && Ho == H && (ldo % 8) == 0) {
+      // whole 16-byte stores
+      for (int c = threadIdx.x * 8; c < H; c += blockDim.x * 8) {
+        uint4 u = make_uint4(0u, 0u, 0u, 0u);
+        if (!pad) {
+          const float4 f = *reinterpret_cast<const float4*>(src + c);
+          const float4 g = *reinterpret_cast<const float4*>(src + c + 4);
+          u = make_uint4(pack_bf16x2(w * f.x, w * f.y), pack_bf16x2(w * f.z, w * f.w),
+                         pack_bf16x2(w * g.x, w * g.y), pack_bf16x2(w * g.z, w * g.w));
+        }
+        *reinterpret_cast<uint4*>(dst + c) = u;
+      }
+      return;
+    }
+  }
   for (int c = threadIdx.x * 4; c < Ho; c += blockDim.x * 4) {
     float4 f = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     if (!pad && vec && c < H) {

@@ -28,7 +28,9 @@ __device__ __forceinline__ void ldv(const float* p, float (&f)[V]) {
 }
 template <int V>
 __device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&f)[V]) {
-  if constexpr (V == 4) {
+  if constexpr (V == 8) {
+    vec8_load<__nv_bfloat16>(p, f);
+  } else if constexpr (V == 4) {
     const uint2 u = *reinterpret_cast<const uint2*>(p);
     const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
     f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
@@ -46,7 +48,9 @@ __device__ __forceinline__ void stv(float* p, const float (&f)[V]) {
 }
 template <int V>
 __device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&f)[V]) {
-  if constexpr (V == 4) {
+  if constexpr (V == 8) {
+    vec8_store<__nv_bfloat16>(p, f);
+  } else if constexpr (V == 4) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
   } else {
     p[0] = __float2bfloat16(f[0]);
@@ -325,7 +329,9 @@ B200_API int b200_sigmoid_gate(const void* o, long long ldo, const void* z, long
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const bool v4 = (D % 4) == 0 && (ldo % 4) == 0 && (ldz % 4) == 0 && (ldout % 4) == 0 &&
                   aligned(o, 16) && aligned(z, dtype == 0 ? 8 : 16) && aligned(out, 16);
-  const long long items = static_cast<long long>(T) * (v4 ? D / 4 : D);
+  const bool v8 = dtype == 0 && v4 && (D % 8) == 0 && (ldo % 8) == 0 && (ldz % 8) == 0 &&
+                  (ldout % 8) == 0 && aligned(z, 16);
+  const long long items = static_cast<long long>(T) * (v8 ? D / 8 : v4 ? D / 4 : D);
   long long blocks = (items + 255) / 256;
   const long long cap = static_cast<long long>(sm_count()) * 16;
   if (blocks > cap) blocks = cap;
@@ -334,7 +340,8 @@ B200_API int b200_sigmoid_gate(const void* o, long long ldo, const void* z, long
     const __nv_bfloat16* po = static_cast<const __nv_bfloat16*>(o);
     const __nv_bfloat16* pz = static_cast<const __nv_bfloat16*>(z);
     __nv_bfloat16* pq = static_cast<__nv_bfloat16*>(out);
-    if (v4) sigmoid_gate_kernel<__nv_bfloat16, 4><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
+    if (v8) sigmoid_gate_kernel<__nv_bfloat16, 8><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
+    else if (v4) sigmoid_gate_kernel<__nv_bfloat16, 4><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
     else sigmoid_gate_kernel<__nv_bfloat16, 1><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
   } else {
     const float* po = static_cast<const float*>(o);

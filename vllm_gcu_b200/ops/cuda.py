@@ -647,7 +647,8 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tens
         global _SM_COUNT
         if _SM_COUNT == 0:
             _SM_COUNT = max(1, int(N.lib().b200_sm_count()))
-        splits = max(1, min(_SM_COUNT // ctas, (max_seq_len + 255) // 256, 16))
+        slots = _SM_COUNT * (2 if L <= 128 else 1)       # narrow latents: two CTAs per SM
+        splits = max(1, min(slots // ctas, (max_seq_len + 255) // 256, 16))
     ws = None
     if splits > 1:
         ws = torch.empty(splits * T * Nh * (L + 1), dtype=torch.float32, device=q.device)
