@@ -32,6 +32,9 @@ CONFIGS = {
     # sizes that are whole tiles nowhere
     "odd": model_config(203, 100, 3.1, 1e-5, [layer(7, 12, 20, 44, 0.25, 9, 4, 20),
                                               layer(3, 28, 12, 52, 0.15, 4, 1, 36)]),
+    # no size is a multiple of anything
+    "prime": model_config(101, 37, 2.6, 1e-4, [layer(3, 5, 7, 9, 0.6, 5, 3, 11),
+                                               layer(1, 3, 11, 13, 0.8, 7, 2, 5)]),
     # wider than one 64-column tile, more heads than a power of two, no feed-forward at the end
     "wide": model_config(500, 192, 2.2, 1e-5, [layer(12, 48, 40, 80, 0.14, 8, 3, 96),
                                                layer(6, 64, 72, 144, 0.12, 12, 2, 64),

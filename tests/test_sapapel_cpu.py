@@ -163,7 +163,8 @@ def test_configuration_reader():
         d["layers"][0].update(bad)
         with pytest.raises(ValueError):
             ModelConfig.from_hf_dict(d)
-    assert preset("tiny-sapapel", num_hidden_layers=5, dtype="float32").num_hidden_layers == 5
+    p = preset("tiny-sapapel", num_hidden_layers=5, dtype="float32")
+    assert p.num_hidden_layers == 5 == len(p.layer_specs)
 
 
 def test_missing_and_extra_tensors(tmp_path):

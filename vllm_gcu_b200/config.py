@@ -100,6 +100,11 @@ class ModelConfig:
 
     def __post_init__(self) -> None:
         self.dtype = to_dtype(self.dtype)
+        if self.layer_specs is not None and len(self.layer_specs) != self.num_hidden_layers:
+            # a shorter or longer model of the same layers
+            n = self.num_hidden_layers
+            reps = -(-n // len(self.layer_specs))
+            self.layer_specs = (tuple(self.layer_specs) * reps)[:n]
         if self.head_dim <= 0:
             self.head_dim = self.hidden_size // self.num_attention_heads
 
@@ -381,10 +386,7 @@ def preset(name: str, **overrides) -> ModelConfig:
                               rope_is_neox=False, dtype="float32"),
     }
     if name in _LAYER_LIST_PRESETS:
-        n = overrides.pop("num_hidden_layers", None)
-        d = _LAYER_LIST_PRESETS[name]
-        layers = d["layers"] if n is None else (d["layers"] * n)[:n]
-        return ModelConfig.from_hf_dict({**d, "layers": layers}, **overrides)
+        return ModelConfig.from_hf_dict(_LAYER_LIST_PRESETS[name], **overrides)
     kw = dict(presets[name])
     kw.update(overrides)
     return ModelConfig(**kw)
@@ -401,8 +403,7 @@ def _sapapel_preset(layers: int, vocab: int, width: int, heads: int, dim: int, v
             "postln_alpha": (2.0 * layers) ** 0.25, "layers": [layer] * layers}
 
 
-#: configurations of designs that are described layer by layer (``num_hidden_layers`` repeats or
-#: truncates the list)
+#: configurations of designs that are described layer by layer
 _LAYER_LIST_PRESETS: dict[str, dict] = {
     "tiny-sapapel": _sapapel_preset(3, 1024, 128, 4, 24, 40, 48, 6, 2, 48),
     # layers of the size of DeepSeek-V2-Lite's

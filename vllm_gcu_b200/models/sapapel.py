@@ -87,7 +87,7 @@ class SapapelLayer(nn.Module):
 class SapapelForCausalLM(DecoderLM):
     # CUDA sources with the kernels of this model (a fresh checkout may build only these)
     native_sources = ("common", "attention_mla", "gemm_bf16", "gemm_pair", "gemm_skinny", "latent",
-                      "moe", "residual", "sampler", "spec", "step", "cache")
+                      "moe", "residual", "sampler", "step", "cache")
     # the shift's state follows the cache blocks; a rejected draft token would leave its row there
     has_block_state = True
 
