@@ -375,3 +375,30 @@ def test_layer_spec_is_frozen():
     assert not LayerSpec("latent_attention", 1, 1, 1, 1, 1.0).has_mlp
     assert layer(1, 1, 1, 1, 1.0)["mlp"] is None
     assert model_config(8, 4, 1.0, 1e-5, [])["layers"] == []
+
+
+@pytest.mark.timeout(120)
+def test_server_from_its_command_line(tmp_path):
+    import argparse
+    import asyncio
+    httpx = pytest.importorskip("httpx")
+    from vllm_gcu_b200.entrypoints.api_server import (ByteTokenizer, add_engine_arguments,
+                                                      build_app, make_engine)
+    cfg, w, path = _checkpoint(tmp_path, "prime", seed=12)
+    ap = argparse.ArgumentParser()
+    add_engine_arguments(ap)
+    eng, mc = make_engine(ap.parse_args(["--model", path, "--device", "cpu", "--dtype", "float32",
+                                         "--max-num-seqs", "4", "--max-model-len", "128"]))
+    app = build_app(eng, ByteTokenizer(mc.vocab_size), "sapapel")
+    prompts = [tokens_for(cfg, n, n) for n in (5, 33)]
+
+    async def call():
+        async with httpx.AsyncClient(transport=httpx.ASGITransport(app=app),
+                                     base_url="http://t") as c:
+            return (await c.post("/v1/completions", json={
+                "prompt": prompts, "max_tokens": 6, "temperature": 0.0, "ignore_eos": True})).json()
+    try:
+        out = asyncio.run(call())
+    finally:
+        eng.shutdown()
+    assert [c["token_ids"] for c in out["choices"]] == [greedy(cfg, w, p, 6) for p in prompts]
