@@ -27,21 +27,62 @@ def to_dtype(x: Any) -> torch.dtype:
 
 
 @dataclass(frozen=True)
+class AttentionSpec:
+    """Attention over keys that are their own values (layers/key_attention.py)."""
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    scale: float                           # score scale
+    rot_dims: int                          # rotated dimensions of every head
+    rot_base: float
+
+
+@dataclass(frozen=True)
+class MemorySpec:
+    """Matrix memory with exponential gates (layers/recurrent.py)."""
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+    gate_cap: float                        # soft cap of the gates' projections
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Gated delta rule with one decay per key channel (layers/recurrent.py)."""
+    num_heads: int
+    num_kv_heads: int                      # query / key heads
+    head_dim: int
+    v_head_dim: int
+    conv_taps: int
+    decay_rank: int                        # inner width of the decay's two-step projection
+    gate_rank: int                         # and of the output gate's
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One layer of a design whose layers differ: mixer type and sizes, feed-forward sizes."""
-    mixer: str                             # "latent_attention"
-    num_heads: int
-    head_dim: int                          # query / key dimensions per head
-    v_head_dim: int
-    kv_lora_rank: int                      # latent width
-    scale: float                           # score scale
-    num_experts: int = 0                   # 0: no feed-forward
+    mixer: str                             # "latent_attention", or with ``parts`` any name
+    num_heads: int = 0
+    head_dim: int = 0                      # query / key dimensions per head
+    v_head_dim: int = 0
+    kv_lora_rank: int = 0                  # latent width
+    scale: float = 1.0                     # score scale
+    num_experts: int = 0
     num_experts_per_tok: int = 0
     moe_intermediate_size: int = 0
+    intermediate_size: int = 0             # dense feed-forward
+    # mixer as a sum of parts: (checkpoint prefix, factor, spec)
+    parts: tuple[tuple[str, float, Any], ...] = ()
 
     @property
     def has_mlp(self) -> bool:
-        return self.num_experts > 0
+        return self.num_experts > 0 or self.intermediate_size > 0
+
+    @property
+    def cached_per_token(self) -> int:
+        """Elements a token leaves in the paged cache."""
+        return self.kv_lora_rank + sum(2 * s.num_kv_heads * s.head_dim for _, _, s in self.parts
+                                       if isinstance(s, AttentionSpec))
 
 
 @dataclass
@@ -96,6 +137,8 @@ class ModelConfig:
     # designs described layer by layer (None: every layer has the sizes above)
     layer_specs: Optional[tuple[LayerSpec, ...]] = None
     residual_alpha: float = 1.0            # norm after the sum: norm(alpha * x + sublayer(x))
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
     extra: dict = field(default_factory=dict)
 
     def __post_init__(self) -> None:
@@ -136,7 +179,7 @@ class ModelConfig:
         es = 1 if self.kv_cache_dtype.startswith("fp8") or self.kv_cache_dtype == "int8" else \
             torch.empty((), dtype=self.dtype).element_size()
         if self.layer_specs is not None:
-            return sum(s.kv_lora_rank for s in self.layer_specs) * es
+            return sum(s.cached_per_token for s in self.layer_specs) * es
         if self.is_mla:
             return self.num_hidden_layers * (self.kv_lora_rank + self.qk_rope_head_dim) * es
         kvh = max(1, self.num_key_value_heads // tp_size)
@@ -182,6 +225,9 @@ class ModelConfig:
         if d.get("architecture") == "Sapapel" or "SapapelForCausalLM" in (
                 d.get("architectures") or ()):
             return cls._from_layer_list(d, **overrides)
+        if d.get("architecture") == "Fizunex" or "FizunexForCausalLM" in (
+                d.get("architectures") or ()):
+            return cls._from_mixer_list(d, **overrides)
         archs = d.get("architectures") or ["LlamaForCausalLM"]
         for nested in ("text_config", "language_config", "llm_config"):
             if isinstance(d.get(nested), dict):
@@ -312,9 +358,69 @@ class ModelConfig:
         return cls(**kw)
 
     @classmethod
+    def _from_mixer_list(cls, d: dict, **overrides) -> "ModelConfig":
+        """Fizunex's ``config.json``: ``vocab``, ``width``, ``norm.eps``, ``embedding.scale``,
+        ``logit_scale`` and one entry of ``layers`` per layer.  The inner widths of a delta layer's
+        two-step projections are no numbers of the file: a checkpoint's tensors give them
+        (``tensor_shapes``), else ``decay_rank`` / ``gate_rank`` of the mixer, else its ``dim``."""
+        shapes = overrides.pop("tensor_shapes", None) or {}
+        specs = []
+        for i, layer in enumerate(d["layers"]):
+            m, f, where = layer["mixer"], layer.get("mlp"), f"layer {i}"
+            ff = 0
+            if f is not None:
+                if f.get("kind", "dense") != "dense":
+                    raise ValueError(f"{where}: unknown feed-forward {f['kind']!r}")
+                ff = int(f["ff"])
+            if layer["type"] == "channel_delta":
+                def rank(tensor: str, key: str) -> int:
+                    s = shapes.get(f"l{i}.mix.{tensor}")
+                    return int(s[0] if s is not None else m.get(key) or m["dim"])
+                parts = (("", 1.0, DeltaSpec(
+                    int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]),
+                    int(m["conv"]), rank("a1", "decay_rank"), rank("g1", "gate_rank"))),)
+            elif layer["type"] == "parallel":
+                a, b = m["left"], m["right"]
+                if int(a.get("vdim", a["dim"])) != int(a["dim"]):
+                    raise ValueError(f"{where}: values are the keys, so {a['vdim']} value "
+                                     f"dimensions cannot differ from {a['dim']} key dimensions")
+                parts = (("left.", float(m["left_scale"]), AttentionSpec(
+                    int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), float(a["scale"]),
+                    int(a["rot"]["dims"]), float(a["rot"]["base"]))),
+                    ("right.", float(m["right_scale"]), MemorySpec(
+                        int(b["heads"]), int(b["dim"]), int(b["vdim"]), float(b["gate_cap"]))))
+            else:
+                raise ValueError(f"{where}: unknown mixer {layer['type']!r}")
+            specs.append(LayerSpec(layer["type"], intermediate_size=ff, parts=parts))
+        if not specs:
+            raise ValueError("the configuration lists no layers")
+        attn = [s for sp in specs for _, _, s in sp.parts if isinstance(s, AttentionSpec)]
+        kw: dict[str, Any] = dict(
+            architecture="FizunexForCausalLM", vocab_size=int(d["vocab"]),
+            hidden_size=int(d["width"]), num_hidden_layers=len(specs),
+            rms_norm_eps=float(d["norm"]["eps"]), layer_specs=tuple(specs),
+            embed_scale=float(d["embedding"]["scale"]), logit_scale=float(d["logit_scale"]),
+            tie_word_embeddings=True,
+            # the largest layer stands for the model where one number is asked for
+            intermediate_size=max(s.intermediate_size for s in specs),
+            num_attention_heads=max((s.num_heads for s in attn), default=1),
+            num_key_value_heads=max((s.num_kv_heads for s in attn), default=1),
+            head_dim=max((s.head_dim for s in attn), default=1),
+            # no limit of the design's own: bounds the rotary and block tables only
+            max_position_embeddings=int(d.get("max_position_embeddings", 131072)),
+            extra={k: v for k, v in d.items() if k not in (
+                "layers", "vocab", "width", "norm", "embedding", "logit_scale", "architecture",
+                "architectures", "max_position_embeddings")})
+        kw.update(overrides)
+        return cls(**kw)
+
+    @classmethod
     def from_pretrained(cls, path: str, **overrides) -> "ModelConfig":
         p = Path(path)
         d = json.loads((p / "config.json").read_text())
+        if d.get("architecture") == "Fizunex":
+            from .utils.weights import tensor_shapes
+            overrides = {"tensor_shapes": tensor_shapes(path), **overrides}
         cfg = cls.from_hf_dict(d, **overrides)
         gpath = p / "generation_config.json"
         if gpath.exists():
@@ -403,11 +509,35 @@ def _sapapel_preset(layers: int, vocab: int, width: int, heads: int, dim: int, v
             "postln_alpha": (2.0 * layers) ** 0.25, "layers": [layer] * layers}
 
 
+def _fizunex_preset(pattern: str, vocab: int, width: int, ff: int, delta: dict, left: dict,
+                    right: dict) -> dict:
+    """``pattern``: one letter per layer, d for a gated delta layer, p for a parallel one."""
+    mlp = {"kind": "dense", "ff": ff}
+    kinds = {"d": {"type": "channel_delta", "mixer": delta, "mlp": mlp},
+             "p": {"type": "parallel", "mlp": mlp,
+                   "mixer": {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7}}}
+    return {"architecture": "Fizunex", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 1.0}, "logit_scale": 1.0, "layers": [kinds[c] for c in pattern]}
+
+
+def _fizunex_mixers(heads: int, kv_heads: int, dim: int, memory_heads: int, memory_dim: int,
+                    memory_vdim: int, conv: int = 4, rot_dims: int = 0) -> tuple[dict, dict, dict]:
+    delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": conv}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+            "rot": {"dims": rot_dims or dim // 2, "base": 500000.0}}
+    right = {"heads": memory_heads, "dim": memory_dim, "vdim": memory_vdim, "gate_cap": 15.0}
+    return delta, left, right
+
+
 #: configurations of designs that are described layer by layer
 _LAYER_LIST_PRESETS: dict[str, dict] = {
     "tiny-sapapel": _sapapel_preset(3, 1024, 128, 4, 24, 40, 48, 6, 2, 48),
     # layers of the size of DeepSeek-V2-Lite's
     "sapapel-16b": _sapapel_preset(27, 102400, 2048, 16, 128, 128, 512, 64, 6, 1408),
+    "tiny-fizunex": _fizunex_preset("dpd", 1024, 128, 192, *_fizunex_mixers(4, 2, 32, 2, 24, 40)),
+    # layers of the size of Llama-3-8B's
+    "fizunex-8b": _fizunex_preset("dddp" * 8, 128256, 4096, 14336,
+                                  *_fizunex_mixers(32, 8, 128, 8, 128, 256)),
 }
 
 

@@ -154,7 +154,17 @@ struct DecodeArgs {
   int B, Hq, Hkv, num_splits;
   float scale;
   const float* alibi;   // optional [Hq] slopes: score += slope * (key position - query position)
+  const float* sink;    // optional [Hq]: exp(sink) joins the softmax denominator, no key behind it
 };
+
+// Weight of the attention output (and the added share of the denominator) once a sink's term has
+// joined a softmax whose log2-domain maximum is M and whose sum relative to it is L.
+__device__ __forceinline__ float sink_share(float M, float L, float sink) {
+  const float s2 = sink * kLog2e;
+  const float top = fmaxf(M, s2);
+  const float keys = L * exp2f(M - top);
+  return keys / (keys + exp2f(s2 - top));
+}
 
 template <typename T, int HD>
 __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs a) {
@@ -345,8 +355,9 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
       L += sm_l[w * 16 + r] * f;
       o += sm_o[(w * 16 + r) * HD + d] * f;
     }
-    const float val = L > 0.0f ? o / L : 0.0f;
+    float val = L > 0.0f ? o / L : 0.0f;
     const int head = kvh * G + r;
+    if (a.sink != nullptr && a.num_splits == 1 && L > 0.0f) val *= sink_share(M, L, a.sink[head]);
     if (a.num_splits > 1) {
       const long long base = (static_cast<long long>(b) * a.Hq + head) * a.num_splits + split;
       a.tmp_out[base * HD + d] = val;
@@ -372,8 +383,9 @@ __global__ void __launch_bounds__(128) decode_reduce_kernel(const DecodeArgs a) 
       wsum += w;
       acc += w * a.tmp_out[(base + s) * HD + d];
     }
-    static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * HD + d] =
-        from_f32<T>(wsum > 0.0f ? acc / wsum : 0.0f);
+    float val = wsum > 0.0f ? acc / wsum : 0.0f;
+    if (a.sink != nullptr && wsum > 0.0f) val *= sink_share(M, wsum, a.sink[head]);
+    static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * HD + d] = from_f32<T>(val);
   }
 }
 
@@ -670,7 +682,7 @@ B200_API int b200_decode_num_splits(int B, int Hkv, int max_seq_len) {
 
 // Decode attention.  Workspace (only read when num_splits > 1):
 //   tmp_out fp32 [B, Hq, num_splits, HD], tmp_lse fp32 [B, Hq, num_splits].
-// dtype 0 bf16 / 1 fp16; HD in {64, 128, 256}; Hq / Hkv <= 16.
+// dtype 0 bf16 / 1 fp16; HD in {64, 128, 256} (bf16 also 96); Hq / Hkv <= 16.
 static int paged_decode_impl(const void* q, long long ldq, void* out, long long ldo,
                              const void* k_cache, const void* v_cache, long long slot_stride,
                              long long head_stride, long long num_slots,
@@ -678,7 +690,8 @@ static int paged_decode_impl(const void* q, long long ldq, void* out, long long 
                              const int* seq_lens, float* tmp_out, float* tmp_lse,
                              int num_splits, int B, int Hq, int Hkv, int HD, float scale,
                              int dtype, int qmode, float k_scale, float v_scale, float k_zp,
-                             float v_zp, void* stream, const float* alibi = nullptr) {
+                             float v_zp, void* stream, const float* alibi = nullptr,
+                             const float* sink = nullptr) {
   if (B <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16) return -2;
   if (num_splits < 1) return -2;
@@ -693,11 +706,13 @@ static int paged_decode_impl(const void* q, long long ldq, void* out, long long 
   a.ldq = ldq; a.ldo = ldo; a.B = B; a.Hq = Hq; a.Hkv = Hkv; a.num_splits = num_splits;
   a.scale = scale;
   a.alibi = alibi;
+  a.sink = sink;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
 #define B200_DEC(TT, H) return launch_decode<TT, H>(a, s)
   if (dtype == 0) {
     if (HD == 128) B200_DEC(__nv_bfloat16, 128);
     if (HD == 64) B200_DEC(__nv_bfloat16, 64);
+    if (HD == 96) B200_DEC(__nv_bfloat16, 96);
     if (HD == 256) B200_DEC(__nv_bfloat16, 256);
   } else if (dtype == 1) {
     if (HD == 128) B200_DEC(__half, 128);
@@ -739,6 +754,22 @@ B200_API int b200_paged_decode_alibi(const void* q, long long ldq, void* out, lo
                            stream, alibi);
 }
 
+// Decode attention with one learnt sink per query head: exp(sink) is added to the softmax
+// denominator; it has no key and no value and is not scaled.
+B200_API int b200_paged_decode_sink(const void* q, long long ldq, void* out, long long ldo,
+                                    const void* k_cache, const void* v_cache,
+                                    long long slot_stride, long long head_stride,
+                                    long long num_slots, const int* block_tables, int max_blocks,
+                                    int block_size, const int* seq_lens, float* tmp_out,
+                                    float* tmp_lse, int num_splits, int B, int Hq, int Hkv,
+                                    int HD, float scale, int dtype, const float* sink,
+                                    void* stream) {
+  return paged_decode_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride, num_slots,
+                           block_tables, max_blocks, block_size, seq_lens, tmp_out, tmp_lse,
+                           num_splits, B, Hq, Hkv, HD, scale, dtype, 0, 1.0f, 1.0f, 0.0f, 0.0f,
+                           stream, nullptr, sink);
+}
+
 // Decode attention over an 8-bit KV cache (same layout, one byte per element; slot_stride and
 // head_stride in bytes).  qmode 1: fp8 e4m3 with per-tensor scales; qmode 2: int8 with scales
 // and zero points (the reference's int8 KV cache, vllm_gcu/kernels/quantization/kv_cache.py:12-61).
@@ -761,9 +792,11 @@ B200_API int b200_paged_decode_q8kv(const void* q, long long ldq, void* out, lon
 // Second pass of split-KV decode: LSE-weighted sum of the per-split partial outputs
 // (tmp_out fp32 [B, Hq, num_splits, HD], tmp_lse fp32 [B, Hq, num_splits], log2 domain).
 B200_API int b200_decode_reduce(void* out, long long ldo, float* tmp_out, float* tmp_lse,
-                                int num_splits, int B, int Hq, int HD, int dtype, void* stream) {
+                                int num_splits, int B, int Hq, int HD, int dtype,
+                                const float* sink, void* stream) {
   if (B <= 0 || num_splits <= 1) return 0;
   DecodeArgs a{};
+  a.sink = sink;
   a.out = out; a.tmp_out = tmp_out; a.tmp_lse = tmp_lse; a.ldo = ldo; a.B = B; a.Hq = Hq;
   a.num_splits = num_splits;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

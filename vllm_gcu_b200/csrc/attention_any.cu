@@ -1,0 +1,374 @@
+// Kernels of key / value attention outside the tensor-core layouts, and the kernel in front of it.
+//
+//   qk_norm_rope_cache  RMS norm of a query and of a key row over the whole projection (all heads
+//                       at once), rotary positions on the first dimensions of every head, queries
+//                       to a padded buffer, keys and values to the paged cache.  Values are a
+//                       projection of their own or the keys as they were before the norm.
+//   any_attention       causal paged attention for any head dimension and group size, fp32 or
+//                       bf16 rows, optional sink: serves models that run in 32-bit and the
+//                       shapes the tensor-core kernels do not cover.
+//
+// Cache layout as in attention.cu: [num_slots, kv_heads, DC] with DC >= D, zeros behind D.
+#include "common.cuh"
+
+namespace b200 {
+namespace anyattn {
+
+constexpr unsigned int kKernelId = 74;
+
+struct PrepArgs {
+  const void* q;             // [T, Hq * D] view, row pitch ldq
+  const void* k;             // [T, Hkv * D]
+  const void* v;             // [T, Hkv * D], or null: the keys before their norm
+  const float* qw;           // [Hq * D] norm weights
+  const float* kw;           // [Hkv * D]
+  const float* sumsq;        // [T, 2] sums of squares of the whole q / k rows, or null: these rows
+  const float* cos_sin;      // [positions, rot] cos | sin
+  const long long* positions;
+  const long long* slots;    // [T] (-1: no cache write)
+  void* qo;                  // [T, Hq, DC]
+  void* kc;                  // [num_slots, Hkv, DC]
+  void* vc;
+  long long ldq, ldk, ldv, num_slots, max_pos;
+  int T, Hq, Hkv, D, DC, rot, q_all, k_all, is_neox;
+  float eps;
+  unsigned int* status;
+};
+
+// Normalised (and rotated) element c of head `h`: x is the projected row, inv its 1 / rms.
+template <typename T>
+__device__ __forceinline__ float rotated(const T* x, const float* w, float inv, int base, int c,
+                                         int rot, int is_neox, const float* cs) {
+  const float self = to_f32<T>(x[base + c]) * inv * w[base + c];
+  if (c >= rot) return self;
+  const int half = rot / 2;
+  int i, mate;
+  bool first;
+  if (is_neox) {
+    first = c < half;
+    i = first ? c : c - half;
+    mate = first ? c + half : c - half;
+  } else {
+    first = (c & 1) == 0;
+    i = c >> 1;
+    mate = c ^ 1;
+  }
+  const float other = to_f32<T>(x[base + mate]) * inv * w[base + mate];
+  const float co = cs[i], si = cs[half + i];
+  return first ? self * co - other * si : self * co + other * si;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) qk_norm_rope_cache_kernel(const PrepArgs a) {
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  const T* q = static_cast<const T*>(a.q) + static_cast<long long>(t) * a.ldq;
+  const T* k = static_cast<const T*>(a.k) + static_cast<long long>(t) * a.ldk;
+  const int nq = a.Hq * a.D, nk = a.Hkv * a.D;
+  float sq = 0.0f, sk = 0.0f;
+  if (a.sumsq != nullptr) {
+    sq = a.sumsq[2 * t];
+    sk = a.sumsq[2 * t + 1];
+  } else {
+    for (int c = threadIdx.x; c < nq; c += blockDim.x) {
+      const float f = to_f32<T>(q[c]);
+      sq += f * f;
+    }
+    for (int c = threadIdx.x; c < nk; c += blockDim.x) {
+      const float f = to_f32<T>(k[c]);
+      sk += f * f;
+    }
+    sq = block_sum(sq, red);
+    sk = block_sum(sk, red);
+  }
+  const float qi = 1.0f / sqrtf(sq / static_cast<float>(a.q_all) + a.eps);
+  const float ki = 1.0f / sqrtf(sk / static_cast<float>(a.k_all) + a.eps);
+  long long pos = a.positions[t];
+  if (pos < 0 || pos >= a.max_pos) {
+    if (threadIdx.x == 0)
+      report_status(a.status, kStatusBounds, kKernelId, static_cast<unsigned int>(t));
+    pos = 0;
+  }
+  const float* cs = a.cos_sin + pos * a.rot;
+  T* qo = static_cast<T*>(a.qo) + static_cast<long long>(t) * a.Hq * a.DC;
+  for (int e = threadIdx.x; e < a.Hq * a.DC; e += blockDim.x) {
+    const int h = e / a.DC, c = e - h * a.DC;
+    qo[e] = from_f32<T>(c < a.D ? rotated<T>(q, a.qw, qi, h * a.D, c, a.rot, a.is_neox, cs) : 0.0f);
+  }
+  const long long slot = a.slots[t];
+  if (slot < 0) return;
+  if (slot >= a.num_slots) {
+    if (threadIdx.x == 0)
+      report_status(a.status, kStatusBounds, kKernelId + 1, static_cast<unsigned int>(t));
+    return;
+  }
+  const T* v = a.v != nullptr ? static_cast<const T*>(a.v) + static_cast<long long>(t) * a.ldv : k;
+  T* kc = static_cast<T*>(a.kc) + slot * a.Hkv * a.DC;
+  T* vc = static_cast<T*>(a.vc) + slot * a.Hkv * a.DC;
+  for (int e = threadIdx.x; e < a.Hkv * a.DC; e += blockDim.x) {
+    const int h = e / a.DC, c = e - h * a.DC;
+    const bool in = c < a.D;
+    kc[e] = from_f32<T>(in ? rotated<T>(k, a.kw, ki, h * a.D, c, a.rot, a.is_neox, cs) : 0.0f);
+    vc[e] = in ? v[h * a.D + c] : from_f32<T>(0.0f);
+  }
+}
+
+// The same for bf16 rows, two neighbouring elements per thread (D, DC and rot even, pairs of
+// neighbours rotated together).
+__global__ void __launch_bounds__(256) qk_norm_rope_cache_pairs_kernel(const PrepArgs a) {
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  const __nv_bfloat16* q =
+      static_cast<const __nv_bfloat16*>(a.q) + static_cast<long long>(t) * a.ldq;
+  const __nv_bfloat16* k =
+      static_cast<const __nv_bfloat16*>(a.k) + static_cast<long long>(t) * a.ldk;
+  auto pair = [](const __nv_bfloat16* p, int i) {
+    return unpack_bf16x2(reinterpret_cast<const uint32_t*>(p)[i]);
+  };
+  const int nq = a.Hq * a.D / 2, nk = a.Hkv * a.D / 2;
+  float sq = 0.0f, sk = 0.0f;
+  if (a.sumsq != nullptr) {
+    sq = a.sumsq[2 * t];
+    sk = a.sumsq[2 * t + 1];
+  } else {
+    for (int i = threadIdx.x; i < nq; i += blockDim.x) {
+      const float2 f = pair(q, i);
+      sq += f.x * f.x + f.y * f.y;
+    }
+    for (int i = threadIdx.x; i < nk; i += blockDim.x) {
+      const float2 f = pair(k, i);
+      sk += f.x * f.x + f.y * f.y;
+    }
+    sq = block_sum(sq, red);
+    sk = block_sum(sk, red);
+  }
+  const float qi = 1.0f / sqrtf(sq / static_cast<float>(a.q_all) + a.eps);
+  const float ki = 1.0f / sqrtf(sk / static_cast<float>(a.k_all) + a.eps);
+  long long pos = a.positions[t];
+  if (pos < 0 || pos >= a.max_pos) {
+    if (threadIdx.x == 0)
+      report_status(a.status, kStatusBounds, kKernelId, static_cast<unsigned int>(t));
+    pos = 0;
+  }
+  const float* cs = a.cos_sin + pos * a.rot;
+  const int half = a.rot / 2, dp = a.D / 2, dcp = a.DC / 2;
+  auto turned = [&](const __nv_bfloat16* x, const float* w, float inv, int i, int c) {
+    const float2 f = pair(x, i);
+    const float2 g = reinterpret_cast<const float2*>(w)[i];
+    const float u = f.x * inv * g.x, v = f.y * inv * g.y;
+    if (c >= half) return pack_bf16x2(u, v);
+    const float co = cs[c], si = cs[half + c];
+    return pack_bf16x2(u * co - v * si, v * co + u * si);
+  };
+  uint32_t* qo = reinterpret_cast<uint32_t*>(a.qo) + static_cast<long long>(t) * a.Hq * dcp;
+  for (int e = threadIdx.x; e < a.Hq * dcp; e += blockDim.x) {
+    const int h = e / dcp, c = e - h * dcp;
+    qo[e] = c < dp ? turned(q, a.qw, qi, h * dp + c, c) : 0u;
+  }
+  const long long slot = a.slots[t];
+  if (slot < 0) return;
+  if (slot >= a.num_slots) {
+    if (threadIdx.x == 0)
+      report_status(a.status, kStatusBounds, kKernelId + 1, static_cast<unsigned int>(t));
+    return;
+  }
+  const uint32_t* v = reinterpret_cast<const uint32_t*>(
+      a.v != nullptr ? static_cast<const __nv_bfloat16*>(a.v) + static_cast<long long>(t) * a.ldv
+                     : k);
+  uint32_t* kc = reinterpret_cast<uint32_t*>(a.kc) + slot * a.Hkv * dcp;
+  uint32_t* vc = reinterpret_cast<uint32_t*>(a.vc) + slot * a.Hkv * dcp;
+  for (int e = threadIdx.x; e < a.Hkv * dcp; e += blockDim.x) {
+    const int h = e / dcp, c = e - h * dcp;
+    kc[e] = c < dp ? turned(k, a.kw, ki, h * dp + c, c) : 0u;
+    vc[e] = c < dp ? v[h * dp + c] : 0u;
+  }
+}
+
+// ---------------------------------------------------------------------------
+struct AttnArgs {
+  const void* q;             // [T, Hq, DC]
+  const void* kc;            // [num_slots, Hkv, DC]
+  const void* vc;
+  void* out;                 // [T, Hq, DC]
+  const int* block_tables;   // [B, max_blocks]
+  const int* seq_lens;       // [B]
+  const int* cu_q;           // [num_prefills + 1] relative to token num_decodes, or null
+  const float* sink;         // [Hq] or null
+  long long num_slots;
+  int T, Hq, Hkv, DC, num_decodes, num_prefills, max_blocks, block_size;
+  float scale;
+  unsigned int* status;
+};
+
+constexpr int kWarps = 4;      // warps that share the keys of one (token, head)
+constexpr int kBatch = 4;      // keys a warp has in flight
+
+template <typename T, int NC>
+__global__ void __launch_bounds__(kWarps * 32) any_attention_kernel(const AttnArgs a) {
+  __shared__ float s_m[kWarps], s_l[kWarps];
+  __shared__ float s_o[kWarps][NC * 32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x, head = blockIdx.y;
+  const int kvh = head / (a.Hq / a.Hkv);
+  const TokenPlace pl = token_place(t, a.num_decodes, a.num_prefills, a.cu_q);
+  int keys = 0;
+  if (pl.req >= 0) {
+    keys = a.seq_lens[pl.req];
+    if (t >= a.num_decodes)      // tokens of the request behind this one in the step
+      keys -= a.cu_q[pl.req - a.num_decodes + 1] - (t - a.num_decodes) - 1;
+  }
+  if (keys > a.max_blocks * a.block_size) {
+    if (threadIdx.x == 0)
+      report_status(a.status, kStatusBounds, kKernelId + 2, static_cast<unsigned int>(t));
+    keys = 0;
+  }
+  const long long row = (static_cast<long long>(t) * a.Hq + head) * a.DC;
+  float q[NC], acc[NC];
+#pragma unroll
+  for (int i = 0; i < NC; ++i) {
+    const int c = lane + 32 * i;
+    q[i] = c < a.DC ? to_f32<T>(static_cast<const T*>(a.q)[row + c]) : 0.0f;
+    acc[i] = 0.0f;
+  }
+  float m = -INFINITY, l = 0.0f;
+  const int* bt = a.block_tables + static_cast<long long>(pl.req < 0 ? 0 : pl.req) * a.max_blocks;
+  for (int k0 = warp * kBatch; k0 < keys; k0 += kWarps * kBatch) {
+    float s[kBatch], v[kBatch][NC];
+#pragma unroll
+    for (int b = 0; b < kBatch; ++b) {
+      const int key = k0 + b;
+      long long slot = -1;
+      if (key < keys) {
+        slot = static_cast<long long>(bt[key / a.block_size]) * a.block_size + key % a.block_size;
+        if (slot < 0 || slot >= a.num_slots) {
+          if (lane == 0)
+            report_status(a.status, kStatusBounds, kKernelId + 3, static_cast<unsigned int>(t));
+          slot = -1;
+        }
+      }
+      const long long at = (slot * a.Hkv + kvh) * a.DC;
+      float d = 0.0f;
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        const int c = lane + 32 * i;
+        const bool in = slot >= 0 && c < a.DC;
+        d += in ? q[i] * to_f32<T>(static_cast<const T*>(a.kc)[at + c]) : 0.0f;
+        v[b][i] = in ? to_f32<T>(static_cast<const T*>(a.vc)[at + c]) : 0.0f;
+      }
+      s[b] = d;
+    }
+    float top = m;
+#pragma unroll
+    for (int b = 0; b < kBatch; ++b) {
+      s[b] = k0 + b < keys ? warp_sum(s[b]) * a.scale : -INFINITY;
+      top = fmaxf(top, s[b]);
+    }
+    const float al = expf(m - top);            // top is finite: key k0 is visible
+    m = top;
+    l *= al;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) acc[i] *= al;
+#pragma unroll
+    for (int b = 0; b < kBatch; ++b) {
+      const float p = expf(s[b] - m);
+      l += p;
+#pragma unroll
+      for (int i = 0; i < NC; ++i) acc[i] += p * v[b][i];
+    }
+  }
+  if (lane == 0) {
+    s_m[warp] = m;
+    s_l[warp] = l;
+  }
+#pragma unroll
+  for (int i = 0; i < NC; ++i) s_o[warp][lane + 32 * i] = acc[i];
+  __syncthreads();
+  float top = a.sink != nullptr ? a.sink[head] : -INFINITY;
+  const float sink = top;
+#pragma unroll
+  for (int w = 0; w < kWarps; ++w) top = fmaxf(top, s_m[w]);
+  float f[kWarps], den = a.sink != nullptr ? expf(sink - top) : 0.0f;
+#pragma unroll
+  for (int w = 0; w < kWarps; ++w) {
+    f[w] = s_m[w] == -INFINITY ? 0.0f : expf(s_m[w] - top);
+    den += s_l[w] * f[w];
+  }
+  const float inv = keys > 0 ? 1.0f / den : 0.0f;
+  for (int c = threadIdx.x; c < a.DC; c += blockDim.x) {
+    float o = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kWarps; ++w) o += s_o[w][c] * f[w];
+    static_cast<T*>(a.out)[row + c] = from_f32<T>(o * inv);
+  }
+}
+
+template <typename T>
+static int dispatch_attention(const AttnArgs& a, cudaStream_t s) {
+  const int nc = (a.DC + 31) / 32;
+  dim3 grid(a.T, a.Hq);
+  if (nc <= 2) any_attention_kernel<T, 2><<<grid, kWarps * 32, 0, s>>>(a);
+  else if (nc <= 4) any_attention_kernel<T, 4><<<grid, kWarps * 32, 0, s>>>(a);
+  else if (nc <= 8) any_attention_kernel<T, 8><<<grid, kWarps * 32, 0, s>>>(a);
+  else if (nc <= 16) any_attention_kernel<T, 16><<<grid, kWarps * 32, 0, s>>>(a);
+  else return -20;
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace anyattn
+}  // namespace b200
+
+using namespace b200;
+using namespace b200::anyattn;
+
+// dtype (rows and caches): 0 bf16, 2 fp32.  rot even, <= D.  q_all / k_all: number of elements a
+// norm runs over (with sumsq, rows of other ranks included).
+B200_API int b200_qk_norm_rope_cache(const void* q, long long ldq, const void* k, long long ldk,
+                                     const void* v, long long ldv, const float* qw, const float* kw,
+                                     const float* sumsq, int q_all, int k_all, float eps,
+                                     const float* cos_sin, int rot, long long max_pos, int is_neox,
+                                     const long long* positions, const long long* slots, void* qo,
+                                     void* kc, void* vc, long long num_slots, int T, int Hq,
+                                     int Hkv, int D, int DC, int dtype, void* stream) {
+  if (T <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || D <= 0 || DC < D || rot < 0 || rot > D || (rot & 1) != 0 ||
+      (dtype != 0 && dtype != 2))
+    return -2;
+  PrepArgs a;
+  a.q = q; a.k = k; a.v = v; a.qw = qw; a.kw = kw; a.sumsq = sumsq; a.cos_sin = cos_sin;
+  a.positions = positions; a.slots = slots; a.qo = qo; a.kc = kc; a.vc = vc; a.ldq = ldq;
+  a.ldk = ldk; a.ldv = ldv; a.num_slots = num_slots; a.max_pos = max_pos; a.T = T; a.Hq = Hq;
+  a.Hkv = Hkv; a.D = D; a.DC = DC; a.rot = rot; a.q_all = q_all; a.k_all = k_all;
+  a.is_neox = is_neox; a.eps = eps; a.status = status_ptr();
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const auto even = [](const void* p, int bytes) {
+    return (reinterpret_cast<uintptr_t>(p) % bytes) == 0;
+  };
+  if (dtype == 2)
+    qk_norm_rope_cache_kernel<float><<<T, 256, 0, s>>>(a);
+  else if (!is_neox && (D & 1) == 0 && (DC & 1) == 0 && (ldq & 1) == 0 && (ldk & 1) == 0 &&
+           (ldv & 1) == 0 && even(q, 4) && even(k, 4) && even(v, 4) && even(qw, 8) &&
+           even(kw, 8) && even(qo, 4) && even(kc, 4) && even(vc, 4))
+    qk_norm_rope_cache_pairs_kernel<<<T, 256, 0, s>>>(a);
+  else
+    qk_norm_rope_cache_kernel<__nv_bfloat16><<<T, 256, 0, s>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// q / out [T, Hq, DC]; -20: a head dimension the kernel does not cover (> 512).
+B200_API int b200_any_attention(const void* q, const void* kc, const void* vc, long long num_slots,
+                                void* out, const int* block_tables, int max_blocks, int block_size,
+                                const int* seq_lens, const int* cu_q, const float* sink, int T,
+                                int Hq, int Hkv, int DC, int num_decodes, int num_prefills,
+                                float scale, int dtype, void* stream) {
+  if (T <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || Hq % Hkv != 0 || DC <= 0 || block_size <= 0 || Hq > 65535 ||
+      (dtype != 0 && dtype != 2))
+    return -2;
+  AttnArgs a;
+  a.q = q; a.kc = kc; a.vc = vc; a.out = out; a.block_tables = block_tables;
+  a.seq_lens = seq_lens; a.cu_q = cu_q; a.sink = sink; a.num_slots = num_slots; a.T = T; a.Hq = Hq;
+  a.Hkv = Hkv; a.DC = DC; a.num_decodes = num_decodes; a.num_prefills = num_prefills;
+  a.max_blocks = max_blocks; a.block_size = block_size; a.scale = scale; a.status = status_ptr();
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return dtype == 0 ? dispatch_attention<__nv_bfloat16>(a, s) : dispatch_attention<float>(a, s);
+}

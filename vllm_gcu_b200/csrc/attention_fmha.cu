@@ -1,6 +1,6 @@
 // Prefill / chunked-prefill / prefix attention on the 5th-generation tensor cores.
 //
-// One CTA = 128 query rows of one head.  Per tile of 128 keys:
+// One CTA = 128 query rows of one head (head dimension 64, 96 or 128).  Per tile of 128 keys:
 //   S = Q K^T      tcgen05.mma, Q and K tiles K-major in shared memory (TMA, 128-byte swizzle),
 //                  fp32 scores in tensor memory (two buffers);
 //   softmax        eight warps, two threads per query row (64 keys each): two passes over the
@@ -31,7 +31,6 @@ namespace fmha {
 constexpr unsigned int kKernelId = 21;
 constexpr int BQ = 128;      // query rows per CTA
 constexpr int BKV = 128;     // keys per tile
-constexpr int HD = 128;      // head dimension
 constexpr int kPage = 16;    // tokens per TMA copy (divides the cache block size)
 constexpr int kThreads = 320;   // TMA warp, MMA warp, 2 x 4 softmax warps
 constexpr int kSub = BQ * 64 * 2;          // one [128 x 64] bf16 sub-tile: 16 KB
@@ -59,8 +58,9 @@ __device__ __forceinline__ float ex2_approx(float x) {
 }
 
 struct Args {
-  __nv_bfloat16* out;      // [T, Hq * 128], row pitch ldo
-  float* lse;              // optional [Hq, T]
+  __nv_bfloat16* out;      // [T, Hq * HD], row pitch ldo
+  float* lse;              // optional [Hq, T] (without the sink's term)
+  const float* sink;       // optional [Hq]: exp(sink) joins the denominator
   const int* cu_q;         // [B + 1]
   const int* seq_lens;     // [B]
   const int* block_tables; // [B, max_blocks]
@@ -70,6 +70,9 @@ struct Args {
   unsigned int* status;
 };
 
+// HD below 128 uses the same tiles: the second 64-column half then carries columns of the next
+// head (or zeros) behind HD, which no contraction step and no store touches.
+template <int HD>
 __global__ void __launch_bounds__(kThreads, 1)
     fmha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ,
                         const __grid_constant__ CUtensorMap tmK,
@@ -91,6 +94,8 @@ __global__ void __launch_bounds__(kThreads, 1)
   volatile uint32_t* abort_flag = tmem_slot + 1;
   int* s_info = reinterpret_cast<int*>(tmem_slot + 2);   // [0] sequence, [1] q tile in sequence
 
+  static_assert(HD == 64 || HD == 96 || HD == 128, "head dimensions of this kernel");
+  constexpr uint32_t kLoadBytes = HD > 64 ? kTile : kSub;
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
   const int head = blockIdx.y;
@@ -172,9 +177,10 @@ __global__ void __launch_bounds__(kThreads, 1)
   if (warp == 0) {
     // ---------------- TMA producer ----------------
     if (elect_one()) {
-      mbar_expect_tx(q_full, kTile);
+      mbar_expect_tx(q_full, kLoadBytes);
       tma_load_2d(smem + kOffQ, &tmQ, q_full, head * HD, q_start + q0);
-      tma_load_2d(smem + kOffQ + kSub, &tmQ, q_full, head * HD + 64, q_start + q0);
+      if (HD > 64)
+        tma_load_2d(smem + kOffQ + kSub, &tmQ, q_full, head * HD + 64, q_start + q0);
       const int* bt = a.block_tables + static_cast<long long>(seq) * a.max_blocks;
       const int last_tok = seq_len - 1;
       bool ok = true;
@@ -191,14 +197,14 @@ __global__ void __launch_bounds__(kThreads, 1)
             ok = false;
             break;
           }
-          mbar_expect_tx(full, kTile);
+          mbar_expect_tx(full, kLoadBytes);
           for (int c = 0; c < BKV / kPage; ++c) {
             const int tok = min(key0 + c * kPage, last_tok);   // pages past the end: any valid page
             const int blk = bt[tok / a.block_size];
             const int y = blk * a.block_size + ((key0 + c * kPage) % a.block_size);
             const int x = kvh * HD;
             tma_load_2d(dst + c * (kPage * 128), tm, full, x, y);
-            tma_load_2d(dst + kSub + c * (kPage * 128), tm, full, x + 64, y);
+            if (HD > 64) tma_load_2d(dst + kSub + c * (kPage * 128), tm, full, x + 64, y);
           }
         }
       }
@@ -369,7 +375,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         tc_fence_after();
         if (ok && __any_sync(0xffffffffu, alpha != 1.0f)) {
 #pragma unroll 1
-          for (int c = 0; c < 2; ++c) {
+          for (int c = 0; c < 2 && g * 64 + c * 32 < HD; ++c) {
             uint32_t v[32];
             tmem_ld_32x32(lane_addr + kColO + g * 64 + c * 32, v);
             tmem_ld_wait();
@@ -399,12 +405,15 @@ __global__ void __launch_bounds__(kThreads, 1)
     l += xch[(g ^ 1) * BQ + r];
     if (ok && mbar_wait(o_done, (nt - 1) & 1, a.status, kKernelId, 0x320u, abort_flag)) {
       tc_fence_after();
-      const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+      float den = l;
+      if (a.sink != nullptr)       // relative to the running maximum, like the row sum
+        den += exp2f(fmaf(-m_used, sl2, a.sink[head] * 1.4426950408889634f));
+      const float inv = l > 0.0f ? 1.0f / den : 0.0f;
       const bool row_ok = r < rows;
       __nv_bfloat16* orow =
           a.out + static_cast<long long>(q_start + q0 + r) * a.ldo + head * HD + g * 64;
 #pragma unroll 1
-      for (int c = 0; c < 2; ++c) {
+      for (int c = 0; c < 2 && g * 64 + c * 32 < HD; ++c) {
         uint32_t v[32];
         tmem_ld_32x32(lane_addr + kColO + g * 64 + c * 32, v);
         tmem_ld_wait();
@@ -474,29 +483,53 @@ static int get_map(const void* base, unsigned long long rows, unsigned long long
 }  // namespace fmha
 }  // namespace b200
 
-// Same contract as b200_varlen_prefill for bf16, head_dim 128, caches laid out as
-// [num_slots, Hkv * 128] rows and a block size that is a multiple of 16; num_q_tiles must be
-// >= sum_b ceil(q_len_b / 128).  Returns -20 when the layout does not qualify (callers use
-// b200_varlen_prefill).
-B200_API int b200_fmha_prefill(const void* q, long long ldq, void* out, long long ldo, float* lse,
-                               const int* cu_q, const int* seq_lens, const void* k_cache,
-                               const void* v_cache, long long slot_stride, long long head_stride,
-                               long long num_slots, const int* block_tables, int max_blocks,
-                               int block_size, int B, int T, int num_q_tiles, int Hq, int Hkv,
-                               int HD, float scale, int causal, int window, int dtype,
-                               void* stream) {
+namespace b200 {
+namespace fmha {
+
+template <int HD>
+static int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
+                  const Args& a, int num_q_tiles, cudaStream_t s) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev >= 0 && dev < 64 && !configured[dev]) {
+    cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel<HD>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured[dev] = true;
+  }
+  dim3 grid(num_q_tiles, a.Hq);
+  fmha_prefill_kernel<HD><<<grid, kThreads, kSmemBytes, s>>>(tmQ, tmK, tmV, a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace fmha
+}  // namespace b200
+
+// Same contract as b200_varlen_prefill for bf16, head_dim 64, 96 or 128, caches laid out as
+// [num_slots, Hkv * HD] rows and a block size that is a multiple of 16; num_q_tiles must be
+// >= sum_b ceil(q_len_b / 128).  `sink`: optional [Hq], exp(sink) is added to the softmax
+// denominator.  Returns -20 when the layout does not qualify (callers use another kernel).
+B200_API int b200_fmha_prefill_sink(const void* q, long long ldq, void* out, long long ldo,
+                                    float* lse, const int* cu_q, const int* seq_lens,
+                                    const void* k_cache, const void* v_cache,
+                                    long long slot_stride, long long head_stride,
+                                    long long num_slots, const int* block_tables, int max_blocks,
+                                    int block_size, int B, int T, int num_q_tiles, int Hq, int Hkv,
+                                    int HD, float scale, int causal, int window, int dtype,
+                                    const float* sink, void* stream) {
   using namespace b200;
   using namespace b200::fmha;
   if (B <= 0 || T <= 0 || num_q_tiles <= 0) return 0;
-  if (dtype != 0 || HD != fmha::HD || (block_size % kPage) != 0 || head_stride != fmha::HD ||
-      slot_stride != static_cast<long long>(Hkv) * fmha::HD || Hkv <= 0 || Hq % Hkv != 0 ||
-      (ldq % 8) != 0 || (ldo % 8) != 0 ||
+  if (dtype != 0 || (HD != 64 && HD != 96 && HD != 128) || (block_size % kPage) != 0 ||
+      head_stride != HD || slot_stride != static_cast<long long>(Hkv) * HD || Hkv <= 0 ||
+      Hq % Hkv != 0 || (ldq % 8) != 0 || (ldo % 8) != 0 ||
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out) |
         reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15))
     return -20;
   CUtensorMap tmQ, tmK, tmV;
-  const unsigned long long cols = static_cast<unsigned long long>(Hkv) * fmha::HD;
-  int r = get_map(q, static_cast<unsigned long long>(T), static_cast<unsigned long long>(Hq) * fmha::HD,
+  const unsigned long long cols = static_cast<unsigned long long>(Hkv) * HD;
+  int r = get_map(q, static_cast<unsigned long long>(T), static_cast<unsigned long long>(Hq) * HD,
                   static_cast<unsigned long long>(ldq) * 2, BQ, false, &tmQ);
   if (r != 0) return r < 0 ? -6 : r;
   r = get_map(k_cache, static_cast<unsigned long long>(num_slots), cols, cols * 2, kPage, true, &tmK);
@@ -505,21 +538,25 @@ B200_API int b200_fmha_prefill(const void* q, long long ldq, void* out, long lon
   if (r != 0) return r < 0 ? -6 : r;
   Args a;
   a.out = static_cast<__nv_bfloat16*>(out);
-  a.lse = lse; a.cu_q = cu_q; a.seq_lens = seq_lens; a.block_tables = block_tables;
+  a.lse = lse; a.sink = sink; a.cu_q = cu_q; a.seq_lens = seq_lens; a.block_tables = block_tables;
   a.ldo = ldo; a.B = B; a.T = T; a.Hq = Hq; a.Hkv = Hkv; a.max_blocks = max_blocks;
   a.block_size = block_size; a.causal = causal; a.window = window; a.scale = scale;
   a.status = status_ptr();
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev >= 0 && dev < 64 && !configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    configured[dev] = true;
-  }
-  dim3 grid(num_q_tiles, Hq);
-  fmha_prefill_kernel<<<grid, kThreads, kSmemBytes, static_cast<cudaStream_t>(stream)>>>(
-      tmQ, tmK, tmV, a);
-  return static_cast<int>(cudaGetLastError());
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (HD == 64) return launch<64>(tmQ, tmK, tmV, a, num_q_tiles, s);
+  if (HD == 96) return launch<96>(tmQ, tmK, tmV, a, num_q_tiles, s);
+  return launch<128>(tmQ, tmK, tmV, a, num_q_tiles, s);
+}
+
+B200_API int b200_fmha_prefill(const void* q, long long ldq, void* out, long long ldo, float* lse,
+                               const int* cu_q, const int* seq_lens, const void* k_cache,
+                               const void* v_cache, long long slot_stride, long long head_stride,
+                               long long num_slots, const int* block_tables, int max_blocks,
+                               int block_size, int B, int T, int num_q_tiles, int Hq, int Hkv,
+                               int HD, float scale, int causal, int window, int dtype,
+                               void* stream) {
+  return b200_fmha_prefill_sink(q, ldq, out, ldo, lse, cu_q, seq_lens, k_cache, v_cache,
+                                slot_stride, head_stride, num_slots, block_tables, max_blocks,
+                                block_size, B, T, num_q_tiles, Hq, Hkv, HD, scale, causal, window,
+                                dtype, nullptr, stream);
 }

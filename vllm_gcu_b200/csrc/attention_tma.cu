@@ -79,6 +79,7 @@ struct Args {
   long long ldq, ldo;
   int B, Hq, Hkv, num_splits, max_blocks, block_size;
   float scale;
+  const float* sink;     // optional [Hq], see b200_paged_decode_sink
   unsigned int* status;
 };
 
@@ -304,8 +305,14 @@ __global__ void __launch_bounds__(kThreads)
       L += sm_l[w * 16 + r] * f;
       o += sm_o[(w * 16 + r) * HD + d] * f;
     }
-    const float val = (ok && L > 0.0f) ? o / L : 0.0f;
+    float val = (ok && L > 0.0f) ? o / L : 0.0f;
     const int head = kvh * G + r;
+    if (a.sink != nullptr && a.num_splits == 1 && ok && L > 0.0f) {
+      const float s2 = a.sink[head] * kLog2e;
+      const float top = fmaxf(M, s2);
+      const float keys = L * exp2f(M - top);
+      val *= keys / (keys + exp2f(s2 - top));
+    }
     if (a.num_splits > 1) {
       const long long base = (static_cast<long long>(b) * a.Hq + head) * a.num_splits + split;
       a.tmp_out[base * HD + d] = val;
@@ -358,19 +365,20 @@ static int get_map(const void* base, unsigned long long rows, unsigned long long
 }  // namespace b200
 
 B200_API int b200_decode_reduce(void* out, long long ldo, float* tmp_out, float* tmp_lse,
-                                int num_splits, int B, int Hq, int HD, int dtype, void* stream);
+                                int num_splits, int B, int Hq, int HD, int dtype,
+                                const float* sink, void* stream);
 
 // Same contract as b200_paged_decode for head_dim 128 with the caches laid out as
 // [num_slots, Hkv * 128] rows (slot_stride == Hkv * 128, head_stride == 128) and a block size
 // that is a multiple of 16.  Returns -20 when the layout does not qualify (callers fall back
 // to b200_paged_decode).
-B200_API int b200_paged_decode_tma(const void* q, long long ldq, void* out, long long ldo,
-                                   const void* k_cache, const void* v_cache,
-                                   long long slot_stride, long long head_stride,
-                                   long long num_slots, const int* block_tables, int max_blocks,
-                                   int block_size, const int* seq_lens, float* tmp_out,
-                                   float* tmp_lse, int num_splits, int B, int Hq, int Hkv, int HD,
-                                   float scale, int dtype, void* stream) {
+static int paged_decode_tma_impl(const void* q, long long ldq, void* out, long long ldo,
+                                 const void* k_cache, const void* v_cache, long long slot_stride,
+                                 long long head_stride, long long num_slots,
+                                 const int* block_tables, int max_blocks, int block_size,
+                                 const int* seq_lens, float* tmp_out, float* tmp_lse,
+                                 int num_splits, int B, int Hq, int Hkv, int HD, float scale,
+                                 int dtype, const float* sink, void* stream) {
   using namespace b200;
   using namespace b200::attn_tma;
   if (B <= 0) return 0;
@@ -391,7 +399,7 @@ B200_API int b200_paged_decode_tma(const void* q, long long ldq, void* out, long
   a.q = q; a.out = out; a.tmp_out = tmp_out; a.tmp_lse = tmp_lse; a.seq_lens = seq_lens;
   a.block_tables = block_tables; a.ldq = ldq; a.ldo = ldo; a.B = B; a.Hq = Hq; a.Hkv = Hkv;
   a.num_splits = num_splits; a.max_blocks = max_blocks; a.block_size = block_size;
-  a.scale = scale; a.status = status_ptr();
+  a.scale = scale; a.sink = sink; a.status = status_ptr();
   constexpr int smem = kStages * kStageBytes + 256 + 1024;
   static_assert(kStages * kStageBytes >= (128 + 4 * 16 * b200::attn_tma::HD) * 4,
                 "merge buffer must fit");
@@ -419,5 +427,32 @@ B200_API int b200_paged_decode_tma(const void* q, long long ldq, void* out, long
   }
   int e = static_cast<int>(cudaGetLastError());
   if (e != 0 || num_splits <= 1) return e;
-  return b200_decode_reduce(out, ldo, tmp_out, tmp_lse, num_splits, B, Hq, HD, dtype, stream);
+  return b200_decode_reduce(out, ldo, tmp_out, tmp_lse, num_splits, B, Hq, HD, dtype, sink,
+                            stream);
+}
+
+B200_API int b200_paged_decode_tma(const void* q, long long ldq, void* out, long long ldo,
+                                   const void* k_cache, const void* v_cache,
+                                   long long slot_stride, long long head_stride,
+                                   long long num_slots, const int* block_tables, int max_blocks,
+                                   int block_size, const int* seq_lens, float* tmp_out,
+                                   float* tmp_lse, int num_splits, int B, int Hq, int Hkv, int HD,
+                                   float scale, int dtype, void* stream) {
+  return paged_decode_tma_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride,
+                               num_slots, block_tables, max_blocks, block_size, seq_lens, tmp_out,
+                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, nullptr, stream);
+}
+
+// The same with one learnt sink per query head (see b200_paged_decode_sink).
+B200_API int b200_paged_decode_tma_sink(const void* q, long long ldq, void* out, long long ldo,
+                                        const void* k_cache, const void* v_cache,
+                                        long long slot_stride, long long head_stride,
+                                        long long num_slots, const int* block_tables,
+                                        int max_blocks, int block_size, const int* seq_lens,
+                                        float* tmp_out, float* tmp_lse, int num_splits, int B,
+                                        int Hq, int Hkv, int HD, float scale, int dtype,
+                                        const float* sink, void* stream) {
+  return paged_decode_tma_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride,
+                               num_slots, block_tables, max_blocks, block_size, seq_lens, tmp_out,
+                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, sink, stream);
 }

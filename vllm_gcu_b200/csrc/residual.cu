@@ -9,6 +9,14 @@
 //                   results X_j of the layers so far, and by the final norm of that row
 //   sigmoid_gate    o = o * sigmoid(z), z a strided view of a wider projection
 //
+// and around one whose norms sit on the sublayers' outputs only:
+//
+//   start_rows      x = s * embedding row
+//   add_normed      x = x + norm(y) with a layer norm or an RMS norm (weight, optional bias);
+//                   optionally the final norm of the new row in the same pass
+//   silu_mul_rows   h = silu(g) * u of rows [g | u], any width
+//   head_gate       o = o * sigmoid(z) * s from rows whose heads are padded
+//
 // The residual stream, the statistics and the averages are fp32; LO is the type of the rows that
 // feed matrix products (bf16, or fp32 when the whole model runs in 32-bit).  One CTA per row,
 // vectors of V elements (4 where every row is 4-aligned, else 1).
@@ -240,6 +248,143 @@ __global__ void __launch_bounds__(256)
   }
 }
 
+// ---------------------------------------------------------------------------
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+    start_rows_kernel(const T* e, long long lde, float scale, float* x, T* lo, int H) {
+  const long long t = blockIdx.x;
+  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+    float f[V];
+    ldv<V>(e + t * lde + c, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] *= scale;
+    stv<V>(x + t * H + c, f);
+    stv<V>(lo + t * H + c, f);
+  }
+}
+
+struct AddNormArgs {
+  const float* x;        // [T, H] residual stream
+  const void* y;         // [T, ldy] sublayer output
+  const float* w;        // [H] norm weight
+  const float* b;        // [H] norm bias, or null
+  const float* fw;       // [H] final norm's weight, or null
+  const float* fb;       // [H] final norm's bias, or null
+  float* xo;             // [T, H] the sum (may be x), or null
+  void* lo;              // [T, H] LO copy: of the sum, or of its final norm times fscale
+  long long ldy;
+  int T, H, centred;     // centred: layer norm (mean taken off), else RMS norm
+  float eps, fscale;
+};
+
+// 1 / root of the mean square of z (minus its mean if `centred`); returns the mean in `mean`.
+template <int V>
+__device__ __forceinline__ float row_stats(const float* z, float sum, int H, int centred, float eps,
+                                           float* red, float& mean) {
+  mean = centred ? block_sum(sum, red) / static_cast<float>(H) : 0.0f;
+  float ss = 0.0f;
+  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+    float f[V];
+    ldv<V>(z + c, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += (f[i] - mean) * (f[i] - mean);
+  }
+  ss = block_sum(ss, red);
+  return 1.0f / sqrtf(ss / static_cast<float>(H) + eps);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(512) add_normed_kernel(const AddNormArgs a) {
+  extern __shared__ float z[];       // [H]; every thread reads back only what it wrote
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  const long long row = t * a.H;
+  const T* y = static_cast<const T*>(a.y) + t * a.ldy;
+  float sum = 0.0f;
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
+    float f[V];
+    ldv<V>(y + c, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) sum += f[i];
+    stv<V>(z + c, f);
+  }
+  float mean;
+  const float inv = row_stats<V>(z, sum, a.H, a.centred, a.eps, red, mean);
+  T* lo = static_cast<T*>(a.lo) + row;
+  sum = 0.0f;
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
+    float f[V], x[V], w[V], b[V];
+    ldv<V>(z + c, f);
+    ldv<V>(a.x + row + c, x);
+    ldv<V>(a.w + c, w);
+    if (a.b != nullptr) {
+      ldv<V>(a.b + c, b);
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) b[i] = 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      x[i] += (f[i] - mean) * inv * w[i] + b[i];
+      sum += x[i];
+    }
+    if (a.xo != nullptr) stv<V>(a.xo + row + c, x);
+    if (a.fw == nullptr) stv<V>(lo + c, x);
+    else stv<V>(z + c, x);
+  }
+  if (a.fw == nullptr) return;
+  const float inv2 = row_stats<V>(z, sum, a.H, a.centred, a.eps, red, mean);
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
+    float f[V], w[V], b[V];
+    ldv<V>(z + c, f);
+    ldv<V>(a.fw + c, w);
+    if (a.fb != nullptr) {
+      ldv<V>(a.fb + c, b);
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) b[i] = 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] = ((f[i] - mean) * inv2 * w[i] + b[i]) * a.fscale;
+    stv<V>(lo + c, f);
+  }
+}
+
+// out[t, h * D + c] = o[t, h * DC + c] * sigmoid(z[t, h * D + c]) * scale
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+    head_gate_kernel(const T* o, int DC, const T* z, long long ldz, float scale, T* out,
+                     long long ldout, long long rows, int N, int D) {
+  const int nv = N * D / V;
+  const long long n = rows * nv;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / nv;
+    const int e = static_cast<int>(i - t * nv) * V;
+    const int h = e / D, c = e - h * D;
+    float a[V], g[V];
+    ldv<V>(o + (t * N + h) * DC + c, a);
+    ldv<V>(z + t * ldz + e, g);
+#pragma unroll
+    for (int k = 0; k < V; ++k) a[k] = a[k] * scale / (1.0f + expf(-g[k]));
+    stv<V>(out + t * ldout + e, a);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+    silu_mul_rows_kernel(const T* x, long long ldx, T* out, long long ldo, int D) {
+  const T* g = x + blockIdx.x * ldx;
+  for (int c = threadIdx.x * V; c < D; c += blockDim.x * V) {
+    float a[V], b[V];
+    ldv<V>(g + c, a);
+    ldv<V>(g + D + c, b);
+#pragma unroll
+    for (int i = 0; i < V; ++i) a[i] = a[i] / (1.0f + expf(-a[i])) * b[i];
+    stv<V>(out + blockIdx.x * ldo + c, a);
+  }
+}
+
 static int row_threads(int H, int V, int most) {
   int n = (H / V + 31) / 32 * 32;
   return n < 32 ? 32 : (n > most ? most : n);
@@ -258,6 +403,21 @@ static int launch_post_norm(const PostNormArgs& a, cudaStream_t s) {
   // few rows: more threads per row, so that a row's loads are in flight together
   const int threads = row_threads(a.H, V, a.T < 2 * sm_count() ? 512 : 256);
   post_norm_kernel<Y, LO, V><<<a.T, threads, smem, s>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int V>
+static int launch_add_normed(const AddNormArgs& a, cudaStream_t s) {
+  const size_t smem = static_cast<size_t>(a.H) * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(add_normed_kernel<T, V>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  const int threads = row_threads(a.H, V, a.T < 2 * sm_count() ? 512 : 256);
+  add_normed_kernel<T, V><<<a.T, threads, smem, s>>>(a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -349,6 +509,106 @@ B200_API int b200_sigmoid_gate(const void* o, long long ldo, const void* z, long
     float* pq = static_cast<float*>(out);
     if (v4) sigmoid_gate_kernel<float, 4><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
     else sigmoid_gate_kernel<float, 1><<<g, 256, 0, s>>>(po, ldo, pz, ldz, pq, ldout, T, D);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+// x = scale * e (fp32) and its copy `lo` in e's type; dtype (of e and lo): 0 bf16, 2 fp32.
+B200_API int b200_start_rows(const void* e, long long lde, float scale, float* x, void* lo, int T,
+                             int H, int dtype, void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || (dtype != 0 && dtype != 2)) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (H % 4) == 0 && (lde % 4) == 0 && aligned(e, 16) && aligned(x, 16) &&
+                  aligned(lo, 16);
+  const int th = row_threads(H, v4 ? 4 : 1, 256);
+  if (dtype == 0) {
+    const __nv_bfloat16* pe = static_cast<const __nv_bfloat16*>(e);
+    __nv_bfloat16* pl = static_cast<__nv_bfloat16*>(lo);
+    if (v4) start_rows_kernel<__nv_bfloat16, 4><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
+    else start_rows_kernel<__nv_bfloat16, 1><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
+  } else {
+    const float* pe = static_cast<const float*>(e);
+    float* pl = static_cast<float*>(lo);
+    if (v4) start_rows_kernel<float, 4><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
+    else start_rows_kernel<float, 1><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+// xo = x + norm(y) * w + b; lo: the sum, or with fw (norm(sum) * fw + fb) * fscale.  centred 1:
+// layer norm, 0: RMS norm.  dtype (of y and lo): 0 bf16, 2 fp32.
+B200_API int b200_add_normed(const float* x, const void* y, long long ldy, const float* w,
+                             const float* b, int centred, float eps, float* xo, const float* fw,
+                             const float* fb, float fscale, void* lo, int T, int H, int dtype,
+                             void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || (dtype != 0 && dtype != 2) || lo == nullptr) return -2;
+  AddNormArgs a;
+  a.x = x; a.y = y; a.w = w; a.b = b; a.fw = fw; a.fb = fb; a.xo = xo; a.lo = lo; a.ldy = ldy;
+  a.T = T; a.H = H; a.centred = centred; a.eps = eps; a.fscale = fscale;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (H % 4) == 0 && (ldy % 4) == 0 && aligned(x, 16) && aligned(y, 16) &&
+                  aligned(w, 16) && aligned(b, 16) && aligned(fw, 16) && aligned(fb, 16) &&
+                  aligned(xo, 16) && aligned(lo, 16);
+  if (dtype == 0)
+    return v4 ? launch_add_normed<__nv_bfloat16, 4>(a, s) : launch_add_normed<__nv_bfloat16, 1>(a, s);
+  return v4 ? launch_add_normed<float, 4>(a, s) : launch_add_normed<float, 1>(a, s);
+}
+
+// o [T, N, DC] -> out [T, N * D]: times sigmoid(z) and scale.
+B200_API int b200_head_gate(const void* o, int DC, const void* z, long long ldz, float scale,
+                            void* out, long long ldout, int T, int N, int D, int dtype,
+                            void* stream) {
+  if (T <= 0 || N <= 0 || D <= 0) return 0;
+  if (DC < D || (dtype != 0 && dtype != 2)) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (D % 4) == 0 && (DC % 4) == 0 && (ldz % 4) == 0 && (ldout % 4) == 0 &&
+                  aligned(o, 16) && aligned(z, dtype == 0 ? 8 : 16) &&
+                  aligned(out, dtype == 0 ? 8 : 16);
+  const bool v8 = dtype == 0 && v4 && (D % 8) == 0 && (DC % 8) == 0 && (ldz % 8) == 0 &&
+                  (ldout % 8) == 0 && aligned(z, 16) && aligned(out, 16);
+  const long long items = static_cast<long long>(T) * N * D / (v8 ? 8 : v4 ? 4 : 1);
+  long long blocks = (items + 255) / 256;
+  const long long cap = static_cast<long long>(sm_count()) * 16;
+  if (blocks > cap) blocks = cap;
+  const int g = static_cast<int>(blocks);
+  if (dtype == 0) {
+    const __nv_bfloat16* po = static_cast<const __nv_bfloat16*>(o);
+    const __nv_bfloat16* pz = static_cast<const __nv_bfloat16*>(z);
+    __nv_bfloat16* pq = static_cast<__nv_bfloat16*>(out);
+    if (v8) head_gate_kernel<__nv_bfloat16, 8><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
+    else if (v4) head_gate_kernel<__nv_bfloat16, 4><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
+    else head_gate_kernel<__nv_bfloat16, 1><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
+  } else {
+    const float* po = static_cast<const float*>(o);
+    const float* pz = static_cast<const float*>(z);
+    float* pq = static_cast<float*>(out);
+    if (v4) head_gate_kernel<float, 4><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
+    else head_gate_kernel<float, 1><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+// out [T, D] = silu(x[:, :D]) * x[:, D:]; dtype 0 bf16, 2 fp32.
+B200_API int b200_silu_mul_rows(const void* x, long long ldx, void* out, long long ldo, int T, int D,
+                                int dtype, void* stream) {
+  if (T <= 0 || D <= 0) return 0;
+  if (dtype != 0 && dtype != 2) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (D % 4) == 0 && (ldx % 4) == 0 && (ldo % 4) == 0 && aligned(x, 16) &&
+                  aligned(out, 16);
+  const int th = row_threads(D, v4 ? 4 : 1, 256);
+  if (dtype == 0) {
+    const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(x);
+    __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
+    if (v4) silu_mul_rows_kernel<__nv_bfloat16, 4><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
+    else silu_mul_rows_kernel<__nv_bfloat16, 1><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
+  } else {
+    const float* p = static_cast<const float*>(x);
+    float* o = static_cast<float*>(out);
+    if (v4) silu_mul_rows_kernel<float, 4><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
+    else silu_mul_rows_kernel<float, 1><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
   }
   return static_cast<int>(cudaGetLastError());
 }

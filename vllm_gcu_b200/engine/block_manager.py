@@ -149,13 +149,16 @@ class BlockPool:
 
 
 class KVCacheManager:
-    """Per-request block bookkeeping on top of a :class:`BlockPool`."""
+    """Per-request block bookkeeping on top of a :class:`BlockPool`; with ``num_state_slots`` a
+    request also holds one slot of recurrent state from its first blocks to its end."""
 
     def __init__(self, num_blocks: int, block_size: int, enable_prefix_caching: bool = True,
-                 watermark_blocks: int = 0):
+                 watermark_blocks: int = 0, num_state_slots: int = 0):
         self.pool = BlockPool(num_blocks, block_size, enable_prefix_caching)
         self.block_size = block_size
         self.watermark = watermark_blocks
+        self.has_state = num_state_slots > 0
+        self.free_slots = list(range(num_state_slots - 1, -1, -1))
 
     @staticmethod
     def _extra(req) -> tuple:
@@ -189,6 +192,10 @@ class KVCacheManager:
         if need + idle_hits > self.pool.num_free_blocks - (self.watermark if not req.block_ids
                                                             else 0):
             return None
+        if self.has_state and req.state_slot < 0:
+            if not self.free_slots:
+                return None
+            req.state_slot = self.free_slots.pop()
         if new_computed_blocks:
             self.pool.touch(new_computed_blocks)
             req.block_ids.extend(new_computed_blocks)
@@ -238,6 +245,9 @@ class KVCacheManager:
         req.block_ids = []
         req._hashed_blocks = 0
         req._last_hash = None
+        if req.state_slot >= 0:
+            self.free_slots.append(req.state_slot)
+            req.state_slot = -1
 
     @property
     def usage(self) -> float:

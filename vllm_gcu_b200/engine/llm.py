@@ -82,9 +82,15 @@ class LLMEngine:
         self.proposer = None
         self.spec_metrics = None
         sp = cfg.speculative
-        if sp.method and getattr(self.model, "has_block_state", False):
-            raise ValueError(f"{cfg.model.architecture} keeps recurrent state with its cache "
-                             "blocks: draft tokens cannot be taken back")
+        has_slots = getattr(self.model, "has_request_state", False)
+        if sp.method and (has_slots or getattr(self.model, "has_block_state", False)):
+            raise ValueError(f"{cfg.model.architecture} keeps recurrent state with its requests: "
+                             "draft tokens cannot be taken back")
+        if has_slots:
+            # the state behind a cached block, or beside swapped ones, is not kept: prompts start
+            # at their first token, and a preempted request is computed again
+            cfg.cache.enable_prefix_caching = False
+            cfg.cache.num_cpu_blocks = 0
         if sp.method:
             from ..spec import NgramProposer, SpecMetrics
             self.spec_metrics = SpecMetrics()
@@ -140,7 +146,9 @@ class LLMEngine:
                                    separate_prefill_decode=bool(
                                        cfg.additional_config.get("separate_prefill_decode")),
                                    num_lookahead_tokens=sp.num_speculative_tokens
-                                   if sp.method else 0)
+                                   if sp.method else 0,
+                                   num_state_slots=cfg.scheduler.max_num_seqs
+                                   if has_slots else 0)
         self._ids = itertools.count()
         self._want_sync = False
         self.disagg = None               # set by attach_kv_connector()
@@ -279,9 +287,10 @@ class LLMEngine:
         """Disaggregated prefill: requests with ``kv_transfer_params`` send their KV to /
         take their KV from the peer instance through ``connector`` (engine/kv_disagg.py)."""
         from .kv_disagg import DisaggCoordinator
-        if getattr(self.model, "has_block_state", False):
-            raise ValueError(f"{self.cfg.model.architecture} keeps recurrent state with its cache "
-                             "blocks, which the connector does not ship")
+        if getattr(self.model, "has_block_state", False) \
+                or getattr(self.model, "has_request_state", False):
+            raise ValueError(f"{self.cfg.model.architecture} keeps recurrent state with its "
+                             "requests, which the connector does not ship")
         self.disagg = DisaggCoordinator(self, connector, recv_timeout_s)
         self.scheduler.on_free = self.disagg.before_free
         return self.disagg

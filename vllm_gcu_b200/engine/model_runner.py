@@ -17,6 +17,7 @@ vllm_gcu/v1/gcu_async_model_runner.py:99-1081):
 """
 from __future__ import annotations
 
+import math
 import time
 import zlib
 from dataclasses import dataclass, field
@@ -99,6 +100,7 @@ class ModelRunner:
         self.max_blocks = -(-sc.max_model_len // self.block_size) + 1
         self.kv_caches: list[torch.Tensor] = []
         self.block_state: list[torch.Tensor] = []
+        self.request_state: list[dict] = []        # per layer, [slots, ...] tensors
         self.num_blocks = 0
         tp = cfg.parallel.tensor_parallel_size
         # under tensor parallelism every rank samples its slice of the batch rows and the ids
@@ -156,11 +158,11 @@ class ModelRunner:
                            "sample_indices": (3 * T, S * W), "seeds": (3 * T + S * W, S),
                            "mtp_ids": (3 * T + S * W + S, T if self.max_spec else 0)}
         n64 = 3 * T + S * W + S + (T if self.max_spec else 0)
-        # int32 block: seq_lens | cu_q | feed_dst | feed_src | top_k | num_draft | draft_ids |
+        # int32 block: seq_lens | state_slots | cu_q | feed_dst | feed_src | top_k | num_draft | draft_ids |
         #              block_tables
         o = 0
         self.i32_layout = {}
-        for name, n in (("seq_lens", S), ("cu_q", S + 1), ("feed_dst", S), ("feed_src", S),
+        for name, n in (("seq_lens", S), ("state_slots", S), ("cu_q", S + 1), ("feed_dst", S), ("feed_src", S),
                         ("top_k", S), ("num_draft", S), ("draft_ids", S * max(self.max_spec, 1)),
                         ("block_tables", S * MB)):
             self.i32_layout[name] = (o, n)
@@ -188,6 +190,7 @@ class ModelRunner:
         self.slot_mapping, self.sample_indices = v64("slot_mapping"), v64("sample_indices")
         self.seeds = v64("seeds")
         self.seq_lens, self.cu_q = v32("seq_lens"), v32("cu_q")
+        self.state_slots = v32("state_slots")
         self.feed_dst, self.feed_src, self.top_k = v32("feed_dst"), v32("feed_src"), v32("top_k")
         self.block_tables = v32("block_tables").view(S, MB)
         self.temperature, self.top_p = self.d_f32[:S], self.d_f32[S:]
@@ -218,6 +221,10 @@ class ModelRunner:
             bytes_per_block = self.block_size * sum(spec["widths"]) \
                 * torch.empty((), dtype=self.cfg.model.dtype).element_size() \
                 + 4 * sum(spec.get("block_state", ()))
+        elif "layer_shapes" in spec:
+            bytes_per_block = max(1, 2 * self.block_size * sum(
+                h * d for h, d in (s for s in spec["layer_shapes"] if s is not None))
+                * torch.empty((), dtype=self.cfg.model.dtype).element_size())
         else:
             bytes_per_block = self.cfg.model.kv_bytes_per_token(
                 self.cfg.parallel.tensor_parallel_size) * self.block_size
@@ -233,9 +240,12 @@ class ModelRunner:
         free, total = torch.cuda.mem_get_info()
         torch.cuda.empty_cache()
         weights_and_act = peak
-        budget = int(total * cc.gpu_memory_utilization) - weights_and_act
+        state_bytes = self.max_seqs * sum(
+            math.prod(shape) * torch.empty((), dtype=dt).element_size()
+            for layer in spec.get("request_state", ()) for shape, dt in layer.values())
+        budget = int(total * cc.gpu_memory_utilization) - weights_and_act - state_bytes
         # the dummy forward is gone but other processes may hold memory too
-        budget = min(budget, int(torch.cuda.mem_get_info()[0] * 0.97))
+        budget = min(budget, int(torch.cuda.mem_get_info()[0] * 0.97) - state_bytes)
         n = budget // bytes_per_block
         if n < 16:
             raise RuntimeError(f"not enough GPU memory for the KV cache ({budget} bytes)")
@@ -268,6 +278,12 @@ class ModelRunner:
             widths = spec.get("widths") or [spec["width"]] * spec["layers"]
             self.kv_caches = [torch.zeros(num_blocks, self.block_size, w, dtype=dt,
                                           device=self.device) for w in widths]
+        elif "layer_shapes" in spec:       # sizes per layer; layers without a cache hold nothing
+            if self.is_cuda and dt != mc.dtype:
+                raise ValueError(f"{mc.architecture} has no 8-bit KV cache")
+            self.kv_caches = [torch.zeros(2, num_blocks if s else 0, self.block_size,
+                                          *(s or (1, 1)), dtype=dt, device=self.device)
+                              for s in spec["layer_shapes"]]
         else:
             self.kv_caches = [torch.zeros(2, num_blocks, self.block_size, spec["kv_heads"],
                                           spec["head_dim"], dtype=dt, device=self.device)
@@ -275,6 +291,10 @@ class ModelRunner:
         # recurrent rows that live with the cache blocks (token shift): one per block and layer
         self.block_state = [torch.zeros(num_blocks, w, dtype=torch.float32, device=self.device)
                             for w in spec.get("block_state", ())]
+        # recurrent state with one slot per running request
+        self.request_state = [{k: torch.zeros(self.max_seqs, *shape, dtype=d, device=self.device)
+                               for k, (shape, d) in layer.items()}
+                              for layer in spec.get("request_state", ())]
         self.num_blocks = num_blocks
         if self.drafter is not None:
             ds = self.drafter.kv_cache_spec()
@@ -287,7 +307,8 @@ class ModelRunner:
                                                    ds["head_dim"], dtype=dt, device=self.device)
                                        for _ in range(ds["layers"])]
         if self.is_cuda and spec["type"] == "gqa":
-            Hq = mc.num_attention_heads // self.cfg.parallel.tensor_parallel_size
+            Hq = spec.get("q_heads") or \
+                mc.num_attention_heads // self.cfg.parallel.tensor_parallel_size
             ns = 32
             self.decode_ws = (
                 torch.empty(self.max_seqs * Hq * ns * spec["head_dim"] // 8 + 1024,
@@ -299,10 +320,13 @@ class ModelRunner:
         if not self.is_cuda or self.model.kv_cache_spec()["type"] != "gqa":
             return 1
         from ..ops import cuda as C
-        kvh = self.model.kv_cache_spec()["kv_heads"]
-        s = C.decode_num_splits(batch, kvh, max_seq_len)
-        Hq = self.cfg.model.num_attention_heads // self.cfg.parallel.tensor_parallel_size
-        while s > 1 and batch * Hq * s * self.cfg.model.head_dim > self.decode_ws[0].numel():
+        spec = self.model.kv_cache_spec()
+        s = C.decode_num_splits(batch, spec["kv_heads"], max_seq_len)
+        Hq = spec.get("q_heads") or \
+            self.cfg.model.num_attention_heads // self.cfg.parallel.tensor_parallel_size
+        D = max(self.cfg.model.head_dim, spec["head_dim"])
+        while s > 1 and (batch * Hq * s * D > self.decode_ws[0].numel()
+                         or batch * Hq * s > self.decode_ws[1].numel()):
             s -= 1
         return s
 
@@ -553,8 +577,11 @@ class ModelRunner:
                 i64[o_seed + r] = (base * 1000003 + order[j].sample_index) & 0x7FFFFFFFFFFFFFFF
         # per-sequence metadata
         i32[o_sl:o_sl + B] = seq_after
+        o_ss = self.i32_layout["state_slots"][0]
+        i32[o_ss:o_ss + B] = [s.state_slot for s in order]
         if B_pad > B:
             i32[o_sl + B:o_sl + B_pad] = 0
+            i32[o_ss + B:o_ss + B_pad] = -1
         cu = np.zeros(npf + 1, dtype=np.int64)
         if npf:
             np.cumsum(ntok[nd:], out=cu[1:])
@@ -627,6 +654,7 @@ class ModelRunner:
             sample_indices=self.sample_indices[:max(ns * width, 1)],
             q_lens_cpu=[int(x) for x in ntok], seq_lens_cpu=[int(x) for x in seq_after],
             common_prefix_len=common_prefix, block_state=self.block_state,
+            request_state=self.request_state, state_slots=self.state_slots[:max(B_pad, B)],
             cu_q_all=torch.tensor(tok_off, dtype=torch.int32, device=self.device)
             if common_prefix else None)
 
@@ -1027,6 +1055,7 @@ class ModelRunner:
             sizes.append(self.max_seqs)
         self.graph_sizes = sizes
         self.seq_lens.zero_()
+        self.state_slots.fill_(-1)
         self.slot_mapping.fill_(-1)
         torch.cuda.synchronize()
         stream = torch.cuda.Stream()
@@ -1045,7 +1074,8 @@ class ModelRunner:
                             decode_splits=self._decode_splits(Bp, self.cfg.scheduler.max_model_len),
                             decode_workspace=self.decode_ws,
                             sample_indices=self.sample_indices[:Bp],
-                            block_state=self.block_state)
+                            block_state=self.block_state, request_state=self.request_state,
+                            state_slots=self.state_slots[:Bp])
                         # warm-up outside the graph (lazy initialisation, autotuning)
                         self._forward_and_sample(md, Bp, Bp, self.sampled[cur], greedy)
                         stream.synchronize()

@@ -125,6 +125,7 @@ class Request:
     num_cached_tokens: int = 0                # prefix-cache hit length (first schedule)
     spec_token_ids: list[int] = field(default_factory=list)
     block_ids: list[int] = field(default_factory=list)
+    state_slot: int = -1                      # slot of its recurrent state (-1: none held)
     num_preemptions: int = 0
     first_token_time: Optional[float] = None
     finish_time: Optional[float] = None

@@ -36,6 +36,7 @@ class ScheduledRequest:
     will_sample: bool = False  # this step produces the next token(s) of the request
     epoch: int = 0             # the request's preemption count when this step was planned
     sample_index: int = 0      # index of the first output token this step produces
+    state_slot: int = -1       # recurrent state of the request (KVCacheManager)
     # offsets among this step's tokens whose logits go back to the caller
     logit_rows: list[int] = field(default_factory=list)
 
@@ -59,11 +60,13 @@ class SchedulerOutput:
 
 class Scheduler:
     def __init__(self, sched_cfg: SchedulerConfig, cache_cfg: CacheConfig, num_blocks: int,
-                 separate_prefill_decode: bool = False, num_lookahead_tokens: int = 0):
+                 separate_prefill_decode: bool = False, num_lookahead_tokens: int = 0,
+                 num_state_slots: int = 0):
         self.cfg = sched_cfg
         self.block_size = cache_cfg.block_size
         self.kv = KVCacheManager(num_blocks, cache_cfg.block_size,
-                                 cache_cfg.enable_prefix_caching)
+                                 cache_cfg.enable_prefix_caching,
+                                 num_state_slots=num_state_slots)
         self.waiting: deque[Request] = deque()
         self.running: list[Request] = []
         self.requests: dict[str, Request] = {}
@@ -381,6 +384,7 @@ class Scheduler:
         for s in out.scheduled:
             req = s.req
             s.epoch = getattr(req, "preempt_epoch", 0)
+            s.state_slot = req.state_slot
             req.num_computed_tokens += s.num_tokens
             will_sample = req.num_computed_tokens >= (req.num_tokens_with_placeholders
                                                       + len(s.spec_token_ids))

@@ -59,6 +59,10 @@ class AttentionMetadata:
     # per layer [num_blocks, width] fp32: state rows that models with ``has_block_state`` keep
     # with every cache block
     block_state: Optional[list] = None
+    # per layer, a dict of tensors ``[slots, ...]``: recurrent state of models with
+    # ``has_request_state``, and the slot of every request of the step ``[B]`` int32 (-1: padding)
+    request_state: Optional[list] = None
+    state_slots: Optional[torch.Tensor] = None
     cu_q_all: Optional[torch.Tensor] = None
 
 

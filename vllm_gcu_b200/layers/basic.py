@@ -68,6 +68,26 @@ class ScalarGain(nn.Module):
         self.gain.data.copy_(full.reshape(()))
 
 
+class LayerNormParams(nn.Module):
+    """fp32 weight and bias of a layer norm that is fused with a residual sum."""
+
+    def __init__(self, hidden_size: int, device=None):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=torch.float32, device=device),
+                                   requires_grad=False)
+        self.bias = nn.Parameter(torch.zeros(hidden_size, dtype=torch.float32, device=device),
+                                 requires_grad=False)
+
+    def add(self, ops_, x: torch.Tensor, y: torch.Tensor, eps: float, lo: torch.Tensor,
+            end: dict) -> None:
+        """``x += norm(y)``, ``lo`` in y's type; ``end``: the final norm's operands, if it follows
+        (see ``ops.cuda.add_normed``; x is then not needed any more)."""
+        ops_.add_normed(x, y, self.weight, self.bias, eps, lo, out=None if end else x, **end)
+
+    def load_weight(self, name: str, full: torch.Tensor, shard_id=None) -> None:
+        getattr(self, name).data.copy_(full)
+
+
 def _yarn_find_correction_dim(num_rot, dim, base, max_pos):
     return (dim * math.log(max_pos / (num_rot * 2 * math.pi))) / (2 * math.log(base))
 

@@ -1,0 +1,118 @@
+"""Attention whose queries and keys are normalised over the whole projection, with attention
+sinks and an output gate; the values are the projected keys themselves.
+
+Paged cache ``[2, blocks, block_size, kv_heads, DC]`` as in ``PagedAttention``: rotated keys and
+raw keys (the values), heads padded to a width the tensor-core kernels take.  On the GPU one kernel
+normalises, rotates and writes the cache; decode rows run through the split-KV kernels, portions
+through the tcgen05 prefill kernel, everything else (32-bit models, wide heads, large groups)
+through the general kernel of csrc/attention_any.cu.
+"""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from .. import ops
+from ..config import AttentionSpec
+from ..ops import cuda as C
+from ..ops import ref
+from ..parallel.communicator import get_comm
+from ..parallel.state import tp_size
+from .attention import AttentionMetadata
+from .basic import RotaryEmbedding
+from .mixer import MixerPart
+
+#: query heads per key head the decode kernels take
+MAX_DECODE_GROUP = 16
+MAX_HEAD_DIM = 512
+
+
+def cached_head_dim(head_dim: int, dtype: torch.dtype) -> int:
+    """Width of a cached head: one the tensor-core kernels cover where that is possible."""
+    if dtype == torch.bfloat16:
+        for n in (64, 96, 128):
+            if head_dim <= n:
+                return n
+    return -(-head_dim // 4) * 4
+
+
+class KeyAttention(MixerPart):
+    def __init__(self, spec: AttentionSpec, eps: float, dtype, device, prefix: str,
+                 rotary: RotaryEmbedding):
+        super().__init__()
+        self.spec, self.eps, self.rotary = spec, eps, rotary
+        H, G, D = spec.num_heads, spec.num_kv_heads, spec.head_dim
+        tp = tp_size()
+        if H % G:
+            raise ValueError(f"{prefix}: {H} query heads over {G} key heads")
+        if H % tp or G % tp:
+            raise ValueError(f"{prefix}: {H} query and {G} key heads over {tp} ranks")
+        if D > MAX_HEAD_DIM:
+            raise ValueError(f"{prefix}: heads of {D} dimensions, at most {MAX_HEAD_DIM}")
+        if spec.rot_dims % 2 or not 0 <= spec.rot_dims <= D:
+            raise ValueError(f"{prefix}: {spec.rot_dims} rotated of {D} dimensions")
+        self.H, self.G, self.DC = H // tp, G // tp, cached_head_dim(D, dtype)
+        self.width = H * D
+        self.projections = [("q", H * D, True), ("k", G * D, True), ("g", H * D, True)]
+        self.q_norm = self.new(self.H * D, device=device)
+        self.k_norm = self.new(self.G * D, device=device)
+        self.sink = self.new(self.H, device=device)
+
+    def cache_shape(self) -> tuple[int, int]:
+        return self.G, self.DC
+
+    _OWN = {"q.norm": "q_norm", "k.norm": "k_norm", "sink": "sink"}
+
+    def own_tensors(self) -> set[str]:
+        return set(self._OWN)
+
+    def load(self, name: str, full: torch.Tensor) -> bool:
+        if name not in self._OWN:
+            return False
+        getattr(self, self._OWN[name]).data.copy_(self.shard(full))
+        return True
+
+    def _attend(self, q: torch.Tensor, cache: torch.Tensor, md: AttentionMetadata) -> torch.Tensor:
+        s = self.spec
+        kc, vc = cache[0], cache[1]
+        nd, npf, nr = md.num_decode_tokens, md.num_prefills, md.num_decodes
+        if not ops.use_native(q):
+            return ref.any_attention(q, kc, vc, md.block_tables, md.seq_lens, nd, md.cu_q_prefill,
+                                     s.scale, self.sink)
+        rest = dict(scale=s.scale, sink=self.sink)
+        tensor_cores = q.dtype == torch.bfloat16 and self.DC in (64, 96, 128)
+        if not tensor_cores:
+            return C.any_attention(q, kc, vc, md.block_tables, md.seq_lens, nd, md.cu_q_prefill,
+                                   **rest)
+        out = torch.empty_like(q)
+        if nd > 0:
+            if self.H // self.G <= MAX_DECODE_GROUP:
+                C.paged_decode(q[:nd], kc, vc, md.block_tables[:nd], md.seq_lens[:nd], out=out[:nd],
+                               num_splits=md.decode_splits, workspace=md.decode_workspace, **rest)
+            else:
+                C.any_attention(q[:nd], kc, vc, md.block_tables[:nd], md.seq_lens[:nd], nd, None,
+                                out=out[:nd], **rest)
+        if npf > 0:
+            bt, sl = md.block_tables[nr:nr + npf], md.seq_lens[nr:nr + npf]
+            if C.fmha_prefill_sink(q[nd:], kc, vc, bt, md.cu_q_prefill, sl,
+                                   num_q_tiles_128=md.num_q_tiles_128, out=out[nd:], **rest) is None:
+                C.any_attention(q[nd:], kc, vc, bt, sl, 0, md.cu_q_prefill, out=out[nd:], **rest)
+        return out
+
+    def mix(self, y, f, md: AttentionMetadata, cache: Optional[torch.Tensor],
+            state: Optional[dict], scale: float, out: torch.Tensor) -> None:
+        D = self.spec.head_dim
+        if cache is None or md.is_dummy:
+            out.zero_()
+            return
+        o_ = C if ops.use_native(out) else ref
+        q, k = y["q"][:, :self.H * D], y["k"][:, :self.G * D]
+        tp, sumsq = tp_size(), None
+        if tp > 1:          # the norm runs over the heads of all ranks
+            sumsq = get_comm("tp").all_reduce(torch.stack(
+                [q.float().pow(2).sum(-1), k.float().pow(2).sum(-1)], dim=1).contiguous())
+        qn = o_.qk_norm_rope_cache(q, k, None, self.q_norm, self.k_norm, self.eps,
+                                   self.rotary.cos_sin_cache, self.rotary.is_neox, md.positions,
+                                   md.slot_mapping, cache[0], cache[1], D, sumsq, tp)
+        o_.head_gate(self._attend(qn, cache, md), y["g"][:, :self.H * D], scale, D, out)

@@ -12,6 +12,7 @@ vllm_gcu/models/deepseek_v3/deepseek_v3.py:1037-1173):
   (``gate_up_proj``); with ``fuse_silu`` the gate/up rows are interleaved in blocks
   of 128 at load time and SiLU(gate)*up runs in the GEMM epilogue
 * ``QKVParallelLinear``           – fused q/k/v with GQA-aware sharding
+* ``MixedRowParallelLinear``      – several sharded inputs side by side into one output
 * ``RowParallelLinear``           – input sharded, output all-reduced (or left partial /
   reduce-scattered for sequence parallelism)
 * ``ReplicatedLinear`` / ``MergedReplicatedLinear`` – unsharded (router gate, MLA
@@ -61,7 +62,8 @@ class UnquantizedLinearMethod(LinearMethod):
         if getattr(layer, "fuse_silu", False) and not getattr(layer, "_interleaved", False):
             w = layer.weight.data
             half = w.shape[0] // 2
-            if half % ref.GATE_UP_BLOCK == 0 and w.dtype == torch.bfloat16:
+            if half % ref.GATE_UP_BLOCK == 0 and w.dtype == torch.bfloat16 and w.is_cuda \
+                    and w.shape[1] % 8 == 0:
                 layer.weight.data = ref.interleave_gate_up(w[:half], w[half:]).contiguous()
                 layer._interleaved = True
 
@@ -81,13 +83,14 @@ class UnquantizedLinearMethod(LinearMethod):
                 else:
                     y = C.gemm_bf16(x2, w, bias=bias, residual=residual)
                 if getattr(layer, "fuse_silu", False):
-                    y = C.activation(y, "silu")
+                    y = C.activation(y, "silu") if y.shape[-1] % 16 == 0 else C.silu_mul_rows(y)
             return y.view(*shape[:-1], y.shape[-1])
         y = F.linear(x, w, bias)
         if residual is not None:
             y = y + residual
         if getattr(layer, "fuse_silu", False):
-            y = ref.silu_and_mul(y)
+            y = C.silu_mul_rows(y) if y.dtype == torch.float32 and ops.use_native(y) \
+                else ref.silu_and_mul(y)
         return y
 
 
@@ -195,24 +198,45 @@ class ColumnParallelLinear(LinearBase):
 
 class MixedParallelLinear(LinearBase):
     """Projections of one input stacked along the output dim, each either sharded over TP
-    (``sharded[i]``) or replicated; ``split(y)`` gives the views of an output row."""
+    (``sharded[i]``) or replicated; ``split(y)`` gives the views of an output row.  With ``align``
+    every projection starts at a multiple of that many columns (zero rows in between)."""
 
     def __init__(self, in_features, output_sizes: Sequence[int], sharded: Sequence[bool],
-                 dtype=torch.bfloat16, device=None, quant_method=None, prefix=""):
+                 dtype=torch.bfloat16, device=None, quant_method=None, prefix="", align: int = 1):
         tp = tp_size()
-        assert all(n % tp == 0 for n, s in zip(output_sizes, sharded) if s)
+        if any(n % tp for n, s in zip(output_sizes, sharded) if s):
+            raise ValueError(f"{prefix}: output sizes {list(output_sizes)} over {tp} ranks")
         self.sharded = list(sharded)
         self.local_sizes = [n // tp if s else n for n, s in zip(output_sizes, sharded)]
-        super().__init__(in_features, sum(output_sizes), in_features, sum(self.local_sizes), False,
+        self.padded_sizes = [-(-n // align) * align for n in self.local_sizes]
+        super().__init__(in_features, sum(output_sizes), in_features, sum(self.padded_sizes), False,
                          dtype, device, quant_method, prefix)
+        if self.padded_sizes != self.local_sizes:
+            self.weight.data.zero_()
 
     def shard_spec(self, shard_id=None):
         n = self.local_sizes[shard_id]
         src = tp_rank() * n if self.sharded[shard_id] else 0
-        return [(src, n, sum(self.local_sizes[:shard_id]))], None
+        return [(src, n, sum(self.padded_sizes[:shard_id]))], None
 
-    def split(self, y: torch.Tensor):
-        return y.split(self.local_sizes, dim=-1)
+    def split(self, y: torch.Tensor, padded: bool = False):
+        parts = y.split(self.padded_sizes, dim=-1)
+        return parts if padded else tuple(p[..., :n] for p, n in zip(parts, self.local_sizes))
+
+    def finalize(self) -> None:
+        at = 0
+        for n, p in zip(self.local_sizes, self.padded_sizes):
+            self.weight.data[at + n:at + p] = 0
+            at += p
+        super().finalize()
+
+
+def linear_fp32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``x @ weight^T`` with an fp32 result: rows that the consumer needs unrounded (router scores,
+    gates of a recurrence)."""
+    if ops.use_native(x) and x.dtype == torch.bfloat16:
+        return C.gemm_bf16(x, weight, epilogue=C.EPI_FP32)
+    return F.linear(x.float(), weight.float())
 
 
 class MergedColumnParallelLinear(LinearBase):
@@ -308,3 +332,18 @@ class RowParallelLinear(LinearBase):
         if self.bias is not None:   # added once, after the reduction
             y = y + self.bias
         return y
+
+
+class MixedRowParallelLinear(RowParallelLinear):
+    """Projections of several sharded inputs that lie side by side, summed by one GEMM."""
+
+    def __init__(self, input_sizes: Sequence[int], out_features, **kw):
+        tp = tp_size()
+        if any(n % tp for n in input_sizes):
+            raise ValueError(f"{kw.get('prefix')}: input sizes {list(input_sizes)} over {tp} ranks")
+        self.local_sizes = [n // tp for n in input_sizes]
+        super().__init__(sum(input_sizes), out_features, **kw)
+
+    def load_weight(self, name: str, full: torch.Tensor, shard_id=None) -> None:
+        n, at = self.local_sizes[shard_id], sum(self.local_sizes[:shard_id])
+        self.weight.data[:, at:at + n].copy_(full[:, tp_rank() * n:(tp_rank() + 1) * n])

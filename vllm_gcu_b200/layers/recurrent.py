@@ -1,0 +1,151 @@
+"""Mixer parts with a matrix state per head: gated delta rule and matrix memory.
+
+Their state belongs to a request, not to its cache blocks: it lives in the request's state slot
+(``AttentionMetadata.state_slots``) in fp32 and is updated in place by every step.  A portion at
+position 0 starts from zeros, so slots are handed on without clearing.  See csrc/recurrent.cu for
+the layout.
+"""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from .. import ops
+from ..config import DeltaSpec, MemorySpec
+from ..ops import cuda as C
+from ..ops import ref
+from ..parallel.state import tp_size
+from .attention import AttentionMetadata
+from .linear import linear_fp32
+from .mixer import MixerPart, linear
+
+#: padded key dimensions of the scan kernel
+STATE_ROWS = (32, 64, 96, 128, 192, 256)
+MAX_TAPS = 8
+
+
+def state_rows(head_dim: int, prefix: str) -> int:
+    for n in STATE_ROWS:
+        if head_dim <= n:
+            return n
+    raise ValueError(f"{prefix}: a state with {head_dim} keys per head, at most {STATE_ROWS[-1]}")
+
+
+def _local_heads(heads: int, prefix: str) -> int:
+    tp = tp_size()
+    if heads % tp:
+        raise ValueError(f"{prefix}: {heads} heads over {tp} ranks")
+    return heads // tp
+
+
+class GatedDelta(MixerPart):
+    """Gated delta rule with one decay per head and key channel.  Queries, keys and values pass a
+    short causal convolution and SiLU; decays and the output gate come from two-step projections."""
+
+    def __init__(self, spec: DeltaSpec, eps: float, dtype, device, prefix: str):
+        super().__init__()
+        self.spec, self.eps, self.dtype = spec, eps, dtype
+        N, G, D, V = spec.num_heads, spec.num_kv_heads, spec.head_dim, spec.v_head_dim
+        if N % G:
+            raise ValueError(f"{prefix}: {N} heads over {G} query / key heads")
+        if not 1 <= spec.conv_taps <= MAX_TAPS:
+            raise ValueError(f"{prefix}: a convolution of {spec.conv_taps} taps, at most {MAX_TAPS}")
+        self.N, self.G = _local_heads(N, prefix), _local_heads(G, prefix)
+        self.rows = state_rows(D, prefix)
+        self.width = N * V
+        self.projections = [("q", G * D, True), ("k", G * D, True), ("v", N * V, True),
+                            ("a1", spec.decay_rank, False), ("g1", spec.gate_rank, False)]
+        self.fp32_projections = [("b", N, True)]
+        new = lambda *s, dt=torch.float32: self.new(*s, dtype=dt, device=device)  # noqa: E731
+        self.conv_q, self.conv_k = (new(self.G * D, spec.conv_taps) for _ in range(2))
+        self.conv_v = new(self.N * V, spec.conv_taps)
+        self.a_log, self.dt_bias = new(self.N), new(self.N * D)
+        self.norm = new(V)
+        pad = lambda n: -(-n // 8) * 8  # noqa: E731
+        self.a2 = new(self.N * D, pad(spec.decay_rank), dt=dtype)      # columns behind the rank
+        self.g2 = new(self.N * V, pad(spec.gate_rank), dt=dtype)       # stay zero
+
+    def state_shapes(self) -> dict:
+        s = self.spec
+        C_ = 2 * self.G * s.head_dim + self.N * s.v_head_dim
+        return {"matrix": ((self.N, s.v_head_dim, self.rows), torch.float32),
+                "taps": ((s.conv_taps, C_), self.dtype)}
+
+    _OWN = {"q.conv": "conv_q", "k.conv": "conv_k", "v.conv": "conv_v", "A_log": "a_log",
+            "dt_bias": "dt_bias", "norm": "norm", "a2": "a2", "g2": "g2"}
+
+    def own_tensors(self) -> set[str]:
+        return set(self._OWN)
+
+    def load(self, name: str, full: torch.Tensor) -> bool:
+        if name not in self._OWN:
+            return False
+        p = getattr(self, self._OWN[name]).data
+        t = full if name == "norm" else self.shard(full)
+        (p[:, :t.shape[1]] if name in ("a2", "g2") else p).copy_(t)
+        return True
+
+    def finalize(self) -> None:
+        self.a2.data[:, self.spec.decay_rank:] = 0
+        self.g2.data[:, self.spec.gate_rank:] = 0
+
+    def mix(self, y, f, md: AttentionMetadata, cache, state: Optional[dict], scale: float,
+            out: torch.Tensor) -> None:
+        s = self.spec
+        o_ = C if ops.use_native(out) else ref
+        n = self.N * s.v_head_dim
+        if md.is_dummy:
+            state = None
+        o = o_.delta_rule(y["q"][:, :self.G * s.head_dim], y["k"][:, :self.G * s.head_dim],
+                          y["v"][:, :n], linear_fp32(y["a1"], self.a2), f["b"],
+                          (self.conv_q, self.conv_k, self.conv_v), self.dt_bias, self.a_log,
+                          s.head_dim, s.v_head_dim, self.rows, md, state)
+        o_.head_norm_gate(o, self.norm, linear(y["g1"], self.g2), self.eps, scale, out)
+
+
+class MatrixMemory(MixerPart):
+    """Matrix memory of an mLSTM: exponential input gate, forget gate in log space, a running
+    maximum that keeps both in range, and a normaliser vector."""
+
+    def __init__(self, spec: MemorySpec, eps: float, dtype, device, prefix: str):
+        super().__init__()
+        self.spec, self.eps = spec, eps
+        N, D, V = spec.num_heads, spec.head_dim, spec.v_head_dim
+        self.N = _local_heads(N, prefix)
+        self.rows = state_rows(D, prefix)
+        self.width = N * V
+        self.projections = [("q", N * D, True), ("k", N * D, True), ("v", N * V, True),
+                            ("g", N * V, True)]
+        self.fp32_projections = [("i", N, True), ("f", N, True)]
+        self.i_bias, self.f_bias = self.new(self.N, device=device), self.new(self.N, device=device)
+        self.norm = self.new(self.N * V, device=device)
+
+    def state_shapes(self) -> dict:
+        f32 = torch.float32
+        return {"matrix": ((self.N, self.spec.v_head_dim, self.rows), f32),
+                "vector": ((self.N, self.rows), f32), "scalar": ((self.N,), f32)}
+
+    _OWN = {"i.b": "i_bias", "f.b": "f_bias", "norm": "norm"}
+
+    def own_tensors(self) -> set[str]:
+        return set(self._OWN)
+
+    def load(self, name: str, full: torch.Tensor) -> bool:
+        if name not in self._OWN:
+            return False
+        getattr(self, self._OWN[name]).data.copy_(self.shard(full))
+        return True
+
+    def mix(self, y, f, md: AttentionMetadata, cache, state: Optional[dict], scale: float,
+            out: torch.Tensor) -> None:
+        s = self.spec
+        o_ = C if ops.use_native(out) else ref
+        nk, nv = self.N * s.head_dim, self.N * s.v_head_dim
+        if md.is_dummy:
+            state = None
+        # (a head count of one makes the norm weight per head and shared at once)
+        o = o_.matrix_memory(y["q"][:, :nk], y["k"][:, :nk], y["v"][:, :nv], f["i"], f["f"],
+                             self.i_bias, self.f_bias, s.gate_cap, s.head_dim, s.v_head_dim,
+                             self.rows, md, state)
+        o_.head_norm_gate(o, self.norm, y["g"][:, :nv], self.eps, scale, out)

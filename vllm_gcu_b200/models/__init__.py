@@ -51,6 +51,7 @@ _REGISTRY: dict[str, str] = {
     "DeepseekV3ForCausalLM": "vllm_gcu_b200.models.deepseek:DeepseekV3ForCausalLM",
     "DeepseekVLV2ForCausalLM": "vllm_gcu_b200.models.deepseek_vl2:DeepseekVLV2ForCausalLM",
     "SapapelForCausalLM": "vllm_gcu_b200.models.sapapel:SapapelForCausalLM",
+    "FizunexForCausalLM": "vllm_gcu_b200.models.fizunex:FizunexForCausalLM",
     "DeepSeekMTPModel": "vllm_gcu_b200.models.deepseek_mtp:DeepSeekMTP",
     # pooling models (no KV cache; built by build_pooling_model)
     "XLMRobertaForSequenceClassification":

@@ -129,6 +129,27 @@ class _Sigs:
     b200_token_shift = [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P]
     b200_post_norm = [P, P, L, P, I, P, F, F, P, P, L, I, P, P, P, P, I, I, I, P]
     b200_sigmoid_gate = [P, L, P, L, P, L, I, I, I, P]
+    b200_silu_mul_rows = [P, L, P, L, I, I, I, P]
+    b200_start_rows = [P, L, F, P, P, I, I, I, P]
+    b200_add_normed = [P, P, L, P, P, I, F, P, P, P, F, P, I, I, I, P]
+    b200_head_gate = [P, I, P, L, F, P, L, I, I, I, I, P]
+    b200_qk_norm_rope_cache = [P, L, P, L, P, L, P, P, P, I, I, F, P, I, L, I, P, P, P, P, P, L, I,
+                               I, I, I, I, I, P]
+    b200_any_attention = [P, P, P, L, P, P, I, I, P, P, P, I, I, I, I, I, I, F, I, P]
+    b200_paged_decode_sink = [P, L, P, L, P, P, L, L, L, P, I, I, P, P, P, I, I, I, I, I, F, I, P,
+                              P]
+    b200_paged_decode_tma_sink = [P, L, P, L, P, P, L, L, L, P, I, I, P, P, P, I, I, I, I, I, F, I,
+                                  P, P]
+    b200_fmha_prefill_sink = [P, L, P, L, P, P, P, P, P, L, L, L, P, I, I, I, I, I, I, I, I, F,
+                              I, I, I, P, P]
+    b200_recurrent_rows = [I]
+    b200_delta_inputs = [P, P, P, L, P, P, P, I, P, I, P, L, P, L, P, P, P, P, P, P, P, P, P, P,
+                         I, I, I, I, I, I, I, I, I, I, P]
+    b200_memory_inputs = [P, P, P, L, P, P, L, P, P, F, F, P, P, P, P, P, I, I, I, I, I, I, I, P]
+    b200_delta_scan = [P, P, P, P, P, P, P, P, P, P, L, P, I, P, P, I, P, I, I, I, I, I, I, I, I,
+                       I, P]
+    b200_memory_scan = [P, P, P, P, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, P]
+    b200_head_norm_gate = [P, P, I, P, L, P, L, F, F, I, I, I, I, P]
     b200_gemm_wna16 = [P, L, P, P, P, P, P, L, I, I, I, I, I, P, P]
     b200_gemm_wna16_workspace = [I, I, I]
     b200_gemm_wna16_grouped = [P, L, P, P, P, P, L, I, I, I, I, I, I, P, P, P, P]

@@ -448,10 +448,12 @@ def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                  out: Optional[torch.Tensor] = None, num_splits: int = 0,
                  workspace: Optional[tuple[torch.Tensor, torch.Tensor]] = None,
                  max_seq_len: int = 0, kv_quant: Optional[tuple] = None,
-                 alibi_slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 alibi_slopes: Optional[torch.Tensor] = None,
+                 sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     res = _paged_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, out, num_splits,
-                        workspace, max_seq_len, kv_quant, alibi_slopes)
+                        workspace, max_seq_len, kv_quant, alibi_slopes, sink)
     if (oracle_enabled("paged_decode") and k_cache.element_size() > 1 and alibi_slopes is None
+            and sink is None
             and not torch.cuda.is_current_stream_capturing()):
         from . import ref
         live = seq_lens > 0
@@ -466,11 +468,12 @@ def _paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                   out: Optional[torch.Tensor] = None, num_splits: int = 0,
                   workspace: Optional[tuple[torch.Tensor, torch.Tensor]] = None,
                   max_seq_len: int = 0, kv_quant: Optional[tuple] = None,
-                  alibi_slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  alibi_slopes: Optional[torch.Tensor] = None,
+                  sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q ``[B, Hq, D]`` (row stride free), caches ``[blocks, bs, Hkv, D]``.  For fp8 / int8
     caches ``kv_quant = (k_scale, v_scale, k_zero_point, v_zero_point)`` (floats).
     ``alibi_slopes`` fp32 ``[Hq]`` adds slope * (key position - query position) to the scores
-    (bf16 / fp16 caches)."""
+    (bf16 / fp16 caches).  ``sink`` fp32 ``[Hq]``: exp(sink) joins the softmax denominator."""
     B, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
     assert q.stride(2) == 1 and q.stride(1) == D
@@ -496,6 +499,21 @@ def _paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
             raise NotImplementedError("ALiBi attention over an 8-bit KV cache")
         assert alibi_slopes.dtype == torch.float32 and alibi_slopes.numel() == Hq
         call("b200_paged_decode_alibi", *args[:-1], ptr(alibi_slopes), stream_ptr())
+        return out
+    if sink is not None:
+        if k_cache.element_size() == 1:
+            raise NotImplementedError("attention sinks over an 8-bit KV cache")
+        assert sink.dtype == torch.float32 and sink.numel() == Hq
+        tail = (ptr(sink), stream_ptr())
+        if USE_TMA_DECODE and D == 128 and bs % 16 == 0 and k_cache.stride(2) == 128 \
+                and k_cache.stride(1) == Hkv * 128:
+            rc = N.lib().b200_paged_decode_tma_sink(*args[:-1], *tail)
+            N.launch_count += 1
+            if rc == 0:
+                return out
+            if rc != -20:
+                raise N.NativeError(f"b200_paged_decode_tma_sink failed with code {rc}")
+        call("b200_paged_decode_sink", *args[:-1], *tail)
         return out
     if k_cache.element_size() == 1:
         ks, vs, kz, vz = kv_quant or (1.0, 1.0, 0.0, 0.0)
@@ -588,6 +606,76 @@ def _varlen_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
          num_q_tiles, Hq, Hkv, D, float(scale), int(causal), int(window),
          DTYPE_CODE[q.dtype], stream_ptr())
     return (out, lse) if return_lse else out
+
+
+def fmha_prefill_sink(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                      block_tables: torch.Tensor, cu_q: torch.Tensor, seq_lens: torch.Tensor,
+                      scale: float, num_q_tiles_128: int, sink: Optional[torch.Tensor],
+                      out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """Causal tcgen05 prefill attention for head dimensions 64, 96 and 128 with optional sinks
+    (see ``paged_decode``); None when the layout is not covered (then use ``any_attention``)."""
+    T, Hq, D = q.shape
+    nb, bs, Hkv, _ = k_cache.shape
+    assert q.stride(2) == 1 and q.stride(1) == D
+    if out is None:
+        out = torch.empty((T, Hq, D), device=q.device, dtype=q.dtype)
+    rc = N.lib().b200_fmha_prefill_sink(
+        ptr(q), q.stride(0), ptr(out), out.stride(0), None, ptr(cu_q), ptr(seq_lens), ptr(k_cache),
+        ptr(v_cache), k_cache.stride(1), k_cache.stride(2), nb * bs, ptr(block_tables),
+        block_tables.stride(0), bs, block_tables.shape[0], T, num_q_tiles_128, Hq, Hkv, D,
+        float(scale), 1, 0, DTYPE_CODE[q.dtype], ptr(sink), stream_ptr())
+    N.launch_count += 1
+    if rc == -20:
+        return None
+    if rc != 0:
+        raise N.NativeError(f"b200_fmha_prefill_sink failed with code {rc}")
+    return out
+
+
+def any_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                  block_tables: torch.Tensor, seq_lens: torch.Tensor, num_decodes: int,
+                  cu_q: Optional[torch.Tensor], scale: float, sink: Optional[torch.Tensor] = None,
+                  out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal paged attention for any head dimension (<= 512) and group size, fp32 or bf16
+    (csrc/attention_any.cu): q ``[T, Hq, D]``, the first ``num_decodes`` tokens one per request,
+    the rest by ``cu_q``."""
+    T, Hq, D = q.shape
+    nb, bs, Hkv, _ = k_cache.shape
+    assert q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.dtype == q.dtype and k_cache.shape[3] == D
+    if out is None:
+        out = torch.empty_like(q)
+    call("b200_any_attention", ptr(q), ptr(k_cache), ptr(v_cache), nb * bs, ptr(out),
+         ptr(block_tables), block_tables.stride(0), bs, ptr(seq_lens), ptr(cu_q), ptr(sink), T, Hq,
+         Hkv, D, num_decodes, cu_q.shape[0] - 1 if cu_q is not None else 0, float(scale),
+         DTYPE_CODE[q.dtype], stream_ptr())
+    return out
+
+
+def qk_norm_rope_cache(q: torch.Tensor, k: torch.Tensor, v: Optional[torch.Tensor],
+                       q_weight: torch.Tensor, k_weight: torch.Tensor, eps: float,
+                       cos_sin: torch.Tensor, is_neox: bool, positions: torch.Tensor,
+                       slot_mapping: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                       head_dim: int, sumsq: Optional[torch.Tensor] = None, ranks: int = 1
+                       ) -> torch.Tensor:
+    """RMS norm of the query rows ``q [T, Hq * D]`` and key rows ``k [T, Hkv * D]`` over the whole
+    projection, rotary positions on the first ``cos_sin.shape[1]`` dimensions of every head, keys
+    and values (``v``, or the keys before their norm) into the paged caches ``[blocks, bs, Hkv, DC
+    >= D]``.  Returns the queries ``[T, Hq, DC]``.  ``sumsq [T, 2]``: sums of squares over the rows
+    of all ``ranks`` ranks that share the projections."""
+    T = q.shape[0]
+    nb, bs, Hkv, DC = k_cache.shape
+    D = head_dim
+    Hq = q.shape[1] // D
+    assert q.stride(1) == 1 and k.stride(1) == 1 and cos_sin.dtype == torch.float32
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == q.dtype
+    out = torch.empty((T, Hq, DC), dtype=q.dtype, device=q.device)
+    call("b200_qk_norm_rope_cache", ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v),
+         v.stride(0) if v is not None else 0, ptr(q_weight), ptr(k_weight), ptr(sumsq),
+         Hq * D * ranks, Hkv * D * ranks, float(eps), ptr(cos_sin), cos_sin.shape[1],
+         cos_sin.shape[0], int(is_neox), ptr(positions), ptr(slot_mapping), ptr(out), ptr(k_cache),
+         ptr(v_cache), nb * bs, T, Hq, Hkv, D, DC, DTYPE_CODE[q.dtype], stream_ptr())
+    return out
 
 
 WNA16_FUSED_MAX_M = 256
@@ -739,6 +827,135 @@ def sigmoid_gate(o: torch.Tensor, z: torch.Tensor, out: Optional[torch.Tensor] =
         out = torch.empty((T, D), dtype=o.dtype, device=o.device)
     call("b200_sigmoid_gate", ptr(o), o.stride(0), ptr(z), z.stride(0), ptr(out), out.stride(0), T,
          D, DTYPE_CODE[o.dtype], stream_ptr())
+    return out
+
+
+def start_rows(e: torch.Tensor, scale: float) -> tuple[torch.Tensor, torch.Tensor]:
+    """``(scale * e`` in fp32, the same in ``e``'s type)."""
+    T, H = e.shape
+    x = torch.empty((T, H), dtype=torch.float32, device=e.device)
+    lo = torch.empty((T, H), dtype=e.dtype, device=e.device)
+    call("b200_start_rows", ptr(e), e.stride(0), float(scale), ptr(x), ptr(lo), T, H,
+         DTYPE_CODE[e.dtype], stream_ptr())
+    return x, lo
+
+
+def add_normed(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor,
+               bias: Optional[torch.Tensor], eps: float, lo: torch.Tensor,
+               out: Optional[torch.Tensor] = None, layer_norm: bool = True,
+               final_weight: Optional[torch.Tensor] = None,
+               final_bias: Optional[torch.Tensor] = None, final_scale: float = 1.0) -> None:
+    """``s = x + norm(y) * weight + bias`` over fp32 rows ``x [T, H]`` (layer norm or RMS norm);
+    ``out`` takes s (may be ``x``), ``lo`` takes s in ``y``'s type, or with ``final_weight`` its
+    norm ``(norm(s) * final_weight + final_bias) * final_scale``."""
+    T, H = x.shape
+    call("b200_add_normed", ptr(x), ptr(y), y.stride(0), ptr(weight), ptr(bias), int(layer_norm),
+         float(eps), ptr(out), ptr(final_weight), ptr(final_bias), float(final_scale), ptr(lo), T, H,
+         DTYPE_CODE[y.dtype], stream_ptr())
+
+
+def head_gate(o: torch.Tensor, z: torch.Tensor, scale: float, head_dim: int, out: torch.Tensor
+              ) -> torch.Tensor:
+    """``out = o * sigmoid(z) * scale`` with ``o [T, N, DC >= head_dim]`` and ``z``, ``out``
+    ``[T, N * head_dim]`` (row-strided views are fine)."""
+    T, Nh, DC = o.shape
+    assert o.is_contiguous() and z.stride(1) == 1 and out.stride(1) == 1
+    call("b200_head_gate", ptr(o), DC, ptr(z), z.stride(0), float(scale), ptr(out), out.stride(0),
+         T, Nh, head_dim, DTYPE_CODE[o.dtype], stream_ptr())
+    return out
+
+
+# ---------------------------------------------------------------------------
+# gated activation of any width
+# ---------------------------------------------------------------------------
+def silu_mul_rows(x: torch.Tensor) -> torch.Tensor:
+    """``silu(x[:, :D]) * x[:, D:]`` for rows of any width, bf16 or fp32."""
+    shape = x.shape
+    x2 = _rowmajor_2d(x)
+    T, D = x2.shape[0], x2.shape[1] // 2
+    out = torch.empty((T, D), dtype=x.dtype, device=x.device)
+    call("b200_silu_mul_rows", ptr(x2), x2.stride(0), ptr(out), D, T, D, DTYPE_CODE[x.dtype],
+         stream_ptr())
+    return out.view(*shape[:-1], D)
+
+
+# ---------------------------------------------------------------------------
+# recurrences with a matrix state per head (csrc/recurrent.cu)
+# ---------------------------------------------------------------------------
+def _scan_place(md):
+    cu = md.cu_q_prefill
+    return md.num_decode_tokens, (cu.shape[0] - 1 if cu is not None else 0), cu
+
+
+def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
+               b: torch.Tensor, conv: Sequence[torch.Tensor], dt_bias: torch.Tensor,
+               a_log: torch.Tensor, head_dim: int, v_dim: int, rows: int, md,
+               state: Optional[dict]) -> torch.Tensor:
+    """Gated delta rule with one decay per key channel over the portions of a step: q, k ``[T, G *
+    head_dim]`` and v ``[T, N * v_dim]`` are projections (views of one row), ``z [T, N * head_dim]``
+    and ``b [T, N]`` fp32.  ``state``: ``matrix [slots, N, v_dim, rows]`` fp32 and ``taps [slots,
+    taps, channels]``, addressed by ``md.state_slots``.  Returns fp32 ``[T, N, v_dim]``."""
+    T, D, V = q.shape[0], head_dim, v_dim
+    G, Nh = q.shape[1] // D, v.shape[1] // V
+    VP = -(-V // 4) * 4
+    ntaps = conv[0].shape[1]
+    assert q.stride(0) == k.stride(0) == v.stride(0) and z.dtype == b.dtype == torch.float32
+    new = lambda *s: torch.empty(s, dtype=torch.float32, device=q.device)  # noqa: E731
+    qo, ko, go, vo, beta = new(T, G, rows), new(T, G, rows), new(T, Nh, rows), new(T, Nh, VP), \
+        new(T, Nh)
+    out = new(T, Nh, V)
+    if state is None:
+        return out.zero_()
+    nd, npf, cu = _scan_place(md)
+    S, taps, slots = state["matrix"], state["taps"], md.state_slots
+    call("b200_delta_inputs", ptr(q), ptr(k), ptr(v), q.stride(0), ptr(conv[0]), ptr(conv[1]),
+         ptr(conv[2]), ntaps, ptr(taps), taps.shape[0], ptr(z), z.stride(0), ptr(b), b.stride(0),
+         ptr(dt_bias), ptr(a_log), ptr(qo), ptr(ko), ptr(go), ptr(vo), ptr(beta),
+         ptr(md.positions), ptr(slots), ptr(cu), T, G, Nh, D, V, rows, VP, nd, npf,
+         DTYPE_CODE[q.dtype], stream_ptr())
+    call("b200_delta_scan", ptr(qo), ptr(ko), ptr(go), ptr(vo), ptr(beta), ptr(out), ptr(S), ptr(q),
+         ptr(k), ptr(v), q.stride(0), ptr(taps), ntaps, ptr(md.positions), ptr(slots),
+         taps.shape[0], ptr(cu), G, Nh, D, V, rows, VP, nd, npf, q.element_size(), stream_ptr())
+    return out
+
+
+def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, zi: torch.Tensor,
+                  zf: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
+                  head_dim: int, v_dim: int, rows: int, md, state: Optional[dict]) -> torch.Tensor:
+    """Matrix memory with exponential gates (mLSTM) over the portions of a step: q, k, v
+    projections ``[T, N * dim]`` (views of one row), ``zi`` / ``zf`` fp32 ``[T, N]`` gate
+    projections.  ``state``: ``matrix [slots, N, v_dim, rows]``, ``vector [slots, N, rows]``,
+    ``scalar [slots, N]`` fp32.  Returns fp32 ``[T, N, v_dim]``."""
+    T, D, V = q.shape[0], head_dim, v_dim
+    Nh = q.shape[1] // D
+    VP = -(-V // 4) * 4
+    assert q.stride(0) == k.stride(0) == v.stride(0) and zi.stride(0) == zf.stride(0)
+    assert zi.dtype == zf.dtype == torch.float32
+    new = lambda *s: torch.empty(s, dtype=torch.float32, device=q.device)  # noqa: E731
+    qo, ko, vo, li, lf = new(T, Nh, rows), new(T, Nh, rows), new(T, Nh, VP), new(T, Nh), new(T, Nh)
+    out = new(T, Nh, V)
+    if state is None:
+        return out.zero_()
+    nd, npf, cu = _scan_place(md)
+    S = state["matrix"]
+    call("b200_memory_inputs", ptr(q), ptr(k), ptr(v), q.stride(0), ptr(zi), ptr(zf), zi.stride(0),
+         ptr(i_bias), ptr(f_bias), float(cap), float(D ** -0.5), ptr(qo), ptr(ko), ptr(vo), ptr(li),
+         ptr(lf), T, Nh, D, V, rows, VP, DTYPE_CODE[q.dtype], stream_ptr())
+    call("b200_memory_scan", ptr(qo), ptr(ko), ptr(vo), ptr(li), ptr(lf), ptr(out), ptr(S),
+         ptr(state["vector"]), ptr(state["scalar"]), ptr(md.positions), ptr(md.state_slots),
+         S.shape[0], ptr(cu), Nh, D, V, rows, VP, nd, npf, stream_ptr())
+    return out
+
+
+def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, z: torch.Tensor, eps: float,
+                   scale: float, out: torch.Tensor) -> torch.Tensor:
+    """``out = o / rms(o) * weight * sigmoid(z) * scale`` with ``o [T, N, V]`` fp32 normalised per
+    head, ``weight`` ``[V]`` or ``[N * V]``, ``z`` and ``out`` ``[T, N * V]`` (views are fine)."""
+    T, Nh, V = o.shape
+    assert z.stride(1) == 1 and out.stride(1) == 1 and z.dtype == out.dtype
+    call("b200_head_norm_gate", ptr(o), ptr(weight), int(weight.numel() != V), ptr(z), z.stride(0),
+         ptr(out), out.stride(0), float(eps), float(scale), T, Nh, V, DTYPE_CODE[out.dtype],
+         stream_ptr())
     return out
 
 

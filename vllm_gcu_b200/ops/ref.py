@@ -676,6 +676,168 @@ def sigmoid_gate(o: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
     return (o.float() * torch.sigmoid(z.float())).to(o.dtype)
 
 
+def start_rows(e: torch.Tensor, scale: float) -> tuple[torch.Tensor, torch.Tensor]:
+    """See ``ops.cuda.start_rows``."""
+    x = e.float() * scale
+    return x, x.to(e.dtype)
+
+
+def add_normed(x, y, weight, bias, eps, lo, out=None, layer_norm=True, final_weight=None,
+               final_bias=None, final_scale=1.0) -> None:
+    """See ``ops.cuda.add_normed``."""
+    def norm(r, w, b):
+        if layer_norm:
+            r = r - r.mean(-1, keepdim=True)
+        r = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps) * w
+        return r if b is None else r + b
+
+    s = x + norm(y.float(), weight, bias)
+    if out is not None:
+        out.copy_(s)
+    lo.copy_(s if final_weight is None else norm(s, final_weight, final_bias) * final_scale)
+
+
+def head_gate(o, z, scale, head_dim, out) -> torch.Tensor:
+    """See ``ops.cuda.head_gate``."""
+    out.copy_(o[..., :head_dim].flatten(1).float() * torch.sigmoid(z.float()) * scale)
+    return out
+
+
+def qk_norm_rope_cache(q, k, v, q_weight, k_weight, eps, cos_sin, is_neox, positions, slot_mapping,
+                       k_cache, v_cache, head_dim, sumsq=None, ranks=1) -> torch.Tensor:
+    """See ``ops.cuda.qk_norm_rope_cache``."""
+    T, D = q.shape[0], head_dim
+    nb, bs, Hkv, DC = k_cache.shape
+
+    def norm(x, w, ss):
+        f = x.float()
+        ss = f.pow(2).sum(-1) if ss is None else ss
+        return f * torch.rsqrt(ss[:, None] / (x.shape[1] * ranks) + eps) * w
+
+    qn = norm(q, q_weight, None if sumsq is None else sumsq[:, 0])
+    kn = norm(k, k_weight, None if sumsq is None else sumsq[:, 1])
+    qn, kn = rotary_embedding(positions, qn, kn, D, cos_sin, is_neox)
+    pad = lambda x: torch.nn.functional.pad(x.reshape(T, -1, D), (0, DC - D))  # noqa: E731
+    ok = slot_mapping >= 0
+    at = slot_mapping[ok].long()
+    k_cache.view(nb * bs, Hkv, DC)[at] = pad(kn)[ok].to(k_cache.dtype)
+    v_cache.view(nb * bs, Hkv, DC)[at] = pad(k if v is None else v)[ok].to(v_cache.dtype)
+    return pad(qn).to(q.dtype)
+
+
+def any_attention(q, k_cache, v_cache, block_tables, seq_lens, num_decodes, cu_q, scale, sink=None,
+                  out=None) -> torch.Tensor:
+    """See ``ops.cuda.any_attention``."""
+    T, Hq, D = q.shape
+    out = torch.zeros_like(q) if out is None else out
+    for r, (lo, hi) in enumerate(_portions(T, num_decodes, cu_q)):
+        n = int(seq_lens[r])
+        if n == 0 or hi == lo:
+            continue
+        k, v = _gather_kv(k_cache, v_cache, block_tables[r], n)
+        G = Hq // k.shape[1]
+        k, v = k.repeat_interleave(G, dim=1), v.repeat_interleave(G, dim=1)
+        s = torch.einsum("qhd,nhd->hqn", q[lo:hi].float(), k) * scale
+        qpos = torch.arange(n - (hi - lo), n, device=q.device)[:, None]
+        s = s.masked_fill((torch.arange(n, device=q.device)[None, :] > qpos)[None], float("-inf"))
+        if sink is not None:
+            s = torch.cat([s, sink.float()[:, None, None].expand(-1, hi - lo, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :n]
+        out[lo:hi] = torch.einsum("hqn,nhd->qhd", p, v).to(out.dtype)
+    return out
+
+
+# ---------------------------------------------------------------------------
+# recurrences with a matrix state per head
+# ---------------------------------------------------------------------------
+def _recurrent_portions(T, md):
+    """(first, end, state slot, starts at position 0) of every request of a step."""
+    for r, (lo, hi) in enumerate(_portions(T, md.num_decode_tokens, md.cu_q_prefill)):
+        slot = int(md.state_slots[r])
+        if hi > lo and slot >= 0:
+            yield lo, hi, slot, int(md.positions[lo]) == 0
+
+
+def delta_rule(q, k, v, z, b, conv, dt_bias, a_log, head_dim, v_dim, rows, md, state
+               ) -> torch.Tensor:
+    """See ``ops.cuda.delta_rule``."""
+    T, D, V = q.shape[0], head_dim, v_dim
+    G, Nh = q.shape[1] // D, v.shape[1] // V
+    out = torch.zeros(T, Nh, V, dtype=torch.float32, device=q.device)
+    if state is None:
+        return out
+    n = conv[0].shape[1]
+    taps = torch.cat(list(conv)).float()                      # [channels, n]
+    x = torch.cat([q, k, v], dim=1)
+    decay = torch.exp(-torch.exp(a_log.float())[None, :, None] * torch.nn.functional.softplus(
+        z + dt_bias).view(T, Nh, D))
+    beta = torch.sigmoid(b)
+    unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)  # noqa: E731
+    for lo, hi, slot, fresh in _recurrent_portions(T, md):
+        p0 = int(md.positions[lo])
+        ring = state["taps"][slot]
+        past = [ring[p % n].float() if p >= 0 else torch.zeros_like(taps[:, 0])
+                for p in range(p0 - n + 1, p0)]
+        seq = torch.cat([torch.stack(past), x[lo:hi].float()]) if past else x[lo:hi].float()
+        c = sum(seq[j:j + hi - lo] * taps[:, j] for j in range(n))
+        c = torch.nn.functional.silu(c)
+        qc = unit(c[:, :G * D].view(-1, G, D)) * D ** -0.5
+        kc = unit(c[:, G * D:2 * G * D].view(-1, G, D))
+        vc = c[:, 2 * G * D:].view(-1, Nh, V)
+        S = state["matrix"][slot, :, :, :D]                    # [N, V, D], a view
+        S = torch.zeros_like(S) if fresh else S.clone()
+        for i in range(hi - lo):
+            kt, qt = (t[i].repeat_interleave(Nh // G, dim=0)[:, None, :] for t in (kc, qc))
+            S = S * decay[lo + i][:, None, :]
+            u = beta[lo + i][:, None] * (vc[i] - (S * kt).sum(-1))
+            S = S + u[:, :, None] * kt
+            out[lo + i] = (S * qt).sum(-1)
+        state["matrix"][slot, :, :, :D] = S
+        for t in range(max(lo, hi - n + 1), hi):
+            ring[(p0 + t - lo) % n] = x[t]
+    return out
+
+
+def matrix_memory(q, k, v, zi, zf, i_bias, f_bias, cap, head_dim, v_dim, rows, md, state
+                  ) -> torch.Tensor:
+    """See ``ops.cuda.matrix_memory``."""
+    T, D, V = q.shape[0], head_dim, v_dim
+    Nh = q.shape[1] // D
+    out = torch.zeros(T, Nh, V, dtype=torch.float32, device=q.device)
+    if state is None:
+        return out
+    li = cap * torch.tanh((zi + i_bias) / cap)
+    lf = torch.nn.functional.logsigmoid(cap * torch.tanh((zf + f_bias) / cap))
+    qf, kf = q.float().view(T, Nh, D) * D ** -0.5, k.float().view(T, Nh, D)
+    vf = v.float().view(T, Nh, V)
+    for lo, hi, slot, fresh in _recurrent_portions(T, md):
+        S, nv, m = (state["matrix"][slot, :, :, :D].clone(), state["vector"][slot, :, :D].clone(),
+                    state["scalar"][slot].clone())
+        if fresh:
+            S, nv, m = torch.zeros_like(S), torch.zeros_like(nv), torch.zeros_like(m)
+        for t in range(lo, hi):
+            new = torch.maximum(lf[t] + m, li[t])
+            keep, add = torch.exp(lf[t] + m - new), torch.exp(li[t] - new)
+            m = new
+            S = keep[:, None, None] * S + add[:, None, None] * vf[t][:, :, None] * kf[t][:, None, :]
+            nv = keep[:, None] * nv + add[:, None] * kf[t]
+            den = torch.maximum((nv * qf[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            out[t] = (S * qf[t][:, None, :]).sum(-1) / den[:, None]
+        state["matrix"][slot, :, :, :D] = S
+        state["vector"][slot, :, :D] = nv
+        state["scalar"][slot] = m
+    return out
+
+
+def head_norm_gate(o, weight, z, eps, scale, out) -> torch.Tensor:
+    """See ``ops.cuda.head_norm_gate``."""
+    T, Nh, V = o.shape
+    r = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+    r = r * (weight.view(Nh, V) if weight.numel() != V else weight)
+    out.copy_(r.flatten(1) * torch.sigmoid(z.float()) * scale)
+    return out
+
+
 def input_weighted_experts(x, w13, w2, topk_w, topk_ids) -> tuple[torch.Tensor, torch.Tensor]:
     """See ``ops.cuda.input_weighted_experts`` (gate rows first in ``w13``); one output row per
     (token, slot) pair, so ``pos_of`` is the identity."""

@@ -65,6 +65,16 @@ def write_safetensors(path: str, tensors: dict[str, torch.Tensor], metadata: dic
             f.write(b)
 
 
+def tensor_shapes(model_dir: str) -> dict[str, tuple[int, ...]]:
+    """Names and shapes of the tensors in a folder's ``*.safetensors`` files (headers only)."""
+    out: dict[str, tuple[int, ...]] = {}
+    for path in sorted(Path(model_dir).glob("*.safetensors")):
+        with open(path, "rb") as f:
+            header = json.loads(f.read(struct.unpack("<Q", f.read(8))[0]))
+        out.update({k: tuple(v["shape"]) for k, v in header.items() if k != "__metadata__"})
+    return out
+
+
 def iter_safetensors(model_dir: str) -> Iterator[tuple[str, torch.Tensor]]:
     """Yields (name, tensor) for every tensor of the checkpoint in ``model_dir``."""
     d = Path(model_dir)
