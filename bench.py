@@ -23,7 +23,8 @@ Launch: ``python bench.py`` (1 GPU) or
 ``--impl reference`` reports why the reference cannot run on this hardware;
 ``--impl vllm-stock`` runs the same workload through stock vLLM on the CUDA platform (the
 stand-in baseline, benchmarks/baseline_vllm_stock.py).
-``--workload sapapel`` runs another measurement instead: one model family beside another.
+``--workload fizunex`` / ``sapapel`` runs another measurement instead: one model family beside
+another.
 """
 from __future__ import annotations
 
@@ -119,13 +120,14 @@ def main() -> None:
     ap.add_argument("--no-async", action="store_true")
     ap.add_argument("--eager", action="store_true")
     ap.add_argument("--layers", type=int, default=0, help="debug only: truncate the model")
-    ap.add_argument("--workload", default="default", choices=["default", "sapapel"],
-                    help="sapapel: prefill / decode throughput of Sapapel layers beside DeepSeek's "
-                         "at equal sizes (benchmarks/bench_family_pair.py), one line per size")
+    ap.add_argument("--workload", default="default", choices=["default", "sapapel", "fizunex"],
+                    help="prefill / decode throughput of Fizunex layers beside Llama's or of "
+                         "Sapapel layers beside DeepSeek's at equal sizes "
+                         "(benchmarks/bench_family_pair.py), one line per size")
     args = ap.parse_args()
-    if args.workload == "sapapel":
+    if args.workload != "default":
         from benchmarks.bench_family_pair import main as family_pair
-        family_pair(["--warmup", str(max(3, args.warmup)), "--steps", str(max(1, args.steps))])
+        family_pair(["--pair", args.workload, "--warmup", str(max(3, args.warmup)), "--steps", str(max(1, args.steps))])
         return
     if args.impl == "reference":
         run_reference(args)

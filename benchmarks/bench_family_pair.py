@@ -1,14 +1,19 @@
-"""Prefill and decode throughput of a Sapapel model beside DeepSeek (the closest other family:
-latent attention over a paged latent cache, routed experts) at equal layer sizes.
+"""Prefill and decode throughput of one model family beside the closest other one at equal layer
+sizes, both through ``LLM.generate`` with random weights.
 
-Both run through ``LLM.generate`` with random weights: same width, heads, latent rank, experts,
-experts per token, expert width, layers and vocabulary; DeepSeek's rows have 64 rotary columns more
-and it has neither the output gate nor the depth average.  Timed on the device: the CUDA events
-that bracket every engine step.  Prefill: ``prompts x input_len`` tokens in steps of 8192, one
-output token.  Decode: the steps of ``batch`` requests behind a prompt of ``input_len``.
+* Sapapel beside DeepSeek (latent attention over a paged latent cache, routed experts): same width,
+  heads, latent rank, experts, experts per token, expert width, layers and vocabulary; DeepSeek's
+  rows have 64 rotary columns more and it has neither the output gate nor the depth average.
+* Fizunex beside Llama (grouped-query attention, dense feed-forward): same width, heads, head
+  dimension, feed-forward, layers and vocabulary.  Half of Fizunex's layers are gated delta layers
+  (full query / key heads), the others run attention with Llama's heads and a matrix memory.
 
-    python bench.py --workload sapapel                    (all sizes, one JSON line each)
-    python benchmarks/bench_family_pair.py --sizes 2048 --no-decode
+Timed on the device: the CUDA events that bracket every engine step.  Prefill: ``prompts x
+input_len`` tokens in steps of 8192, one output token.  Decode: the steps of ``batch`` requests
+behind a prompt of ``input_len``.
+
+    python bench.py --workload fizunex                    (all sizes, one JSON line each)
+    python benchmarks/bench_family_pair.py --pair sapapel --sizes 2048 --no-decode
 """
 from __future__ import annotations
 
@@ -20,18 +25,39 @@ import sys
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
-#: width -> heads, head dims, latent rank, experts, experts per token, expert width, layers
-SIZES = {
+#: per pair, width -> heads, head dims, latent rank, experts, experts per token, expert width,
+#: layers; or heads, key heads, head dims, memory heads and dims, feed-forward, layers
+SIZES = {"sapapel": {
     2048: dict(heads=16, dim=128, rank=512, experts=64, top=6, ff=1408, layers=8),
     4096: dict(heads=32, dim=128, rank=512, experts=32, top=4, ff=1536, layers=6),
     7168: dict(heads=128, dim=128, rank=512, experts=64, top=8, ff=2048, layers=3),
-}
+}, "fizunex": {
+    2048: dict(heads=16, kv_heads=4, dim=128, mem_heads=4, mem_dim=128, mem_vdim=256, ff=8192,
+               layers=8),
+    4096: dict(heads=32, kv_heads=8, dim=128, mem_heads=8, mem_dim=128, mem_vdim=256, ff=14336,
+               layers=8),
+    8192: dict(heads=64, kv_heads=8, dim=128, mem_heads=16, mem_dim=128, mem_vdim=256, ff=28672,
+               layers=4),
+}}
+PAIRS = {"sapapel": ("sapapel", "deepseek"), "fizunex": ("fizunex", "llama")}
 VOCAB = 32768
 
 
-def model_config(family: str, width: int):
+def model_config(pair: str, family: str, width: int):
     from vllm_gcu_b200.config import ModelConfig
-    s = SIZES[width]
+    s = SIZES[pair][width]
+    if family == "fizunex":
+        from vllm_gcu_b200.config import _fizunex_mixers, _fizunex_preset
+        mixers = _fizunex_mixers(s["heads"], s["kv_heads"], s["dim"], s["mem_heads"],
+                                 s["mem_dim"], s["mem_vdim"])
+        return ModelConfig.from_hf_dict(_fizunex_preset(
+            ("dp" * s["layers"])[:s["layers"]], VOCAB, width, s["ff"], *mixers), dtype="bfloat16")
+    if family == "llama":
+        return ModelConfig(
+            architecture="LlamaForCausalLM", vocab_size=VOCAB, hidden_size=width,
+            intermediate_size=s["ff"], num_hidden_layers=s["layers"],
+            num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"],
+            head_dim=s["dim"], tie_word_embeddings=True, dtype="bfloat16")
     if family == "sapapel":
         layer = {"type": "latent_attention",
                  "mixer": {"heads": s["heads"], "dim": s["dim"], "vdim": s["dim"],
@@ -52,14 +78,14 @@ def model_config(family: str, width: int):
         rope_is_neox=False, dtype="bfloat16")
 
 
-def measure(family: str, width: int, prompts: int, input_len: int, batch: int, output_len: int,
+def measure(pair: str, family: str, width: int, prompts: int, input_len: int, batch: int, output_len: int,
             warmup: int, steps: int, decode: bool = True, profile: str | None = None) -> dict:
     import torch
     from vllm_gcu_b200.engine.llm import LLM
     from vllm_gcu_b200.engine.request import SamplingParams
     from vllm_gcu_b200.ops import _native
     n = max(prompts, batch)
-    llm = LLM(model_config(family, width), max_num_seqs=n, max_num_batched_tokens=8192,
+    llm = LLM(model_config(pair, family, width), max_num_seqs=n, max_num_batched_tokens=8192,
               max_model_len=input_len + output_len + 16, async_scheduling=True,
               enable_prefix_caching=False, cuda_graph_sizes=[batch],
               num_gpu_blocks=n * (-(-(input_len + output_len) // 16) + 2))
@@ -108,28 +134,29 @@ def measure(family: str, width: int, prompts: int, input_len: int, batch: int, o
 def main(argv=None) -> None:
     ap = argparse.ArgumentParser(description=__doc__,
                                  formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--sizes", type=int, nargs="*", default=sorted(SIZES))
+    ap.add_argument("--pair", default="fizunex", choices=sorted(PAIRS))
+    ap.add_argument("--sizes", type=int, nargs="*", default=None)
     ap.add_argument("--prompts", type=int, default=16)
     ap.add_argument("--input-len", type=int, default=1024)
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--output-len", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--steps", type=int, default=3)
-    ap.add_argument("--families", nargs="*", default=["sapapel", "deepseek"])
+    ap.add_argument("--families", nargs="*", default=None)
     ap.add_argument("--no-decode", action="store_true")
     ap.add_argument("--profile", default=None, metavar="PREFIX",
                     help="also write a kernel table per family and phase (numbers under a "
                          "profiler: for shares only)")
     a = ap.parse_args(argv)
-    for width in a.sizes:
+    for width in a.sizes or sorted(SIZES[a.pair]):
         line = {"metric": "prefill and decode tok/s, device time", "unit": "tok/s", "n_gpus": 1,
                 "dtype": "bf16", "data": "synthetic (random ids, random weights)",
-                "config": {"width": width, **SIZES[width], "vocab": VOCAB, "prompts": a.prompts,
+                "config": {"width": width, **SIZES[a.pair][width], "vocab": VOCAB, "prompts": a.prompts,
                            "input_len": a.input_len, "decode_batch": a.batch,
                            "output_len": a.output_len,
                            "l2_policy": "weights and cache larger than L2"}}
-        for fam in a.families:
-            line[fam] = measure(fam, width, a.prompts, a.input_len, a.batch, a.output_len,
+        for fam in a.families or PAIRS[a.pair]:
+            line[fam] = measure(a.pair, fam, width, a.prompts, a.input_len, a.batch, a.output_len,
                                 a.warmup, a.steps, not a.no_decode, a.profile)
         print(json.dumps(line), flush=True)
 

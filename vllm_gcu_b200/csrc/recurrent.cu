@@ -394,7 +394,7 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
       const float mt = fmaxf(m + F, M);
       float before = __shfl_up_sync(0xffffffffu, mt, 1);
       if (lane == 0) before = m;
-      keep = expf(f + before - mt);
+      keep = expf(f + (before - mt));        // the difference of the maxima is (nearly) exact
       add = expf(ig - mt);
       floor_den = expf(-mt);
       m = __shfl_sync(0xffffffffu, mt, n - 1);

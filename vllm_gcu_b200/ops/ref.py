@@ -817,7 +817,7 @@ def matrix_memory(q, k, v, zi, zf, i_bias, f_bias, cap, head_dim, v_dim, rows, m
             S, nv, m = torch.zeros_like(S), torch.zeros_like(nv), torch.zeros_like(m)
         for t in range(lo, hi):
             new = torch.maximum(lf[t] + m, li[t])
-            keep, add = torch.exp(lf[t] + m - new), torch.exp(li[t] - new)
+            keep, add = torch.exp(lf[t] + (m - new)), torch.exp(li[t] - new)
             m = new
             S = keep[:, None, None] * S + add[:, None, None] * vf[t][:, :, None] * kf[t][:, None, :]
             nv = keep[:, None] * nv + add[:, None] * kf[t]
