@@ -80,7 +80,14 @@ def cases(lens: list[int], ctx: int, decode: bool, H: int, N: int, G: int, D: in
     gate, nw = rnd(T, N * D).to(bf), torch.ones(D, device=dev)
     res = torch.empty(T, N * D, device=dev, dtype=bf)
 
+    a2, g2, wb1 = rnd(N * D, 128).to(bf), rnd(N * D, 128).to(bf), rnd(N, H).to(bf)
+
     def delta():
+        if decode:
+            C.delta_step(xb, q, k, v, wide[:, 3 * N * D:3 * N * D + 128],
+                         wide[:, 3 * N * D + 128:], a2, g2, wb1, conv, dtb, alog, nw, D, D, D,
+                         md.positions, md.state_slots, st, 1e-5, 1.0, res)
+            return
         o = C.delta_rule(q, k, v, z, bz, conv, dtb, alog, D, D, D, md, st)
         C.head_norm_gate(o, nw, gate, 1e-5, 1.0, res)
     out.append(("delta (inputs, scan, norm)", "attention", delta, io + stb, T * N * D * D * 8,
@@ -95,9 +102,15 @@ def cases(lens: list[int], ctx: int, decode: bool, H: int, N: int, G: int, D: in
     mnw = torch.ones(MN * MV, device=dev)
     mres = torch.empty(T, MN * MV, device=dev, dtype=bf)
 
+    wi, wf = rnd(MN, H).to(bf), rnd(MN, H).to(bf)
+
     def memory():
-        o = C.matrix_memory(mq, mk, mv, zi, zf, ib, fb, 15.0, MD, MV, MD, md, ms)
-        C.head_norm_gate(o, mnw, mg, 1e-5, 1.0, mres)
+        if decode:
+            C.memory_step(xb, mq, mk, mv, mg, wi, wf, ib, fb, 15.0, mnw, MD, MV, MD, md.positions,
+                          md.state_slots, ms, 1e-5, 1.0, mres)
+            return
+        o, nq, low = C.matrix_memory(mq, mk, mv, zi, zf, ib, fb, 15.0, MD, MV, MD, md, ms)
+        C.head_norm_gate(o, mnw, mg, 1e-5, 1.0, mres, nq, low)
     out.append(("memory (inputs, scan, norm)", "attention", memory,
                 T * MN * (2 * MD + 3 * MV) * 2 + B * MN * MD * MV * 4 * (2 if decode else 1),
                 T * MN * MD * MV * 6, FP32_TFLOPS))

@@ -184,6 +184,114 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_pairs_kernel(const Pre
   }
 }
 
+// The same for bf16 rows of whole 16-byte vectors (D, DC and rot multiples of 8): NV vectors per
+// thread, queries then keys, read once and kept in registers.
+template <int NV>
+__global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const PrepArgs a) {
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  const __nv_bfloat16* q =
+      static_cast<const __nv_bfloat16*>(a.q) + static_cast<long long>(t) * a.ldq;
+  const __nv_bfloat16* k =
+      static_cast<const __nv_bfloat16*>(a.k) + static_cast<long long>(t) * a.ldk;
+  const int dv = a.D / 8, dcv = a.DC / 8;
+  const int vq = a.Hq * dv, vk = a.Hkv * dv;
+  uint4 raw[NV];
+  float sq = 0.0f, sk = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int e = threadIdx.x + i * 256;
+    if (e >= vq + vk) continue;
+    raw[i] = e < vq ? reinterpret_cast<const uint4*>(q)[e]
+                    : reinterpret_cast<const uint4*>(k)[e - vq];
+    const uint32_t w[4] = {raw[i].x, raw[i].y, raw[i].z, raw[i].w};
+    float s = 0.0f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(w[j]);
+      s += f.x * f.x + f.y * f.y;
+    }
+    if (e < vq) sq += s;
+    else sk += s;
+  }
+  if (a.sumsq != nullptr) {
+    sq = a.sumsq[2 * t];
+    sk = a.sumsq[2 * t + 1];
+  } else {
+    sq = block_sum(sq, red);
+    sk = block_sum(sk, red);
+  }
+  const float qi = 1.0f / sqrtf(sq / static_cast<float>(a.q_all) + a.eps);
+  const float ki = 1.0f / sqrtf(sk / static_cast<float>(a.k_all) + a.eps);
+  long long pos = a.positions[t];
+  if (pos < 0 || pos >= a.max_pos) {
+    if (threadIdx.x == 0)
+      report_status(a.status, kStatusBounds, kKernelId, static_cast<unsigned int>(t));
+    pos = 0;
+  }
+  long long slot = a.slots[t];
+  if (slot >= a.num_slots) {
+    if (threadIdx.x == 0)
+      report_status(a.status, kStatusBounds, kKernelId + 1, static_cast<unsigned int>(t));
+    slot = -1;
+  }
+  const float* cs = a.cos_sin + pos * a.rot;
+  uint4* qo = static_cast<uint4*>(a.qo) + static_cast<long long>(t) * a.Hq * dcv;
+  uint4* kc = static_cast<uint4*>(a.kc) + slot * a.Hkv * dcv;
+  uint4* vc = static_cast<uint4*>(a.vc) + slot * a.Hkv * dcv;
+  const uint4* v = a.v != nullptr
+      ? reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.v) +
+                                       static_cast<long long>(t) * a.ldv) : nullptr;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int e = threadIdx.x + i * 256;
+    if (e >= vq + vk) continue;
+    const bool is_q = e < vq;
+    const int x = is_q ? e : e - vq;
+    if (!is_q && slot < 0) continue;
+    const float inv = is_q ? qi : ki;
+    const float4* w4 = reinterpret_cast<const float4*>(is_q ? a.qw : a.kw) + 2 * x;
+    const float4 wa = w4[0], wb = w4[1];
+    const float w[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
+    const uint32_t in[4] = {raw[i].x, raw[i].y, raw[i].z, raw[i].w};
+    const int h = x / dv, c = x - h * dv;            // c: vector inside the head
+    float co[4] = {1.0f, 1.0f, 1.0f, 1.0f}, si[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    if (c * 8 < a.rot) {
+      const float4 cv = *reinterpret_cast<const float4*>(cs + c * 4);
+      const float4 sv = *reinterpret_cast<const float4*>(cs + a.rot / 2 + c * 4);
+      co[0] = cv.x; co[1] = cv.y; co[2] = cv.z; co[3] = cv.w;
+      si[0] = sv.x; si[1] = sv.y; si[2] = sv.z; si[3] = sv.w;
+    }
+    uint32_t out[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = unpack_bf16x2(in[j]);
+      const float u = f.x * inv * w[2 * j], y = f.y * inv * w[2 * j + 1];
+      out[j] = pack_bf16x2(u * co[j] - y * si[j], y * co[j] + u * si[j]);
+    }
+    const uint4 res = make_uint4(out[0], out[1], out[2], out[3]);
+    const int at = h * dcv + c;
+    if (is_q) {
+      qo[at] = res;
+    } else {
+      kc[at] = res;
+      vc[at] = v != nullptr ? v[x] : raw[i];
+    }
+  }
+  if (dcv == dv) return;
+  const int pad = dcv - dv;
+  for (int e = threadIdx.x; e < (a.Hq + a.Hkv) * pad; e += 256) {
+    const int h = e / pad, c = dv + e - h * pad;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    if (h < a.Hq) {
+      qo[h * dcv + c] = zero;
+    } else if (slot >= 0) {
+      kc[(h - a.Hq) * dcv + c] = zero;
+      vc[(h - a.Hq) * dcv + c] = zero;
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------
 struct AttnArgs {
   const void* q;             // [T, Hq, DC]
@@ -343,7 +451,18 @@ B200_API int b200_qk_norm_rope_cache(const void* q, long long ldq, const void* k
   const auto even = [](const void* p, int bytes) {
     return (reinterpret_cast<uintptr_t>(p) % bytes) == 0;
   };
-  if (dtype == 2)
+  const int vectors = (Hq + Hkv) * D / 8;
+  const bool vec = dtype == 0 && !is_neox && (D % 8) == 0 && (DC % 8) == 0 && (rot % 8) == 0 &&
+                   (ldq % 8) == 0 && (ldk % 8) == 0 && (ldv % 8) == 0 && even(q, 16) &&
+                   even(k, 16) && even(v, 16) && even(qw, 16) && even(kw, 16) &&
+                   even(cos_sin, 16) && even(qo, 16) && even(kc, 16) && even(vc, 16) &&
+                   vectors <= 8 * 256;
+  if (vec) {
+    if (vectors <= 256) qk_norm_rope_cache_vec_kernel<1><<<T, 256, 0, s>>>(a);
+    else if (vectors <= 512) qk_norm_rope_cache_vec_kernel<2><<<T, 256, 0, s>>>(a);
+    else if (vectors <= 1024) qk_norm_rope_cache_vec_kernel<4><<<T, 256, 0, s>>>(a);
+    else qk_norm_rope_cache_vec_kernel<8><<<T, 256, 0, s>>>(a);
+  } else if (dtype == 2)
     qk_norm_rope_cache_kernel<float><<<T, 256, 0, s>>>(a);
   else if (!is_neox && (D & 1) == 0 && (DC & 1) == 0 && (ldq & 1) == 0 && (ldk & 1) == 0 &&
            (ldv & 1) == 0 && even(q, 4) && even(k, 4) && even(v, 4) && even(qw, 8) &&

@@ -3,30 +3,32 @@
 //
 //   delta_inputs    short causal convolution + SiLU of q, k, v, unit vectors, decays, step sizes
 //   memory_inputs   q (scaled), k, v in fp32, log gates of the matrix memory
-//   recurrent_scan  the recurrence itself, for every request of a step: portions of prompts and
-//                   single tokens alike
+//   recurrent_scan  the recurrence over portions of prompts
 //   head_norm_gate  o / rms(o) per head, times the norm weight, a sigmoid gate and a factor
+//   recurrent_step  all of these (and the narrow projections in front of them) for requests that
+//                   bring a single token: one CTA per request and head
 //
 // State of a request, addressed by its state slot, fp32 throughout:
 //   matrix  [slot, head, vdim, DP]      S transposed: a value column's key entries are contiguous
 //   vector  [slot, head, DP], scalar [slot, head]      (matrix memory: normaliser n, maximum m)
 //   taps    [slot, taps, channels] in the model's type: row p % taps holds the convolution input
 //           of position p.  A step reads the rows of positions in front of its portion before
-//           the scan overwrites them.
+//           the scan overwrites them; a single token writes a row that no one reads in its step.
 // A portion that starts at position 0 starts from zeros whatever the slot holds, so slots need no
-// clearing.  DP is the head dimension rounded up to 8 * RPL; the padding stays zero.
+// clearing.  DP is the head dimension rounded up (b200_recurrent_rows); the padding stays zero.
 //
-// The scan splits a head's value columns over threads: they are independent of each other.  Eight
+// The scan splits a head's value columns over threads: they are independent of each other.  LPC
 // lanes share a column (RPL key rows each, in registers), CPT columns per lane group; a CTA holds a
 // block of columns of one head of one request and walks its tokens in order, inputs staged through
-// shared memory by cp.async one chunk ahead.  The result of a token does not depend on where the
-// prompt was cut.
+// shared memory by cp.async one chunk ahead.  Two lanes per column keep the arithmetic units busy
+// when there are heads enough for every scheduler; eight shorten the chain from token to token when
+// there are few.  The normaliser of the matrix memory is one more column whose value is always 1.
+// The result of a token does not depend on where the prompt was cut.
 #include "common.cuh"
 
 namespace b200 {
 namespace recurrent {
 
-constexpr unsigned int kKernelId = 80;
 constexpr int kDelta = 0, kMemory = 1;
 
 // fp32 pairs: two multiply-adds per instruction
@@ -101,88 +103,160 @@ struct DeltaIn {
   int T, G, N, D, V, DP, VP, ntaps, num_slots, nd, np;
 };
 
-// Rows of the convolution window of one token: [o] = input of `o` tokens ago, null for none.
 constexpr int kMaxTaps = 8;
-template <typename T>
-struct Window {
-  const T* row[kMaxTaps];
-};
+constexpr int kStrip = 16;       // tokens one warp walks
 
-template <typename T>
-__device__ __forceinline__ float conv_silu(const Window<T>& w, const float* taps, int ntaps, int c) {
-  float s = 0.0f;
-#pragma unroll
-  for (int o = kMaxTaps - 1; o >= 0; --o) {
-    if (o >= ntaps || w.row[o] == nullptr) continue;
-    s += taps[c * ntaps + (ntaps - 1 - o)] * to_f32<T>(w.row[o][c]);
+template <typename T, int V>
+__device__ __forceinline__ void load_n(const T* p, float (&f)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else if constexpr (V == 4) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
+  } else {
+    f[0] = to_f32<T>(p[0]);
   }
-  return s / (1.0f + expf(-s));
+}
+template <int V>
+__device__ __forceinline__ void store_n(float* p, const float (&f)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else p[0] = f[0];
+}
+// SiLU at the precision of the model's type
+template <typename T>
+__device__ __forceinline__ float silu(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.0f + __expf(-x));
+  else return x / (1.0f + expf(-x));
 }
 
-template <typename T>
+// One warp: kStrip tokens of one item, V neighbouring channels per lane (32 V channels at a time).
+// Items: [0, G) q heads, [G, 2G) k heads, [2G, 2G + N) v heads, [2G + N, 2G + 2N) decays.
+template <typename T, int NT, int V>
 __global__ void __launch_bounds__(256) delta_inputs_kernel(const DeltaIn a) {
-  const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int item = blockIdx.y * 8 + warp;          // [0, G): q and k heads; [G, G + N): v heads
-  if (item >= a.G + a.N) return;
-  const TokenPlace pl = token_place(t, a.nd, a.np, a.cu_q);
-  if (pl.req < 0) return;
-  const Portion po = portion_of(pl.req, a.nd, a.cu_q);
-  const long long pos = a.positions[t];
-  const int slot = a.slots[pl.req];
-  const int C = 2 * a.G * a.D + a.N * a.V;
-  auto window = [&](int which) {
-    Window<T> w;
-    const T* x = static_cast<const T*>(a.x[which]);
-    const int off = which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D;
+  const int item = blockIdx.y * 8 + warp;
+  const int t0 = blockIdx.x * kStrip;
+  if (item >= 2 * a.G + 2 * a.N || t0 >= a.T) return;
+  const int t1 = min(t0 + kStrip, a.T);
+  if (item >= 2 * a.G + a.N) {                   // decays and step sizes
+    const int h = item - 2 * a.G - a.N;
+    const float rate = expf(a.a_log[h]);
+    for (int d = lane * V; d < a.DP; d += 32 * V) {
+      float bias[V];
 #pragma unroll
-    for (int o = 0; o < kMaxTaps; ++o) {
-      w.row[o] = nullptr;
-      if (o >= a.ntaps || pos - o < 0) continue;
-      if (t - o >= po.first) {
-        w.row[o] = x + static_cast<long long>(t - o) * a.ld;
-      } else if (slot >= 0 && slot < a.num_slots) {
-        w.row[o] = static_cast<const T*>(a.taps) +
-                   (static_cast<long long>(slot) * a.ntaps + (pos - o) % a.ntaps) * C + off;
+      for (int i = 0; i < V; ++i) bias[i] = d + i < a.D ? a.dt_bias[h * a.D + d + i] : 0.0f;
+      for (int t = t0; t < t1; ++t) {
+        float g[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) g[i] = 0.0f;
+        if (d < a.D) {
+          load_n<float, V>(a.z + t * a.ldz + h * a.D + d, g);
+#pragma unroll
+          for (int i = 0; i < V; ++i) g[i] = expf(-rate * softplus(g[i] + bias[i]));
+        }
+        store_n<V>(a.g + (static_cast<long long>(t) * a.N + h) * a.DP + d, g);
       }
     }
-    return w;
-  };
-  if (item < a.G) {
-    constexpr int kMax = 8;                        // DP <= 256
-#pragma unroll
-    for (int which = 0; which < 2; ++which) {
-      const Window<T> w = window(which);
-      float f[kMax], ss = 0.0f;
-#pragma unroll
-      for (int i = 0; i < kMax; ++i) {
-        const int d = lane + 32 * i;
-        f[i] = d < a.D ? conv_silu<T>(w, a.taps_w[which], a.ntaps, item * a.D + d) : 0.0f;
-        ss += f[i] * f[i];
-      }
-      float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
-      if (which == 0) inv *= 1.0f / sqrtf(static_cast<float>(a.D));
-      float* out = (which == 0 ? a.q : a.k) + (static_cast<long long>(t) * a.G + item) * a.DP;
-#pragma unroll
-      for (int i = 0; i < kMax; ++i) {
-        const int d = lane + 32 * i;
-        if (d < a.DP) out[d] = f[i] * inv;
-      }
-    }
+    for (int t = t0 + lane; t < t1; t += 32)
+      a.beta[static_cast<long long>(t) * a.N + h] = sigmoid(a.bz[t * a.ldb + h]);
     return;
   }
-  const int h = item - a.G;
-  const Window<T> w = window(2);
-  float* v = a.v + (static_cast<long long>(t) * a.N + h) * a.VP;
-  for (int d = lane; d < a.VP; d += 32)
-    v[d] = d < a.V ? conv_silu<T>(w, a.taps_w[2], a.ntaps, h * a.V + d) : 0.0f;
-  float* g = a.g + (static_cast<long long>(t) * a.N + h) * a.DP;
-  const float* z = a.z + t * a.ldz + h * a.D;
-  const float rate = expf(a.a_log[h]);
-  for (int d = lane; d < a.DP; d += 32)
-    g[d] = d < a.D ? expf(-rate * softplus(z[d] + a.dt_bias[h * a.D + d])) : 0.0f;
-  if (lane == 0)
-    a.beta[static_cast<long long>(t) * a.N + h] = sigmoid(a.bz[t * a.ldb + h]);
+  const int which = item < a.G ? 0 : item < 2 * a.G ? 1 : 2;
+  const int head = which == 0 ? item : which == 1 ? item - a.G : item - 2 * a.G;
+  const int dim = which == 2 ? a.V : a.D, pitch = which == 2 ? a.VP : a.DP;
+  const int C = 2 * a.G * a.D + a.N * a.V;
+  const int ring_off = (which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D) + head * dim;
+  const T* x = static_cast<const T*>(a.x[which]) + head * dim;
+  const float* wt = a.taps_w[which] + static_cast<long long>(head) * dim * a.ntaps;
+  float* out = (which == 0 ? a.q : which == 1 ? a.k : a.v) + head * pitch;
+  const long long ldo = static_cast<long long>(which == 2 ? a.N : a.G) * pitch;
+  const int passes = (pitch + 32 * V - 1) / (32 * V);
+  float inv_sum[kStrip];
+  // q and k of more channels than one pass holds: a first walk over all passes for the norms
+  const bool unit = which < 2;
+  for (int walk = unit && passes > 1 ? 0 : 1; walk < 2; ++walk) {
+    for (int ps = 0; ps < passes; ++ps) {
+      const int d = (ps * 32 + lane) * V;
+      const bool in = d < dim;
+      float w[NT][V];                              // [o]: tap that meets the input of o tokens ago
+#pragma unroll
+      for (int o = 0; o < NT; ++o) {
+#pragma unroll
+        for (int i = 0; i < V; ++i)
+          w[o][i] = in && o < a.ntaps ? wt[(d + i) * a.ntaps + a.ntaps - 1 - o] : 0.0f;
+      }
+      float past[NT][V];                           // [o]: input of o tokens ago
+#pragma unroll
+      for (int o = 0; o < NT; ++o) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) past[o][i] = 0.0f;
+      }
+      int end = -1;                                // end of the portion the walk is in
+      for (int t = t0; t < t1; ++t) {
+        if (t >= end) {                            // first token of the strip or of a portion
+          const TokenPlace pl = token_place(t, a.nd, a.np, a.cu_q);
+          if (pl.req < 0) return;                  // padding rows end the step
+          const Portion po = portion_of(pl.req, a.nd, a.cu_q);
+          end = po.first + po.count;
+          const long long pos = a.positions[t];
+          const int slot = a.slots[pl.req];
+#pragma unroll
+          for (int o = 1; o < NT; ++o) {
+#pragma unroll
+            for (int i = 0; i < V; ++i) past[o - 1][i] = 0.0f;
+            if (!in || o >= a.ntaps || pos - o < 0) continue;
+            if (t - o >= po.first) {
+              load_n<T, V>(x + static_cast<long long>(t - o) * a.ld + d, past[o - 1]);
+            } else if (slot >= 0 && slot < a.num_slots) {
+              load_n<T, V>(static_cast<const T*>(a.taps) +
+                               (static_cast<long long>(slot) * a.ntaps + (pos - o) % a.ntaps) * C +
+                               ring_off + d, past[o - 1]);
+            }
+          }
+        }
+#pragma unroll
+        for (int o = NT - 1; o > 0; --o) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) past[o][i] = past[o - 1][i];
+        }
+        if (in) load_n<T, V>(x + static_cast<long long>(t) * a.ld + d, past[0]);
+        float f[V], ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+          float c = 0.0f;
+#pragma unroll
+          for (int o = NT - 1; o >= 0; --o) c += w[o][i] * past[o][i];
+          f[i] = silu<T>(c);
+          ss += f[i] * f[i];
+        }
+        if (unit) {
+          float inv;
+          if (passes == 1) {
+            inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
+          } else if (walk == 0) {
+            // (a static index keeps the sums in registers)
+            const float sum = warp_sum(ss);
+#pragma unroll
+            for (int u = 0; u < kStrip; ++u)
+              if (u == t - t0) inv_sum[u] = ps == 0 ? sum : inv_sum[u] + sum;
+            continue;
+          } else {
+            float sum = 0.0f;
+#pragma unroll
+            for (int u = 0; u < kStrip; ++u)
+              if (u == t - t0) sum = inv_sum[u];
+            inv = 1.0f / sqrtf(sum + 1e-6f);
+          }
+          if (which == 0) inv *= 1.0f / sqrtf(static_cast<float>(a.D));
+#pragma unroll
+          for (int i = 0; i < V; ++i) f[i] *= inv;
+        }
+        if (d < pitch) store_n<V>(out + t * ldo + d, f);
+      }
+    }
+  }
 }
 
 // ---------------------------------------------------------------------------
@@ -190,36 +264,59 @@ struct MemoryIn {
   const void *q, *k, *v;     // [T, channels] views, row pitch ld
   const float *zi, *zf;      // [T, N] input and forget gate projections, row pitch ldg
   const float *ib, *fb;      // [N] biases
+  const float* scalar;       // state m [slots, N]
   float *qo, *ko;            // out: [T, N, DP]
-  float* vo;                 // out: [T, N, VP]
+  float* vo;                 // out: [T, N, VP], column V: 1
   float *io, *fo;            // out: [T, N] log gates
+  float* m0;                 // out: [requests, N] m in front of the portion
+  const long long* positions;
+  const int* slots;
+  const int* cu_q;
   long long ld, ldg;
-  int T, N, D, V, DP, VP;
+  int T, N, D, V, DP, VP, num_slots, nd, np;
   float cap, qscale;
 };
 
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
 
-template <typename T>
+template <typename T, int W>
 __global__ void __launch_bounds__(256) memory_inputs_kernel(const MemoryIn a) {
   const long long t = blockIdx.x;
-  const int nq = a.N * a.DP, nv = a.N * a.VP;
-  const T* q = static_cast<const T*>(a.q) + t * a.ld;
-  const T* k = static_cast<const T*>(a.k) + t * a.ld;
-  const T* v = static_cast<const T*>(a.v) + t * a.ld;
-  for (int e = threadIdx.x; e < nq; e += blockDim.x) {
-    const int h = e / a.DP, d = e - h * a.DP;
-    const bool in = d < a.D;
-    a.qo[t * nq + e] = in ? to_f32<T>(q[h * a.D + d]) * a.qscale : 0.0f;
-    a.ko[t * nq + e] = in ? to_f32<T>(k[h * a.D + d]) : 0.0f;
+  const int kd = a.DP / W, kv = a.VP / W;
+  const int nq = a.N * kd, nv = a.N * kv;
+  for (int e = threadIdx.x; e < 2 * nq + nv; e += blockDim.x) {
+    const int which = e < nq ? 0 : e < 2 * nq ? 1 : 2;
+    const int r = which == 0 ? e : which == 1 ? e - nq : e - 2 * nq;
+    const int per = which == 2 ? kv : kd, dim = which == 2 ? a.V : a.D;
+    const int h = r / per, d = (r - h * per) * W;
+    const T* x = static_cast<const T*>(which == 0 ? a.q : which == 1 ? a.k : a.v) + t * a.ld +
+                 h * dim;
+    float f[W];
+#pragma unroll
+    for (int i = 0; i < W; ++i) f[i] = 0.0f;
+    if (d < dim) load_n<T, W>(x + d, f);
+    if (which == 0) {
+#pragma unroll
+      for (int i = 0; i < W; ++i) f[i] *= a.qscale;
+    }
+    if (which == 2) {
+#pragma unroll
+      for (int i = 0; i < W; ++i)
+        if (d + i == a.V) f[i] = 1.0f;
+    }
+    float* out = which == 0 ? a.qo : which == 1 ? a.ko : a.vo;
+    store_n<W>(out + (t * a.N + h) * (which == 2 ? a.VP : a.DP) + d, f);
   }
-  for (int e = threadIdx.x; e < nv; e += blockDim.x) {
-    const int h = e / a.VP, d = e - h * a.VP;
-    a.vo[t * nv + e] = d < a.V ? to_f32<T>(v[h * a.V + d]) : 0.0f;
-  }
+  const TokenPlace pl = token_place(static_cast<int>(t), a.nd, a.np, a.cu_q);
   for (int h = threadIdx.x; h < a.N; h += blockDim.x) {
     a.io[t * a.N + h] = soft_cap(a.zi[t * a.ldg + h] + a.ib[h], a.cap);
     a.fo[t * a.N + h] = -softplus(-soft_cap(a.zf[t * a.ldg + h] + a.fb[h], a.cap));
+    if (pl.req >= 0 && pl.first) {
+      const int slot = a.slots[pl.req];
+      a.m0[static_cast<long long>(pl.req) * a.N + h] =
+          a.positions[t] == 0 || slot < 0 || slot >= a.num_slots
+              ? 0.0f : a.scalar[static_cast<long long>(slot) * a.N + h];
+    }
   }
 }
 
@@ -231,7 +328,9 @@ struct ScanArgs {
   const float* g;            // delta: decays [T, N, DP]
   const float* v;            // [T, N, VP]
   const float *s0, *s1;      // delta: step sizes | memory: log input gate, log forget gate [T, N]
-  float* out;                // [T, N, V]
+  float* out;                // [T, N, V] (memory: not yet divided)
+  float *nq, *low;           // memory: [T, N] normaliser . q, exp(-m)
+  const float* m0;           // memory: [requests, N] m in front of the portion
   float* matrix;             // state, see the head of the file
   float* vector;
   float* scalar;
@@ -267,34 +366,44 @@ __device__ void keep_taps(const ScanArgs& a, const Portion& po, int slot, int h)
   }
 }
 
-template <int MODE, int RPL>
+template <int MODE, int DP>
 __host__ __device__ constexpr int stage_floats(int cols) {
-  return kChunk * ((MODE == kDelta ? 3 : 2) * 8 * RPL + cols + 4);
+  return kChunk * ((MODE == kDelta ? 3 : 2) * DP + cols + 4);
 }
 
-template <int MODE, int RPL, int CPT>
-__global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
-  constexpr int DP = 8 * RPL, P = RPL / 2;       // P: row pairs per lane
+template <int MODE, int LPC, int RPL, int CPT>
+__global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
+  constexpr int DP = LPC * RPL, P = RPL / 2;     // P: row pairs per lane
   constexpr int kRows = MODE == kDelta ? 3 : 2;  // staged rows of DP floats per token
+  constexpr int kGroups = 32 / LPC;              // columns groups of a warp
   extern __shared__ float4 smem4[];
   float* smem = reinterpret_cast<float*>(smem4);
-  const int stage = stage_floats<MODE, RPL>(a.cols);
+  const int stage = stage_floats<MODE, DP>(a.cols);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int l = lane & 7;
+  const int l = lane & (LPC - 1);
   const int r = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
   const int kvh = h / (a.N / a.G);
   const Portion po = portion_of(r, a.nd, a.cu_q);
   const int slot = a.slots[r];
-  const int c_loc = (warp * 4 + (lane >> 3)) * CPT;      // first column of this lane, in the CTA's block
+  const int c_loc = (warp * kGroups + lane / LPC) * CPT;   // first column of this lane in the block
   const int c0 = z * a.cols + c_loc;
-  if (slot < 0 || slot >= a.num_slots) {                 // padding of a captured batch
+  const int columns = MODE == kMemory ? a.V + 1 : a.V;     // the last one of a memory: normaliser
+  if (slot < 0 || slot >= a.num_slots) {                   // padding of a captured batch
     for (int i = 0; i < po.count; ++i)
       for (int c = threadIdx.x; c < a.cols; c += blockDim.x)
         if (z * a.cols + c < a.V)
           a.out[(static_cast<long long>(po.first + i) * a.N + h) * a.V + z * a.cols + c] = 0.0f;
+    if (MODE == kMemory && z == 0) {
+      for (int i = threadIdx.x; i < po.count; i += blockDim.x) {
+        const long long at = static_cast<long long>(po.first + i) * a.N + h;
+        a.nq[at] = 0.0f;
+        a.low[at] = 1.0f;
+      }
+    }
     return;
   }
   const bool fresh = a.positions[po.first] == 0;
+  const bool warp_on = z * a.cols + warp * kGroups * CPT < columns;    // a column for this warp
 
   // tokens [i0, i0 + kChunk) of the portion -> stage b
   auto fetch = [&](int i0, int b) {
@@ -332,33 +441,26 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
   fetch(0, 0);
   copy_commit();
 
-  // state -> registers: lane l holds rows 4 (l + 8 i) .. + 3 of its columns
-  uint64_t S[CPT][P], nv[MODE == kMemory ? P : 1];
-  float m = 0.0f;
+  // state -> registers: lane l holds rows 4 (l + LPC i) .. + 3 of its columns
+  uint64_t S[CPT][P];
   const long long head_at = static_cast<long long>(slot) * a.N + h;
+  auto column_state = [&](int c) {
+    return MODE == kMemory && c == a.V ? a.vector + head_at * DP
+                                       : a.matrix + (head_at * a.V + c) * DP;
+  };
 #pragma unroll
   for (int j = 0; j < CPT; ++j) {
-    const bool in = !fresh && c0 + j < a.V;
-    const float* src = a.matrix + (head_at * a.V + c0 + j) * DP + 4 * l;
+    const bool in = !fresh && c0 + j < columns;
+    const float* src = column_state(c0 + j) + 4 * l;
 #pragma unroll
     for (int i = 0; i < P / 2; ++i) {
       ulonglong2 u = make_ulonglong2(0, 0);
-      if (in) u = *reinterpret_cast<const ulonglong2*>(src + 32 * i);
+      if (in) u = *reinterpret_cast<const ulonglong2*>(src + 4 * LPC * i);
       S[j][2 * i] = u.x;
       S[j][2 * i + 1] = u.y;
     }
   }
-  if (MODE == kMemory) {
-#pragma unroll
-    for (int i = 0; i < P / 2; ++i) {
-      ulonglong2 u = make_ulonglong2(0, 0);
-      if (!fresh)
-        u = *reinterpret_cast<const ulonglong2*>(a.vector + head_at * DP + 4 * l + 32 * i);
-      nv[2 * i] = u.x;
-      nv[2 * i + 1] = u.y;
-    }
-    if (!fresh) m = a.scalar[head_at];
-  }
+  float m = MODE == kMemory ? a.m0[static_cast<long long>(r) * a.N + h] : 0.0f;
 
   for (int i0 = 0; i0 < po.count; i0 += kChunk) {
     const int b = (i0 / kChunk) & 1;
@@ -367,15 +469,15 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
     copy_wait<1>();
     __syncthreads();
     const int n = min(kChunk, po.count - i0);
-    const float* sq = smem + b * stage;
+    const float* sq = smem + b * stage + 4 * l;
     const float* sk = sq + kChunk * DP;
     const float* sg = sk + kChunk * DP;                         // delta only
-    const float* sv = sq + kRows * kChunk * DP;
+    const float* sv = smem + b * stage + kRows * kChunk * DP;
     const float* ss = sv + kChunk * a.cols;
 
     // matrix memory: running maximum and the two factors of every token of the chunk, lane t
     // computing token t's
-    float keep = 0.0f, add = 0.0f, floor_den = 0.0f;
+    float keep = 0.0f, add = 0.0f, low = 0.0f;
     if (MODE == kMemory) {
       float f = 0.0f, F = 0.0f, M = -INFINITY, ig = -INFINITY;
       if (lane < n) {
@@ -396,22 +498,23 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
       if (lane == 0) before = m;
       keep = expf(f + (before - mt));        // the difference of the maxima is (nearly) exact
       add = expf(ig - mt);
-      floor_den = expf(-mt);
+      low = expf(-mt);
       m = __shfl_sync(0xffffffffu, mt, n - 1);
     }
 
-    for (int i = 0; i < n; ++i) {
-      uint64_t kk[P], qq[P];
-#pragma unroll
-      for (int u = 0; u < P / 2; ++u) {
-        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(sk + i * DP + 4 * l + 32 * u);
-        const ulonglong2 y = *reinterpret_cast<const ulonglong2*>(sq + i * DP + 4 * l + 32 * u);
-        kk[2 * u] = x.x; kk[2 * u + 1] = x.y;
-        qq[2 * u] = y.x; qq[2 * u + 1] = y.y;
-      }
+    for (int i = 0; i < (warp_on ? n : 0); ++i) {
       float v[CPT], o[CPT];
 #pragma unroll
       for (int j = 0; j < CPT; ++j) v[j] = sv[i * a.cols + c_loc + j];
+      uint64_t kk[P];
+#pragma unroll
+      for (int u = 0; u < P / 2; ++u) {
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(sk + i * DP + 4 * LPC * u);
+        kk[2 * u] = x.x; kk[2 * u + 1] = x.y;
+      }
+      uint64_t e0[CPT], e1[CPT];
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) e0[j] = e1[j] = 0;
       if (MODE == kDelta) {
         const float beta = ss[i];
         uint64_t d0[CPT], d1[CPT];
@@ -419,7 +522,7 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
         for (int j = 0; j < CPT; ++j) d0[j] = d1[j] = 0;
 #pragma unroll
         for (int u = 0; u < P / 2; ++u) {
-          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(sg + i * DP + 4 * l + 32 * u);
+          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(sg + i * DP + 4 * LPC * u);
 #pragma unroll
           for (int j = 0; j < CPT; ++j) {
             S[j][2 * u] = mul2(S[j][2 * u], g.x);
@@ -428,146 +531,130 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
             d1[j] = fma2(S[j][2 * u + 1], kk[2 * u + 1], d1[j]);
           }
         }
+        uint64_t u2[CPT];
         float d[CPT];
 #pragma unroll
         for (int j = 0; j < CPT; ++j) d[j] = halves_sum(d0[j]) + halves_sum(d1[j]);
 #pragma unroll
-        for (int w = 1; w < 8; w <<= 1) {
+        for (int w = 1; w < LPC; w <<= 1) {
 #pragma unroll
           for (int j = 0; j < CPT; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], w);
         }
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) {
-          const uint64_t u2 = both(beta * (v[j] - d[j]));
-          uint64_t e0 = 0, e1 = 0;
+        for (int j = 0; j < CPT; ++j) u2[j] = both(beta * (v[j] - d[j]));
 #pragma unroll
-          for (int u = 0; u < P; u += 2) {
-            S[j][u] = fma2(kk[u], u2, S[j][u]);
-            S[j][u + 1] = fma2(kk[u + 1], u2, S[j][u + 1]);
-            e0 = fma2(S[j][u], qq[u], e0);
-            e1 = fma2(S[j][u + 1], qq[u + 1], e1);
+        for (int u = 0; u < P / 2; ++u) {
+          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(sq + i * DP + 4 * LPC * u);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            S[j][2 * u] = fma2(kk[2 * u], u2[j], S[j][2 * u]);
+            S[j][2 * u + 1] = fma2(kk[2 * u + 1], u2[j], S[j][2 * u + 1]);
+            e0[j] = fma2(S[j][2 * u], q.x, e0[j]);
+            e1[j] = fma2(S[j][2 * u + 1], q.y, e1[j]);
           }
-          o[j] = halves_sum(e0) + halves_sum(e1);
-        }
-#pragma unroll
-        for (int w = 1; w < 8; w <<= 1) {
-#pragma unroll
-          for (int j = 0; j < CPT; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
         }
       } else {
         const uint64_t a2 = both(__shfl_sync(0xffffffffu, keep, i));
-        const uint64_t b2 = both(__shfl_sync(0xffffffffu, add, i));
-        const float low = __shfl_sync(0xffffffffu, floor_den, i);
-        uint64_t e = 0;
+        const float b1 = __shfl_sync(0xffffffffu, add, i);
+        uint64_t v2[CPT];
 #pragma unroll
-        for (int u = 0; u < P; ++u) {
-          kk[u] = mul2(kk[u], b2);
-          nv[u] = fma2(nv[u], a2, kk[u]);
-          e = fma2(nv[u], qq[u], e);
-        }
-        float den = halves_sum(e);
+        for (int j = 0; j < CPT; ++j) v2[j] = both(b1 * v[j]);
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) {
-          const uint64_t v2 = both(v[j]);
-          uint64_t e0 = 0, e1 = 0;
+        for (int u = 0; u < P / 2; ++u) {
+          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(sq + i * DP + 4 * LPC * u);
 #pragma unroll
-          for (int u = 0; u < P; u += 2) {
-            S[j][u] = fma2(kk[u], v2, mul2(S[j][u], a2));
-            S[j][u + 1] = fma2(kk[u + 1], v2, mul2(S[j][u + 1], a2));
-            e0 = fma2(S[j][u], qq[u], e0);
-            e1 = fma2(S[j][u + 1], qq[u + 1], e1);
+          for (int j = 0; j < CPT; ++j) {
+            S[j][2 * u] = fma2(kk[2 * u], v2[j], mul2(S[j][2 * u], a2));
+            S[j][2 * u + 1] = fma2(kk[2 * u + 1], v2[j], mul2(S[j][2 * u + 1], a2));
+            e0[j] = fma2(S[j][2 * u], q.x, e0[j]);
+            e1[j] = fma2(S[j][2 * u + 1], q.y, e1[j]);
           }
-          o[j] = halves_sum(e0) + halves_sum(e1);
         }
-#pragma unroll
-        for (int w = 1; w < 8; w <<= 1) {
-          den += __shfl_xor_sync(0xffffffffu, den, w);
-#pragma unroll
-          for (int j = 0; j < CPT; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
-        }
-        den = fmaxf(fabsf(den), low) + 1e-6f;
-#pragma unroll
-        for (int j = 0; j < CPT; ++j) o[j] /= den;
       }
-      float* dst = a.out + (static_cast<long long>(po.first + i0 + i) * a.N + h) * a.V + c0;
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) o[j] = halves_sum(e0[j]) + halves_sum(e1[j]);
+#pragma unroll
+      for (int w = 1; w < LPC; w <<= 1) {
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
+      }
+      const long long at = static_cast<long long>(po.first + i0 + i) * a.N + h;
       if (l == 0) {
 #pragma unroll
-        for (int j = 0; j < CPT; ++j)
-          if (c0 + j < a.V) dst[j] = o[j];
+        for (int j = 0; j < CPT; ++j) {
+          if (c0 + j < a.V) a.out[at * a.V + c0 + j] = o[j];
+          else if (MODE == kMemory && c0 + j == a.V) a.nq[at] = o[j];
+        }
       }
     }
+    if (MODE == kMemory && z == 0 && warp == 0 && lane < n)
+      a.low[static_cast<long long>(po.first + i0 + lane) * a.N + h] = low;
     __syncthreads();           // stage b is refilled next
   }
 
   // registers -> state
 #pragma unroll
   for (int j = 0; j < CPT; ++j) {
-    if (c0 + j >= a.V) continue;
-    float* dst = a.matrix + (head_at * a.V + c0 + j) * DP + 4 * l;
+    if (c0 + j >= columns) continue;
+    float* dst = column_state(c0 + j) + 4 * l;
 #pragma unroll
     for (int i = 0; i < P / 2; ++i)
-      *reinterpret_cast<ulonglong2*>(dst + 32 * i) = make_ulonglong2(S[j][2 * i], S[j][2 * i + 1]);
+      *reinterpret_cast<ulonglong2*>(dst + 4 * LPC * i) =
+          make_ulonglong2(S[j][2 * i], S[j][2 * i + 1]);
   }
   if (MODE == kMemory) {
-    if (z == 0 && threadIdx.x < 8) {
-#pragma unroll
-      for (int i = 0; i < P / 2; ++i)
-        *reinterpret_cast<ulonglong2*>(a.vector + head_at * DP + 4 * l + 32 * i) =
-            make_ulonglong2(nv[2 * i], nv[2 * i + 1]);
-      if (threadIdx.x == 0) a.scalar[head_at] = m;
-    }
+    if (z == 0 && threadIdx.x == 0) a.scalar[head_at] = m;
   } else if (z == 0 && a.ntaps > 1) {
     if (a.elt == 2) keep_taps<uint16_t>(a, po, slot, h);
     else keep_taps<uint32_t>(a, po, slot, h);
   }
 }
 
-template <int MODE, int RPL, int CPT>
-static int launch_scan(const ScanArgs& a, int requests, cudaStream_t s) {
-  const int smem = 2 * stage_floats<MODE, RPL>(a.cols) * static_cast<int>(sizeof(float));
+template <int MODE, int LPC, int RPL, int CPT>
+static int launch_scan(ScanArgs& a, int requests, int warps, cudaStream_t s) {
+  constexpr int kPerWarp = 32 / LPC * CPT;
+  const int columns = MODE == kMemory ? a.V + 1 : a.V;
+  const int want = (columns + kPerWarp - 1) / kPerWarp;
+  if (warps > want) warps = want;
+  a.cols = warps * kPerWarp;
+  const int smem = 2 * stage_floats<MODE, LPC * RPL>(a.cols) * static_cast<int>(sizeof(float));
   static bool done[64] = {false};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -9;
   if (!done[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(recurrent_scan_kernel<MODE, RPL, CPT>,
+    cudaError_t e = cudaFuncSetAttribute(recurrent_scan_kernel<MODE, LPC, RPL, CPT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
     done[dev] = true;
   }
-  dim3 grid(requests, a.N, (a.V + a.cols - 1) / a.cols);
-  recurrent_scan_kernel<MODE, RPL, CPT><<<grid, a.cols / CPT * 8, smem, s>>>(a);
+  dim3 grid(requests, a.N, (columns + a.cols - 1) / a.cols);
+  recurrent_scan_kernel<MODE, LPC, RPL, CPT><<<grid, warps * 32, smem, s>>>(a);
   return static_cast<int>(cudaGetLastError());
 }
 
-// Columns per CTA: as many as leave two CTAs for every SM.
-static int scan_columns(int V, int ctas_per_block, int most) {
-  int cols = 16;
-  while (cols < most && cols < V) cols *= 2;
-  while (cols > 16 && static_cast<long long>(ctas_per_block) * ((V + cols - 1) / cols) <
-                          2ll * sm_count())
-    cols /= 2;
-  return cols;
-}
-
-template <int MODE, int RPL>
+// A warp of the wide form walks 32 (DP <= 128) or 16 columns, one of the narrow forms 8 or 4: the
+// widest form that gives every scheduler of the GPU a warp.
+template <int MODE, int DP>
 static int dispatch_scan(ScanArgs& a, int requests, cudaStream_t s) {
-  a.cols = scan_columns(a.V, requests * a.N, RPL > 16 ? 64 : 128);
-  if constexpr (RPL <= 16) {
-    if (a.cols >= 64) return launch_scan<MODE, RPL, 4>(a, requests, s);
-  }
-  if (a.cols >= 32) return launch_scan<MODE, RPL, 2>(a, requests, s);
-  return launch_scan<MODE, RPL, 1>(a, requests, s);
+  constexpr int kWide = DP <= 128 ? 2 : 4;
+  const long long heads = static_cast<long long>(requests) * a.N;
+  const long long schedulers = 4ll * sm_count();
+  const auto warps = [&](int per) { return heads * ((a.V + per - 1) / per); };
+  if (warps(64 / kWide) >= schedulers)
+    return launch_scan<MODE, kWide, DP / kWide, 2>(a, requests, 4, s);
+  if (warps(8) >= schedulers) return launch_scan<MODE, 8, DP / 8, 2>(a, requests, 4, s);
+  return launch_scan<MODE, 8, DP / 8, 1>(a, requests, 4, s);
 }
 
 template <int MODE>
 static int dispatch_scan(ScanArgs& a, int DP, int requests, cudaStream_t s) {
   switch (DP) {
-    case 32: return dispatch_scan<MODE, 4>(a, requests, s);
-    case 64: return dispatch_scan<MODE, 8>(a, requests, s);
-    case 96: return dispatch_scan<MODE, 12>(a, requests, s);
-    case 128: return dispatch_scan<MODE, 16>(a, requests, s);
-    case 192: return dispatch_scan<MODE, 24>(a, requests, s);
-    case 256: return dispatch_scan<MODE, 32>(a, requests, s);
+    case 32: return dispatch_scan<MODE, 32>(a, requests, s);
+    case 64: return dispatch_scan<MODE, 64>(a, requests, s);
+    case 96: return dispatch_scan<MODE, 96>(a, requests, s);
+    case 128: return dispatch_scan<MODE, 128>(a, requests, s);
+    case 192: return dispatch_scan<MODE, 192>(a, requests, s);
+    case 256: return dispatch_scan<MODE, 256>(a, requests, s);
   }
   return -20;
 }
@@ -575,6 +662,7 @@ static int dispatch_scan(ScanArgs& a, int DP, int requests, cudaStream_t s) {
 // ---------------------------------------------------------------------------
 struct HeadNormArgs {
   const float* o;            // [T, N, V]
+  const float *nq, *low;     // [T, N]: o is divided by max(|nq|, low) + 1e-6 first, or null
   const float* w;            // norm weight: [V] shared by the heads, or [N * V]
   const void* z;             // [T, N * V] gate projection, row pitch ldz
   void* out;                 // [T, N * V], row pitch ldo
@@ -583,7 +671,19 @@ struct HeadNormArgs {
   float eps, scale;
 };
 
-template <typename T>
+template <typename T, int W>
+__device__ __forceinline__ void store_t(T* p, const float (&f)[W]) {
+  if constexpr (W == 4 && sizeof(T) == 2) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+  } else if constexpr (W == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    p[0] = from_f32<T>(f[0]);
+  }
+}
+
+// One warp per row and head.
+template <typename T, int W>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs a) {
   const int lane = threadIdx.x & 31;
   const long long row = blockIdx.x * 8ll + (threadIdx.x >> 5);
@@ -591,14 +691,364 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs 
   const long long t = row / a.N;
   const int h = static_cast<int>(row - t * a.N);
   const float* o = a.o + row * a.V;
-  float ss = 0.0f;
-  for (int c = lane; c < a.V; c += 32) ss += o[c] * o[c];
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(a.V) + a.eps) * a.scale;
+  constexpr int kKeep = W == 4 ? 4 : 8;          // vectors per lane that stay in registers
+  float f[kKeep][W], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (lane + 32 * i) * W;
+    if (c >= a.V) continue;
+    load_n<float, W>(o + c, f[i]);
+#pragma unroll
+    for (int j = 0; j < W; ++j) ss += f[i][j] * f[i][j];
+  }
+  for (int c = (lane + 32 * kKeep) * W; c < a.V; c += 32 * W) {
+    float x[W];
+    load_n<float, W>(o + c, x);
+#pragma unroll
+    for (int j = 0; j < W; ++j) ss += x[j] * x[j];
+  }
+  const float den = a.nq != nullptr ? 1.0f / (fmaxf(fabsf(a.nq[row]), a.low[row]) + 1e-6f) : 1.0f;
+  const float inv =
+      den * (1.0f / sqrtf(warp_sum(ss) * den * den / static_cast<float>(a.V) + a.eps)) * a.scale;
   const float* w = a.w + (a.per_head ? h * a.V : 0);
   const T* z = static_cast<const T*>(a.z) + t * a.ldz + h * a.V;
   T* out = static_cast<T*>(a.out) + t * a.ldo + h * a.V;
-  for (int c = lane; c < a.V; c += 32)
-    out[c] = from_f32<T>(o[c] * inv * w[c] * sigmoid(to_f32<T>(z[c])));
+  auto put = [&](int c, float (&x)[W]) {
+    float g[W], b[W];
+    load_n<T, W>(z + c, g);
+    load_n<float, W>(w + c, b);
+#pragma unroll
+    for (int j = 0; j < W; ++j) x[j] = x[j] * inv * b[j] * sigmoid(g[j]);
+    store_t<T, W>(out + c, x);
+  };
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (lane + 32 * i) * W;
+    if (c < a.V) put(c, f[i]);
+  }
+  for (int c = (lane + 32 * kKeep) * W; c < a.V; c += 32 * W) {
+    float x[W];
+    load_n<float, W>(o + c, x);
+    put(c, x);
+  }
+}
+
+// ---------------------------------------------------------------------------
+// Requests that bring one token: everything between the wide projections and the output projection
+// in one CTA per (request, head), 256 threads.
+struct StepArgs {
+  const void* hrow;          // [nd, H] mixer input, row pitch ldh
+  const void* x[3];          // q, k, v projections, row pitch ld
+  const void* gate;          // memory: [nd, N V] gate projection, row pitch ld
+  const void *r1, *g1;       // delta: first steps of the decay / gate projections, row pitch ld
+  const void *r2, *g2;       // delta: second steps [N D, R], [N V, RG]
+  const void *w0, *w1;       // rows [N, H]: delta step size, - ; memory input gate, forget gate
+  const float *b0, *b1;      // memory: their biases [N]
+  const float* taps_w[3];    // delta: convolution weights
+  const float *dt_bias, *a_log;
+  const float* norm;         // [V], or [N V] with per_head
+  void* taps;
+  float *matrix, *vector, *scalar;
+  void* out;                 // [nd, N V], row pitch ldo
+  const long long* positions;
+  const int* slots;
+  long long ldh, ld, ldo;
+  int H, G, N, D, V, R, RG, ntaps, num_slots, per_head;
+  float cap, qscale, eps, scale;
+};
+
+// 8 elements as floats (16-byte aligned)
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&f)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    vec8_load<T>(p, f);
+  } else {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    const float4 b = *reinterpret_cast<const float4*>(p + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  }
+}
+
+// This thread's share of x . w over n elements (vec: both 16-byte aligned and n a multiple of 8).
+template <typename T>
+__device__ __forceinline__ float dot_share(const T* x, const T* w, int n, bool vec) {
+  float s = 0.0f;
+  if (vec) {
+    for (int c = threadIdx.x * 8; c < n; c += blockDim.x * 8) {
+      float f[8], g[8];
+      load8<T>(x + c, f);
+      load8<T>(w + c, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s += f[i] * g[i];
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += blockDim.x) s += to_f32<T>(x[c]) * to_f32<T>(w[c]);
+  }
+  return s;
+}
+
+// Four lanes: row . x for x of n (multiple of 8) floats in shared memory.
+template <typename T>
+__device__ __forceinline__ float quad_dot(const T* row, const float* x, int n, int q) {
+  float s = 0.0f;
+  for (int c = q * 8; c < n; c += 32) {
+    float f[8];
+    load8<T>(row + c, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) s += f[i] * x[c + i];
+  }
+  s += __shfl_xor_sync(0xffffffffu, s, 1);
+  s += __shfl_xor_sync(0xffffffffu, s, 2);
+  return s;
+}
+
+__host__ __device__ inline int step_floats(int DP, int V, int R, int RG) {
+  return 3 * DP + 3 * ((V + 3) / 4 * 4) + R + RG + 64;
+}
+
+template <typename T, int MODE, int RPL, int CPT>
+__global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(const StepArgs a) {
+  constexpr int DP = 8 * RPL, P = RPL / 2;
+  constexpr int kCols = 8 * 4 * CPT;              // columns per pass
+  extern __shared__ float4 smem4[];
+  float* sq = reinterpret_cast<float*>(smem4);    // [DP]
+  float* sk = sq + DP;                            // [DP]
+  float* sg = sk + DP;                            // [DP] decays (delta), normaliser products (memory)
+  const int VS = (a.V + 3) / 4 * 4;
+  float* sv = sg + DP;                            // [V]
+  float* so = sv + VS;                            // [V]
+  float* sz = so + VS;                            // [V] output gate
+  float* s1 = sz + VS;                            // [R] [RG]
+  float* red = s1 + a.R + a.RG;                   // [64]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & 7;
+  const int r = blockIdx.x, h = blockIdx.y;
+  const int kvh = h / (a.N / a.G);
+  T* out = static_cast<T*>(a.out) + static_cast<long long>(r) * a.ldo + h * a.V;
+  const int slot = a.slots[r];
+  if (slot < 0 || slot >= a.num_slots) {          // padding of a captured batch
+    for (int c = tid; c < a.V; c += blockDim.x) out[c] = from_f32<T>(0.0f);
+    return;
+  }
+  const long long pos = a.positions[r];
+  const bool fresh = pos == 0;
+  const long long head_at = static_cast<long long>(slot) * a.N + h;
+  const int c_warp = (warp * 4 + (lane >> 3)) * CPT;
+
+  uint64_t S[CPT][P];
+  auto load_state = [&](int base) {
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      const int c = base + c_warp + j;
+      const bool in = !fresh && c < a.V;
+      const float* src = a.matrix + (head_at * a.V + c) * DP + 4 * l;
+#pragma unroll
+      for (int i = 0; i < P / 2; ++i) {
+        ulonglong2 u = make_ulonglong2(0, 0);
+        if (in) u = *reinterpret_cast<const ulonglong2*>(src + 32 * i);
+        S[j][2 * i] = u.x;
+        S[j][2 * i + 1] = u.y;
+      }
+    }
+  };
+  load_state(0);                                  // in flight while the inputs are computed
+
+  const T* hr = static_cast<const T*>(a.hrow) + static_cast<long long>(r) * a.ldh;
+  const bool vec = (a.H % 8) == 0 && ((reinterpret_cast<uintptr_t>(hr) |
+                                       reinterpret_cast<uintptr_t>(a.w0) |
+                                       reinterpret_cast<uintptr_t>(a.w1)) & 15) == 0;
+  const long long xrow = static_cast<long long>(r) * a.ld;
+  const float d0 = dot_share<T>(hr, static_cast<const T*>(a.w0) + static_cast<long long>(h) * a.H,
+                                a.H, vec);
+  float d1 = 0.0f;
+  if (MODE == kMemory)
+    d1 = dot_share<T>(hr, static_cast<const T*>(a.w1) + static_cast<long long>(h) * a.H, a.H, vec);
+
+  if (MODE == kDelta) {
+    const int C = 2 * a.G * a.D + a.N * a.V;
+    T* ring = static_cast<T*>(a.taps) + static_cast<long long>(slot) * a.ntaps * C;
+    for (int e = tid; e < 2 * DP + a.V; e += blockDim.x) {
+      const int which = e < DP ? 0 : e < 2 * DP ? 1 : 2;
+      const int d = which == 0 ? e : which == 1 ? e - DP : e - 2 * DP;
+      const int head = which == 2 ? h : kvh, dim = which == 2 ? a.V : a.D;
+      float f = 0.0f;
+      if (d < dim) {
+        const int ch = head * dim + d;
+        const int at = ch + (which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D);
+        const float* w = a.taps_w[which] + static_cast<long long>(ch) * a.ntaps;
+        const T now = static_cast<const T*>(a.x[which])[xrow + ch];
+        float s = w[a.ntaps - 1] * to_f32<T>(now);
+        for (int o = 1; o < a.ntaps; ++o)
+          if (pos - o >= 0)
+            s += w[a.ntaps - 1 - o] * to_f32<T>(ring[(pos - o) % a.ntaps * C + at]);
+        f = silu<T>(s);
+        if (a.ntaps > 1 && (which == 2 || h % (a.N / a.G) == 0)) ring[pos % a.ntaps * C + at] = now;
+      }
+      (which == 0 ? sq : which == 1 ? sk : sv)[d] = f;
+    }
+    for (int e = tid; e < a.R; e += blockDim.x) s1[e] = to_f32<T>(static_cast<const T*>(a.r1)[xrow + e]);
+    for (int e = tid; e < a.RG; e += blockDim.x)
+      s1[a.R + e] = to_f32<T>(static_cast<const T*>(a.g1)[xrow + e]);
+  } else {
+    for (int d = tid; d < DP; d += blockDim.x) {
+      const bool in = d < a.D;
+      sq[d] = in ? to_f32<T>(static_cast<const T*>(a.x[0])[xrow + h * a.D + d]) * a.qscale : 0.0f;
+      sk[d] = in ? to_f32<T>(static_cast<const T*>(a.x[1])[xrow + h * a.D + d]) : 0.0f;
+    }
+    for (int c = tid; c < a.V; c += blockDim.x) {
+      sv[c] = to_f32<T>(static_cast<const T*>(a.x[2])[xrow + h * a.V + c]);
+      sz[c] = sigmoid(to_f32<T>(static_cast<const T*>(a.gate)[xrow + h * a.V + c]));
+    }
+  }
+  const float z0 = block_sum(d0, red);            // (synchronises: the shared rows are complete)
+  const float z1 = MODE == kMemory ? block_sum(d1, red) : 0.0f;
+
+  float beta = 0.0f, keep = 0.0f, add = 0.0f, den = 1.0f;
+  if (MODE == kDelta) {
+    beta = sigmoid(z0);
+    // unit vectors (warps 0 and 1), then decays and the output gate, four lanes per row
+    if (warp < 2) {
+      float* x = warp == 0 ? sq : sk;
+      float ss = 0.0f;
+      for (int d = lane; d < DP; d += 32) ss += x[d] * x[d];
+      float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
+      if (warp == 0) inv *= 1.0f / sqrtf(static_cast<float>(a.D));
+      for (int d = lane; d < DP; d += 32) x[d] *= inv;
+    }
+    const float rate = expf(a.a_log[h]);
+    const int rows = DP + a.V, quad = lane >> 2;
+    for (int e0 = warp * 8; e0 < rows; e0 += 64) {
+      const int e = e0 + quad;
+      const bool decay = e < DP;
+      const int d = decay ? e : e - DP;
+      const bool in = decay ? d < a.D : e < rows;
+      // rows outside read row 0 of the head, so that all four lanes take part in the sum
+      const T* row = decay ? static_cast<const T*>(a.r2) +
+                                 (static_cast<long long>(h) * a.D + (in ? d : 0)) * a.R
+                           : static_cast<const T*>(a.g2) +
+                                 (static_cast<long long>(h) * a.V + (in ? d : 0)) * a.RG;
+      const float s = quad_dot<T>(row, decay ? s1 : s1 + a.R, decay ? a.R : a.RG, lane & 3);
+      if ((lane & 3) == 0) {
+        if (decay) sg[d] = in ? expf(-rate * softplus(s + a.dt_bias[h * a.D + d])) : 0.0f;
+        else if (in) sz[d] = sigmoid(to_f32<T>(from_f32<T>(s)));
+      }
+    }
+    __syncthreads();
+  } else {
+    const float li = soft_cap(z0 + a.b0[h], a.cap);
+    const float lf = -softplus(-soft_cap(z1 + a.b1[h], a.cap));
+    const float m = fresh ? 0.0f : a.scalar[head_at];
+    const float mt = fmaxf(lf + m, li);
+    keep = expf(lf + (m - mt));
+    add = expf(li - mt);
+    float part = 0.0f;
+    for (int d = tid; d < DP; d += blockDim.x) {
+      float* n = a.vector + head_at * DP + d;
+      const float v = (fresh ? 0.0f : keep * *n) + add * sk[d];
+      *n = v;
+      part += v * sq[d];
+    }
+    den = 1.0f / (fmaxf(fabsf(block_sum(part, red)), expf(-mt)) + 1e-6f);
+    if (tid == 0) a.scalar[head_at] = mt;         // every thread has read m (block_sum)
+  }
+
+  float ss = 0.0f;
+  for (int base = 0; base < a.V; base += kCols) {
+    if (base > 0) load_state(base);
+    const int c0 = base + c_warp;
+    float v[CPT], o[CPT], d[CPT];
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      v[j] = c0 + j < a.V ? sv[c0 + j] : 0.0f;
+      uint64_t e0 = 0, e1 = 0;
+      if (MODE == kDelta) {
+#pragma unroll
+        for (int u = 0; u < P / 2; ++u) {
+          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(sg + 4 * l + 32 * u);
+          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(sk + 4 * l + 32 * u);
+          S[j][2 * u] = mul2(S[j][2 * u], g.x);
+          S[j][2 * u + 1] = mul2(S[j][2 * u + 1], g.y);
+          e0 = fma2(S[j][2 * u], k.x, e0);
+          e1 = fma2(S[j][2 * u + 1], k.y, e1);
+        }
+      }
+      d[j] = halves_sum(e0) + halves_sum(e1);
+    }
+    if (MODE == kDelta) {
+#pragma unroll
+      for (int w = 1; w < 8; w <<= 1) {
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], w);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      const uint64_t u2 = both(MODE == kDelta ? beta * (v[j] - d[j]) : add * v[j]);
+      const uint64_t a2 = both(keep);
+      uint64_t e0 = 0, e1 = 0;
+#pragma unroll
+      for (int u = 0; u < P / 2; ++u) {
+        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(sk + 4 * l + 32 * u);
+        const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(sq + 4 * l + 32 * u);
+        if (MODE == kMemory) {
+          S[j][2 * u] = mul2(S[j][2 * u], a2);
+          S[j][2 * u + 1] = mul2(S[j][2 * u + 1], a2);
+        }
+        S[j][2 * u] = fma2(k.x, u2, S[j][2 * u]);
+        S[j][2 * u + 1] = fma2(k.y, u2, S[j][2 * u + 1]);
+        e0 = fma2(S[j][2 * u], q.x, e0);
+        e1 = fma2(S[j][2 * u + 1], q.y, e1);
+      }
+      o[j] = halves_sum(e0) + halves_sum(e1);
+      if (c0 + j < a.V) {
+        float* dst = a.matrix + (head_at * a.V + c0 + j) * DP + 4 * l;
+#pragma unroll
+        for (int i = 0; i < P / 2; ++i)
+          *reinterpret_cast<ulonglong2*>(dst + 32 * i) =
+              make_ulonglong2(S[j][2 * i], S[j][2 * i + 1]);
+      }
+    }
+#pragma unroll
+    for (int w = 1; w < 8; w <<= 1) {
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
+    }
+    if (l == 0) {
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) {
+        if (c0 + j >= a.V) continue;
+        o[j] *= den;
+        so[c0 + j] = o[j];
+        ss += o[j] * o[j];
+      }
+    }
+  }
+  ss = block_sum(ss, red);                        // (synchronises: so is complete)
+  const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.V) + a.eps) * a.scale;
+  const float* nw = a.norm + (a.per_head ? h * a.V : 0);
+  for (int c = tid; c < a.V; c += blockDim.x)
+    out[c] = from_f32<T>(so[c] * inv * nw[c] * sz[c]);
+}
+
+template <typename T, int MODE, int RPL, int CPT>
+static int launch_step(const StepArgs& a, int requests, cudaStream_t s) {
+  const int smem = step_floats(8 * RPL, a.V, a.R, a.RG) * static_cast<int>(sizeof(float));
+  if (smem > 48 * 1024) return -20;
+  recurrent_step_kernel<T, MODE, RPL, CPT><<<dim3(requests, a.N), 256, smem, s>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int MODE>
+static int dispatch_step(const StepArgs& a, int DP, int requests, cudaStream_t s) {
+  switch (DP) {
+    case 32: return launch_step<T, MODE, 4, 4>(a, requests, s);
+    case 64: return launch_step<T, MODE, 8, 4>(a, requests, s);
+    case 96: return launch_step<T, MODE, 12, 4>(a, requests, s);
+    case 128: return launch_step<T, MODE, 16, 4>(a, requests, s);
+    case 192: return launch_step<T, MODE, 24, 2>(a, requests, s);
+    case 256: return launch_step<T, MODE, 32, 2>(a, requests, s);
+  }
+  return -20;
 }
 
 }  // namespace recurrent
@@ -636,27 +1086,57 @@ B200_API int b200_delta_inputs(const void* xq, const void* xk, const void* xv, l
   a.ld = ld; a.ldz = ldz; a.ldb = ldb; a.T = T; a.G = G; a.N = N; a.D = D; a.V = V; a.DP = DP;
   a.VP = VP; a.ntaps = ntaps; a.num_slots = num_slots; a.nd = nd; a.np = np;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  dim3 grid(T, (G + N + 7) / 8);
-  if (dtype == 0) delta_inputs_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(a);
-  else delta_inputs_kernel<float><<<grid, 256, 0, s>>>(a);
+  const dim3 grid((T + kStrip - 1) / kStrip, (2 * G + 2 * N + 7) / 8);
+  const uintptr_t x = reinterpret_cast<uintptr_t>(xq) | reinterpret_cast<uintptr_t>(xk) |
+                      reinterpret_cast<uintptr_t>(xv) | reinterpret_cast<uintptr_t>(taps);
+  const bool v4 = (D % 4) == 0 && (V % 4) == 0 && (VP % 4) == 0 && (ld % 4) == 0 &&
+                  (ldz % 4) == 0 && (x % (dtype == 0 ? 8 : 16)) == 0 &&
+                  (reinterpret_cast<uintptr_t>(z) % 16) == 0;
+#define B200_IN(NT, W)                                                             \
+  do {                                                                             \
+    if (dtype == 0) delta_inputs_kernel<__nv_bfloat16, NT, W><<<grid, 256, 0, s>>>(a); \
+    else delta_inputs_kernel<float, NT, W><<<grid, 256, 0, s>>>(a);                 \
+  } while (0)
+  if (ntaps <= 4) {
+    if (v4) B200_IN(4, 4);
+    else B200_IN(4, 1);
+  } else {
+    if (v4) B200_IN(8, 4);
+    else B200_IN(8, 1);
+  }
+#undef B200_IN
   return static_cast<int>(cudaGetLastError());
 }
 
-// fp32 inputs and log gates of the matrix memory.  dtype (of q, k, v): 0 bf16, 2 fp32.
+// fp32 inputs and log gates of the matrix memory; VP > V (column V of vo is the normaliser's 1).
+// dtype (of q, k, v): 0 bf16, 2 fp32.
 B200_API int b200_memory_inputs(const void* q, const void* k, const void* v, long long ld,
                                 const float* zi, const float* zf, long long ldg, const float* ib,
-                                const float* fb, float cap, float qscale, float* qo, float* ko, float* vo,
-                                float* io, float* fo, int T, int N, int D, int V, int DP, int VP,
-                                int dtype, void* stream) {
+                                const float* fb, const float* scalar, float cap, float qscale,
+                                float* qo, float* ko, float* vo, float* io, float* fo, float* m0,
+                                const long long* positions, const int* slots, int num_slots,
+                                const int* cu_q, int T, int N, int D, int V, int DP, int VP,
+                                int nd, int np, int dtype, void* stream) {
   if (T <= 0) return 0;
-  if (N <= 0 || D <= 0 || D > DP || V <= 0 || V > VP || (dtype != 0 && dtype != 2)) return -2;
+  if (N <= 0 || D <= 0 || D > DP || V <= 0 || V >= VP || (dtype != 0 && dtype != 2)) return -2;
   MemoryIn a;
-  a.q = q; a.k = k; a.v = v; a.zi = zi; a.zf = zf; a.ib = ib; a.fb = fb; a.qo = qo; a.ko = ko; a.vo = vo;
-  a.io = io; a.fo = fo; a.ld = ld; a.ldg = ldg; a.T = T; a.N = N; a.D = D; a.V = V; a.DP = DP;
-  a.VP = VP; a.cap = cap; a.qscale = qscale;
+  a.q = q; a.k = k; a.v = v; a.zi = zi; a.zf = zf; a.ib = ib; a.fb = fb; a.scalar = scalar;
+  a.qo = qo; a.ko = ko; a.vo = vo; a.io = io; a.fo = fo; a.m0 = m0; a.positions = positions;
+  a.slots = slots; a.cu_q = cu_q; a.ld = ld; a.ldg = ldg; a.T = T; a.N = N; a.D = D; a.V = V;
+  a.DP = DP; a.VP = VP; a.num_slots = num_slots; a.nd = nd; a.np = np; a.cap = cap;
+  a.qscale = qscale;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == 0) memory_inputs_kernel<__nv_bfloat16><<<T, 256, 0, s>>>(a);
-  else memory_inputs_kernel<float><<<T, 256, 0, s>>>(a);
+  const uintptr_t x = reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) |
+                      reinterpret_cast<uintptr_t>(v);
+  const bool v4 = (D % 4) == 0 && (V % 4) == 0 && (VP % 4) == 0 && (ld % 4) == 0 &&
+                  (x % (dtype == 0 ? 8 : 16)) == 0;
+  if (dtype == 0) {
+    if (v4) memory_inputs_kernel<__nv_bfloat16, 4><<<T, 256, 0, s>>>(a);
+    else memory_inputs_kernel<__nv_bfloat16, 1><<<T, 256, 0, s>>>(a);
+  } else {
+    if (v4) memory_inputs_kernel<float, 4><<<T, 256, 0, s>>>(a);
+    else memory_inputs_kernel<float, 1><<<T, 256, 0, s>>>(a);
+  }
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -678,35 +1158,99 @@ B200_API int b200_delta_scan(const float* q, const float* k, const float* g, con
   return dispatch_scan<kDelta>(a, DP, nd + np, static_cast<cudaStream_t>(stream));
 }
 
-// Matrix memory over the portions of a step; the state is (matrix, vector n, scalar m).
+// Matrix memory over the portions of a step; the state is (matrix, vector n, scalar m).  `out` is
+// the undivided read-out, nq and low what b200_head_norm_gate divides it by.
 B200_API int b200_memory_scan(const float* q, const float* k, const float* v, const float* li,
-                              const float* lf, float* out, float* matrix, float* vector,
-                              float* scalar, const long long* positions, const int* slots,
-                              int num_slots, const int* cu_q, int N, int D, int V, int DP, int VP,
-                              int nd, int np, void* stream) {
+                              const float* lf, const float* m0, float* out, float* nq, float* low,
+                              float* matrix, float* vector, float* scalar,
+                              const long long* positions, const int* slots, int num_slots,
+                              const int* cu_q, int N, int D, int V, int DP, int VP, int nd, int np,
+                              void* stream) {
   if (nd + np <= 0) return 0;
-  if (N <= 0 || (VP % 4) != 0) return -2;
+  if (N <= 0 || (VP % 4) != 0 || VP <= V) return -2;
   ScanArgs a{};
-  a.q = q; a.k = k; a.v = v; a.s0 = li; a.s1 = lf; a.out = out; a.matrix = matrix;
-  a.vector = vector; a.scalar = scalar; a.positions = positions; a.slots = slots;
-  a.num_slots = num_slots; a.cu_q = cu_q; a.G = N; a.N = N; a.D = D; a.V = V; a.VP = VP; a.nd = nd;
-  a.np = np; a.ntaps = 1;
+  a.q = q; a.k = k; a.v = v; a.s0 = li; a.s1 = lf; a.m0 = m0; a.out = out; a.nq = nq; a.low = low;
+  a.matrix = matrix; a.vector = vector; a.scalar = scalar; a.positions = positions;
+  a.slots = slots; a.num_slots = num_slots; a.cu_q = cu_q; a.G = N; a.N = N; a.D = D; a.V = V;
+  a.VP = VP; a.nd = nd; a.np = np; a.ntaps = 1;
   return dispatch_scan<kMemory>(a, DP, nd + np, static_cast<cudaStream_t>(stream));
 }
 
-// out = o / rms(o) per head * w * sigmoid(z) * scale.  per_head: w is [N * V], else [V].  dtype (of
-// z and out): 0 bf16, 2 fp32.
-B200_API int b200_head_norm_gate(const float* o, const float* w, int per_head, const void* z,
-                                 long long ldz, void* out, long long ldo, float eps, float scale,
-                                 int T, int N, int V, int dtype, void* stream) {
+// out = o' / rms(o') per head * w * sigmoid(z) * scale with o' = o, or with nq and low
+// o / (max(|nq|, low) + 1e-6).  per_head: w is [N * V], else [V].  dtype (of z and out): 0 bf16,
+// 2 fp32.
+B200_API int b200_head_norm_gate(const float* o, const float* nq, const float* low, const float* w,
+                                 int per_head, const void* z, long long ldz, void* out,
+                                 long long ldo, float eps, float scale, int T, int N, int V,
+                                 int dtype, void* stream) {
   if (T <= 0) return 0;
   if (N <= 0 || V <= 0 || (dtype != 0 && dtype != 2)) return -2;
   HeadNormArgs a;
-  a.o = o; a.w = w; a.z = z; a.out = out; a.ldz = ldz; a.ldo = ldo; a.T = T; a.N = N; a.V = V;
-  a.per_head = per_head; a.eps = eps; a.scale = scale;
+  a.o = o; a.nq = nq; a.low = low; a.w = w; a.z = z; a.out = out; a.ldz = ldz; a.ldo = ldo;
+  a.T = T; a.N = N; a.V = V; a.per_head = per_head; a.eps = eps; a.scale = scale;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const long long blocks = (static_cast<long long>(T) * N + 7) / 8;
-  if (dtype == 0) head_norm_gate_kernel<__nv_bfloat16><<<static_cast<int>(blocks), 256, 0, s>>>(a);
-  else head_norm_gate_kernel<float><<<static_cast<int>(blocks), 256, 0, s>>>(a);
+  const int blocks = static_cast<int>((static_cast<long long>(T) * N + 7) / 8);
+  const uintptr_t lo = reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out);
+  const uintptr_t hi = reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w);
+  const bool v4 = (V % 4) == 0 && (ldz % 4) == 0 && (ldo % 4) == 0 && (hi % 16) == 0 &&
+                  (lo % (dtype == 0 ? 8 : 16)) == 0;
+  if (dtype == 0) {
+    if (v4) head_norm_gate_kernel<__nv_bfloat16, 4><<<blocks, 256, 0, s>>>(a);
+    else head_norm_gate_kernel<__nv_bfloat16, 1><<<blocks, 256, 0, s>>>(a);
+  } else {
+    if (v4) head_norm_gate_kernel<float, 4><<<blocks, 256, 0, s>>>(a);
+    else head_norm_gate_kernel<float, 1><<<blocks, 256, 0, s>>>(a);
+  }
   return static_cast<int>(cudaGetLastError());
+}
+
+// One token of `nd` requests through the gated delta rule, from the wide projections to the gated
+// output: r1 / g1 (views of the same rows as q, k, v, R and RG columns, multiples of 8) are the
+// first steps of the decay and gate projections, r2 [N D, R] and g2 [N V, RG] the second ones,
+// wb [N, H] the step size's.  dtype: 0 bf16, 2 fp32.  -20: not covered (very wide second steps).
+B200_API int b200_delta_step(const void* h, long long ldh, int H, const void* xq, const void* xk,
+                             const void* xv, const void* r1, const void* g1, long long ld,
+                             const void* r2, int R, const void* g2, int RG, const void* wb,
+                             const float* wq, const float* wk, const float* wv, int ntaps,
+                             const float* dt_bias, const float* a_log, const float* norm,
+                             void* taps, float* matrix, const long long* positions,
+                             const int* slots, int num_slots, void* out, long long ldo, float eps,
+                             float scale, int nd, int G, int N, int D, int V, int DP, int dtype,
+                             void* stream) {
+  if (nd <= 0) return 0;
+  if (G <= 0 || N <= 0 || N % G != 0 || D <= 0 || D > DP || V <= 0 || H <= 0 || (R % 8) != 0 ||
+      (RG % 8) != 0 || ntaps < 1 || (dtype != 0 && dtype != 2))
+    return -2;
+  StepArgs a{};
+  a.hrow = h; a.ldh = ldh; a.H = H; a.x[0] = xq; a.x[1] = xk; a.x[2] = xv; a.r1 = r1; a.g1 = g1;
+  a.ld = ld; a.r2 = r2; a.R = R; a.g2 = g2; a.RG = RG; a.w0 = wb; a.taps_w[0] = wq;
+  a.taps_w[1] = wk; a.taps_w[2] = wv; a.ntaps = ntaps; a.dt_bias = dt_bias; a.a_log = a_log;
+  a.norm = norm; a.taps = taps; a.matrix = matrix; a.positions = positions; a.slots = slots;
+  a.num_slots = num_slots; a.out = out; a.ldo = ldo; a.eps = eps; a.scale = scale; a.G = G;
+  a.N = N; a.D = D; a.V = V;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return dtype == 0 ? dispatch_step<__nv_bfloat16, kDelta>(a, DP, nd, s)
+                    : dispatch_step<float, kDelta>(a, DP, nd, s);
+}
+
+// The same for the matrix memory: wi, wf [N, H] are the gates' projections, `gate` (a view of the
+// same rows as q, k, v) the output gate's result.
+B200_API int b200_memory_step(const void* h, long long ldh, int H, const void* xq, const void* xk,
+                              const void* xv, const void* gate, long long ld, const void* wi,
+                              const void* wf, const float* ib, const float* fb, float cap,
+                              float qscale, const float* norm, float* matrix, float* vector,
+                              float* scalar, const long long* positions, const int* slots,
+                              int num_slots, void* out, long long ldo, float eps, float scale,
+                              int nd, int N, int D, int V, int DP, int dtype, void* stream) {
+  if (nd <= 0) return 0;
+  if (N <= 0 || D <= 0 || D > DP || V <= 0 || H <= 0 || (dtype != 0 && dtype != 2)) return -2;
+  StepArgs a{};
+  a.hrow = h; a.ldh = ldh; a.H = H; a.x[0] = xq; a.x[1] = xk; a.x[2] = xv; a.gate = gate;
+  a.ld = ld; a.w0 = wi; a.w1 = wf; a.b0 = ib; a.b1 = fb; a.cap = cap; a.qscale = qscale;
+  a.norm = norm; a.per_head = 1; a.matrix = matrix; a.vector = vector; a.scalar = scalar;
+  a.positions = positions; a.slots = slots; a.num_slots = num_slots; a.out = out; a.ldo = ldo;
+  a.eps = eps; a.scale = scale; a.G = N; a.N = N; a.D = D; a.V = V;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return dtype == 0 ? dispatch_step<__nv_bfloat16, kMemory>(a, DP, nd, s)
+                    : dispatch_step<float, kMemory>(a, DP, nd, s);
 }

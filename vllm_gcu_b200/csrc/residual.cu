@@ -352,15 +352,13 @@ __global__ void __launch_bounds__(512) add_normed_kernel(const AddNormArgs a) {
 
 // out[t, h * D + c] = o[t, h * DC + c] * sigmoid(z[t, h * D + c]) * scale
 template <typename T, int V>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(512)
     head_gate_kernel(const T* o, int DC, const T* z, long long ldz, float scale, T* out,
-                     long long ldout, long long rows, int N, int D) {
+                     long long ldout, int N, int D) {
+  const long long t = blockIdx.x;
   const int nv = N * D / V;
-  const long long n = rows * nv;
-  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
-       i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long t = i / nv;
-    const int e = static_cast<int>(i - t * nv) * V;
+  for (int i = threadIdx.x; i < nv; i += blockDim.x) {
+    const int e = i * V;
     const int h = e / D, c = e - h * D;
     float a[V], g[V];
     ldv<V>(o + (t * N + h) * DC + c, a);
@@ -568,24 +566,20 @@ B200_API int b200_head_gate(const void* o, int DC, const void* z, long long ldz,
                   aligned(out, dtype == 0 ? 8 : 16);
   const bool v8 = dtype == 0 && v4 && (D % 8) == 0 && (DC % 8) == 0 && (ldz % 8) == 0 &&
                   (ldout % 8) == 0 && aligned(z, 16) && aligned(out, 16);
-  const long long items = static_cast<long long>(T) * N * D / (v8 ? 8 : v4 ? 4 : 1);
-  long long blocks = (items + 255) / 256;
-  const long long cap = static_cast<long long>(sm_count()) * 16;
-  if (blocks > cap) blocks = cap;
-  const int g = static_cast<int>(blocks);
+  const int th = row_threads(N * D, v8 ? 8 : v4 ? 4 : 1, 512);
   if (dtype == 0) {
     const __nv_bfloat16* po = static_cast<const __nv_bfloat16*>(o);
     const __nv_bfloat16* pz = static_cast<const __nv_bfloat16*>(z);
     __nv_bfloat16* pq = static_cast<__nv_bfloat16*>(out);
-    if (v8) head_gate_kernel<__nv_bfloat16, 8><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
-    else if (v4) head_gate_kernel<__nv_bfloat16, 4><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
-    else head_gate_kernel<__nv_bfloat16, 1><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
+    if (v8) head_gate_kernel<__nv_bfloat16, 8><<<T, th, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, N, D);
+    else if (v4) head_gate_kernel<__nv_bfloat16, 4><<<T, th, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, N, D);
+    else head_gate_kernel<__nv_bfloat16, 1><<<T, th, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, N, D);
   } else {
     const float* po = static_cast<const float*>(o);
     const float* pz = static_cast<const float*>(z);
     float* pq = static_cast<float*>(out);
-    if (v4) head_gate_kernel<float, 4><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
-    else head_gate_kernel<float, 1><<<g, 256, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, T, N, D);
+    if (v4) head_gate_kernel<float, 4><<<T, th, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, N, D);
+    else head_gate_kernel<float, 1><<<T, th, 0, s>>>(po, DC, pz, ldz, scale, pq, ldout, N, D);
   }
   return static_cast<int>(cudaGetLastError());
 }

@@ -100,7 +100,7 @@ class KeyAttention(MixerPart):
                 C.any_attention(q[nd:], kc, vc, bt, sl, 0, md.cu_q_prefill, out=out[nd:], **rest)
         return out
 
-    def mix(self, y, f, md: AttentionMetadata, cache: Optional[torch.Tensor],
+    def mix(self, h, y, f, fw, md: AttentionMetadata, cache: Optional[torch.Tensor],
             state: Optional[dict], scale: float, out: torch.Tensor) -> None:
         D = self.spec.head_dim
         if cache is None or md.is_dummy:

@@ -4,7 +4,8 @@ A part (key attention, matrix memory, gated delta rule) names the projections it
 ``MixerBlock`` stacks those of all its parts into one GEMM, hands every part its views, and lets
 the parts write their gated results side by side into one buffer that a single output GEMM sums.
 A part's factor in the sum is applied when it writes, in 32-bit.  Projections whose results enter
-a recurrence's gates unrounded come from a second, narrow GEMM with fp32 results.
+a recurrence's gates unrounded come from a second, narrow GEMM with fp32 results; single tokens on
+the GPU do without it (the parts' fused kernels take its weights).
 """
 from __future__ import annotations
 
@@ -61,11 +62,19 @@ class MixerPart(nn.Module):
         """Names that :meth:`load` takes."""
         return set()
 
-    def mix(self, y: dict, f: dict, md: AttentionMetadata, cache: Optional[torch.Tensor],
-            state: Optional[dict], scale: float, out: torch.Tensor) -> None:
-        """Writes ``scale`` times the part's result into ``out [T, local width]``; ``y`` / ``f``:
-        views of its projections."""
+    def mix(self, h: torch.Tensor, y: dict, f: dict, fw: dict, md: AttentionMetadata,
+            cache: Optional[torch.Tensor], state: Optional[dict], scale: float, out: torch.Tensor
+            ) -> None:
+        """Writes ``scale`` times the part's result into ``out [T, local width]``.  ``y``: views of
+        its projections of the mixer's input ``h`` (padded to multiples of 8 columns); ``f``: of its
+        fp32 projections, without the rows of single tokens where :func:`fused_tokens` says so;
+        ``fw``: the latter's weights."""
         raise NotImplementedError
+
+
+def fused_tokens(h: torch.Tensor, md: AttentionMetadata) -> int:
+    """Leading tokens of a step that fused single-token kernels take."""
+    return md.num_decode_tokens if ops.use_native(h) and not md.is_dummy else 0
 
 
 class MixerBlock(nn.Module):
@@ -126,16 +135,23 @@ class MixerBlock(nn.Module):
                 state: Optional[dict]) -> torch.Tensor:
         T = h.shape[0]
         ys = self.in_proj.split(self.in_proj(h), padded=True)
-        fs = self.fp32_proj.split(linear_fp32(h, self.fp32_proj.weight)) \
-            if self.fp32_proj is not None else ()
+        n1 = fused_tokens(h, md)
+        fs, fws = (), ()
+        if self.fp32_proj is not None:
+            w = self.fp32_proj.weight
+            fws = [v[:n] for v, n in zip(w.split(self.fp32_proj.padded_sizes),
+                                         self.fp32_proj.local_sizes)]
+            if n1 < T:
+                fs = self.fp32_proj.split(linear_fp32(h[n1:], w))
         out = torch.empty(T, self.o_proj.in_per_rank, dtype=h.dtype, device=h.device)
         at = 0
         for i, part in enumerate(self.parts):
             y = {n: v for (j, n), v in zip(self.slots, ys) if j == i}
             f = {n: v for (j, n), v in zip(self.fp32_slots, fs) if j == i}
+            fw = {n: v for (j, n), v in zip(self.fp32_slots, fws) if j == i}
             st = {k.partition(".")[2]: v for k, v in state.items()
                   if k.partition(".")[0] == str(i)} if state is not None else None
             w = self.o_proj.local_sizes[i]
-            part.mix(y, f, md, cache, st or None, self.scales[i], out[:, at:at + w])
+            part.mix(h, y, f, fw, md, cache, st or None, self.scales[i], out[:, at:at + w])
             at += w
         return self.o_proj(out)

@@ -7,6 +7,7 @@ the layout.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -18,11 +19,26 @@ from ..ops import ref
 from ..parallel.state import tp_size
 from .attention import AttentionMetadata
 from .linear import linear_fp32
-from .mixer import MixerPart, linear
+from .mixer import MixerPart, fused_tokens, linear
 
 #: padded key dimensions of the scan kernel
 STATE_ROWS = (32, 64, 96, 128, 192, 256)
 MAX_TAPS = 8
+
+
+@dataclass
+class Place:
+    """What the scans need to know of a step (or of its rows behind the single tokens)."""
+    positions: torch.Tensor
+    state_slots: Optional[torch.Tensor]
+    num_decode_tokens: int
+    cu_q_prefill: Optional[torch.Tensor]
+
+    @staticmethod
+    def behind(md: AttentionMetadata, n: int) -> "Place":
+        """``n``: 0 or all single tokens of the step (one request each)."""
+        slots = md.state_slots[n:] if md.state_slots is not None else None
+        return Place(md.positions[n:], slots, md.num_decode_tokens - n, md.cu_q_prefill)
 
 
 def state_rows(head_dim: int, prefix: str) -> int:
@@ -90,18 +106,25 @@ class GatedDelta(MixerPart):
         self.a2.data[:, self.spec.decay_rank:] = 0
         self.g2.data[:, self.spec.gate_rank:] = 0
 
-    def mix(self, y, f, md: AttentionMetadata, cache, state: Optional[dict], scale: float,
+    def mix(self, h, y, f, fw, md: AttentionMetadata, cache, state: Optional[dict], scale: float,
             out: torch.Tensor) -> None:
         s = self.spec
+        nk, nv = self.G * s.head_dim, self.N * s.v_head_dim
+        q, k, v, a1, g1 = y["q"][:, :nk], y["k"][:, :nk], y["v"][:, :nv], y["a1"], y["g1"]
+        conv = (self.conv_q, self.conv_k, self.conv_v)
+        sizes = s.head_dim, s.v_head_dim, self.rows
+        n1 = fused_tokens(h, md)
+        if n1:
+            C.delta_step(h[:n1], q[:n1], k[:n1], v[:n1], a1[:n1], g1[:n1], self.a2, self.g2,
+                         fw["b"], conv, self.dt_bias, self.a_log, self.norm, *sizes, md.positions,
+                         md.state_slots, state, self.eps, scale, out[:n1])
+        if n1 == h.shape[0]:
+            return
         o_ = C if ops.use_native(out) else ref
-        n = self.N * s.v_head_dim
-        if md.is_dummy:
-            state = None
-        o = o_.delta_rule(y["q"][:, :self.G * s.head_dim], y["k"][:, :self.G * s.head_dim],
-                          y["v"][:, :n], linear_fp32(y["a1"], self.a2), f["b"],
-                          (self.conv_q, self.conv_k, self.conv_v), self.dt_bias, self.a_log,
-                          s.head_dim, s.v_head_dim, self.rows, md, state)
-        o_.head_norm_gate(o, self.norm, linear(y["g1"], self.g2), self.eps, scale, out)
+        o = o_.delta_rule(q[n1:], k[n1:], v[n1:], linear_fp32(a1[n1:], self.a2), f["b"], conv,
+                          self.dt_bias, self.a_log, *sizes, Place.behind(md, n1),
+                          None if md.is_dummy else state)
+        o_.head_norm_gate(o, self.norm, linear(g1[n1:], self.g2), self.eps, scale, out[n1:])
 
 
 class MatrixMemory(MixerPart):
@@ -137,15 +160,21 @@ class MatrixMemory(MixerPart):
         getattr(self, self._OWN[name]).data.copy_(self.shard(full))
         return True
 
-    def mix(self, y, f, md: AttentionMetadata, cache, state: Optional[dict], scale: float,
+    def mix(self, h, y, f, fw, md: AttentionMetadata, cache, state: Optional[dict], scale: float,
             out: torch.Tensor) -> None:
         s = self.spec
-        o_ = C if ops.use_native(out) else ref
         nk, nv = self.N * s.head_dim, self.N * s.v_head_dim
-        if md.is_dummy:
-            state = None
-        # (a head count of one makes the norm weight per head and shared at once)
-        o = o_.matrix_memory(y["q"][:, :nk], y["k"][:, :nk], y["v"][:, :nv], f["i"], f["f"],
-                             self.i_bias, self.f_bias, s.gate_cap, s.head_dim, s.v_head_dim,
-                             self.rows, md, state)
-        o_.head_norm_gate(o, self.norm, y["g"][:, :nv], self.eps, scale, out)
+        q, k, v, g = y["q"][:, :nk], y["k"][:, :nk], y["v"][:, :nv], y["g"][:, :nv]
+        sizes = s.head_dim, s.v_head_dim, self.rows
+        n1 = fused_tokens(h, md)
+        if n1:
+            C.memory_step(h[:n1], q[:n1], k[:n1], v[:n1], g[:n1], fw["i"], fw["f"], self.i_bias,
+                          self.f_bias, s.gate_cap, self.norm, *sizes, md.positions,
+                          md.state_slots, state, self.eps, scale, out[:n1])
+        if n1 == h.shape[0]:
+            return
+        o_ = C if ops.use_native(out) else ref
+        o, nq, low = o_.matrix_memory(q[n1:], k[n1:], v[n1:], f["i"], f["f"], self.i_bias,
+                                      self.f_bias, s.gate_cap, *sizes, Place.behind(md, n1),
+                                      None if md.is_dummy else state)
+        o_.head_norm_gate(o, self.norm, g[n1:], self.eps, scale, out[n1:], nq, low)

@@ -894,7 +894,8 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tenso
     """Gated delta rule with one decay per key channel over the portions of a step: q, k ``[T, G *
     head_dim]`` and v ``[T, N * v_dim]`` are projections (views of one row), ``z [T, N * head_dim]``
     and ``b [T, N]`` fp32.  ``state``: ``matrix [slots, N, v_dim, rows]`` fp32 and ``taps [slots,
-    taps, channels]``, addressed by ``md.state_slots``.  Returns fp32 ``[T, N, v_dim]``."""
+    taps, channels]``, addressed by ``md.state_slots``; ``md`` also gives ``positions``,
+    ``num_decode_tokens`` and ``cu_q_prefill``.  Returns fp32 ``[T, N, v_dim]``."""
     T, D, V = q.shape[0], head_dim, v_dim
     G, Nh = q.shape[1] // D, v.shape[1] // V
     VP = -(-V // 4) * 4
@@ -921,41 +922,94 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tenso
 
 def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, zi: torch.Tensor,
                   zf: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
-                  head_dim: int, v_dim: int, rows: int, md, state: Optional[dict]) -> torch.Tensor:
+                  head_dim: int, v_dim: int, rows: int, md, state: Optional[dict]
+                  ) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
     """Matrix memory with exponential gates (mLSTM) over the portions of a step: q, k, v
     projections ``[T, N * dim]`` (views of one row), ``zi`` / ``zf`` fp32 ``[T, N]`` gate
     projections.  ``state``: ``matrix [slots, N, v_dim, rows]``, ``vector [slots, N, rows]``,
-    ``scalar [slots, N]`` fp32.  Returns fp32 ``[T, N, v_dim]``."""
+    ``scalar [slots, N]`` fp32.  Returns fp32 ``o [T, N, v_dim]``, ``nq`` and ``low`` ``[T, N]``; the
+    result is ``o / (max(|nq|, low) + 1e-6)`` (:func:`head_norm_gate`)."""
     T, D, V = q.shape[0], head_dim, v_dim
     Nh = q.shape[1] // D
-    VP = -(-V // 4) * 4
+    VP = V // 4 * 4 + 4
     assert q.stride(0) == k.stride(0) == v.stride(0) and zi.stride(0) == zf.stride(0)
     assert zi.dtype == zf.dtype == torch.float32
     new = lambda *s: torch.empty(s, dtype=torch.float32, device=q.device)  # noqa: E731
     qo, ko, vo, li, lf = new(T, Nh, rows), new(T, Nh, rows), new(T, Nh, VP), new(T, Nh), new(T, Nh)
-    out = new(T, Nh, V)
+    out, nq, low = new(T, Nh, V), new(T, Nh), new(T, Nh)
     if state is None:
-        return out.zero_()
+        return out.zero_(), nq.zero_(), low.fill_(1.0)
     nd, npf, cu = _scan_place(md)
-    S = state["matrix"]
+    S, slots = state["matrix"], md.state_slots
+    m0 = new(nd + npf, Nh)
     call("b200_memory_inputs", ptr(q), ptr(k), ptr(v), q.stride(0), ptr(zi), ptr(zf), zi.stride(0),
-         ptr(i_bias), ptr(f_bias), float(cap), float(D ** -0.5), ptr(qo), ptr(ko), ptr(vo), ptr(li),
-         ptr(lf), T, Nh, D, V, rows, VP, DTYPE_CODE[q.dtype], stream_ptr())
-    call("b200_memory_scan", ptr(qo), ptr(ko), ptr(vo), ptr(li), ptr(lf), ptr(out), ptr(S),
-         ptr(state["vector"]), ptr(state["scalar"]), ptr(md.positions), ptr(md.state_slots),
-         S.shape[0], ptr(cu), Nh, D, V, rows, VP, nd, npf, stream_ptr())
-    return out
+         ptr(i_bias), ptr(f_bias), ptr(state["scalar"]), float(cap), float(D ** -0.5), ptr(qo),
+         ptr(ko), ptr(vo), ptr(li), ptr(lf), ptr(m0), ptr(md.positions), ptr(slots), S.shape[0],
+         ptr(cu), T, Nh, D, V, rows, VP, nd, npf, DTYPE_CODE[q.dtype], stream_ptr())
+    call("b200_memory_scan", ptr(qo), ptr(ko), ptr(vo), ptr(li), ptr(lf), ptr(m0), ptr(out),
+         ptr(nq), ptr(low), ptr(S), ptr(state["vector"]), ptr(state["scalar"]), ptr(md.positions),
+         ptr(slots), S.shape[0], ptr(cu), Nh, D, V, rows, VP, nd, npf, stream_ptr())
+    return out, nq, low
 
 
 def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, z: torch.Tensor, eps: float,
-                   scale: float, out: torch.Tensor) -> torch.Tensor:
+                   scale: float, out: torch.Tensor, nq: Optional[torch.Tensor] = None,
+                   low: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out = o / rms(o) * weight * sigmoid(z) * scale`` with ``o [T, N, V]`` fp32 normalised per
-    head, ``weight`` ``[V]`` or ``[N * V]``, ``z`` and ``out`` ``[T, N * V]`` (views are fine)."""
+    head, ``weight`` ``[V]`` or ``[N * V]``, ``z`` and ``out`` ``[T, N * V]`` (views are fine).  With
+    ``nq`` and ``low`` (:func:`matrix_memory`) o is divided first."""
     T, Nh, V = o.shape
     assert z.stride(1) == 1 and out.stride(1) == 1 and z.dtype == out.dtype
-    call("b200_head_norm_gate", ptr(o), ptr(weight), int(weight.numel() != V), ptr(z), z.stride(0),
-         ptr(out), out.stride(0), float(eps), float(scale), T, Nh, V, DTYPE_CODE[out.dtype],
+    call("b200_head_norm_gate", ptr(o), ptr(nq), ptr(low), ptr(weight), int(weight.numel() != V),
+         ptr(z), z.stride(0), ptr(out), out.stride(0), float(eps), float(scale), T, Nh, V,
+         DTYPE_CODE[out.dtype], stream_ptr())
+    return out
+
+
+def delta_step(h: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
+               a1: torch.Tensor, g1: torch.Tensor, a2: torch.Tensor, g2: torch.Tensor,
+               b_weight: torch.Tensor, conv: Sequence[torch.Tensor], dt_bias: torch.Tensor,
+               a_log: torch.Tensor, norm: torch.Tensor, head_dim: int, v_dim: int, rows: int,
+               positions: torch.Tensor, slots: torch.Tensor, state: dict, eps: float, scale: float,
+               out: torch.Tensor) -> torch.Tensor:
+    """One token of every request through the gated delta rule in one kernel: :func:`delta_rule`
+    and :func:`head_norm_gate` with the step sizes (``b_weight [N, H]`` on the mixer's input ``h``),
+    the second steps of the decay and gate projections (``a2``, ``g2``; ``a1``, ``g1`` their inputs,
+    padded to multiples of 8 columns) included."""
+    nd, D, V = h.shape[0], head_dim, v_dim
+    G, Nh = q.shape[1] // D, v.shape[1] // V
+    ld = q.stride(0)
+    assert all(t.stride(0) == ld and t.stride(1) == 1 for t in (k, v, a1, g1))
+    assert a1.shape[1] == a2.shape[1] and g1.shape[1] == g2.shape[1] and b_weight.is_contiguous()
+    taps = state["taps"]
+    call("b200_delta_step", ptr(h), h.stride(0), h.shape[1], ptr(q), ptr(k), ptr(v), ptr(a1),
+         ptr(g1), ld, ptr(a2), a2.shape[1], ptr(g2), g2.shape[1], ptr(b_weight), ptr(conv[0]),
+         ptr(conv[1]), ptr(conv[2]), conv[0].shape[1], ptr(dt_bias), ptr(a_log), ptr(norm),
+         ptr(taps), ptr(state["matrix"]), ptr(positions), ptr(slots), taps.shape[0], ptr(out),
+         out.stride(0), float(eps), float(scale), nd, G, Nh, D, V, rows, DTYPE_CODE[h.dtype],
          stream_ptr())
+    return out
+
+
+def memory_step(h: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
+                gate: torch.Tensor, i_weight: torch.Tensor, f_weight: torch.Tensor,
+                i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, norm: torch.Tensor,
+                head_dim: int, v_dim: int, rows: int, positions: torch.Tensor,
+                slots: torch.Tensor, state: dict, eps: float, scale: float, out: torch.Tensor
+                ) -> torch.Tensor:
+    """One token of every request through the matrix memory in one kernel: :func:`matrix_memory`
+    and :func:`head_norm_gate` with the gates' projections of the mixer's input ``h`` included."""
+    nd, D, V = h.shape[0], head_dim, v_dim
+    Nh = q.shape[1] // D
+    ld = q.stride(0)
+    assert all(t.stride(0) == ld and t.stride(1) == 1 for t in (k, v, gate))
+    assert i_weight.is_contiguous() and f_weight.is_contiguous()
+    S = state["matrix"]
+    call("b200_memory_step", ptr(h), h.stride(0), h.shape[1], ptr(q), ptr(k), ptr(v), ptr(gate), ld,
+         ptr(i_weight), ptr(f_weight), ptr(i_bias), ptr(f_bias), float(cap), float(D ** -0.5),
+         ptr(norm), ptr(S), ptr(state["vector"]), ptr(state["scalar"]), ptr(positions), ptr(slots),
+         S.shape[0], ptr(out), out.stride(0), float(eps), float(scale), nd, Nh, D, V, rows,
+         DTYPE_CODE[h.dtype], stream_ptr())
     return out
 
 

@@ -804,8 +804,9 @@ def matrix_memory(q, k, v, zi, zf, i_bias, f_bias, cap, head_dim, v_dim, rows, m
     T, D, V = q.shape[0], head_dim, v_dim
     Nh = q.shape[1] // D
     out = torch.zeros(T, Nh, V, dtype=torch.float32, device=q.device)
+    nqs, low = torch.zeros_like(out[..., 0]), torch.ones_like(out[..., 0])
     if state is None:
-        return out
+        return out, nqs, low
     li = cap * torch.tanh((zi + i_bias) / cap)
     lf = torch.nn.functional.logsigmoid(cap * torch.tanh((zf + f_bias) / cap))
     qf, kf = q.float().view(T, Nh, D) * D ** -0.5, k.float().view(T, Nh, D)
@@ -821,17 +822,19 @@ def matrix_memory(q, k, v, zi, zf, i_bias, f_bias, cap, head_dim, v_dim, rows, m
             m = new
             S = keep[:, None, None] * S + add[:, None, None] * vf[t][:, :, None] * kf[t][:, None, :]
             nv = keep[:, None] * nv + add[:, None] * kf[t]
-            den = torch.maximum((nv * qf[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
-            out[t] = (S * qf[t][:, None, :]).sum(-1) / den[:, None]
+            nqs[t], low[t] = (nv * qf[t]).sum(-1), torch.exp(-m)
+            out[t] = (S * qf[t][:, None, :]).sum(-1)
         state["matrix"][slot, :, :, :D] = S
         state["vector"][slot, :, :D] = nv
         state["scalar"][slot] = m
-    return out
+    return out, nqs, low
 
 
-def head_norm_gate(o, weight, z, eps, scale, out) -> torch.Tensor:
+def head_norm_gate(o, weight, z, eps, scale, out, nq=None, low=None) -> torch.Tensor:
     """See ``ops.cuda.head_norm_gate``."""
     T, Nh, V = o.shape
+    if nq is not None:
+        o = o / (torch.maximum(nq.abs(), low) + 1e-6).unsqueeze(-1)
     r = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
     r = r * (weight.view(Nh, V) if weight.numel() != V else weight)
     out.copy_(r.flatten(1) * torch.sigmoid(z.float()) * scale)
