@@ -80,13 +80,12 @@ def cases(lens: list[int], ctx: int, decode: bool, H: int, N: int, G: int, D: in
     gate, nw = rnd(T, N * D).to(bf), torch.ones(D, device=dev)
     res = torch.empty(T, N * D, device=dev, dtype=bf)
 
-    a2, g2, wb1 = rnd(N * D, 128).to(bf), rnd(N * D, 128).to(bf), rnd(N, H).to(bf)
+    wb1 = rnd(N, H).to(bf)
 
     def delta():
         if decode:
-            C.delta_step(xb, q, k, v, wide[:, 3 * N * D:3 * N * D + 128],
-                         wide[:, 3 * N * D + 128:], a2, g2, wb1, conv, dtb, alog, nw, D, D, D,
-                         md.positions, md.state_slots, st, 1e-5, 1.0, res)
+            C.delta_step(xb, q, k, v, z, gate, wb1, conv, dtb, alog, nw, D, D, D, md.positions,
+                         md.state_slots, st, 1e-5, 1.0, res)
             return
         o = C.delta_rule(q, k, v, z, bz, conv, dtb, alog, D, D, D, md, st)
         C.head_norm_gate(o, nw, gate, 1e-5, 1.0, res)

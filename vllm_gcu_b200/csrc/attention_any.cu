@@ -188,7 +188,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_pairs_kernel(const Pre
 // thread, queries then keys, read once and kept in registers.
 template <int NV>
 __global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const PrepArgs a) {
-  __shared__ float red[32];
+  __shared__ float red[2][8];
   const int t = blockIdx.x;
   const __nv_bfloat16* q =
       static_cast<const __nv_bfloat16*>(a.q) + static_cast<long long>(t) * a.ldq;
@@ -218,8 +218,19 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const PrepA
     sq = a.sumsq[2 * t];
     sk = a.sumsq[2 * t + 1];
   } else {
-    sq = block_sum(sq, red);
-    sk = block_sum(sk, red);
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) {
+      red[0][threadIdx.x >> 5] = sq;
+      red[1][threadIdx.x >> 5] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+      sq += red[0][w];
+      sk += red[1][w];
+    }
   }
   const float qi = 1.0f / sqrtf(sq / static_cast<float>(a.q_all) + a.eps);
   const float ki = 1.0f / sqrtf(sk / static_cast<float>(a.k_all) + a.eps);

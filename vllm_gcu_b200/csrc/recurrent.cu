@@ -32,30 +32,40 @@ namespace recurrent {
 constexpr int kDelta = 0, kMemory = 1;
 
 // fp32 pairs: two multiply-adds per instruction
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ uint64_t both(float x) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "f"(x));
-  return d;
-}
-__device__ __forceinline__ float halves_sum(uint64_t x) {
-  float lo, hi;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(x));
-  return lo + hi;
-}
+struct __align__(16) Quad {
+  float2 x, y;
+};
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __ffma2_rn(a, b, c); }
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) { return __fmul2_rn(a, b); }
+__device__ __forceinline__ float2 both(float x) { return make_float2(x, x); }
+__device__ __forceinline__ float halves_sum(float2 x) { return x.x + x.y; }
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus(float z) {
   return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)));
+}
+// fp32 forms for 16-bit models: the fast exponential and division, relative errors near 1e-6; the
+// logarithm of 1 + e switches to its series where e would be rounded away
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.0f, 1.0f + __expf(-z));
+  else return sigmoid(z);
+}
+template <typename T>
+__device__ __forceinline__ float softplus_t(float z) {
+  if constexpr (sizeof(T) == 2) {
+    const float e = __expf(-fabsf(z));
+    const float l = e < 0.02f ? e * (1.0f - e * (0.5f - e * (1.0f / 3.0f - e * 0.25f)))
+                              : __logf(1.0f + e);
+    return fmaxf(z, 0.0f) + l;
+  } else {
+    return softplus(z);
+  }
+}
+template <typename T>
+__device__ __forceinline__ float exp_t(float z) {
+  if constexpr (sizeof(T) == 2) return __expf(z);
+  else return expf(z);
 }
 
 __device__ __forceinline__ void copy16(void* dst, const void* src) {
@@ -104,7 +114,7 @@ struct DeltaIn {
 };
 
 constexpr int kMaxTaps = 8;
-constexpr int kStrip = 16;       // tokens one warp walks
+constexpr int kStrip = 8;        // tokens one warp walks
 
 template <typename T, int V>
 __device__ __forceinline__ void load_n(const T* p, float (&f)[V]) {
@@ -131,129 +141,150 @@ __device__ __forceinline__ float silu(float x) {
   else return x / (1.0f + expf(-x));
 }
 
-// One warp: kStrip tokens of one item, V neighbouring channels per lane (32 V channels at a time).
-// Items: [0, G) q heads, [G, 2G) k heads, [2G, 2G + N) v heads, [2G + N, 2G + 2N) decays.
+// A CTA: kStrip tokens; every warp walks its items, V neighbouring channels per lane (32 V channels
+// at a time).  Items: [0, G) q heads, [G, 2G) k heads, [2G, 2G + N) v heads, [2G + N, 2G + 2N)
+// decays.
 template <typename T, int NT, int V>
-__global__ void __launch_bounds__(256) delta_inputs_kernel(const DeltaIn a) {
+__global__ void __launch_bounds__(256, 2) delta_inputs_kernel(const DeltaIn a) {
+  __shared__ int s_first[kStrip], s_slot[kStrip];   // portion's first token (-1: none), its slot
+  __shared__ long long s_pos[kStrip];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int item = blockIdx.y * 8 + warp;
   const int t0 = blockIdx.x * kStrip;
-  if (item >= 2 * a.G + 2 * a.N || t0 >= a.T) return;
   const int t1 = min(t0 + kStrip, a.T);
-  if (item >= 2 * a.G + a.N) {                   // decays and step sizes
-    const int h = item - 2 * a.G - a.N;
-    const float rate = expf(a.a_log[h]);
-    for (int d = lane * V; d < a.DP; d += 32 * V) {
-      float bias[V];
-#pragma unroll
-      for (int i = 0; i < V; ++i) bias[i] = d + i < a.D ? a.dt_bias[h * a.D + d + i] : 0.0f;
-      for (int t = t0; t < t1; ++t) {
-        float g[V];
-#pragma unroll
-        for (int i = 0; i < V; ++i) g[i] = 0.0f;
-        if (d < a.D) {
-          load_n<float, V>(a.z + t * a.ldz + h * a.D + d, g);
-#pragma unroll
-          for (int i = 0; i < V; ++i) g[i] = expf(-rate * softplus(g[i] + bias[i]));
-        }
-        store_n<V>(a.g + (static_cast<long long>(t) * a.N + h) * a.DP + d, g);
+  if (threadIdx.x < kStrip) {
+    const int t = t0 + threadIdx.x;
+    s_first[threadIdx.x] = -1;
+    if (t < t1) {
+      const TokenPlace pl = token_place(t, a.nd, a.np, a.cu_q);
+      if (pl.req >= 0) {
+        s_first[threadIdx.x] = portion_of(pl.req, a.nd, a.cu_q).first;
+        s_slot[threadIdx.x] = a.slots[pl.req];
+        s_pos[threadIdx.x] = a.positions[t];
       }
     }
-    for (int t = t0 + lane; t < t1; t += 32)
-      a.beta[static_cast<long long>(t) * a.N + h] = sigmoid(a.bz[t * a.ldb + h]);
-    return;
   }
-  const int which = item < a.G ? 0 : item < 2 * a.G ? 1 : 2;
-  const int head = which == 0 ? item : which == 1 ? item - a.G : item - 2 * a.G;
-  const int dim = which == 2 ? a.V : a.D, pitch = which == 2 ? a.VP : a.DP;
+  __syncthreads();
   const int C = 2 * a.G * a.D + a.N * a.V;
-  const int ring_off = (which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D) + head * dim;
-  const T* x = static_cast<const T*>(a.x[which]) + head * dim;
-  const float* wt = a.taps_w[which] + static_cast<long long>(head) * dim * a.ntaps;
-  float* out = (which == 0 ? a.q : which == 1 ? a.k : a.v) + head * pitch;
-  const long long ldo = static_cast<long long>(which == 2 ? a.N : a.G) * pitch;
-  const int passes = (pitch + 32 * V - 1) / (32 * V);
-  float inv_sum[kStrip];
-  // q and k of more channels than one pass holds: a first walk over all passes for the norms
-  const bool unit = which < 2;
-  for (int walk = unit && passes > 1 ? 0 : 1; walk < 2; ++walk) {
-    for (int ps = 0; ps < passes; ++ps) {
-      const int d = (ps * 32 + lane) * V;
-      const bool in = d < dim;
-      float w[NT][V];                              // [o]: tap that meets the input of o tokens ago
+  for (int item = blockIdx.y * 8 + warp; item < 2 * a.G + 2 * a.N; item += gridDim.y * 8) {
+    if (item >= 2 * a.G + a.N) {                   // decays and step sizes
+      const int h = item - 2 * a.G - a.N;
+      const float rate = expf(a.a_log[h]);
+      for (int d = lane * V; d < a.DP; d += 32 * V) {
+        float bias[V];
 #pragma unroll
-      for (int o = 0; o < NT; ++o) {
+        for (int i = 0; i < V; ++i) bias[i] = d + i < a.D ? a.dt_bias[h * a.D + d + i] : 0.0f;
+        float g[kStrip][V];                        // all rows of the strip in flight at once
 #pragma unroll
-        for (int i = 0; i < V; ++i)
-          w[o][i] = in && o < a.ntaps ? wt[(d + i) * a.ntaps + a.ntaps - 1 - o] : 0.0f;
+        for (int u = 0; u < kStrip; ++u) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) g[u][i] = 0.0f;
+          if (d < a.D && t0 + u < t1) load_n<float, V>(a.z + (t0 + u) * a.ldz + h * a.D + d, g[u]);
+        }
+#pragma unroll
+        for (int u = 0; u < kStrip; ++u) {
+          if (t0 + u >= t1) break;
+#pragma unroll
+          for (int i = 0; i < V; ++i)
+            g[u][i] = d < a.D ? exp_t<T>(-rate * softplus_t<T>(g[u][i] + bias[i])) : 0.0f;
+          store_n<V>(a.g + (static_cast<long long>(t0 + u) * a.N + h) * a.DP + d, g[u]);
+        }
       }
-      float past[NT][V];                           // [o]: input of o tokens ago
+      for (int t = t0 + lane; t < t1; t += 32)
+        a.beta[static_cast<long long>(t) * a.N + h] = sigmoid(a.bz[t * a.ldb + h]);
+      continue;
+    }
+    const int which = item < a.G ? 0 : item < 2 * a.G ? 1 : 2;
+    const int head = which == 0 ? item : which == 1 ? item - a.G : item - 2 * a.G;
+    const int dim = which == 2 ? a.V : a.D, pitch = which == 2 ? a.VP : a.DP;
+    const int ring_off = (which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D) + head * dim;
+    const T* x = static_cast<const T*>(a.x[which]) + head * dim;
+    const float* wt = a.taps_w[which] + static_cast<long long>(head) * dim * a.ntaps;
+    float* out = (which == 0 ? a.q : which == 1 ? a.k : a.v) + head * pitch;
+    const long long ldo = static_cast<long long>(which == 2 ? a.N : a.G) * pitch;
+    const int passes = (pitch + 32 * V - 1) / (32 * V);
+    float inv_sum[kStrip];
+    // q and k of more channels than one pass holds: a first walk over all passes for the norms
+    const bool unit = which < 2;
+    for (int walk = unit && passes > 1 ? 0 : 1; walk < 2; ++walk) {
+      for (int ps = 0; ps < passes; ++ps) {
+        const int d = (ps * 32 + lane) * V;
+        const bool in = d < dim;
+        float rows[kStrip][V];                     // all rows of the strip in flight at once
 #pragma unroll
-      for (int o = 0; o < NT; ++o) {
+        for (int u = 0; u < kStrip; ++u) {
 #pragma unroll
-        for (int i = 0; i < V; ++i) past[o][i] = 0.0f;
-      }
-      int end = -1;                                // end of the portion the walk is in
-      for (int t = t0; t < t1; ++t) {
-        if (t >= end) {                            // first token of the strip or of a portion
-          const TokenPlace pl = token_place(t, a.nd, a.np, a.cu_q);
-          if (pl.req < 0) return;                  // padding rows end the step
-          const Portion po = portion_of(pl.req, a.nd, a.cu_q);
-          end = po.first + po.count;
-          const long long pos = a.positions[t];
-          const int slot = a.slots[pl.req];
+          for (int i = 0; i < V; ++i) rows[u][i] = 0.0f;
+          if (in && t0 + u < t1)
+            load_n<T, V>(x + static_cast<long long>(t0 + u) * a.ld + d, rows[u]);
+        }
+        float w[NT][V];                            // [o]: tap that meets the input of o tokens ago
 #pragma unroll
-          for (int o = 1; o < NT; ++o) {
+        for (int o = 0; o < NT; ++o) {
 #pragma unroll
-            for (int i = 0; i < V; ++i) past[o - 1][i] = 0.0f;
-            if (!in || o >= a.ntaps || pos - o < 0) continue;
-            if (t - o >= po.first) {
-              load_n<T, V>(x + static_cast<long long>(t - o) * a.ld + d, past[o - 1]);
-            } else if (slot >= 0 && slot < a.num_slots) {
-              load_n<T, V>(static_cast<const T*>(a.taps) +
-                               (static_cast<long long>(slot) * a.ntaps + (pos - o) % a.ntaps) * C +
-                               ring_off + d, past[o - 1]);
+          for (int i = 0; i < V; ++i)
+            w[o][i] = in && o < a.ntaps ? wt[(d + i) * a.ntaps + a.ntaps - 1 - o] : 0.0f;
+        }
+        float past[NT][V];                         // [o]: input of o tokens ago
+#pragma unroll
+        for (int o = 0; o < NT; ++o) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) past[o][i] = 0.0f;
+        }
+#pragma unroll
+        for (int u = 0; u < kStrip; ++u) {
+          const int t = t0 + u;
+          const int first = s_first[u];
+          if (t >= t1 || first < 0) break;         // (padding rows end the step)
+          if (u == 0 || t == first) {              // the inputs in front of the walk
+            const long long pos = s_pos[u];
+            const int slot = s_slot[u];
+#pragma unroll
+            for (int o = 1; o < NT; ++o) {
+#pragma unroll
+              for (int i = 0; i < V; ++i) past[o - 1][i] = 0.0f;
+              if (!in || o >= a.ntaps || pos - o < 0) continue;
+              if (t - o >= first) {
+                load_n<T, V>(x + static_cast<long long>(t - o) * a.ld + d, past[o - 1]);
+              } else if (slot >= 0 && slot < a.num_slots) {
+                load_n<T, V>(static_cast<const T*>(a.taps) +
+                                 (static_cast<long long>(slot) * a.ntaps + (pos - o) % a.ntaps) * C +
+                                 ring_off + d, past[o - 1]);
+              }
             }
           }
-        }
 #pragma unroll
-        for (int o = NT - 1; o > 0; --o) {
+          for (int o = NT - 1; o > 0; --o) {
 #pragma unroll
-          for (int i = 0; i < V; ++i) past[o][i] = past[o - 1][i];
-        }
-        if (in) load_n<T, V>(x + static_cast<long long>(t) * a.ld + d, past[0]);
-        float f[V], ss = 0.0f;
-#pragma unroll
-        for (int i = 0; i < V; ++i) {
-          float c = 0.0f;
-#pragma unroll
-          for (int o = NT - 1; o >= 0; --o) c += w[o][i] * past[o][i];
-          f[i] = silu<T>(c);
-          ss += f[i] * f[i];
-        }
-        if (unit) {
-          float inv;
-          if (passes == 1) {
-            inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
-          } else if (walk == 0) {
-            // (a static index keeps the sums in registers)
-            const float sum = warp_sum(ss);
-#pragma unroll
-            for (int u = 0; u < kStrip; ++u)
-              if (u == t - t0) inv_sum[u] = ps == 0 ? sum : inv_sum[u] + sum;
-            continue;
-          } else {
-            float sum = 0.0f;
-#pragma unroll
-            for (int u = 0; u < kStrip; ++u)
-              if (u == t - t0) sum = inv_sum[u];
-            inv = 1.0f / sqrtf(sum + 1e-6f);
+            for (int i = 0; i < V; ++i) past[o][i] = past[o - 1][i];
           }
-          if (which == 0) inv *= 1.0f / sqrtf(static_cast<float>(a.D));
 #pragma unroll
-          for (int i = 0; i < V; ++i) f[i] *= inv;
+          for (int i = 0; i < V; ++i) past[0][i] = rows[u][i];
+          float f[V], ss = 0.0f;
+#pragma unroll
+          for (int i = 0; i < V; ++i) {
+            float c = 0.0f;
+#pragma unroll
+            for (int o = NT - 1; o >= 0; --o) c += w[o][i] * past[o][i];
+            f[i] = silu<T>(c);
+            ss += f[i] * f[i];
+          }
+          if (unit) {
+            float inv;
+            if (passes == 1) {
+              inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
+            } else if (walk == 0) {
+              const float sum = warp_sum(ss);
+              inv_sum[u] = ps == 0 ? sum : inv_sum[u] + sum;
+              continue;
+            } else {
+              inv = 1.0f / sqrtf(inv_sum[u] + 1e-6f);
+            }
+            if (which == 0) inv *= 1.0f / sqrtf(static_cast<float>(a.D));
+#pragma unroll
+            for (int i = 0; i < V; ++i) f[i] *= inv;
+          }
+          if (d < pitch) store_n<V>(out + t * ldo + d, f);
         }
-        if (d < pitch) store_n<V>(out + t * ldo + d, f);
       }
     }
   }
@@ -442,7 +473,7 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
   copy_commit();
 
   // state -> registers: lane l holds rows 4 (l + LPC i) .. + 3 of its columns
-  uint64_t S[CPT][P];
+  float2 S[CPT][P];
   const long long head_at = static_cast<long long>(slot) * a.N + h;
   auto column_state = [&](int c) {
     return MODE == kMemory && c == a.V ? a.vector + head_at * DP
@@ -454,8 +485,8 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
     const float* src = column_state(c0 + j) + 4 * l;
 #pragma unroll
     for (int i = 0; i < P / 2; ++i) {
-      ulonglong2 u = make_ulonglong2(0, 0);
-      if (in) u = *reinterpret_cast<const ulonglong2*>(src + 4 * LPC * i);
+      Quad u = Quad{both(0.0f), both(0.0f)};
+      if (in) u = *reinterpret_cast<const Quad*>(src + 4 * LPC * i);
       S[j][2 * i] = u.x;
       S[j][2 * i + 1] = u.y;
     }
@@ -502,66 +533,92 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
       m = __shfl_sync(0xffffffffu, mt, n - 1);
     }
 
+    // gated delta rule: q . k of every token, so that S'^T q = S^T q + (q . k) u needs no second
+    // reduction behind the update
+    if (MODE == kDelta) {
+      float* sqk = smem + b * stage + kRows * kChunk * DP + kChunk * a.cols + kChunk;
+      for (int e = threadIdx.x; e < n * 8; e += blockDim.x) {    // eight lanes per token
+        const float4* x = reinterpret_cast<const float4*>(smem + b * stage + (e >> 3) * DP);
+        const float4* y = x + kChunk * DP / 4;
+        float d = 0.0f;
+        for (int c = e & 7; c < DP / 4; c += 8) {
+          const float4 f = x[c], g = y[c];
+          d += f.x * g.x + f.y * g.y + f.z * g.z + f.w * g.w;
+        }
+        // (n * 8 is a multiple of 8 and so is the block: whole groups take part)
+        const unsigned int mask = 0xffu << (lane & 24);
+        d += __shfl_xor_sync(mask, d, 1);
+        d += __shfl_xor_sync(mask, d, 2);
+        d += __shfl_xor_sync(mask, d, 4);
+        if ((e & 7) == 0) sqk[e >> 3] = d;
+      }
+      __syncthreads();
+    }
+
+#pragma unroll 2
     for (int i = 0; i < (warp_on ? n : 0); ++i) {
       float v[CPT], o[CPT];
 #pragma unroll
       for (int j = 0; j < CPT; ++j) v[j] = sv[i * a.cols + c_loc + j];
-      uint64_t kk[P];
+      float2 kk[P];
 #pragma unroll
       for (int u = 0; u < P / 2; ++u) {
-        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(sk + i * DP + 4 * LPC * u);
+        const Quad x = *reinterpret_cast<const Quad*>(sk + i * DP + 4 * LPC * u);
         kk[2 * u] = x.x; kk[2 * u + 1] = x.y;
       }
-      uint64_t e0[CPT], e1[CPT];
+      float2 e0[CPT], e1[CPT];
 #pragma unroll
-      for (int j = 0; j < CPT; ++j) e0[j] = e1[j] = 0;
+      for (int j = 0; j < CPT; ++j) e0[j] = e1[j] = both(0.0f);
       if (MODE == kDelta) {
-        const float beta = ss[i];
-        uint64_t d0[CPT], d1[CPT];
+        const float beta = ss[i], qk = ss[kChunk + i];
+        float2 d0[CPT], d1[CPT];
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) d0[j] = d1[j] = 0;
+        for (int j = 0; j < CPT; ++j) d0[j] = d1[j] = both(0.0f);
 #pragma unroll
         for (int u = 0; u < P / 2; ++u) {
-          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(sg + i * DP + 4 * LPC * u);
+          const Quad g = *reinterpret_cast<const Quad*>(sg + i * DP + 4 * LPC * u);
+          const Quad q = *reinterpret_cast<const Quad*>(sq + i * DP + 4 * LPC * u);
 #pragma unroll
           for (int j = 0; j < CPT; ++j) {
             S[j][2 * u] = mul2(S[j][2 * u], g.x);
             S[j][2 * u + 1] = mul2(S[j][2 * u + 1], g.y);
             d0[j] = fma2(S[j][2 * u], kk[2 * u], d0[j]);
             d1[j] = fma2(S[j][2 * u + 1], kk[2 * u + 1], d1[j]);
-          }
-        }
-        uint64_t u2[CPT];
-        float d[CPT];
-#pragma unroll
-        for (int j = 0; j < CPT; ++j) d[j] = halves_sum(d0[j]) + halves_sum(d1[j]);
-#pragma unroll
-        for (int w = 1; w < LPC; w <<= 1) {
-#pragma unroll
-          for (int j = 0; j < CPT; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], w);
-        }
-#pragma unroll
-        for (int j = 0; j < CPT; ++j) u2[j] = both(beta * (v[j] - d[j]));
-#pragma unroll
-        for (int u = 0; u < P / 2; ++u) {
-          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(sq + i * DP + 4 * LPC * u);
-#pragma unroll
-          for (int j = 0; j < CPT; ++j) {
-            S[j][2 * u] = fma2(kk[2 * u], u2[j], S[j][2 * u]);
-            S[j][2 * u + 1] = fma2(kk[2 * u + 1], u2[j], S[j][2 * u + 1]);
             e0[j] = fma2(S[j][2 * u], q.x, e0[j]);
             e1[j] = fma2(S[j][2 * u + 1], q.y, e1[j]);
           }
         }
+        float d[CPT];
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) {
+          d[j] = halves_sum(d0[j]) + halves_sum(d1[j]);
+          o[j] = halves_sum(e0[j]) + halves_sum(e1[j]);
+        }
+#pragma unroll
+        for (int w = 1; w < LPC; w <<= 1) {
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            d[j] += __shfl_xor_sync(0xffffffffu, d[j], w);
+            o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) {
+          const float u1 = beta * (v[j] - d[j]);
+          o[j] += qk * u1;
+          const float2 u2 = both(u1);
+#pragma unroll
+          for (int u = 0; u < P; ++u) S[j][u] = fma2(kk[u], u2, S[j][u]);
+        }
       } else {
-        const uint64_t a2 = both(__shfl_sync(0xffffffffu, keep, i));
+        const float2 a2 = both(__shfl_sync(0xffffffffu, keep, i));
         const float b1 = __shfl_sync(0xffffffffu, add, i);
-        uint64_t v2[CPT];
+        float2 v2[CPT];
 #pragma unroll
         for (int j = 0; j < CPT; ++j) v2[j] = both(b1 * v[j]);
 #pragma unroll
         for (int u = 0; u < P / 2; ++u) {
-          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(sq + i * DP + 4 * LPC * u);
+          const Quad q = *reinterpret_cast<const Quad*>(sq + i * DP + 4 * LPC * u);
 #pragma unroll
           for (int j = 0; j < CPT; ++j) {
             S[j][2 * u] = fma2(kk[2 * u], v2[j], mul2(S[j][2 * u], a2));
@@ -570,13 +627,13 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
             e1[j] = fma2(S[j][2 * u + 1], q.y, e1[j]);
           }
         }
-      }
 #pragma unroll
-      for (int j = 0; j < CPT; ++j) o[j] = halves_sum(e0[j]) + halves_sum(e1[j]);
+        for (int j = 0; j < CPT; ++j) o[j] = halves_sum(e0[j]) + halves_sum(e1[j]);
 #pragma unroll
-      for (int w = 1; w < LPC; w <<= 1) {
+        for (int w = 1; w < LPC; w <<= 1) {
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
+          for (int j = 0; j < CPT; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
+        }
       }
       const long long at = static_cast<long long>(po.first + i0 + i) * a.N + h;
       if (l == 0) {
@@ -599,8 +656,8 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
     float* dst = column_state(c0 + j) + 4 * l;
 #pragma unroll
     for (int i = 0; i < P / 2; ++i)
-      *reinterpret_cast<ulonglong2*>(dst + 4 * LPC * i) =
-          make_ulonglong2(S[j][2 * i], S[j][2 * i + 1]);
+      *reinterpret_cast<Quad*>(dst + 4 * LPC * i) =
+          Quad{S[j][2 * i], S[j][2 * i + 1]};
   }
   if (MODE == kMemory) {
     if (z == 0 && threadIdx.x == 0) a.scalar[head_at] = m;
@@ -691,13 +748,21 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs 
   const long long t = row / a.N;
   const int h = static_cast<int>(row - t * a.N);
   const float* o = a.o + row * a.V;
-  constexpr int kKeep = W == 4 ? 4 : 8;          // vectors per lane that stay in registers
-  float f[kKeep][W], ss = 0.0f;
+  const float* w = a.w + (a.per_head ? h * a.V : 0);
+  const T* z = static_cast<const T*>(a.z) + t * a.ldz + h * a.V;
+  T* out = static_cast<T*>(a.out) + t * a.ldo + h * a.V;
+  constexpr int kKeep = W == 4 ? 2 : 8;          // vectors per lane that stay in registers
+  float f[kKeep][W], g[kKeep][W], ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < kKeep; ++i) {
     const int c = (lane + 32 * i) * W;
     if (c >= a.V) continue;
     load_n<float, W>(o + c, f[i]);
+    load_n<T, W>(z + c, g[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    if ((lane + 32 * i) * W >= a.V) continue;
 #pragma unroll
     for (int j = 0; j < W; ++j) ss += f[i][j] * f[i][j];
   }
@@ -710,26 +775,23 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs 
   const float den = a.nq != nullptr ? 1.0f / (fmaxf(fabsf(a.nq[row]), a.low[row]) + 1e-6f) : 1.0f;
   const float inv =
       den * (1.0f / sqrtf(warp_sum(ss) * den * den / static_cast<float>(a.V) + a.eps)) * a.scale;
-  const float* w = a.w + (a.per_head ? h * a.V : 0);
-  const T* z = static_cast<const T*>(a.z) + t * a.ldz + h * a.V;
-  T* out = static_cast<T*>(a.out) + t * a.ldo + h * a.V;
-  auto put = [&](int c, float (&x)[W]) {
-    float g[W], b[W];
-    load_n<T, W>(z + c, g);
+  auto put = [&](int c, float (&x)[W], const float (&gate)[W]) {
+    float b[W];
     load_n<float, W>(w + c, b);
 #pragma unroll
-    for (int j = 0; j < W; ++j) x[j] = x[j] * inv * b[j] * sigmoid(g[j]);
+    for (int j = 0; j < W; ++j) x[j] = x[j] * inv * b[j] * sigmoid_t<T>(gate[j]);
     store_t<T, W>(out + c, x);
   };
 #pragma unroll
   for (int i = 0; i < kKeep; ++i) {
     const int c = (lane + 32 * i) * W;
-    if (c < a.V) put(c, f[i]);
+    if (c < a.V) put(c, f[i], g[i]);
   }
   for (int c = (lane + 32 * kKeep) * W; c < a.V; c += 32 * W) {
-    float x[W];
+    float x[W], gate[W];
     load_n<float, W>(o + c, x);
-    put(c, x);
+    load_n<T, W>(z + c, gate);
+    put(c, x, gate);
   }
 }
 
@@ -739,9 +801,8 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs 
 struct StepArgs {
   const void* hrow;          // [nd, H] mixer input, row pitch ldh
   const void* x[3];          // q, k, v projections, row pitch ld
-  const void* gate;          // memory: [nd, N V] gate projection, row pitch ld
-  const void *r1, *g1;       // delta: first steps of the decay / gate projections, row pitch ld
-  const void *r2, *g2;       // delta: second steps [N D, R], [N V, RG]
+  const void* gate;          // [nd, N V] output gate projection, row pitch ldg
+  const float* z;            // delta: decay projection [nd, N D], row pitch ldz
   const void *w0, *w1;       // rows [N, H]: delta step size, - ; memory input gate, forget gate
   const float *b0, *b1;      // memory: their biases [N]
   const float* taps_w[3];    // delta: convolution weights
@@ -752,8 +813,8 @@ struct StepArgs {
   void* out;                 // [nd, N V], row pitch ldo
   const long long* positions;
   const int* slots;
-  long long ldh, ld, ldo;
-  int H, G, N, D, V, R, RG, ntaps, num_slots, per_head;
+  long long ldh, ld, ldz, ldg, ldo;
+  int H, G, N, D, V, ntaps, num_slots, per_head;
   float cap, qscale, eps, scale;
 };
 
@@ -788,23 +849,8 @@ __device__ __forceinline__ float dot_share(const T* x, const T* w, int n, bool v
   return s;
 }
 
-// Four lanes: row . x for x of n (multiple of 8) floats in shared memory.
-template <typename T>
-__device__ __forceinline__ float quad_dot(const T* row, const float* x, int n, int q) {
-  float s = 0.0f;
-  for (int c = q * 8; c < n; c += 32) {
-    float f[8];
-    load8<T>(row + c, f);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) s += f[i] * x[c + i];
-  }
-  s += __shfl_xor_sync(0xffffffffu, s, 1);
-  s += __shfl_xor_sync(0xffffffffu, s, 2);
-  return s;
-}
-
-__host__ __device__ inline int step_floats(int DP, int V, int R, int RG) {
-  return 3 * DP + 3 * ((V + 3) / 4 * 4) + R + RG + 64;
+__host__ __device__ inline int step_floats(int DP, int V) {
+  return 3 * DP + 3 * ((V + 3) / 4 * 4) + 64;
 }
 
 template <typename T, int MODE, int RPL, int CPT>
@@ -819,8 +865,7 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
   float* sv = sg + DP;                            // [V]
   float* so = sv + VS;                            // [V]
   float* sz = so + VS;                            // [V] output gate
-  float* s1 = sz + VS;                            // [R] [RG]
-  float* red = s1 + a.R + a.RG;                   // [64]
+  float* red = sz + VS;                           // [64]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & 7;
   const int r = blockIdx.x, h = blockIdx.y;
   const int kvh = h / (a.N / a.G);
@@ -835,7 +880,7 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
   const long long head_at = static_cast<long long>(slot) * a.N + h;
   const int c_warp = (warp * 4 + (lane >> 3)) * CPT;
 
-  uint64_t S[CPT][P];
+  float2 S[CPT][P];
   auto load_state = [&](int base) {
 #pragma unroll
     for (int j = 0; j < CPT; ++j) {
@@ -844,8 +889,8 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
       const float* src = a.matrix + (head_at * a.V + c) * DP + 4 * l;
 #pragma unroll
       for (int i = 0; i < P / 2; ++i) {
-        ulonglong2 u = make_ulonglong2(0, 0);
-        if (in) u = *reinterpret_cast<const ulonglong2*>(src + 32 * i);
+        Quad u = Quad{both(0.0f), both(0.0f)};
+        if (in) u = *reinterpret_cast<const Quad*>(src + 32 * i);
         S[j][2 * i] = u.x;
         S[j][2 * i + 1] = u.y;
       }
@@ -864,9 +909,15 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
   if (MODE == kMemory)
     d1 = dot_share<T>(hr, static_cast<const T*>(a.w1) + static_cast<long long>(h) * a.H, a.H, vec);
 
+  const T* gz = static_cast<const T*>(a.gate) + static_cast<long long>(r) * a.ldg + h * a.V;
+  for (int c = tid; c < a.V; c += blockDim.x) sz[c] = sigmoid_t<T>(to_f32<T>(gz[c]));
   if (MODE == kDelta) {
     const int C = 2 * a.G * a.D + a.N * a.V;
-    T* ring = static_cast<T*>(a.taps) + static_cast<long long>(slot) * a.ntaps * C;
+    const T* ring = static_cast<const T*>(a.taps) + static_cast<long long>(slot) * a.ntaps * C;
+    const float rate = expf(a.a_log[h]);
+    const float* z = a.z + r * a.ldz + h * a.D;
+    for (int d = tid; d < DP; d += blockDim.x)
+      sg[d] = d < a.D ? exp_t<T>(-rate * softplus_t<T>(z[d] + a.dt_bias[h * a.D + d])) : 0.0f;
     for (int e = tid; e < 2 * DP + a.V; e += blockDim.x) {
       const int which = e < DP ? 0 : e < 2 * DP ? 1 : 2;
       const int d = which == 0 ? e : which == 1 ? e - DP : e - 2 * DP;
@@ -876,29 +927,23 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
         const int ch = head * dim + d;
         const int at = ch + (which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D);
         const float* w = a.taps_w[which] + static_cast<long long>(ch) * a.ntaps;
-        const T now = static_cast<const T*>(a.x[which])[xrow + ch];
-        float s = w[a.ntaps - 1] * to_f32<T>(now);
+        float s = w[a.ntaps - 1] * to_f32<T>(static_cast<const T*>(a.x[which])[xrow + ch]);
+#pragma unroll 3
         for (int o = 1; o < a.ntaps; ++o)
           if (pos - o >= 0)
             s += w[a.ntaps - 1 - o] * to_f32<T>(ring[(pos - o) % a.ntaps * C + at]);
         f = silu<T>(s);
-        if (a.ntaps > 1 && (which == 2 || h % (a.N / a.G) == 0)) ring[pos % a.ntaps * C + at] = now;
       }
       (which == 0 ? sq : which == 1 ? sk : sv)[d] = f;
     }
-    for (int e = tid; e < a.R; e += blockDim.x) s1[e] = to_f32<T>(static_cast<const T*>(a.r1)[xrow + e]);
-    for (int e = tid; e < a.RG; e += blockDim.x)
-      s1[a.R + e] = to_f32<T>(static_cast<const T*>(a.g1)[xrow + e]);
   } else {
     for (int d = tid; d < DP; d += blockDim.x) {
       const bool in = d < a.D;
       sq[d] = in ? to_f32<T>(static_cast<const T*>(a.x[0])[xrow + h * a.D + d]) * a.qscale : 0.0f;
       sk[d] = in ? to_f32<T>(static_cast<const T*>(a.x[1])[xrow + h * a.D + d]) : 0.0f;
     }
-    for (int c = tid; c < a.V; c += blockDim.x) {
+    for (int c = tid; c < a.V; c += blockDim.x)
       sv[c] = to_f32<T>(static_cast<const T*>(a.x[2])[xrow + h * a.V + c]);
-      sz[c] = sigmoid(to_f32<T>(static_cast<const T*>(a.gate)[xrow + h * a.V + c]));
-    }
   }
   const float z0 = block_sum(d0, red);            // (synchronises: the shared rows are complete)
   const float z1 = MODE == kMemory ? block_sum(d1, red) : 0.0f;
@@ -906,31 +951,23 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
   float beta = 0.0f, keep = 0.0f, add = 0.0f, den = 1.0f;
   if (MODE == kDelta) {
     beta = sigmoid(z0);
-    // unit vectors (warps 0 and 1), then decays and the output gate, four lanes per row
-    if (warp < 2) {
+    if (warp < 2) {                               // unit vectors
       float* x = warp == 0 ? sq : sk;
       float ss = 0.0f;
       for (int d = lane; d < DP; d += 32) ss += x[d] * x[d];
       float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
       if (warp == 0) inv *= 1.0f / sqrtf(static_cast<float>(a.D));
       for (int d = lane; d < DP; d += 32) x[d] *= inv;
-    }
-    const float rate = expf(a.a_log[h]);
-    const int rows = DP + a.V, quad = lane >> 2;
-    for (int e0 = warp * 8; e0 < rows; e0 += 64) {
-      const int e = e0 + quad;
-      const bool decay = e < DP;
-      const int d = decay ? e : e - DP;
-      const bool in = decay ? d < a.D : e < rows;
-      // rows outside read row 0 of the head, so that all four lanes take part in the sum
-      const T* row = decay ? static_cast<const T*>(a.r2) +
-                                 (static_cast<long long>(h) * a.D + (in ? d : 0)) * a.R
-                           : static_cast<const T*>(a.g2) +
-                                 (static_cast<long long>(h) * a.V + (in ? d : 0)) * a.RG;
-      const float s = quad_dot<T>(row, decay ? s1 : s1 + a.R, decay ? a.R : a.RG, lane & 3);
-      if ((lane & 3) == 0) {
-        if (decay) sg[d] = in ? expf(-rate * softplus(s + a.dt_bias[h * a.D + d])) : 0.0f;
-        else if (in) sz[d] = sigmoid(to_f32<T>(from_f32<T>(s)));
+    } else if (a.ntaps > 1) {                     // this token's row of the convolution state
+      const int C = 2 * a.G * a.D + a.N * a.V;
+      T* row = static_cast<T*>(a.taps) + (static_cast<long long>(slot) * a.ntaps + pos % a.ntaps) * C;
+      for (int d = tid - 64; d < a.V; d += blockDim.x - 64)
+        row[2 * a.G * a.D + h * a.V + d] = static_cast<const T*>(a.x[2])[xrow + h * a.V + d];
+      if (h % (a.N / a.G) == 0) {
+        for (int d = tid - 64; d < a.D; d += blockDim.x - 64) {
+          row[kvh * a.D + d] = static_cast<const T*>(a.x[0])[xrow + kvh * a.D + d];
+          row[(a.G + kvh) * a.D + d] = static_cast<const T*>(a.x[1])[xrow + kvh * a.D + d];
+        }
       }
     }
     __syncthreads();
@@ -960,12 +997,12 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
 #pragma unroll
     for (int j = 0; j < CPT; ++j) {
       v[j] = c0 + j < a.V ? sv[c0 + j] : 0.0f;
-      uint64_t e0 = 0, e1 = 0;
+      float2 e0 = both(0.0f), e1 = both(0.0f);
       if (MODE == kDelta) {
 #pragma unroll
         for (int u = 0; u < P / 2; ++u) {
-          const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(sg + 4 * l + 32 * u);
-          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(sk + 4 * l + 32 * u);
+          const Quad g = *reinterpret_cast<const Quad*>(sg + 4 * l + 32 * u);
+          const Quad k = *reinterpret_cast<const Quad*>(sk + 4 * l + 32 * u);
           S[j][2 * u] = mul2(S[j][2 * u], g.x);
           S[j][2 * u + 1] = mul2(S[j][2 * u + 1], g.y);
           e0 = fma2(S[j][2 * u], k.x, e0);
@@ -983,13 +1020,13 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
     }
 #pragma unroll
     for (int j = 0; j < CPT; ++j) {
-      const uint64_t u2 = both(MODE == kDelta ? beta * (v[j] - d[j]) : add * v[j]);
-      const uint64_t a2 = both(keep);
-      uint64_t e0 = 0, e1 = 0;
+      const float2 u2 = both(MODE == kDelta ? beta * (v[j] - d[j]) : add * v[j]);
+      const float2 a2 = both(keep);
+      float2 e0 = both(0.0f), e1 = both(0.0f);
 #pragma unroll
       for (int u = 0; u < P / 2; ++u) {
-        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(sk + 4 * l + 32 * u);
-        const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(sq + 4 * l + 32 * u);
+        const Quad k = *reinterpret_cast<const Quad*>(sk + 4 * l + 32 * u);
+        const Quad q = *reinterpret_cast<const Quad*>(sq + 4 * l + 32 * u);
         if (MODE == kMemory) {
           S[j][2 * u] = mul2(S[j][2 * u], a2);
           S[j][2 * u + 1] = mul2(S[j][2 * u + 1], a2);
@@ -1004,8 +1041,8 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
         float* dst = a.matrix + (head_at * a.V + c0 + j) * DP + 4 * l;
 #pragma unroll
         for (int i = 0; i < P / 2; ++i)
-          *reinterpret_cast<ulonglong2*>(dst + 32 * i) =
-              make_ulonglong2(S[j][2 * i], S[j][2 * i + 1]);
+          *reinterpret_cast<Quad*>(dst + 32 * i) =
+              Quad{S[j][2 * i], S[j][2 * i + 1]};
       }
     }
 #pragma unroll
@@ -1032,7 +1069,7 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
 
 template <typename T, int MODE, int RPL, int CPT>
 static int launch_step(const StepArgs& a, int requests, cudaStream_t s) {
-  const int smem = step_floats(8 * RPL, a.V, a.R, a.RG) * static_cast<int>(sizeof(float));
+  const int smem = step_floats(8 * RPL, a.V) * static_cast<int>(sizeof(float));
   if (smem > 48 * 1024) return -20;
   recurrent_step_kernel<T, MODE, RPL, CPT><<<dim3(requests, a.N), 256, smem, s>>>(a);
   return static_cast<int>(cudaGetLastError());
@@ -1086,7 +1123,11 @@ B200_API int b200_delta_inputs(const void* xq, const void* xk, const void* xv, l
   a.ld = ld; a.ldz = ldz; a.ldb = ldb; a.T = T; a.G = G; a.N = N; a.D = D; a.V = V; a.DP = DP;
   a.VP = VP; a.ntaps = ntaps; a.num_slots = num_slots; a.nd = nd; a.np = np;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const dim3 grid((T + kStrip - 1) / kStrip, (2 * G + 2 * N + 7) / 8);
+  // few tokens: the items of a strip go to several CTAs
+  const int strips = (T + kStrip - 1) / kStrip, most = (2 * G + 2 * N + 7) / 8;
+  int split = (4 * sm_count() + strips - 1) / strips;
+  if (split > most) split = most;
+  const dim3 grid(strips, split);
   const uintptr_t x = reinterpret_cast<uintptr_t>(xq) | reinterpret_cast<uintptr_t>(xk) |
                       reinterpret_cast<uintptr_t>(xv) | reinterpret_cast<uintptr_t>(taps);
   const bool v4 = (D % 4) == 0 && (V % 4) == 0 && (VP % 4) == 0 && (ld % 4) == 0 &&
@@ -1204,28 +1245,26 @@ B200_API int b200_head_norm_gate(const float* o, const float* nq, const float* l
   return static_cast<int>(cudaGetLastError());
 }
 
-// One token of `nd` requests through the gated delta rule, from the wide projections to the gated
-// output: r1 / g1 (views of the same rows as q, k, v, R and RG columns, multiples of 8) are the
-// first steps of the decay and gate projections, r2 [N D, R] and g2 [N V, RG] the second ones,
-// wb [N, H] the step size's.  dtype: 0 bf16, 2 fp32.  -20: not covered (very wide second steps).
+// One token of `nd` requests through the gated delta rule, from the projections to the gated
+// output: z [nd, N D] fp32 is the decay's projection, gate [nd, N V] the output gate's, wb [N, H] the
+// weights of the step size's.  dtype: 0 bf16, 2 fp32.  -20: not covered (very wide heads).
 B200_API int b200_delta_step(const void* h, long long ldh, int H, const void* xq, const void* xk,
-                             const void* xv, const void* r1, const void* g1, long long ld,
-                             const void* r2, int R, const void* g2, int RG, const void* wb,
-                             const float* wq, const float* wk, const float* wv, int ntaps,
-                             const float* dt_bias, const float* a_log, const float* norm,
-                             void* taps, float* matrix, const long long* positions,
-                             const int* slots, int num_slots, void* out, long long ldo, float eps,
-                             float scale, int nd, int G, int N, int D, int V, int DP, int dtype,
-                             void* stream) {
+                             const void* xv, long long ld, const float* z, long long ldz,
+                             const void* gate, long long ldg, const void* wb, const float* wq,
+                             const float* wk, const float* wv, int ntaps, const float* dt_bias,
+                             const float* a_log, const float* norm, void* taps, float* matrix,
+                             const long long* positions, const int* slots, int num_slots, void* out,
+                             long long ldo, float eps, float scale, int nd, int G, int N, int D,
+                             int V, int DP, int dtype, void* stream) {
   if (nd <= 0) return 0;
-  if (G <= 0 || N <= 0 || N % G != 0 || D <= 0 || D > DP || V <= 0 || H <= 0 || (R % 8) != 0 ||
-      (RG % 8) != 0 || ntaps < 1 || (dtype != 0 && dtype != 2))
+  if (G <= 0 || N <= 0 || N % G != 0 || D <= 0 || D > DP || V <= 0 || H <= 0 || ntaps < 1 ||
+      (dtype != 0 && dtype != 2))
     return -2;
   StepArgs a{};
-  a.hrow = h; a.ldh = ldh; a.H = H; a.x[0] = xq; a.x[1] = xk; a.x[2] = xv; a.r1 = r1; a.g1 = g1;
-  a.ld = ld; a.r2 = r2; a.R = R; a.g2 = g2; a.RG = RG; a.w0 = wb; a.taps_w[0] = wq;
-  a.taps_w[1] = wk; a.taps_w[2] = wv; a.ntaps = ntaps; a.dt_bias = dt_bias; a.a_log = a_log;
-  a.norm = norm; a.taps = taps; a.matrix = matrix; a.positions = positions; a.slots = slots;
+  a.hrow = h; a.ldh = ldh; a.H = H; a.x[0] = xq; a.x[1] = xk; a.x[2] = xv; a.ld = ld; a.z = z;
+  a.ldz = ldz; a.gate = gate; a.ldg = ldg; a.w0 = wb; a.taps_w[0] = wq; a.taps_w[1] = wk;
+  a.taps_w[2] = wv; a.ntaps = ntaps; a.dt_bias = dt_bias; a.a_log = a_log; a.norm = norm;
+  a.taps = taps; a.matrix = matrix; a.positions = positions; a.slots = slots;
   a.num_slots = num_slots; a.out = out; a.ldo = ldo; a.eps = eps; a.scale = scale; a.G = G;
   a.N = N; a.D = D; a.V = V;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -1246,7 +1285,7 @@ B200_API int b200_memory_step(const void* h, long long ldh, int H, const void* x
   if (N <= 0 || D <= 0 || D > DP || V <= 0 || H <= 0 || (dtype != 0 && dtype != 2)) return -2;
   StepArgs a{};
   a.hrow = h; a.ldh = ldh; a.H = H; a.x[0] = xq; a.x[1] = xk; a.x[2] = xv; a.gate = gate;
-  a.ld = ld; a.w0 = wi; a.w1 = wf; a.b0 = ib; a.b1 = fb; a.cap = cap; a.qscale = qscale;
+  a.ldg = ld; a.ld = ld; a.w0 = wi; a.w1 = wf; a.b0 = ib; a.b1 = fb; a.cap = cap; a.qscale = qscale;
   a.norm = norm; a.per_head = 1; a.matrix = matrix; a.vector = vector; a.scalar = scalar;
   a.positions = positions; a.slots = slots; a.num_slots = num_slots; a.out = out; a.ldo = ldo;
   a.eps = eps; a.scale = scale; a.G = N; a.N = N; a.D = D; a.V = V;

@@ -364,7 +364,10 @@ __global__ void __launch_bounds__(512)
     ldv<V>(o + (t * N + h) * DC + c, a);
     ldv<V>(z + t * ldz + e, g);
 #pragma unroll
-    for (int k = 0; k < V; ++k) a[k] = a[k] * scale / (1.0f + expf(-g[k]));
+    for (int k = 0; k < V; ++k) {
+      if constexpr (sizeof(T) == 2) a[k] = __fdividef(a[k] * scale, 1.0f + __expf(-g[k]));
+      else a[k] = a[k] * scale / (1.0f + expf(-g[k]));
+    }
     stv<V>(out + t * ldout + e, a);
   }
 }

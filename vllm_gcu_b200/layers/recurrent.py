@@ -113,18 +113,18 @@ class GatedDelta(MixerPart):
         q, k, v, a1, g1 = y["q"][:, :nk], y["k"][:, :nk], y["v"][:, :nv], y["a1"], y["g1"]
         conv = (self.conv_q, self.conv_k, self.conv_v)
         sizes = s.head_dim, s.v_head_dim, self.rows
+        z, gate = linear_fp32(a1, self.a2), linear(g1, self.g2)
         n1 = fused_tokens(h, md)
         if n1:
-            C.delta_step(h[:n1], q[:n1], k[:n1], v[:n1], a1[:n1], g1[:n1], self.a2, self.g2,
-                         fw["b"], conv, self.dt_bias, self.a_log, self.norm, *sizes, md.positions,
+            C.delta_step(h[:n1], q[:n1], k[:n1], v[:n1], z[:n1], gate[:n1], fw["b"], conv,
+                         self.dt_bias, self.a_log, self.norm, *sizes, md.positions,
                          md.state_slots, state, self.eps, scale, out[:n1])
         if n1 == h.shape[0]:
             return
         o_ = C if ops.use_native(out) else ref
-        o = o_.delta_rule(q[n1:], k[n1:], v[n1:], linear_fp32(a1[n1:], self.a2), f["b"], conv,
-                          self.dt_bias, self.a_log, *sizes, Place.behind(md, n1),
-                          None if md.is_dummy else state)
-        o_.head_norm_gate(o, self.norm, linear(g1[n1:], self.g2), self.eps, scale, out[n1:])
+        o = o_.delta_rule(q[n1:], k[n1:], v[n1:], z[n1:], f["b"], conv, self.dt_bias, self.a_log,
+                          *sizes, Place.behind(md, n1), None if md.is_dummy else state)
+        o_.head_norm_gate(o, self.norm, gate[n1:], self.eps, scale, out[n1:])
 
 
 class MatrixMemory(MixerPart):

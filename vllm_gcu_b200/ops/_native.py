@@ -151,8 +151,8 @@ class _Sigs:
                        I, P]
     b200_memory_scan = [P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, P]
     b200_head_norm_gate = [P, P, P, P, I, P, L, P, L, F, F, I, I, I, I, P]
-    b200_delta_step = [P, L, I, P, P, P, P, P, L, P, I, P, I, P, P, P, P, I, P, P, P, P, P, P, P, I,
-                       P, L, F, F, I, I, I, I, I, I, I, P]
+    b200_delta_step = [P, L, I, P, P, P, L, P, L, P, L, P, P, P, P, I, P, P, P, P, P, P, P, I, P, L,
+                       F, F, I, I, I, I, I, I, I, P]
     b200_memory_step = [P, L, I, P, P, P, P, L, P, P, P, P, F, F, P, P, P, P, P, P, I, P, L, F, F,
                         I, I, I, I, I, I, P]
     b200_gemm_wna16 = [P, L, P, P, P, P, P, L, I, I, I, I, I, P, P]

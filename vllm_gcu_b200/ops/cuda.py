@@ -967,27 +967,25 @@ def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, z: torch.Tensor, eps: 
 
 
 def delta_step(h: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
-               a1: torch.Tensor, g1: torch.Tensor, a2: torch.Tensor, g2: torch.Tensor,
-               b_weight: torch.Tensor, conv: Sequence[torch.Tensor], dt_bias: torch.Tensor,
-               a_log: torch.Tensor, norm: torch.Tensor, head_dim: int, v_dim: int, rows: int,
-               positions: torch.Tensor, slots: torch.Tensor, state: dict, eps: float, scale: float,
-               out: torch.Tensor) -> torch.Tensor:
+               z: torch.Tensor, gate: torch.Tensor, b_weight: torch.Tensor,
+               conv: Sequence[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor,
+               norm: torch.Tensor, head_dim: int, v_dim: int, rows: int, positions: torch.Tensor,
+               slots: torch.Tensor, state: dict, eps: float, scale: float, out: torch.Tensor
+               ) -> torch.Tensor:
     """One token of every request through the gated delta rule in one kernel: :func:`delta_rule`
-    and :func:`head_norm_gate` with the step sizes (``b_weight [N, H]`` on the mixer's input ``h``),
-    the second steps of the decay and gate projections (``a2``, ``g2``; ``a1``, ``g1`` their inputs,
-    padded to multiples of 8 columns) included."""
+    and :func:`head_norm_gate`, with the step sizes (``b_weight [N, H]`` on the mixer's input ``h``)
+    included.  ``z [nd, N * head_dim]`` fp32: decay projection, ``gate [nd, N * v_dim]``: the
+    output gate's."""
     nd, D, V = h.shape[0], head_dim, v_dim
     G, Nh = q.shape[1] // D, v.shape[1] // V
-    ld = q.stride(0)
-    assert all(t.stride(0) == ld and t.stride(1) == 1 for t in (k, v, a1, g1))
-    assert a1.shape[1] == a2.shape[1] and g1.shape[1] == g2.shape[1] and b_weight.is_contiguous()
+    assert q.stride(0) == k.stride(0) == v.stride(0) and z.dtype == torch.float32
+    assert b_weight.is_contiguous() and gate.dtype == h.dtype
     taps = state["taps"]
-    call("b200_delta_step", ptr(h), h.stride(0), h.shape[1], ptr(q), ptr(k), ptr(v), ptr(a1),
-         ptr(g1), ld, ptr(a2), a2.shape[1], ptr(g2), g2.shape[1], ptr(b_weight), ptr(conv[0]),
-         ptr(conv[1]), ptr(conv[2]), conv[0].shape[1], ptr(dt_bias), ptr(a_log), ptr(norm),
-         ptr(taps), ptr(state["matrix"]), ptr(positions), ptr(slots), taps.shape[0], ptr(out),
-         out.stride(0), float(eps), float(scale), nd, G, Nh, D, V, rows, DTYPE_CODE[h.dtype],
-         stream_ptr())
+    call("b200_delta_step", ptr(h), h.stride(0), h.shape[1], ptr(q), ptr(k), ptr(v), q.stride(0),
+         ptr(z), z.stride(0), ptr(gate), gate.stride(0), ptr(b_weight), ptr(conv[0]), ptr(conv[1]),
+         ptr(conv[2]), conv[0].shape[1], ptr(dt_bias), ptr(a_log), ptr(norm), ptr(taps),
+         ptr(state["matrix"]), ptr(positions), ptr(slots), taps.shape[0], ptr(out), out.stride(0),
+         float(eps), float(scale), nd, G, Nh, D, V, rows, DTYPE_CODE[h.dtype], stream_ptr())
     return out
 
 
