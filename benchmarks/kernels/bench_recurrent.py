@@ -71,7 +71,7 @@ def cases(lens: list[int], ctx: int, decode: bool, H: int, N: int, G: int, D: in
     wide = rnd(T, 3 * N * D + 256).to(bf)
     q, k, v = (wide[:, i * N * D:(i + 1) * N * D] for i in range(3))
     z, bz = rnd(T, N * D), rnd(T, N)
-    conv = tuple(rnd(N * D, ntaps) for _ in range(3))
+    conv = tuple(rnd(ntaps, N * D) for _ in range(3))
     st = {"matrix": torch.zeros(B, N, D, D, device=dev),
           "taps": torch.zeros(B, ntaps, 3 * N * D, device=dev, dtype=bf)}
     dtb, alog = torch.full((N * D,), -4.0, device=dev), torch.zeros(N, device=dev)

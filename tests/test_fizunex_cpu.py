@@ -87,7 +87,7 @@ def _delta_inputs(N, G, D, V, taps, T, seed):
     g = gen(seed)
     r = lambda *s: torch.randn(*s, generator=g)  # noqa: E731
     return dict(q=r(T, G * D), k=r(T, G * D), v=r(T, N * V), z=r(T, N * D) - 1, b=r(T, N),
-                conv=tuple(0.7 * r(n, taps) for n in (G * D, G * D, N * V)),
+                conv=tuple(0.7 * r(taps, n) for n in (G * D, G * D, N * V)),
                 dt_bias=r(N * D), a_log=r(N))
 
 
@@ -95,7 +95,7 @@ def _delta_want(x, N, G, D, V):
     d = {k: (tuple(t.double() for t in v) if isinstance(v, tuple) else v.double())
          for k, v in x.items()}
     T = d["q"].shape[0]
-    q, k, v = (O.silu(O.short_conv(d[c], t)) for c, t in zip("qkv", d["conv"]))
+    q, k, v = (O.silu(O.short_conv(d[c], t.T)) for c, t in zip("qkv", d["conv"]))
     step = O.softplus(d["z"] + d["dt_bias"]).view(T, N, D)
     return O.delta_rule(O.unit(q.view(T, G, D)) * D ** -0.5, O.unit(k.view(T, G, D)),
                         v.view(T, N, V), torch.exp(-torch.exp(d["a_log"])[None, :, None] * step),

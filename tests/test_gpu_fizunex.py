@@ -208,7 +208,7 @@ def _delta_case(N, G, D, V, taps, step, dtype, seed):
     pad = (-C_) % 8
     wide = r(step.T, C_ + pad + 8).to(dtype)
     kw = dict(z=r(step.T, N * D) - 1, b=r(step.T, N),
-              conv=tuple(0.7 * r(n, taps) for n in (G * D, G * D, N * V)), dt_bias=r(N * D),
+              conv=tuple(0.7 * r(taps, n) for n in (G * D, G * D, N * V)), dt_bias=r(N * D),
               a_log=r(N))
     state = {"matrix": torch.zeros(8, N, V, rows), "taps": r(8, taps, C_).to(dtype)}
     state["matrix"][..., :D] = r(8, N, V, D)

@@ -55,12 +55,16 @@ template <typename T>
 __device__ __forceinline__ float softplus_t(float z) {
   if constexpr (sizeof(T) == 2) {
     const float e = __expf(-fabsf(z));
-    const float l = e < 0.02f ? e * (1.0f - e * (0.5f - e * (1.0f / 3.0f - e * 0.25f)))
-                              : __logf(1.0f + e);
+    const float l = e < 0.02f ? fmaf(e * e, fmaf(e, 1.0f / 3.0f, -0.5f), e) : __logf(1.0f + e);
     return fmaxf(z, 0.0f) + l;
   } else {
     return softplus(z);
   }
+}
+template <typename T>
+__device__ __forceinline__ float inv_root(float z) {
+  if constexpr (sizeof(T) == 2) return rsqrtf(z);
+  else return 1.0f / sqrtf(z);
 }
 template <typename T>
 __device__ __forceinline__ float exp_t(float z) {
@@ -96,7 +100,7 @@ __device__ __forceinline__ Portion portion_of(int r, int nd, const int* cu_q) {
 // ---------------------------------------------------------------------------
 struct DeltaIn {
   const void* x[3];          // q, k, v projections [T, channels] (views), row pitch ld
-  const float* taps_w[3];    // [channels, taps] convolution weights, last column: current token
+  const float* taps_w[3];    // [taps, channels] convolution weights, last row: current token
   const void* taps;          // state: [slots, taps, C] with C = all channels, q | k | v
   const float* z;            // [T, N * D] decay projection
   const float* bz;           // [T, N] step size projection
@@ -127,6 +131,30 @@ __device__ __forceinline__ void load_n(const T* p, float (&f)[V]) {
     f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
   } else {
     f[0] = to_f32<T>(p[0]);
+  }
+}
+// V elements as they lie in memory
+template <typename T, int V>
+struct Raw {
+  T e;
+};
+template <>
+struct Raw<__nv_bfloat16, 4> {
+  uint2 e;
+};
+template <>
+struct Raw<float, 4> {
+  float4 e;
+};
+template <typename T, int V>
+__device__ __forceinline__ void unpack_raw(const Raw<T, V>& r, float (&f)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    const float2 a = unpack_bf16x2(r.e.x), b = unpack_bf16x2(r.e.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else if constexpr (V == 4) {
+    f[0] = r.e.x; f[1] = r.e.y; f[2] = r.e.z; f[3] = r.e.w;
+  } else {
+    f[0] = to_f32<T>(r.e);
   }
 }
 template <int V>
@@ -165,6 +193,7 @@ __global__ void __launch_bounds__(256, 2) delta_inputs_kernel(const DeltaIn a) {
   }
   __syncthreads();
   const int C = 2 * a.G * a.D + a.N * a.V;
+  const float qscale = 1.0f / sqrtf(static_cast<float>(a.D));
   for (int item = blockIdx.y * 8 + warp; item < 2 * a.G + 2 * a.N; item += gridDim.y * 8) {
     if (item >= 2 * a.G + a.N) {                   // decays and step sizes
       const int h = item - 2 * a.G - a.N;
@@ -198,7 +227,8 @@ __global__ void __launch_bounds__(256, 2) delta_inputs_kernel(const DeltaIn a) {
     const int dim = which == 2 ? a.V : a.D, pitch = which == 2 ? a.VP : a.DP;
     const int ring_off = (which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D) + head * dim;
     const T* x = static_cast<const T*>(a.x[which]) + head * dim;
-    const float* wt = a.taps_w[which] + static_cast<long long>(head) * dim * a.ntaps;
+    const float* wt = a.taps_w[which] + head * dim;
+    const int wld = (which == 2 ? a.N : a.G) * dim;
     float* out = (which == 0 ? a.q : which == 1 ? a.k : a.v) + head * pitch;
     const long long ldo = static_cast<long long>(which == 2 ? a.N : a.G) * pitch;
     const int passes = (pitch + 32 * V - 1) / (32 * V);
@@ -209,20 +239,20 @@ __global__ void __launch_bounds__(256, 2) delta_inputs_kernel(const DeltaIn a) {
       for (int ps = 0; ps < passes; ++ps) {
         const int d = (ps * 32 + lane) * V;
         const bool in = d < dim;
-        float rows[kStrip][V];                     // all rows of the strip in flight at once
+        Raw<T, V> rows[kStrip];                    // all rows of the strip in flight at once
 #pragma unroll
         for (int u = 0; u < kStrip; ++u) {
-#pragma unroll
-          for (int i = 0; i < V; ++i) rows[u][i] = 0.0f;
+          rows[u] = Raw<T, V>{};
           if (in && t0 + u < t1)
-            load_n<T, V>(x + static_cast<long long>(t0 + u) * a.ld + d, rows[u]);
+            rows[u] = *reinterpret_cast<const Raw<T, V>*>(
+                x + static_cast<long long>(t0 + u) * a.ld + d);
         }
         float w[NT][V];                            // [o]: tap that meets the input of o tokens ago
 #pragma unroll
         for (int o = 0; o < NT; ++o) {
 #pragma unroll
-          for (int i = 0; i < V; ++i)
-            w[o][i] = in && o < a.ntaps ? wt[(d + i) * a.ntaps + a.ntaps - 1 - o] : 0.0f;
+          for (int i = 0; i < V; ++i) w[o][i] = 0.0f;
+          if (in && o < a.ntaps) load_n<float, V>(wt + (a.ntaps - 1 - o) * wld + d, w[o]);
         }
         float past[NT][V];                         // [o]: input of o tokens ago
 #pragma unroll
@@ -257,29 +287,38 @@ __global__ void __launch_bounds__(256, 2) delta_inputs_kernel(const DeltaIn a) {
 #pragma unroll
             for (int i = 0; i < V; ++i) past[o][i] = past[o - 1][i];
           }
-#pragma unroll
-          for (int i = 0; i < V; ++i) past[0][i] = rows[u][i];
+          unpack_raw<T, V>(rows[u], past[0]);
           float f[V], ss = 0.0f;
+          if constexpr (V == 4) {
+            float2 c0 = both(0.0f), c1 = both(0.0f);
+#pragma unroll
+            for (int o = NT - 1; o >= 0; --o) {
+              c0 = fma2(make_float2(w[o][0], w[o][1]), make_float2(past[o][0], past[o][1]), c0);
+              c1 = fma2(make_float2(w[o][2], w[o][3]), make_float2(past[o][2], past[o][3]), c1);
+            }
+            f[0] = c0.x; f[1] = c0.y; f[2] = c1.x; f[3] = c1.y;
+          } else {
+            f[0] = 0.0f;
+#pragma unroll
+            for (int o = NT - 1; o >= 0; --o) f[0] += w[o][0] * past[o][0];
+          }
 #pragma unroll
           for (int i = 0; i < V; ++i) {
-            float c = 0.0f;
-#pragma unroll
-            for (int o = NT - 1; o >= 0; --o) c += w[o][i] * past[o][i];
-            f[i] = silu<T>(c);
+            f[i] = silu<T>(f[i]);
             ss += f[i] * f[i];
           }
           if (unit) {
             float inv;
             if (passes == 1) {
-              inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
+              inv = inv_root<T>(warp_sum(ss) + 1e-6f);
             } else if (walk == 0) {
               const float sum = warp_sum(ss);
               inv_sum[u] = ps == 0 ? sum : inv_sum[u] + sum;
               continue;
             } else {
-              inv = 1.0f / sqrtf(inv_sum[u] + 1e-6f);
+              inv = inv_root<T>(inv_sum[u] + 1e-6f);
             }
-            if (which == 0) inv *= 1.0f / sqrtf(static_cast<float>(a.D));
+            if (which == 0) inv *= qscale;
 #pragma unroll
             for (int i = 0; i < V; ++i) f[i] *= inv;
           }
@@ -926,12 +965,13 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
       if (d < dim) {
         const int ch = head * dim + d;
         const int at = ch + (which == 0 ? 0 : which == 1 ? a.G * a.D : 2 * a.G * a.D);
-        const float* w = a.taps_w[which] + static_cast<long long>(ch) * a.ntaps;
-        float s = w[a.ntaps - 1] * to_f32<T>(static_cast<const T*>(a.x[which])[xrow + ch]);
+        const float* w = a.taps_w[which] + ch;
+        const int wld = (which == 2 ? a.N : a.G) * dim;
+        float s = w[(a.ntaps - 1) * wld] * to_f32<T>(static_cast<const T*>(a.x[which])[xrow + ch]);
 #pragma unroll 3
         for (int o = 1; o < a.ntaps; ++o)
           if (pos - o >= 0)
-            s += w[a.ntaps - 1 - o] * to_f32<T>(ring[(pos - o) % a.ntaps * C + at]);
+            s += w[(a.ntaps - 1 - o) * wld] * to_f32<T>(ring[(pos - o) % a.ntaps * C + at]);
         f = silu<T>(s);
       }
       (which == 0 ? sq : which == 1 ? sk : sv)[d] = f;
@@ -1132,7 +1172,8 @@ B200_API int b200_delta_inputs(const void* xq, const void* xk, const void* xv, l
                       reinterpret_cast<uintptr_t>(xv) | reinterpret_cast<uintptr_t>(taps);
   const bool v4 = (D % 4) == 0 && (V % 4) == 0 && (VP % 4) == 0 && (ld % 4) == 0 &&
                   (ldz % 4) == 0 && (x % (dtype == 0 ? 8 : 16)) == 0 &&
-                  (reinterpret_cast<uintptr_t>(z) % 16) == 0;
+                  ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(wq) |
+                    reinterpret_cast<uintptr_t>(wk) | reinterpret_cast<uintptr_t>(wv)) % 16) == 0;
 #define B200_IN(NT, W)                                                             \
   do {                                                                             \
     if (dtype == 0) delta_inputs_kernel<__nv_bfloat16, NT, W><<<grid, 256, 0, s>>>(a); \

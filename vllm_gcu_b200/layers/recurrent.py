@@ -74,8 +74,8 @@ class GatedDelta(MixerPart):
                             ("a1", spec.decay_rank, False), ("g1", spec.gate_rank, False)]
         self.fp32_projections = [("b", N, True)]
         new = lambda *s, dt=torch.float32: self.new(*s, dtype=dt, device=device)  # noqa: E731
-        self.conv_q, self.conv_k = (new(self.G * D, spec.conv_taps) for _ in range(2))
-        self.conv_v = new(self.N * V, spec.conv_taps)
+        self.conv_q, self.conv_k = (new(spec.conv_taps, self.G * D) for _ in range(2))
+        self.conv_v = new(spec.conv_taps, self.N * V)
         self.a_log, self.dt_bias = new(self.N), new(self.N * D)
         self.norm = new(V)
         pad = lambda n: -(-n // 8) * 8  # noqa: E731
@@ -99,6 +99,8 @@ class GatedDelta(MixerPart):
             return False
         p = getattr(self, self._OWN[name]).data
         t = full if name == "norm" else self.shard(full)
+        if name.endswith(".conv"):
+            t = t.t()
         (p[:, :t.shape[1]] if name in ("a2", "g2") else p).copy_(t)
         return True
 

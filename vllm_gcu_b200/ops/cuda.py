@@ -893,13 +893,13 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tenso
                state: Optional[dict]) -> torch.Tensor:
     """Gated delta rule with one decay per key channel over the portions of a step: q, k ``[T, G *
     head_dim]`` and v ``[T, N * v_dim]`` are projections (views of one row), ``z [T, N * head_dim]``
-    and ``b [T, N]`` fp32.  ``state``: ``matrix [slots, N, v_dim, rows]`` fp32 and ``taps [slots,
+    and ``b [T, N]`` fp32, ``conv``: weights ``[taps, channels]`` of q, k and v.  ``state``: ``matrix [slots, N, v_dim, rows]`` fp32 and ``taps [slots,
     taps, channels]``, addressed by ``md.state_slots``; ``md`` also gives ``positions``,
     ``num_decode_tokens`` and ``cu_q_prefill``.  Returns fp32 ``[T, N, v_dim]``."""
     T, D, V = q.shape[0], head_dim, v_dim
     G, Nh = q.shape[1] // D, v.shape[1] // V
     VP = -(-V // 4) * 4
-    ntaps = conv[0].shape[1]
+    ntaps = conv[0].shape[0]
     assert q.stride(0) == k.stride(0) == v.stride(0) and z.dtype == b.dtype == torch.float32
     new = lambda *s: torch.empty(s, dtype=torch.float32, device=q.device)  # noqa: E731
     qo, ko, go, vo, beta = new(T, G, rows), new(T, G, rows), new(T, Nh, rows), new(T, Nh, VP), \
@@ -983,7 +983,7 @@ def delta_step(h: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tenso
     taps = state["taps"]
     call("b200_delta_step", ptr(h), h.stride(0), h.shape[1], ptr(q), ptr(k), ptr(v), q.stride(0),
          ptr(z), z.stride(0), ptr(gate), gate.stride(0), ptr(b_weight), ptr(conv[0]), ptr(conv[1]),
-         ptr(conv[2]), conv[0].shape[1], ptr(dt_bias), ptr(a_log), ptr(norm), ptr(taps),
+         ptr(conv[2]), conv[0].shape[0], ptr(dt_bias), ptr(a_log), ptr(norm), ptr(taps),
          ptr(state["matrix"]), ptr(positions), ptr(slots), taps.shape[0], ptr(out), out.stride(0),
          float(eps), float(scale), nd, G, Nh, D, V, rows, DTYPE_CODE[h.dtype], stream_ptr())
     return out

@@ -766,8 +766,8 @@ def delta_rule(q, k, v, z, b, conv, dt_bias, a_log, head_dim, v_dim, rows, md, s
     out = torch.zeros(T, Nh, V, dtype=torch.float32, device=q.device)
     if state is None:
         return out
-    n = conv[0].shape[1]
-    taps = torch.cat(list(conv)).float()                      # [channels, n]
+    n = conv[0].shape[0]
+    taps = torch.cat(list(conv), dim=1).float()               # [n, channels]
     x = torch.cat([q, k, v], dim=1)
     decay = torch.exp(-torch.exp(a_log.float())[None, :, None] * torch.nn.functional.softplus(
         z + dt_bias).view(T, Nh, D))
@@ -776,10 +776,10 @@ def delta_rule(q, k, v, z, b, conv, dt_bias, a_log, head_dim, v_dim, rows, md, s
     for lo, hi, slot, fresh in _recurrent_portions(T, md):
         p0 = int(md.positions[lo])
         ring = state["taps"][slot]
-        past = [ring[p % n].float() if p >= 0 else torch.zeros_like(taps[:, 0])
+        past = [ring[p % n].float() if p >= 0 else torch.zeros_like(taps[0])
                 for p in range(p0 - n + 1, p0)]
         seq = torch.cat([torch.stack(past), x[lo:hi].float()]) if past else x[lo:hi].float()
-        c = sum(seq[j:j + hi - lo] * taps[:, j] for j in range(n))
+        c = sum(seq[j:j + hi - lo] * taps[j] for j in range(n))
         c = torch.nn.functional.silu(c)
         qc = unit(c[:, :G * D].view(-1, G, D)) * D ** -0.5
         kc = unit(c[:, G * D:2 * G * D].view(-1, G, D))
