@@ -475,36 +475,40 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
   const bool fresh = a.positions[po.first] == 0;
   const bool warp_on = z * a.cols + warp * kGroups * CPT < columns;    // a column for this warp
 
-  // tokens [i0, i0 + kChunk) of the portion -> stage b
+  // tokens [i0, i0 + kChunk) of the portion -> stage b: a warp copies the rows of one token at a
+  // time (address arithmetic counts here: with few heads a warp has a scheduler for itself)
+  const int warps = blockDim.x >> 5;
+  const long long qk_step = static_cast<long long>(a.G) * DP, g_step = static_cast<long long>(a.N) * DP;
+  const long long v_step = static_cast<long long>(a.N) * a.VP;
+  const float* q_src = a.q + po.first * qk_step + kvh * DP + lane * 4;
+  const float* k_src = a.k + po.first * qk_step + kvh * DP + lane * 4;
+  const float* g_src = MODE == kDelta ? a.g + po.first * g_step + h * DP + lane * 4 : nullptr;
+  const float* v_src = a.v + po.first * v_step + static_cast<long long>(h) * a.VP + z * a.cols + lane * 4;
   auto fetch = [&](int i0, int b) {
-    float* s = smem + b * stage;
     const int n = min(kChunk, po.count - i0);
     constexpr int kVec = DP / 4;
-    for (int e = threadIdx.x; e < n * kRows * kVec; e += blockDim.x) {
-      const int i = e / (kRows * kVec), rem = e - i * (kRows * kVec);
-      const int which = rem / kVec, d = (rem - which * kVec) * 4;
-      const long long t = po.first + i0 + i;
-      const float* src = which == 0 ? a.q + (t * a.G + kvh) * DP
-                         : which == 1 ? a.k + (t * a.G + kvh) * DP
-                                      : a.g + (t * a.N + h) * DP;
-      copy16(s + (which * kChunk + i) * DP + d, src + d);
+    float* dst = smem + b * stage + lane * 4;
+#pragma unroll 4
+    for (int i = warp; i < n; i += warps) {
+      const long long t = i0 + i;
+#pragma unroll
+      for (int c = 0; c < kVec; c += 32) {
+        if (kVec % 32 != 0 && lane + c >= kVec) break;
+        copy16(dst + i * DP + c * 4, q_src + t * qk_step + c * 4);
+        copy16(dst + (kChunk + i) * DP + c * 4, k_src + t * qk_step + c * 4);
+        if (MODE == kDelta) copy16(dst + (2 * kChunk + i) * DP + c * 4, g_src + t * g_step + c * 4);
+      }
+      float* dv = dst + kRows * kChunk * DP + i * a.cols;
+      for (int c = lane * 4; c < a.cols; c += 128) {
+        if (z * a.cols + c < a.VP) copy16(dv + c - lane * 4, v_src + t * v_step + c - lane * 4);
+        else *reinterpret_cast<float4*>(dv + c - lane * 4) = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
     }
-    float* sv = s + kRows * kChunk * DP;
-    const int vec = a.cols / 4;
-    for (int e = threadIdx.x; e < n * vec; e += blockDim.x) {
-      const int i = e / vec, c = (e - i * vec) * 4;
-      const int col = z * a.cols + c;
-      if (col < a.VP)
-        copy16(sv + i * a.cols + c,
-               a.v + (static_cast<long long>(po.first + i0 + i) * a.N + h) * a.VP + col);
-      else
-        *reinterpret_cast<float4*>(sv + i * a.cols + c) = make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    float* ss = sv + kChunk * a.cols;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-      const long long at = static_cast<long long>(po.first + i0 + i) * a.N + h;
-      copy4(ss + i, a.s0 + at);
-      if (MODE == kMemory) copy4(ss + kChunk + i, a.s1 + at);
+    float* ss = smem + b * stage + kRows * kChunk * DP + kChunk * a.cols;
+    if (threadIdx.x < n) {
+      const long long at = static_cast<long long>(po.first + i0 + threadIdx.x) * a.N + h;
+      copy4(ss + threadIdx.x, a.s0 + at);
+      if (MODE == kMemory) copy4(ss + kChunk + threadIdx.x, a.s1 + at);
     }
   };
 
