@@ -95,8 +95,9 @@ class KeyAttention(MixerPart):
                                 out=out[:nd], **rest)
         if npf > 0:
             bt, sl = md.block_tables[nr:nr + npf], md.seq_lens[nr:nr + npf]
-            if C.fmha_prefill_sink(q[nd:], kc, vc, bt, md.cu_q_prefill, sl,
-                                   num_q_tiles_128=md.num_q_tiles_128, out=out[nd:], **rest) is None:
+            done = C.fmha_prefill_sink(q[nd:], kc, vc, bt, md.cu_q_prefill, sl, out=out[nd:],
+                                       num_q_tiles_128=md.num_q_tiles_128, **rest)
+            if done is None:
                 C.any_attention(q[nd:], kc, vc, bt, sl, 0, md.cu_q_prefill, out=out[nd:], **rest)
         return out
 

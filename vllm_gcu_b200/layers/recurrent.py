@@ -66,7 +66,8 @@ class GatedDelta(MixerPart):
         if N % G:
             raise ValueError(f"{prefix}: {N} heads over {G} query / key heads")
         if not 1 <= spec.conv_taps <= MAX_TAPS:
-            raise ValueError(f"{prefix}: a convolution of {spec.conv_taps} taps, at most {MAX_TAPS}")
+            raise ValueError(f"{prefix}: a convolution of {spec.conv_taps} taps, at most "
+                             f"{MAX_TAPS}")
         self.N, self.G = _local_heads(N, prefix), _local_heads(G, prefix)
         self.rows = state_rows(D, prefix)
         self.width = N * V
