@@ -28,13 +28,20 @@ def to_dtype(x: Any) -> torch.dtype:
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    """Attention over keys that are their own values (layers/key_attention.py)."""
+    """Attention over cached keys and values (layers/key_attention.py)."""
     num_heads: int
     num_kv_heads: int
     head_dim: int
     scale: float                           # score scale
-    rot_dims: int                          # rotated dimensions of every head
-    rot_base: float
+    rot_dims: int = 0                      # rotated dimensions of every head
+    rot_base: float = 10000.0
+    v_head_dim: int = 0                    # 0: the keys are their own values
+    softcap: float = 0.0                   # scores become softcap * tanh(score / softcap); 0: none
+    chunk: int = 0                         # keys of the query's own chunk of positions; 0: all
+
+    @property
+    def cached_per_token(self) -> int:
+        return self.num_kv_heads * (self.head_dim + (self.v_head_dim or self.head_dim))
 
 
 @dataclass(frozen=True)
@@ -71,6 +78,12 @@ class LayerSpec:
     num_experts_per_tok: int = 0
     moe_intermediate_size: int = 0
     intermediate_size: int = 0             # dense feed-forward
+    shared_intermediate_size: int = 0      # shared expert beside the routed ones
+    router_scale: float = 1.0              # factor of the routing weights
+    rot_dim: int = 0                       # latent attention: rotated query / key dimensions
+    rot_base: float = 10000.0
+    sink: bool = False                     # latent attention: learnt term in the denominator
+    head_gate: bool = False                # latent attention: one gate per head, not per channel
     # mixer as a sum of parts: (checkpoint prefix, factor, spec)
     parts: tuple[tuple[str, float, Any], ...] = ()
 
@@ -81,8 +94,8 @@ class LayerSpec:
     @property
     def cached_per_token(self) -> int:
         """Elements a token leaves in the paged cache."""
-        return self.kv_lora_rank + sum(2 * s.num_kv_heads * s.head_dim for _, _, s in self.parts
-                                       if isinstance(s, AttentionSpec))
+        return self.kv_lora_rank + self.rot_dim + sum(
+            s.cached_per_token for _, _, s in self.parts if isinstance(s, AttentionSpec))
 
 
 @dataclass
@@ -139,6 +152,8 @@ class ModelConfig:
     residual_alpha: float = 1.0            # norm after the sum: norm(alpha * x + sublayer(x))
     embed_scale: float = 1.0
     logit_scale: float = 1.0
+    # (start, stop, times): layers start .. stop - 1 run that often in a row, same weights
+    loop: Optional[tuple[int, int, int]] = None
     extra: dict = field(default_factory=dict)
 
     def __post_init__(self) -> None:
@@ -148,6 +163,10 @@ class ModelConfig:
             n = self.num_hidden_layers
             reps = -(-n // len(self.layer_specs))
             self.layer_specs = (tuple(self.layer_specs) * reps)[:n]
+        if self.loop is not None:
+            start, stop, times = self.loop
+            stop = min(stop, self.num_hidden_layers)
+            self.loop = (start, stop, times) if start < stop else None
         if self.head_dim <= 0:
             self.head_dim = self.hidden_size // self.num_attention_heads
 
@@ -165,6 +184,16 @@ class ModelConfig:
         d = self.qk_rope_head_dim if self.is_mla else self.head_dim
         return int(d * self.partial_rotary_factor)
 
+    @property
+    def layer_runs(self) -> list[tuple[int, Optional[int]]]:
+        """``(layer, pass)`` in the order of execution; ``pass`` is the number of the loop's pass
+        whose first layer this is, else None.  Every run has a cache of its own."""
+        n = self.num_hidden_layers
+        start, stop, times = self.loop or (0, 0, 0)
+        return [(i, None) for i in range(start)] + \
+            [(i, t if i == start else None) for t in range(times) for i in range(start, stop)] + \
+            [(i, None) for i in range(stop, n)]
+
     def is_moe_layer(self, layer_idx: int) -> bool:
         if not self.is_moe or layer_idx < self.first_k_dense_replace \
                 or layer_idx % self.moe_layer_freq != 0:
@@ -179,7 +208,7 @@ class ModelConfig:
         es = 1 if self.kv_cache_dtype.startswith("fp8") or self.kv_cache_dtype == "int8" else \
             torch.empty((), dtype=self.dtype).element_size()
         if self.layer_specs is not None:
-            return sum(s.cached_per_token for s in self.layer_specs) * es
+            return sum(self.layer_specs[i].cached_per_token for i, _ in self.layer_runs) * es
         if self.is_mla:
             return self.num_hidden_layers * (self.kv_lora_rank + self.qk_rope_head_dim) * es
         kvh = max(1, self.num_key_value_heads // tp_size)
@@ -228,6 +257,9 @@ class ModelConfig:
         if d.get("architecture") == "Fizunex" or "FizunexForCausalLM" in (
                 d.get("architectures") or ()):
             return cls._from_mixer_list(d, **overrides)
+        if d.get("architecture") == "Fepopel" or "FepopelForCausalLM" in (
+                d.get("architectures") or ()):
+            return cls._from_looped_list(d, **overrides)
         archs = d.get("architectures") or ["LlamaForCausalLM"]
         for nested in ("text_config", "language_config", "llm_config"):
             if isinstance(d.get(nested), dict):
@@ -415,6 +447,73 @@ class ModelConfig:
         return cls(**kw)
 
     @classmethod
+    def _from_looped_list(cls, d: dict, **overrides) -> "ModelConfig":
+        """Fepopel's ``config.json``: ``vocab``, ``width``, ``norm.eps``, ``embedding.scale``,
+        ``loop`` and one entry of ``layers`` per layer with its mixer's and its feed-forward's
+        sizes."""
+        specs = []
+        for i, layer in enumerate(d["layers"]):
+            m, f, where = layer["mixer"], layer.get("mlp"), f"layer {i}"
+            kw: dict[str, Any] = {}
+            if f is not None and f.get("kind", "dense") == "dense":
+                kw["intermediate_size"] = int(f["ff"])
+            elif f is not None and f["kind"] == "moe":
+                r, shared = f["router"], f.get("shared")
+                kw.update(num_experts=int(r["experts"]), num_experts_per_tok=int(r["top"]),
+                          router_scale=float(r.get("scale", 1.0)),
+                          moe_intermediate_size=int(f["expert"]["ff"]),
+                          shared_intermediate_size=int(shared["ff"]) if shared else 0)
+                if not 0 < kw["num_experts_per_tok"] <= kw["num_experts"]:
+                    raise ValueError(f"{where}: {kw['num_experts_per_tok']} of "
+                                     f"{kw['num_experts']} experts per token")
+            elif f is not None:
+                raise ValueError(f"{where}: unknown feed-forward {f['kind']!r}")
+            if layer["type"] == "latent_attention":
+                rot = m.get("rot") or {}
+                if int(rot.get("dims", m["rot_dim"])) != int(m["rot_dim"]):
+                    raise ValueError(f"{where}: {rot['dims']} of {m['rot_dim']} dimensions rotated")
+                specs.append(LayerSpec(
+                    layer["type"], int(m["heads"]), int(m["dim"]), int(m["vdim"]),
+                    int(m["kv_rank"]), float(m["scale"]), rot_dim=int(m["rot_dim"]),
+                    rot_base=float(rot.get("base", 10000.0)), sink=True, head_gate=True, **kw))
+            elif layer["type"] == "attention":
+                specs.append(LayerSpec(layer["type"], parts=(("", 1.0, AttentionSpec(
+                    int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), float(m["scale"]),
+                    v_head_dim=int(m["vdim"]), softcap=float(m.get("softcap") or 0.0),
+                    chunk=int((m.get("mask") or {}).get("size") or 0))),), **kw))
+            else:
+                raise ValueError(f"{where}: unknown mixer {layer['type']!r}")
+        if not specs:
+            raise ValueError("the configuration lists no layers")
+        loop = d.get("loop")
+        if loop:
+            loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+            if not (0 <= loop[0] < loop[1] <= len(specs) and loop[2] > 0):
+                raise ValueError(f"a loop over layers {loop[0]} to {loop[1]} of {len(specs)}, "
+                                 f"{loop[2]} times")
+        attn = [s for sp in specs for _, _, s in sp.parts]
+        kw = dict(
+            architecture="FepopelForCausalLM", vocab_size=int(d["vocab"]),
+            hidden_size=int(d["width"]), num_hidden_layers=len(specs),
+            rms_norm_eps=float(d["norm"]["eps"]), layer_specs=tuple(specs), loop=loop or None,
+            embed_scale=float(d["embedding"]["scale"]),
+            # the largest layer stands for the model where one number is asked for
+            intermediate_size=max(s.intermediate_size for s in specs),
+            num_attention_heads=max([s.num_heads for s in specs] + [s.num_heads for s in attn]),
+            num_key_value_heads=max((s.num_kv_heads for s in attn), default=1),
+            head_dim=max([s.head_dim + s.rot_dim for s in specs] + [s.head_dim for s in attn]),
+            num_experts=max(s.num_experts for s in specs),
+            num_experts_per_tok=max(s.num_experts_per_tok for s in specs),
+            moe_intermediate_size=max(s.moe_intermediate_size for s in specs),
+            # no limit of the design's own: bounds the rotary and block tables only
+            max_position_embeddings=int(d.get("max_position_embeddings", 131072)),
+            extra={k: v for k, v in d.items() if k not in (
+                "layers", "vocab", "width", "norm", "embedding", "loop", "architecture",
+                "architectures", "max_position_embeddings")})
+        kw.update(overrides)
+        return cls(**kw)
+
+    @classmethod
     def from_pretrained(cls, path: str, **overrides) -> "ModelConfig":
         p = Path(path)
         d = json.loads((p / "config.json").read_text())
@@ -529,11 +628,38 @@ def _fizunex_mixers(heads: int, kv_heads: int, dim: int, memory_heads: int, memo
     return delta, left, right
 
 
+def _fepopel_preset(pattern: str, loop: tuple[int, int, int], vocab: int, width: int, heads: int,
+                    dim: int, rot_dim: int, rank: int, kv_heads: int, chunk: int, ff: int,
+                    experts: int, top: int, expert_ff: int, shared_ff: int) -> dict:
+    """``pattern``: two letters per layer, l for latent or c for chunked attention, then d for a
+    dense feed-forward or e for experts."""
+    mixers = {
+        "l": ("latent_attention", {
+            "heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "kv_rank": rank,
+            "scale": (dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": 500000.0}}),
+        "c": ("attention", {
+            "heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+            "softcap": 50.0, "mask": {"size": chunk}})}
+    mlps = {"d": {"kind": "dense", "ff": ff},
+            "e": {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.0},
+                  "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff}}}
+    return {"architecture": "Fepopel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": width ** 0.5},
+            "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]},
+            "layers": [{"type": mixers[p[0]][0], "mixer": mixers[p[0]][1], "mlp": mlps[p[1]]}
+                       for p in pattern.split()]}
+
+
 #: configurations of designs that are described layer by layer
 _LAYER_LIST_PRESETS: dict[str, dict] = {
     "tiny-sapapel": _sapapel_preset(3, 1024, 128, 4, 24, 40, 48, 6, 2, 48),
     # layers of the size of DeepSeek-V2-Lite's
     "sapapel-16b": _sapapel_preset(27, 102400, 2048, 16, 128, 128, 512, 64, 6, 1408),
+    "tiny-fepopel": _fepopel_preset("ld le ce le", (1, 3, 2), 1024, 128, 4, 24, 8, 48, 2, 32, 192,
+                                    6, 2, 48, 40),
+    # layers of the size of DeepSeek-V2-Lite's
+    "fepopel-16b": _fepopel_preset("ld" + " le ce le" * 8 + " le", (1, 4, 2), 102400, 2048, 16, 128,
+                                   64, 512, 4, 1024, 10944, 64, 6, 1408, 2816),
     "tiny-fizunex": _fizunex_preset("dpd", 1024, 128, 192, *_fizunex_mixers(4, 2, 32, 2, 24, 40)),
     # layers of the size of Llama-3-8B's
     "fizunex-8b": _fizunex_preset("dddp" * 8, 128256, 4096, 14336,

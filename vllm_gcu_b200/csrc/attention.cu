@@ -155,6 +155,10 @@ struct DecodeArgs {
   float scale;
   const float* alibi;   // optional [Hq] slopes: score += slope * (key position - query position)
   const float* sink;    // optional [Hq]: exp(sink) joins the softmax denominator, no key behind it
+  // kShaped kernels only
+  float softcap;        // > 0: scores become softcap * tanh(score / softcap)
+  int chunk;            // > 0: keys of the query's own chunk of that many positions
+  int OD;               // output columns per head (the first of the HD)
 };
 
 // Weight of the attention output (and the added share of the denominator) once a sink's term has
@@ -166,7 +170,8 @@ __device__ __forceinline__ float sink_share(float M, float L, float sink) {
   return keys / (keys + exp2f(s2 - top));
 }
 
-template <typename T, int HD>
+// kShaped: soft cap, chunk and output columns of DecodeArgs are in force
+template <typename T, int HD, bool kShaped = false>
 __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs a) {
   constexpr int kStride = HD + kPad;
   constexpr int kKC = HD / 16;  // k-chunks of the QK product
@@ -181,9 +186,12 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tig = lane & 3;
   const int seq_len = a.seq_lens[b];
-  const int per_split = (seq_len + a.num_splits - 1) / a.num_splits;
+  const int OD = kShaped ? a.OD : HD;
+  // first key the query sees
+  const int first = kShaped && a.chunk > 0 && seq_len > 0 ? (seq_len - 1) / a.chunk * a.chunk : 0;
+  const int per_split = (seq_len - first + a.num_splits - 1) / a.num_splits;
   const int chunk = ((per_split + kTile - 1) / kTile) * kTile;
-  const int start = split * chunk;
+  const int start = first + split * chunk;
   const int end = min(seq_len, start + chunk);
 
   if (start >= end) {  // nothing in this split (or empty sequence)
@@ -193,8 +201,8 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
         if (threadIdx.x == 0)
           a.tmp_lse[(static_cast<long long>(b) * a.Hq + head) * a.num_splits + split] = -INFINITY;
       } else {
-        T* o = static_cast<T*>(a.out) + static_cast<long long>(b) * a.ldo + head * HD;
-        for (int d = threadIdx.x; d < HD; d += kThreads) o[d] = from_f32<T>(0.0f);
+        T* o = static_cast<T*>(a.out) + static_cast<long long>(b) * a.ldo + head * OD;
+        for (int d = threadIdx.x; d < OD; d += kThreads) o[d] = from_f32<T>(0.0f);
       }
     }
     return;
@@ -221,6 +229,8 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.0f, 0.0f};
   const float sl2 = a.scale * kLog2e;
+  const bool capped = kShaped && a.softcap > 0.0f;
+  const float cap2 = capped ? a.softcap * kLog2e : 0.0f, in2 = capped ? a.scale / a.softcap : 0.0f;
   // ALiBi: the query sits at position seq_len - 1 (log2 domain like the scores)
   float al[2] = {0.0f, 0.0f};
   if (a.alibi != nullptr) {
@@ -266,9 +276,10 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int tok = tok0 + j * 8 + 2 * tig + (e & 1);
-          const float v = (tok < end)
-                              ? s[j][e] * sl2 + al[e >> 1] * static_cast<float>(tok - (seq_len - 1))
-                              : -INFINITY;
+          float v = (tok < end)
+                        ? s[j][e] * sl2 + al[e >> 1] * static_cast<float>(tok - (seq_len - 1))
+                        : -INFINITY;
+          if (kShaped && capped && tok < end) v = cap2 * tanh_fast(s[j][e] * in2);
           s[j][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -362,8 +373,8 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
       const long long base = (static_cast<long long>(b) * a.Hq + head) * a.num_splits + split;
       a.tmp_out[base * HD + d] = val;
       if (d == 0) a.tmp_lse[base] = L > 0.0f ? M + log2f(L) : -INFINITY;
-    } else {
-      static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * HD + d] = from_f32<T>(val);
+    } else if (d < OD) {
+      static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * OD + d] = from_f32<T>(val);
     }
   }
 }
@@ -374,7 +385,8 @@ __global__ void __launch_bounds__(128) decode_reduce_kernel(const DecodeArgs a) 
   const long long base = (static_cast<long long>(b) * a.Hq + head) * a.num_splits;
   float M = -INFINITY;
   for (int s = 0; s < a.num_splits; ++s) M = fmaxf(M, a.tmp_lse[base + s]);
-  for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+  const int OD = a.OD > 0 ? a.OD : HD;
+  for (int d = threadIdx.x; d < OD; d += blockDim.x) {
     float acc = 0.0f, wsum = 0.0f;
     for (int s = 0; s < a.num_splits; ++s) {
       const float l = a.tmp_lse[base + s];
@@ -385,7 +397,7 @@ __global__ void __launch_bounds__(128) decode_reduce_kernel(const DecodeArgs a) 
     }
     float val = wsum > 0.0f ? acc / wsum : 0.0f;
     if (a.sink != nullptr && wsum > 0.0f) val *= sink_share(M, wsum, a.sink[head]);
-    static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * HD + d] = from_f32<T>(val);
+    static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * OD + d] = from_f32<T>(val);
   }
 }
 
@@ -633,11 +645,11 @@ int set_smem(KernelT kern, int bytes, bool (&done)[64]) {
   return 0;
 }
 
-template <typename T, int HD>
+template <typename T, int HD, bool kShaped = false>
 int launch_decode(const DecodeArgs& a, cudaStream_t s) {
   constexpr int smem = 2 * 2 * kTile * (HD + kPad) * static_cast<int>(sizeof(T));
   static_assert(smem >= (128 + 4 * 16 * HD) * 4, "merge buffer must fit in the stage memory");
-  auto kern = paged_decode_kernel<T, HD>;
+  auto kern = paged_decode_kernel<T, HD, kShaped>;
   static bool done[64] = {false};
   int e = set_smem(kern, smem, done);
   if (e != 0) return e;
@@ -691,7 +703,8 @@ static int paged_decode_impl(const void* q, long long ldq, void* out, long long 
                              int num_splits, int B, int Hq, int Hkv, int HD, float scale,
                              int dtype, int qmode, float k_scale, float v_scale, float k_zp,
                              float v_zp, void* stream, const float* alibi = nullptr,
-                             const float* sink = nullptr) {
+                             const float* sink = nullptr, float softcap = 0.0f, int chunk = 0,
+                             int OD = 0) {
   if (B <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16) return -2;
   if (num_splits < 1) return -2;
@@ -707,7 +720,14 @@ static int paged_decode_impl(const void* q, long long ldq, void* out, long long 
   a.scale = scale;
   a.alibi = alibi;
   a.sink = sink;
+  a.softcap = softcap; a.chunk = chunk; a.OD = OD > 0 ? OD : HD;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (softcap > 0.0f || chunk > 0 || a.OD != HD) {
+    if (dtype == 0 && HD == 128) return launch_decode<__nv_bfloat16, 128, true>(a, s);
+    if (dtype == 0 && HD == 64) return launch_decode<__nv_bfloat16, 64, true>(a, s);
+    if (dtype == 0 && HD == 96) return launch_decode<__nv_bfloat16, 96, true>(a, s);
+    return -8;
+  }
 #define B200_DEC(TT, H) return launch_decode<TT, H>(a, s)
   if (dtype == 0) {
     if (HD == 128) B200_DEC(__nv_bfloat16, 128);
@@ -754,8 +774,10 @@ B200_API int b200_paged_decode_alibi(const void* q, long long ldq, void* out, lo
                            stream, alibi);
 }
 
-// Decode attention with one learnt sink per query head: exp(sink) is added to the softmax
-// denominator; it has no key and no value and is not scaled.
+// Decode attention with, each optional: one learnt sink per query head (exp(sink) is added to the
+// softmax denominator; it has no key and no value and is not scaled); a soft cap of the scores; only
+// the keys of the query's own chunk of positions, counted from 0; only the first OD columns of a
+// head's output stored, heads side by side.  The last three: bf16, HD 64, 96 or 128.
 B200_API int b200_paged_decode_sink(const void* q, long long ldq, void* out, long long ldo,
                                     const void* k_cache, const void* v_cache,
                                     long long slot_stride, long long head_stride,
@@ -763,11 +785,12 @@ B200_API int b200_paged_decode_sink(const void* q, long long ldq, void* out, lon
                                     int block_size, const int* seq_lens, float* tmp_out,
                                     float* tmp_lse, int num_splits, int B, int Hq, int Hkv,
                                     int HD, float scale, int dtype, const float* sink,
-                                    void* stream) {
+                                    float softcap, int chunk, int OD, void* stream) {
+  if (OD < 0 || OD > HD || chunk < 0) return -2;
   return paged_decode_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride, num_slots,
                            block_tables, max_blocks, block_size, seq_lens, tmp_out, tmp_lse,
                            num_splits, B, Hq, Hkv, HD, scale, dtype, 0, 1.0f, 1.0f, 0.0f, 0.0f,
-                           stream, nullptr, sink);
+                           stream, nullptr, sink, softcap, chunk, OD);
 }
 
 // Decode attention over an 8-bit KV cache (same layout, one byte per element; slot_stride and
@@ -793,10 +816,11 @@ B200_API int b200_paged_decode_q8kv(const void* q, long long ldq, void* out, lon
 // (tmp_out fp32 [B, Hq, num_splits, HD], tmp_lse fp32 [B, Hq, num_splits], log2 domain).
 B200_API int b200_decode_reduce(void* out, long long ldo, float* tmp_out, float* tmp_lse,
                                 int num_splits, int B, int Hq, int HD, int dtype,
-                                const float* sink, void* stream) {
+                                const float* sink, int OD, void* stream) {
   if (B <= 0 || num_splits <= 1) return 0;
   DecodeArgs a{};
   a.sink = sink;
+  a.OD = OD;
   a.out = out; a.tmp_out = tmp_out; a.tmp_lse = tmp_lse; a.ldo = ldo; a.B = B; a.Hq = Hq;
   a.num_splits = num_splits;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

@@ -4,9 +4,12 @@
 //                       at once), rotary positions on the first dimensions of every head, queries
 //                       to a padded buffer, keys and values to the paged cache.  Values are a
 //                       projection of their own or the keys as they were before the norm.
+//   head_norm_cache     RMS norm of every query and key head over its own dimensions with one
+//                       weight for all heads, no positions; queries to a padded buffer, keys and
+//                       values (of another width, if so) to the paged cache.  One warp per head.
 //   any_attention       causal paged attention for any head dimension and group size, fp32 or
-//                       bf16 rows, optional sink: serves models that run in 32-bit and the
-//                       shapes the tensor-core kernels do not cover.
+//                       bf16 rows, optional sink, soft cap and chunks of positions: serves models
+//                       that run in 32-bit and the shapes the tensor-core kernels do not cover.
 //
 // Cache layout as in attention.cu: [num_slots, kv_heads, DC] with DC >= D, zeros behind D.
 #include "common.cuh"
@@ -304,18 +307,136 @@ __global__ void __launch_bounds__(256) qk_norm_rope_cache_vec_kernel(const PrepA
 }
 
 // ---------------------------------------------------------------------------
+struct HeadNormArgs {
+  const void* q;             // [T, Hq * D] view, row pitch ldq
+  const void* k;             // [T, Hkv * D]
+  const void* v;             // [T, Hkv * VD]
+  const float* qw;           // [D]
+  const float* kw;           // [D]
+  const long long* slots;    // [T] (-1: no cache write)
+  void* qo;                  // [T, Hq, DC]
+  void* kc;                  // [num_slots, Hkv, DC]
+  void* vc;
+  long long ldq, ldk, ldv, num_slots;
+  int T, Hq, Hkv, D, VD, DC;
+  float eps;
+  unsigned int* status;
+};
+
+template <typename T, int V>
+__device__ __forceinline__ void load_elems(const T* p, float (&f)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else if constexpr (V == 4) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
+  } else {
+    f[0] = to_f32<T>(p[0]);
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_elems(T* p, const float (&f)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 2)
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+  else if constexpr (V == 4)
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else
+    p[0] = from_f32<T>(f[0]);
+}
+
+constexpr int kHeadWarps = 8;
+
+// NI vectors of V elements per lane cover a head: 32 * V * NI >= DC
+template <typename T, int V, int NI>
+__global__ void __launch_bounds__(kHeadWarps * 32) head_norm_cache_kernel(const HeadNormArgs a) {
+  const int lane = threadIdx.x & 31;
+  const int per_token = a.Hq + 2 * a.Hkv;
+  const long long job = static_cast<long long>(blockIdx.x) * kHeadWarps + (threadIdx.x >> 5);
+  const int t = static_cast<int>(job / per_token);
+  if (t >= a.T) return;
+  const int j = static_cast<int>(job - static_cast<long long>(t) * per_token);
+  const bool is_q = j < a.Hq, is_v = j >= a.Hq + a.Hkv;
+  const int h = is_q ? j : (is_v ? j - a.Hq - a.Hkv : j - a.Hq);
+  const int D = is_v ? a.VD : a.D;
+  long long slot = 0;
+  if (!is_q) {
+    slot = a.slots[t];
+    if (slot < 0) return;
+    if (slot >= a.num_slots) {
+      if (lane == 0)
+        report_status(a.status, kStatusBounds, kKernelId + 1, static_cast<unsigned int>(t));
+      return;
+    }
+  }
+  const T* src = is_q ? static_cast<const T*>(a.q) + t * a.ldq + static_cast<long long>(h) * D
+                      : (is_v ? static_cast<const T*>(a.v) + t * a.ldv + static_cast<long long>(h) * D
+                              : static_cast<const T*>(a.k) + t * a.ldk + static_cast<long long>(h) * D);
+  T* dst = is_q ? static_cast<T*>(a.qo) + (static_cast<long long>(t) * a.Hq + h) * a.DC
+                : static_cast<T*>(is_v ? a.vc : a.kc) + (slot * a.Hkv + h) * a.DC;
+  float x[NI][V];
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int c = (i * 32 + lane) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[i][e] = 0.0f;
+    if (c < D) load_elems<T, V>(src + c, x[i]);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss += x[i][e] * x[i][e];
+  }
+  if (!is_v) {
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(D) + a.eps);
+    const float* w = is_q ? a.qw : a.kw;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = (i * 32 + lane) * V;
+      if (c >= D) continue;
+      float g[V];
+      load_elems<float, V>(w + c, g);
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[i][e] *= inv * g[e];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int c = (i * 32 + lane) * V;
+    if (c < a.DC) store_elems<T, V>(dst + c, x[i]);
+  }
+}
+
+template <typename T>
+static int launch_head_norm(const HeadNormArgs& a, bool v4, cudaStream_t s) {
+  const long long warps = static_cast<long long>(a.T) * (a.Hq + 2 * a.Hkv);
+  const unsigned int grid = static_cast<unsigned int>((warps + kHeadWarps - 1) / kHeadWarps);
+#define B200_HN(V, NI) head_norm_cache_kernel<T, V, NI><<<grid, kHeadWarps * 32, 0, s>>>(a)
+  if (v4) {
+    if (a.DC <= 128) B200_HN(4, 1);
+    else if (a.DC <= 256) B200_HN(4, 2);
+    else B200_HN(4, 4);
+  } else {
+    if (a.DC <= 128) B200_HN(1, 4);
+    else B200_HN(1, 16);
+  }
+#undef B200_HN
+  return static_cast<int>(cudaGetLastError());
+}
+
+// ---------------------------------------------------------------------------
 struct AttnArgs {
   const void* q;             // [T, Hq, DC]
   const void* kc;            // [num_slots, Hkv, DC]
   const void* vc;
-  void* out;                 // [T, Hq, DC]
+  void* out;                 // [T, Hq, OD], row pitch ldo: the first OD of the DC columns
   const int* block_tables;   // [B, max_blocks]
   const int* seq_lens;       // [B]
   const int* cu_q;           // [num_prefills + 1] relative to token num_decodes, or null
   const float* sink;         // [Hq] or null
-  long long num_slots;
-  int T, Hq, Hkv, DC, num_decodes, num_prefills, max_blocks, block_size;
-  float scale;
+  long long num_slots, ldo;
+  int T, Hq, Hkv, DC, OD, num_decodes, num_prefills, max_blocks, block_size;
+  int chunk;                 // > 0: keys of the query's own chunk of that many positions
+  float scale, softcap;      // softcap > 0: scores become softcap * tanh(score / softcap)
   unsigned int* status;
 };
 
@@ -351,7 +472,8 @@ __global__ void __launch_bounds__(kWarps * 32) any_attention_kernel(const AttnAr
   }
   float m = -INFINITY, l = 0.0f;
   const int* bt = a.block_tables + static_cast<long long>(pl.req < 0 ? 0 : pl.req) * a.max_blocks;
-  for (int k0 = warp * kBatch; k0 < keys; k0 += kWarps * kBatch) {
+  const int first = a.chunk > 0 && keys > 0 ? (keys - 1) / a.chunk * a.chunk : 0;
+  for (int k0 = first + warp * kBatch; k0 < keys; k0 += kWarps * kBatch) {
     float s[kBatch], v[kBatch][NC];
 #pragma unroll
     for (int b = 0; b < kBatch; ++b) {
@@ -380,6 +502,7 @@ __global__ void __launch_bounds__(kWarps * 32) any_attention_kernel(const AttnAr
 #pragma unroll
     for (int b = 0; b < kBatch; ++b) {
       s[b] = k0 + b < keys ? warp_sum(s[b]) * a.scale : -INFINITY;
+      if (a.softcap > 0.0f && k0 + b < keys) s[b] = a.softcap * tanhf(s[b] / a.softcap);
       top = fmaxf(top, s[b]);
     }
     const float al = expf(m - top);            // top is finite: key k0 is visible
@@ -413,11 +536,13 @@ __global__ void __launch_bounds__(kWarps * 32) any_attention_kernel(const AttnAr
     den += s_l[w] * f[w];
   }
   const float inv = keys > 0 ? 1.0f / den : 0.0f;
-  for (int c = threadIdx.x; c < a.DC; c += blockDim.x) {
+  T* out = static_cast<T*>(a.out) + static_cast<long long>(t) * a.ldo +
+           static_cast<long long>(head) * a.OD;
+  for (int c = threadIdx.x; c < a.OD; c += blockDim.x) {
     float o = 0.0f;
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) o += s_o[w][c] * f[w];
-    static_cast<T*>(a.out)[row + c] = from_f32<T>(o * inv);
+    out[c] = from_f32<T>(o * inv);
   }
 }
 
@@ -484,21 +609,50 @@ B200_API int b200_qk_norm_rope_cache(const void* q, long long ldq, const void* k
   return static_cast<int>(cudaGetLastError());
 }
 
-// q / out [T, Hq, DC]; -20: a head dimension the kernel does not cover (> 512).
-B200_API int b200_any_attention(const void* q, const void* kc, const void* vc, long long num_slots,
-                                void* out, const int* block_tables, int max_blocks, int block_size,
-                                const int* seq_lens, const int* cu_q, const float* sink, int T,
-                                int Hq, int Hkv, int DC, int num_decodes, int num_prefills,
-                                float scale, int dtype, void* stream) {
+// dtype (rows and caches): 0 bf16, 2 fp32.  q [T, Hq * D], k [T, Hkv * D], v [T, Hkv * VD] views;
+// D, VD <= DC <= 512.
+B200_API int b200_head_norm_cache(const void* q, long long ldq, const void* k, long long ldk,
+                                  const void* v, long long ldv, const float* qw, const float* kw,
+                                  float eps, const long long* slots, void* qo, void* kc, void* vc,
+                                  long long num_slots, int T, int Hq, int Hkv, int D, int VD, int DC,
+                                  int dtype, void* stream) {
   if (T <= 0) return 0;
-  if (Hq <= 0 || Hkv <= 0 || Hq % Hkv != 0 || DC <= 0 || block_size <= 0 || Hq > 65535 ||
+  if (Hq <= 0 || Hkv <= 0 || D <= 0 || VD <= 0 || DC < D || DC < VD || DC > 512 ||
       (dtype != 0 && dtype != 2))
+    return -2;
+  HeadNormArgs a;
+  a.q = q; a.k = k; a.v = v; a.qw = qw; a.kw = kw; a.slots = slots; a.qo = qo; a.kc = kc;
+  a.vc = vc; a.ldq = ldq; a.ldk = ldk; a.ldv = ldv; a.num_slots = num_slots; a.T = T; a.Hq = Hq;
+  a.Hkv = Hkv; a.D = D; a.VD = VD; a.DC = DC; a.eps = eps; a.status = status_ptr();
+  const auto at = [](const void* p, int bytes) {
+    return (reinterpret_cast<uintptr_t>(p) % bytes) == 0;
+  };
+  const int vb = dtype == 0 ? 8 : 16;
+  const bool v4 = (D % 4) == 0 && (VD % 4) == 0 && (DC % 4) == 0 && (ldq % 4) == 0 &&
+                  (ldk % 4) == 0 && (ldv % 4) == 0 && at(q, vb) && at(k, vb) && at(v, vb) &&
+                  at(qo, vb) && at(kc, vb) && at(vc, vb) && at(qw, 16) && at(kw, 16);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return dtype == 0 ? launch_head_norm<__nv_bfloat16>(a, v4, s) : launch_head_norm<float>(a, v4, s);
+}
+
+// q [T, Hq, DC], out [T, Hq, OD] with row pitch ldo (the first OD <= DC columns of a head's value);
+// softcap / chunk 0: none.  -20: a head dimension the kernel does not cover (> 512).
+B200_API int b200_any_attention(const void* q, const void* kc, const void* vc, long long num_slots,
+                                void* out, long long ldo, int OD, const int* block_tables,
+                                int max_blocks, int block_size, const int* seq_lens,
+                                const int* cu_q, const float* sink, int T, int Hq, int Hkv, int DC,
+                                int num_decodes, int num_prefills, float scale, float softcap,
+                                int chunk, int dtype, void* stream) {
+  if (T <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || Hq % Hkv != 0 || DC <= 0 || OD <= 0 || OD > DC || block_size <= 0 ||
+      Hq > 65535 || chunk < 0 || (dtype != 0 && dtype != 2))
     return -2;
   AttnArgs a;
   a.q = q; a.kc = kc; a.vc = vc; a.out = out; a.block_tables = block_tables;
   a.seq_lens = seq_lens; a.cu_q = cu_q; a.sink = sink; a.num_slots = num_slots; a.T = T; a.Hq = Hq;
   a.Hkv = Hkv; a.DC = DC; a.num_decodes = num_decodes; a.num_prefills = num_prefills;
   a.max_blocks = max_blocks; a.block_size = block_size; a.scale = scale; a.status = status_ptr();
+  a.ldo = ldo; a.OD = OD; a.softcap = softcap; a.chunk = chunk;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   return dtype == 0 ? dispatch_attention<__nv_bfloat16>(a, s) : dispatch_attention<float>(a, s);
 }

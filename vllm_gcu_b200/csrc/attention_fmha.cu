@@ -67,12 +67,18 @@ struct Args {
   long long ldo;
   int B, T, Hq, Hkv, max_blocks, block_size, causal, window;
   float scale;
+  // kShaped kernels only
+  float softcap;           // > 0: scores become softcap * tanh(score / softcap)
+  int chunk;               // > 0: keys of the query's own chunk of that many positions
+  int OD;                  // output columns per head (the first of the HD)
   unsigned int* status;
 };
 
 // HD below 128 uses the same tiles: the second 64-column half then carries columns of the next
 // head (or zeros) behind HD, which no contraction step and no store touches.
-template <int HD>
+// kShaped: soft cap, chunk and output columns of Args are in force.  The soft cap is monotonic, so
+// row maxima are taken over uncapped scores.
+template <int HD, bool kShaped>
 __global__ void __launch_bounds__(kThreads, 1)
     fmha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ,
                         const __grid_constant__ CUtensorMap tmK,
@@ -170,6 +176,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   const int kv_hi = a.causal ? min(seq_len, pos0 + rows) : seq_len;
   int kv_lo = 0;
   if (a.window > 0) kv_lo = max(0, pos0 - a.window + 1);
+  if (kShaped && a.chunk > 0) kv_lo = max(kv_lo, pos0 / a.chunk * a.chunk);
   const int t0 = kv_lo / BKV;
   const int nt = (kv_hi + BKV - 1) / BKV - t0;          // >= 1
   const int kvh = head / (a.Hq / a.Hkv);
@@ -274,8 +281,14 @@ __global__ void __launch_bounds__(kThreads, 1)
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(qd * 32) << 16);
     const int pos = pos0 + r;
     const int hi = a.causal ? min(pos, seq_len - 1) : seq_len - 1;      // last visible key
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;       // first visible key
+    int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;             // first visible key
+    if (kShaped && a.chunk > 0) lo = max(lo, pos / a.chunk * a.chunk);
     const float sl2 = a.scale * 1.4426950408889634f;
+    const bool capped = kShaped && a.softcap > 0.0f;
+    const float cap2 = capped ? a.softcap * 1.4426950408889634f : 0.0f;
+    const float in2 = capped ? a.scale / a.softcap : 0.0f;
+    // log2-domain value of a score
+    auto l2 = [&](float raw) { return capped ? cap2 * tanh_fast(raw * in2) : raw * sl2; };
     float m_used = -INFINITY, l = 0.0f;
     uint8_t* sp = smem + kOffP + g * kSub;      // this group's 64-key sub-tile of P
     float* xch = reinterpret_cast<float*>(smem + kOffX);   // [2][128]
@@ -292,7 +305,8 @@ __global__ void __launch_bounds__(kThreads, 1)
       const int tile_key0 = (t0 + j) * BKV;
       const bool need_mask =
           (tile_key0 + BKV - 1 > (a.causal ? min(pos0, seq_len - 1) : seq_len - 1)) ||
-          (a.window > 0 && tile_key0 < pos0 + BQ - a.window);
+          (a.window > 0 && tile_key0 < pos0 + BQ - a.window) ||
+          (kShaped && a.chunk > 0 && tile_key0 < (pos0 + BQ - 1) / a.chunk * a.chunk);
       // pass 1: maximum over this thread's 64 keys
       float mt = -INFINITY;
       if (ok) {
@@ -326,11 +340,28 @@ __global__ void __launch_bounds__(kThreads, 1)
       asm volatile("bar.sync 3, 256;" ::: "memory");       // the slot may be rewritten next tile
       float alpha = 1.0f;
       float m_new = m_used;
-      if (mt > m_used && (m_used == -INFINITY || (mt - m_used) * sl2 > 8.0f)) {
-        m_new = mt;
-        alpha = m_used == -INFINITY ? 0.0f : ex2_approx((m_used - m_new) * sl2);
+      float mb;
+      if constexpr (kShaped) {
+        if (mt > m_used && (m_used == -INFINITY || l2(mt) - l2(m_used) > 8.0f)) {
+          m_new = mt;
+          alpha = m_used == -INFINITY ? 0.0f : ex2_approx(l2(m_used) - l2(m_new));
+        }
+        mb = m_new == -INFINITY ? 0.0f : l2(m_new);
+      } else {
+        if (mt > m_used && (m_used == -INFINITY || (mt - m_used) * sl2 > 8.0f)) {
+          m_new = mt;
+          alpha = m_used == -INFINITY ? 0.0f : ex2_approx((m_used - m_new) * sl2);
+        }
+        mb = (m_new == -INFINITY ? 0.0f : m_new) * sl2;
       }
-      const float mb = (m_new == -INFINITY ? 0.0f : m_new) * sl2;
+      // exponential of a score relative to the running maximum
+      auto prob = [&](uint32_t raw) {
+        const float x = __uint_as_float(raw);
+        if constexpr (kShaped) {
+          if (capped) return ex2_approx(fmaf(cap2, tanh_fast(x * in2), -mb));
+        }
+        return ex2_approx(fmaf(x, sl2, -mb));
+      };
       // pass 2: probabilities (bf16, kept in registers until the P buffer is free) and row sum
       uint32_t pk[32];
       float rs0 = 0.0f, rs1 = 0.0f;
@@ -344,8 +375,8 @@ __global__ void __launch_bounds__(kThreads, 1)
 #pragma unroll
             for (int i = 0; i < 32; i += 2) {
               const int key = key0 + c * 32 + i;
-              float p0 = ex2_approx(fmaf(__uint_as_float(v[i]), sl2, -mb));
-              float p1 = ex2_approx(fmaf(__uint_as_float(v[i + 1]), sl2, -mb));
+              float p0 = prob(v[i]);
+              float p1 = prob(v[i + 1]);
               if (key > hi || key < lo) p0 = 0.0f;
               if (key + 1 > hi || key + 1 < lo) p1 = 0.0f;
               rs0 += p0;
@@ -355,8 +386,8 @@ __global__ void __launch_bounds__(kThreads, 1)
           } else {
 #pragma unroll
             for (int i = 0; i < 32; i += 2) {
-              const float p0 = ex2_approx(fmaf(__uint_as_float(v[i]), sl2, -mb));
-              const float p1 = ex2_approx(fmaf(__uint_as_float(v[i + 1]), sl2, -mb));
+              const float p0 = prob(v[i]);
+              const float p1 = prob(v[i + 1]);
               rs0 += p0;
               rs1 += p1;
               pk[c * 16 + (i >> 1)] = pack_bf16x2(p0, p1);
@@ -407,11 +438,12 @@ __global__ void __launch_bounds__(kThreads, 1)
       tc_fence_after();
       float den = l;
       if (a.sink != nullptr)       // relative to the running maximum, like the row sum
-        den += exp2f(fmaf(-m_used, sl2, a.sink[head] * 1.4426950408889634f));
+        den += exp2f(fmaf(a.sink[head], 1.4426950408889634f, -l2(m_used)));
       const float inv = l > 0.0f ? 1.0f / den : 0.0f;
       const bool row_ok = r < rows;
+      const int OD = kShaped ? a.OD : HD;
       __nv_bfloat16* orow =
-          a.out + static_cast<long long>(q_start + q0 + r) * a.ldo + head * HD + g * 64;
+          a.out + static_cast<long long>(q_start + q0 + r) * a.ldo + head * OD + g * 64;
 #pragma unroll 1
       for (int c = 0; c < 2 && g * 64 + c * 32 < HD; ++c) {
         uint32_t v[32];
@@ -425,13 +457,24 @@ __global__ void __launch_bounds__(kThreads, 1)
             u.y = pack_bf16x2(__uint_as_float(v[i * 8 + 2]) * inv, __uint_as_float(v[i * 8 + 3]) * inv);
             u.z = pack_bf16x2(__uint_as_float(v[i * 8 + 4]) * inv, __uint_as_float(v[i * 8 + 5]) * inv);
             u.w = pack_bf16x2(__uint_as_float(v[i * 8 + 6]) * inv, __uint_as_float(v[i * 8 + 7]) * inv);
+            if constexpr (kShaped) {
+              const int col = g * 64 + c * 32 + i * 8;
+              if ((OD & 7) != 0) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e)
+                  if (col + e < OD)
+                    orow[c * 32 + i * 8 + e] = __float2bfloat16(__uint_as_float(v[i * 8 + e]) * inv);
+                continue;
+              }
+              if (col >= OD) continue;
+            }
             *reinterpret_cast<uint4*>(orow + c * 32 + i * 8) = u;
           }
         }
       }
       if (g == 0 && row_ok && a.lse != nullptr)
         a.lse[static_cast<long long>(head) * a.T + q_start + q0 + r] =
-            l > 0.0f ? m_used * a.scale + logf(l) : -INFINITY;
+            l > 0.0f ? l2(m_used) * 0.6931471805599453f + logf(l) : -INFINITY;
     }
   }
 
@@ -486,20 +529,20 @@ static int get_map(const void* base, unsigned long long rows, unsigned long long
 namespace b200 {
 namespace fmha {
 
-template <int HD>
+template <int HD, bool kShaped>
 static int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                   const Args& a, int num_q_tiles, cudaStream_t s) {
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel<HD>,
+    cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel<HD, kShaped>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev] = true;
   }
   dim3 grid(num_q_tiles, a.Hq);
-  fmha_prefill_kernel<HD><<<grid, kThreads, kSmemBytes, s>>>(tmQ, tmK, tmV, a);
+  fmha_prefill_kernel<HD, kShaped><<<grid, kThreads, kSmemBytes, s>>>(tmQ, tmK, tmV, a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -508,8 +551,8 @@ static int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensor
 
 // Same contract as b200_varlen_prefill for bf16, head_dim 64, 96 or 128, caches laid out as
 // [num_slots, Hkv * HD] rows and a block size that is a multiple of 16; num_q_tiles must be
-// >= sum_b ceil(q_len_b / 128).  `sink`: optional [Hq], exp(sink) is added to the softmax
-// denominator.  Returns -20 when the layout does not qualify (callers use another kernel).
+// >= sum_b ceil(q_len_b / 128).  sink, softcap, chunk and OD: optional, see b200_paged_decode_sink
+// (OD that is no multiple of 8 is stored element by element).  Returns -20 when the layout does not qualify (callers use another kernel).
 B200_API int b200_fmha_prefill_sink(const void* q, long long ldq, void* out, long long ldo,
                                     float* lse, const int* cu_q, const int* seq_lens,
                                     const void* k_cache, const void* v_cache,
@@ -517,14 +560,18 @@ B200_API int b200_fmha_prefill_sink(const void* q, long long ldq, void* out, lon
                                     long long num_slots, const int* block_tables, int max_blocks,
                                     int block_size, int B, int T, int num_q_tiles, int Hq, int Hkv,
                                     int HD, float scale, int causal, int window, int dtype,
-                                    const float* sink, void* stream) {
+                                    const float* sink, float softcap, int chunk, int OD,
+                                    void* stream) {
   using namespace b200;
   using namespace b200::fmha;
   if (B <= 0 || T <= 0 || num_q_tiles <= 0) return 0;
+  if (OD <= 0) OD = HD;
+  if (OD > HD || chunk < 0) return -2;
   if (dtype != 0 || (HD != 64 && HD != 96 && HD != 128) || (block_size % kPage) != 0 ||
       head_stride != HD || slot_stride != static_cast<long long>(Hkv) * HD || Hkv <= 0 ||
-      Hq % Hkv != 0 || (ldq % 8) != 0 || (ldo % 8) != 0 ||
-      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out) |
+      Hq % Hkv != 0 || (ldq % 8) != 0 || ((OD % 8) == 0 && (ldo % 8) != 0) ||
+      ((OD % 8) == 0 && (reinterpret_cast<uintptr_t>(out) & 15)) ||
+      ((reinterpret_cast<uintptr_t>(q) |
         reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15))
     return -20;
   CUtensorMap tmQ, tmK, tmV;
@@ -541,11 +588,17 @@ B200_API int b200_fmha_prefill_sink(const void* q, long long ldq, void* out, lon
   a.lse = lse; a.sink = sink; a.cu_q = cu_q; a.seq_lens = seq_lens; a.block_tables = block_tables;
   a.ldo = ldo; a.B = B; a.T = T; a.Hq = Hq; a.Hkv = Hkv; a.max_blocks = max_blocks;
   a.block_size = block_size; a.causal = causal; a.window = window; a.scale = scale;
+  a.softcap = softcap; a.chunk = chunk; a.OD = OD;
   a.status = status_ptr();
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (HD == 64) return launch<64>(tmQ, tmK, tmV, a, num_q_tiles, s);
-  if (HD == 96) return launch<96>(tmQ, tmK, tmV, a, num_q_tiles, s);
-  return launch<128>(tmQ, tmK, tmV, a, num_q_tiles, s);
+  if (softcap > 0.0f || chunk > 0 || OD != HD) {
+    if (HD == 64) return launch<64, true>(tmQ, tmK, tmV, a, num_q_tiles, s);
+    if (HD == 96) return launch<96, true>(tmQ, tmK, tmV, a, num_q_tiles, s);
+    return launch<128, true>(tmQ, tmK, tmV, a, num_q_tiles, s);
+  }
+  if (HD == 64) return launch<64, false>(tmQ, tmK, tmV, a, num_q_tiles, s);
+  if (HD == 96) return launch<96, false>(tmQ, tmK, tmV, a, num_q_tiles, s);
+  return launch<128, false>(tmQ, tmK, tmV, a, num_q_tiles, s);
 }
 
 B200_API int b200_fmha_prefill(const void* q, long long ldq, void* out, long long ldo, float* lse,
@@ -558,5 +611,5 @@ B200_API int b200_fmha_prefill(const void* q, long long ldq, void* out, long lon
   return b200_fmha_prefill_sink(q, ldq, out, ldo, lse, cu_q, seq_lens, k_cache, v_cache,
                                 slot_stride, head_stride, num_slots, block_tables, max_blocks,
                                 block_size, B, T, num_q_tiles, Hq, Hkv, HD, scale, causal, window,
-                                dtype, nullptr, stream);
+                                dtype, nullptr, 0.0f, 0, 0, stream);
 }

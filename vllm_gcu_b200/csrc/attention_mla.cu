@@ -29,7 +29,9 @@
 //                follows in shared memory for the others; rows are independent and the
 //                surplus ones are never stored), which leaves room for two stages at any W.
 // Long contexts are split over blockIdx.y; the partial results (normalised output +
-// log-sum-exp per row) are merged by mla_combine_kernel.
+// log-sum-exp per row) are merged by mla_combine_kernel.  Whichever writes the result also applies
+// what a design may have at this point, in fp32: a learnt sink per head in the denominator and an
+// output gate per token and head.
 //
 // Warp roles: warp 0 TMA producer, warp 1 MMA issuer and TMEM owner, warps 2..9 softmax and
 // epilogue.  Every wait is bounded and reports through the status word.
@@ -94,8 +96,18 @@ struct Args {
   int off_k, off_p;        // shared-memory layout
   uint32_t tmem_cols;
   float scale;
+  const float* sink;         // [N]: exp(sink) joins the softmax denominator, or null
+  const __nv_bfloat16* gate; // [T, ldg]: head h's output times sigmoid(gate[t, h]), or null
+  long long ldg;
   unsigned int* status;
 };
+
+__device__ __forceinline__ float head_gate(const __nv_bfloat16* gate, long long ldg, long long row,
+                                           int N) {
+  if (gate == nullptr) return 1.0f;
+  const long long t = row / N;
+  return 1.0f / (1.0f + __expf(-__bfloat162float(gate[t * ldg + (row - t * N)])));
+}
 
 // kResident CTAs share an SM: two where shared and tensor memory allow it (narrow latents, whose
 // tiles are too small to hide the latency of the chain loads -> scores -> softmax -> output)
@@ -446,8 +458,13 @@ __global__ void __launch_bounds__(kThreads, kResident)
     l += xch[(g ^ 1) * BQ + r];
     if (ok && mbar_wait(o_done, (nt - 1) & 1, a.status, kKernelId, 0x320u, abort_flag)) {
       tc_fence_after();
-      const float inv = l > 0.0f ? 1.0f / l : 0.0f;
       const long long grow = row0 + r;
+      float inv = l > 0.0f ? 1.0f / l : 0.0f;
+      if (a.splits == 1 && row_ok && l > 0.0f) {
+        if (a.sink != nullptr)       // relative to the running maximum, like the row sum
+          inv = 1.0f / (l + exp2f(fmaf(-m_used, sl2, a.sink[r % a.N] * 1.4426950408889634f)));
+        inv *= head_gate(a.gate, a.ldg, grow, a.N);
+      }
       const int col0 = c0 * 64 + g * nc * 32;
 #pragma unroll 1
       for (int c = 0; c < nc; ++c) {
@@ -486,14 +503,21 @@ __global__ void __launch_bounds__(kThreads, kResident)
   if (warp == 1) tmem_dealloc(tmem_base, a.tmem_cols);
 }
 
-// out[row] = sum_z w_z * ws_o[z][row],  w_z = exp(lse_z - max) / sum exp(lse - max)
+// out[row] = sum_z w_z * ws_o[z][row],  w_z = exp(lse_z - max) / sum exp(lse - max), where the sum
+// takes in the sink's term, times the gate
 __global__ void __launch_bounds__(128)
     mla_combine_kernel(const float* ws_o, const float* ws_lse, __nv_bfloat16* out,
-                       long long rows_total, int splits, int L) {
+                       long long rows_total, int splits, int L, int N, const float* sink,
+                       const __nv_bfloat16* gate, long long ldg) {
   const long long row = blockIdx.x;
   float mx = -INFINITY;
   for (int z = 0; z < splits; ++z) mx = fmaxf(mx, ws_lse[z * rows_total + row]);
   float den = 0.0f;
+  if (sink != nullptr && mx > -INFINITY) {
+    const float s = sink[row % N];
+    mx = fmaxf(mx, s);
+    den = __expf(s - mx);
+  }
   for (int z = 0; z < splits; ++z) {
     const float v = ws_lse[z * rows_total + row];
     den += v == -INFINITY ? 0.0f : __expf(v - mx);
@@ -501,10 +525,11 @@ __global__ void __launch_bounds__(128)
   const int c = threadIdx.x * 4;
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
   if (den > 0.0f) {
+    const float g = head_gate(gate, ldg, row, N) / den;
     for (int z = 0; z < splits; ++z) {
       const float v = ws_lse[z * rows_total + row];
       if (v == -INFINITY) continue;
-      const float w = __expf(v - mx) / den;
+      const float w = __expf(v - mx) * g;
       const float4 o = *reinterpret_cast<const float4*>(ws_o + (z * rows_total + row) * L + c);
       acc.x += w * o.x; acc.y += w * o.y; acc.z += w * o.z; acc.w += w * o.w;
     }
@@ -584,12 +609,14 @@ static int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const Args& a,
 // cache:[num_slots, W] bf16 (block b, offset o -> row b * block_size + o)
 // out:  [T, N, L] bf16.  cu_q null = one query token per request (decode, T == B).
 // splits > 1: workspace of splits * T * N * (L + 1) floats.
+// sink [N] fp32 and gate [T, ldg] bf16 (one logit per head): optional.
 // num_tiles >= sum_b ceil(q_len_b / floor(128 / N)).  N at most 128, L and W multiples of 64 with
 // L <= 512, L <= W <= 576, and the block size a multiple of 16; otherwise -20 (callers fall back).
 B200_API int b200_mla_attention(const void* q, void* out, const void* cache, long long num_slots,
                                 const int* cu_q, const int* seq_lens, const int* block_tables,
                                 int max_blocks, int block_size, int B, int T, int N, int W, int L,
                                 int num_tiles, int splits, float* workspace, float scale,
+                                const float* sink, const void* gate, long long ldg,
                                 void* stream) {
   using namespace b200;
   using namespace b200::mla;
@@ -632,6 +659,7 @@ B200_API int b200_mla_attention(const void* q, void* out, const void* cache, lon
   a.L = L; a.n_w = n_w; a.n_l = n_l; a.halves = n_l > 4 ? 2 : 1;
   a.off_k = lay.off_k; a.off_p = lay.off_p;
   a.tmem_cols = (a.halves == 2 ? (n_l + 1) / 2 : n_l) <= 2 ? 256 : 512;
+  a.sink = sink; a.gate = static_cast<const __nv_bfloat16*>(gate); a.ldg = ldg;
   a.status = status_ptr();
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   dim3 grid(num_tiles * a.halves, splits);
@@ -644,6 +672,6 @@ B200_API int b200_mla_attention(const void* q, void* out, const void* cache, lon
   else e = launch<BQ, 1, 1>(tmQ, tmK, a, grid, lay.bytes, s);
   if (e != 0 || splits == 1) return e;
   mla_combine_kernel<<<static_cast<unsigned>(rows_total), L / 4, 0, s>>>(
-      a.ws_o, a.ws_lse, a.out, rows_total, splits, L);
+      a.ws_o, a.ws_lse, a.out, rows_total, splits, L, N, a.sink, a.gate, ldg);
   return static_cast<int>(cudaGetLastError());
 }

@@ -80,10 +80,13 @@ struct Args {
   int B, Hq, Hkv, num_splits, max_blocks, block_size;
   float scale;
   const float* sink;     // optional [Hq], see b200_paged_decode_sink
+  float softcap;         // kShaped kernels: see b200_paged_decode_sink
+  int chunk, OD;
   unsigned int* status;
 };
 
-template <typename T>
+// kShaped: soft cap, chunk and output columns are in force
+template <typename T, bool kShaped>
 __global__ void __launch_bounds__(kThreads)
     paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK,
                             const __grid_constant__ CUtensorMap tmV, const Args a) {
@@ -98,9 +101,13 @@ __global__ void __launch_bounds__(kThreads)
   const int G = a.Hq / a.Hkv;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq_len = a.seq_lens[b];
-  const int per_split = (seq_len + a.num_splits - 1) / a.num_splits;
+  const int OD = kShaped ? a.OD : HD;
+  // first key the query sees; copies start at whole boxes, the keys in front of it are masked
+  const int lo = kShaped && a.chunk > 0 && seq_len > 0 ? (seq_len - 1) / a.chunk * a.chunk : 0;
+  const int first = lo / kChunk * kChunk;
+  const int per_split = (seq_len - first + a.num_splits - 1) / a.num_splits;
   const int chunk = ((per_split + kTile - 1) / kTile) * kTile;
-  const int start = split * chunk;
+  const int start = first + split * chunk;
   const int end = min(seq_len, start + chunk);
 
   if (start >= end) {
@@ -110,8 +117,8 @@ __global__ void __launch_bounds__(kThreads)
         if (threadIdx.x == 0)
           a.tmp_lse[(static_cast<long long>(b) * a.Hq + head) * a.num_splits + split] = -INFINITY;
       } else {
-        T* o = static_cast<T*>(a.out) + static_cast<long long>(b) * a.ldo + head * HD;
-        for (int d = threadIdx.x; d < HD; d += kThreads) o[d] = from_f32<T>(0.0f);
+        T* o = static_cast<T*>(a.out) + static_cast<long long>(b) * a.ldo + head * OD;
+        for (int d = threadIdx.x; d < OD; d += kThreads) o[d] = from_f32<T>(0.0f);
       }
     }
     return;
@@ -182,6 +189,8 @@ __global__ void __launch_bounds__(kThreads)
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.0f, 0.0f};
   const float sl2 = a.scale * kLog2e;
+  const bool capped = kShaped && a.softcap > 0.0f;
+  const float cap2 = capped ? a.softcap * kLog2e : 0.0f, in2 = capped ? a.scale / a.softcap : 0.0f;
   const uint32_t smem_base = smem_u32(smem);
 
   int stage = 0;
@@ -217,7 +226,9 @@ __global__ void __launch_bounds__(kThreads)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int tok = tok0 + j * 8 + 2 * tig + (e & 1);
-          const float v = (tok < end) ? s[j][e] * sl2 : -INFINITY;
+          float v = s[j][e] * sl2;
+          if (kShaped && capped) v = cap2 * tanh_fast(s[j][e] * in2);
+          if (tok >= end || (kShaped && tok < lo)) v = -INFINITY;
           s[j][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -317,8 +328,8 @@ __global__ void __launch_bounds__(kThreads)
       const long long base = (static_cast<long long>(b) * a.Hq + head) * a.num_splits + split;
       a.tmp_out[base * HD + d] = val;
       if (d == 0) a.tmp_lse[base] = (ok && L > 0.0f) ? M + log2f(L) : -INFINITY;
-    } else {
-      static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * HD + d] = from_f32<T>(val);
+    } else if (d < OD) {
+      static_cast<T*>(a.out)[static_cast<long long>(b) * a.ldo + head * OD + d] = from_f32<T>(val);
     }
   }
 }
@@ -366,7 +377,7 @@ static int get_map(const void* base, unsigned long long rows, unsigned long long
 
 B200_API int b200_decode_reduce(void* out, long long ldo, float* tmp_out, float* tmp_lse,
                                 int num_splits, int B, int Hq, int HD, int dtype,
-                                const float* sink, void* stream);
+                                const float* sink, int OD, void* stream);
 
 // Same contract as b200_paged_decode for head_dim 128 with the caches laid out as
 // [num_slots, Hkv * 128] rows (slot_stride == Hkv * 128, head_stride == 128) and a block size
@@ -378,7 +389,8 @@ static int paged_decode_tma_impl(const void* q, long long ldq, void* out, long l
                                  const int* block_tables, int max_blocks, int block_size,
                                  const int* seq_lens, float* tmp_out, float* tmp_lse,
                                  int num_splits, int B, int Hq, int Hkv, int HD, float scale,
-                                 int dtype, const float* sink, void* stream) {
+                                 int dtype, const float* sink, float softcap, int chunk, int OD,
+                                 void* stream) {
   using namespace b200;
   using namespace b200::attn_tma;
   if (B <= 0) return 0;
@@ -399,17 +411,28 @@ static int paged_decode_tma_impl(const void* q, long long ldq, void* out, long l
   a.q = q; a.out = out; a.tmp_out = tmp_out; a.tmp_lse = tmp_lse; a.seq_lens = seq_lens;
   a.block_tables = block_tables; a.ldq = ldq; a.ldo = ldo; a.B = B; a.Hq = Hq; a.Hkv = Hkv;
   a.num_splits = num_splits; a.max_blocks = max_blocks; a.block_size = block_size;
-  a.scale = scale; a.sink = sink; a.status = status_ptr();
+  a.scale = scale; a.sink = sink; a.softcap = softcap; a.chunk = chunk; a.OD = OD > 0 ? OD : HD;
+  a.status = status_ptr();
+  const bool shaped = softcap > 0.0f || chunk > 0 || a.OD != HD;
+  if (shaped && dtype != 0) return -20;
   constexpr int smem = kStages * kStageBytes + 256 + 1024;
   static_assert(kStages * kStageBytes >= (128 + 4 * 16 * b200::attn_tma::HD) * 4,
                 "merge buffer must fit");
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   dim3 grid(B, Hkv, num_splits);
-  static bool done0[64] = {false}, done1[64] = {false};
+  static bool done0[64] = {false}, done1[64] = {false}, done2[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
-  if (dtype == 0) {
-    auto kern = paged_decode_tma_kernel<__nv_bfloat16>;
+  if (shaped) {
+    auto kern = paged_decode_tma_kernel<__nv_bfloat16, true>;
+    if (dev >= 0 && dev < 64 && !done2[dev]) {
+      cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+      if (e != cudaSuccess) return static_cast<int>(e);
+      done2[dev] = true;
+    }
+    kern<<<grid, kThreads, smem, s>>>(tmK, tmV, a);
+  } else if (dtype == 0) {
+    auto kern = paged_decode_tma_kernel<__nv_bfloat16, false>;
     if (dev >= 0 && dev < 64 && !done0[dev]) {
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
       if (e != cudaSuccess) return static_cast<int>(e);
@@ -417,7 +440,7 @@ static int paged_decode_tma_impl(const void* q, long long ldq, void* out, long l
     }
     kern<<<grid, kThreads, smem, s>>>(tmK, tmV, a);
   } else {
-    auto kern = paged_decode_tma_kernel<__half>;
+    auto kern = paged_decode_tma_kernel<__half, false>;
     if (dev >= 0 && dev < 64 && !done1[dev]) {
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
       if (e != cudaSuccess) return static_cast<int>(e);
@@ -428,7 +451,7 @@ static int paged_decode_tma_impl(const void* q, long long ldq, void* out, long l
   int e = static_cast<int>(cudaGetLastError());
   if (e != 0 || num_splits <= 1) return e;
   return b200_decode_reduce(out, ldo, tmp_out, tmp_lse, num_splits, B, Hq, HD, dtype, sink,
-                            stream);
+                            a.OD, stream);
 }
 
 B200_API int b200_paged_decode_tma(const void* q, long long ldq, void* out, long long ldo,
@@ -440,10 +463,11 @@ B200_API int b200_paged_decode_tma(const void* q, long long ldq, void* out, long
                                    float scale, int dtype, void* stream) {
   return paged_decode_tma_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride,
                                num_slots, block_tables, max_blocks, block_size, seq_lens, tmp_out,
-                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, nullptr, stream);
+                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, nullptr, 0.0f, 0, 0,
+                               stream);
 }
 
-// The same with one learnt sink per query head (see b200_paged_decode_sink).
+// The same with sinks, soft cap, chunk and output columns (see b200_paged_decode_sink).
 B200_API int b200_paged_decode_tma_sink(const void* q, long long ldq, void* out, long long ldo,
                                         const void* k_cache, const void* v_cache,
                                         long long slot_stride, long long head_stride,
@@ -451,8 +475,11 @@ B200_API int b200_paged_decode_tma_sink(const void* q, long long ldq, void* out,
                                         int max_blocks, int block_size, const int* seq_lens,
                                         float* tmp_out, float* tmp_lse, int num_splits, int B,
                                         int Hq, int Hkv, int HD, float scale, int dtype,
-                                        const float* sink, void* stream) {
+                                        const float* sink, float softcap, int chunk, int OD,
+                                        void* stream) {
+  if (OD < 0 || OD > HD || chunk < 0) return -2;
   return paged_decode_tma_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride,
                                num_slots, block_tables, max_blocks, block_size, seq_lens, tmp_out,
-                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, sink, stream);
+                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, sink, softcap, chunk, OD,
+                               stream);
 }

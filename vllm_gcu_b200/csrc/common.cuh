@@ -347,6 +347,15 @@ __device__ __forceinline__ float2 unpack_bf16x2(uint32_t u) {
   return __bfloat1622float2(v);
 }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
+// tanh through one exponential and one division: absolute error below 1e-6, exact limits
+__device__ __forceinline__ float tanh_fast(float x) {
+  return 1.0f - __fdividef(2.0f, __expf(2.0f * x) + 1.0f);
+}
+// square of the rectified value
+__device__ __forceinline__ float relu2_f(float x) {
+  const float r = fmaxf(x, 0.0f);
+  return r * r;
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

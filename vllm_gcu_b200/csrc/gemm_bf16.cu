@@ -37,6 +37,7 @@ enum Epilogue : int {
   kEpiAllGather = 6,  // column-parallel shard -> every peer's full-width output (peer stores)
   kEpiGatherA = 7,    // A rows are gathered from the peers' shards by extra warps of this kernel
   kEpiReduceNorm = 8, // row-parallel partial -> row owners reduce (+ residual, RMSNorm) and broadcast
+  kEpiRelu2 = 9,      // max(x, 0)^2
 };
 
 template <int EPI>
@@ -1322,6 +1323,10 @@ __global__ void __launch_bounds__(kThreadsFor<EPI>, 1)
           float v[32];
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+          if constexpr (EPI == kEpiRelu2) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
+          }
           if (p.row_scale != nullptr) {
             const float rs = p.row_scale[row];
 #pragma unroll
@@ -1506,6 +1511,7 @@ B200_API int b200_gemm_bf16(const void* A, long long lda, const void* B, long lo
     B200_GEMM_CASE(kEpiBias)
     B200_GEMM_CASE(kEpiResidual)
     B200_GEMM_CASE(kEpiFp32)
+    B200_GEMM_CASE(kEpiRelu2)
     case kEpiSiluMul:
       if (bn == 64) return launch<64, 8, kEpiSiluMul>(tmA, tmB, a, s);
       if (bn == 128) return launch<128, 6, kEpiSiluMul>(tmA, tmB, a, s);
@@ -1839,8 +1845,8 @@ B200_API int b200_gemm_bf16_gather_a(void* const* shard, long long lds, const in
 // tiles at or past *num_valid_rows are skipped, so M_cap may be a static upper bound).
 // epi 0: C[M_cap, N] = A * B_e^T (optionally scaled per row by row_scale);
 // epi 2: SiLU(gate) * up with the gate / up rows of every expert interleaved in blocks of
-// 32 (C is [M_cap, N / 2]).  N must be a multiple of the tile width (256 for epi 2,
-// else 128 or 64).
+// 32 (C is [M_cap, N / 2]); epi 9: max(x, 0)^2.  N must be a multiple of the tile width (256 for
+// epi 2, else 128 or 64).
 B200_API int b200_gemm_bf16_grouped(const void* A, long long lda, const void* B, long long ldb,
                                     void* C, long long ldc, int M_cap, int N, int K, int E,
                                     const int* expert_ids, const int* num_valid_rows,
@@ -1855,8 +1861,8 @@ B200_API int b200_gemm_bf16_grouped(const void* A, long long lda, const void* B,
   if (epi == kEpiSiluMul) {
     if ((N % 256) != 0) return -4;
     bn = 256;
-  } else if (epi == kEpiNone) {
-    bn = (N % 128) == 0 ? 128 : 64;
+  } else if (epi == kEpiNone || epi == kEpiRelu2) {
+    bn = epi == kEpiRelu2 && (N % 256) == 0 ? 256 : (N % 128) == 0 ? 128 : 64;
     if ((N % bn) != 0) return -4;
   } else {
     return -7;
@@ -1889,6 +1895,11 @@ B200_API int b200_gemm_bf16_grouped(const void* A, long long lda, const void* B,
   a.ar = ArArgs{};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (epi == kEpiSiluMul) return launch<256, 4, kEpiSiluMul>(tmA, tmB, a, s);
+  if (epi == kEpiRelu2) {
+    if (bn == 256) return launch<256, 4, kEpiRelu2>(tmA, tmB, a, s);
+    if (bn == 128) return launch<128, 6, kEpiRelu2>(tmA, tmB, a, s);
+    return launch<64, 8, kEpiRelu2>(tmA, tmB, a, s);
+  }
   if (bn == 128) return launch<128, 6, kEpiNone>(tmA, tmB, a, s);
   return launch<64, 8, kEpiNone>(tmA, tmB, a, s);
 }

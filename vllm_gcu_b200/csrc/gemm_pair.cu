@@ -49,7 +49,7 @@ constexpr int BK = 64;
 constexpr int UMMA_K = 16;
 constexpr int kThreads = 192;
 
-enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2 };
+enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kRelu2 = 9 };
 
 struct Args {
   __nv_bfloat16* C;
@@ -347,6 +347,10 @@ __global__ void __launch_bounds__(kThreads, 1)
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+            if constexpr (EPI == kRelu2) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
+            }
             if constexpr (EPI == kBias) {
 #pragma unroll
               for (int i = 0; i < 32; ++i) v[i] += __bfloat162float(p.bias[col + i]);
@@ -707,7 +711,7 @@ B200_API int b200_gemm_pair(const void* A, long long lda, const void* B, long lo
   using namespace b200;
   using namespace b200::pair;
   if (M <= 0 || N <= 0) return 0;
-  if ((N % 256) != 0 || (K % BK) != 0 || K <= 0 || epi < 0 || epi > 2) return -20;
+  if ((N % 256) != 0 || (K % BK) != 0 || K <= 0 || (epi != kRelu2 && (epi < 0 || epi > 2))) return -20;
   if ((lda % 8) != 0 || (ldb % 8) != 0 || (ldc % 8) != 0) return -2;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B) |
        reinterpret_cast<uintptr_t>(C)) & 15)
@@ -745,10 +749,12 @@ B200_API int b200_gemm_pair(const void* A, long long lda, const void* B, long lo
   if (mt == 1) {
     if (epi == kSiluMul) return launch<kSiluMul, 1>(tmA, tmB, a, s);
     if (epi == kBias) return launch<kBias, 1>(tmA, tmB, a, s);
+    if (epi == kRelu2) return launch<kRelu2, 1>(tmA, tmB, a, s);
     return launch<kNone, 1>(tmA, tmB, a, s);
   }
   if (epi == kSiluMul) return launch<kSiluMul, 2>(tmA, tmB, a, s);
   if (epi == kBias) return launch<kBias, 2>(tmA, tmB, a, s);
+  if (epi == kRelu2) return launch<kRelu2, 2>(tmA, tmB, a, s);
   return launch<kNone, 2>(tmA, tmB, a, s);
 }
 

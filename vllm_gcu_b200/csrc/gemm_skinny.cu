@@ -16,7 +16,8 @@
 //     (o_proj, down_proj).  The CTAs of a column tile write fp32 partial sums to an L2-resident
 //     workspace, meet at a counter (bounded wait), and each reduces a row slice of the tile
 //     in a fixed order (bitwise reproducible), applying the epilogue;
-//   * epilogues: none, + bias, SiLU(gate) * up (gate / up interleaved in blocks of 32 rows).
+//   * epilogues: none, + bias, max(x, 0)^2, SiLU(gate) * up (gate / up interleaved in blocks of 32
+//     rows).
 //
 // Replaces the vendor matmul behind the decode path of every unquantised linear layer of the
 // reference (vllm_gcu/kernels/linear.py; SiluAndMul of vllm_gcu/kernels/activation.py:20-32
@@ -34,7 +35,7 @@ constexpr int BK = 64;
 constexpr int UMMA_K = 16;
 constexpr int kThreads = 192;
 
-enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2 };
+enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kRelu2 = 9 };
 
 struct Args {
   __nv_bfloat16* C;
@@ -212,6 +213,10 @@ __global__ void __launch_bounds__(kThreads, 1)
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+            if constexpr (EPI == kRelu2) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
+            }
             __nv_bfloat16* crow = p.C + static_cast<long long>(row) * p.ldc + col;
             if (col + 32 <= p.N) {
               if constexpr (EPI == kBias) {
@@ -314,6 +319,10 @@ __global__ void __launch_bounds__(kThreads, 1)
             }
             const int col = n0 + c4;
             if (col >= p.N) continue;
+            if constexpr (EPI == kRelu2) {
+              acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y);
+              acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w);
+            }
             if constexpr (EPI == kBias) {
               acc.x += __bfloat162float(p.bias[col]);
               acc.y += __bfloat162float(p.bias[col + 1]);
@@ -600,7 +609,8 @@ struct Plan {
 // a column tile lie one after the other, [tile][slice][R x bn]; fixed summation order.
 __global__ void __launch_bounds__(256)
     skinny_reduce_kernel(const float* ws, __nv_bfloat16* C, long long ldc,
-                         const __nv_bfloat16* bias, int M, int N, int bn, int R, int splits) {
+                         const __nv_bfloat16* bias, int relu2, int M, int N, int bn, int R,
+                         int splits) {
   const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   const int n4 = N >> 2;
   if (idx >= static_cast<long long>(M) * n4) return;
@@ -618,6 +628,10 @@ __global__ void __launch_bounds__(256)
     acc.y += __bfloat162float(bias[col + 1]);
     acc.z += __bfloat162float(bias[col + 2]);
     acc.w += __bfloat162float(bias[col + 3]);
+  }
+  if (relu2) {
+    acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y);
+    acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w);
   }
   uint2 o;
   o.x = pack_bf16x2(acc.x, acc.y);
@@ -698,7 +712,7 @@ B200_API int b200_gemm_skinny_workspace(int N, long long* ws_bytes, int* ctr_wor
 }
 
 // C[M,N] (bf16) = A[M,K] * B[N,K]^T for M <= 256 with epilogue epi: 0 none, 1 + bias[N],
-// 2 SiLU(gate)*up (B rows interleaved gate/up in blocks of 32; C is [M, N/2]).
+// 2 SiLU(gate)*up (B rows interleaved gate/up in blocks of 32; C is [M, N/2]), 9 max(x, 0)^2.
 // Row pitches in elements; K, lda, ldb, N, ldc multiples of 8; 16-byte aligned pointers.
 // ws / ctr: see b200_gemm_skinny_workspace (ctr must be zero before the first call; the kernel
 // leaves it zero).  Launches on one stream may share the workspace; concurrent streams need
@@ -720,7 +734,7 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
     return -3;
   if (epi == kSiluMul && (N % 256) != 0) return -4;
   if (epi == kBias && bias == nullptr) return -5;
-  if (epi < 0 || epi > 2) return -20;
+  if (epi != kRelu2 && (epi < 0 || epi > 2)) return -20;
   const int sms = sm_count();
   Plan pl = allow_split == 2 ? make_plan2(M, N, K, epi, sms) : make_plan(M, N, K, epi, sms);
   if (allow_split == 2 && pl.splits == 1) {
@@ -768,6 +782,11 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
   switch (epi) {                                                                    \
     case kNone: rc = launch<BN_, MT_, ST_, kNone>(tmA, tmB, a, units, s); break;    \
     case kBias: rc = launch<BN_, MT_, ST_, kBias>(tmA, tmB, a, units, s); break;    \
+    case kRelu2:                                                                    \
+      rc = a.splits > 1 && a.ctr == nullptr                                         \
+               ? launch<BN_, MT_, ST_, kNone>(tmA, tmB, a, units, s)                \
+               : launch<BN_, MT_, ST_, kRelu2>(tmA, tmB, a, units, s);              \
+      break;                                                                        \
     default: break;                                                                 \
   }
   if (epi == kSiluMul) {
@@ -786,7 +805,7 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
   // two-kernel K split: add the partial sums
   const long long work = static_cast<long long>(M) * (N / 4);
   skinny_reduce_kernel<<<static_cast<unsigned>((work + 255) / 256), 256, 0, s>>>(
-      a.ws, a.C, a.ldc, epi == kBias ? a.bias : nullptr, M, N, pl.bn, mt * BM, a.splits);
+      a.ws, a.C, a.ldc, epi == kBias ? a.bias : nullptr, epi == kRelu2, M, N, pl.bn, mt * BM, a.splits);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -8,6 +8,7 @@
 //                     the expert of every tile, the padded row count and the inverse map
 //   moe_permute       gathers activation rows into expert-sorted order (the A operand of
 //                     the grouped tcgen05 GEMM in gemm_bf16.cu)
+//   moe_permute_any   the same for rows of any width, bf16 or fp32, padded with zeros
 //   moe_permute_weighted  the same from an fp32 stream, every row scaled by its routing weight
 //                     (designs whose weight multiplies the expert's input)
 //   grouped_gemm_f32  the expert products of models that run in 32-bit
@@ -246,6 +247,20 @@ __global__ void __launch_bounds__(256)
   for (int v = threadIdx.x; v < nvec; v += blockDim.x) dst[v] = src[v];
 }
 
+// The same for rows of any width: H columns, zeros behind them up to Ho.
+template <typename T>
+__global__ void __launch_bounds__(256)
+    moe_permute_any_kernel(const T* x, long long ldx, T* out, long long ldo, const int* sorted_ids,
+                           const int* num_post_pad, int numel, int k, int H, int Ho) {
+  const int pos = blockIdx.x;
+  if (pos >= *num_post_pad) return;
+  const int pair = sorted_ids[pos];
+  T* dst = out + static_cast<long long>(pos) * ldo;
+  const T* src = x + static_cast<long long>(pair >= numel ? 0 : pair / k) * ldx;
+  for (int c = threadIdx.x; c < Ho; c += blockDim.x)
+    dst[c] = (pair < numel && c < H) ? src[c] : from_f32<T>(0.0f);
+}
+
 // A_sorted[pos] = weight(pair) * x[pair / k] from an fp32 stream: routing that weights the
 // expert's input.  One rounding, to the type of the expert GEMM's operand.
 template <typename T>
@@ -353,6 +368,15 @@ __global__ void __launch_bounds__(256)
   const float* g = u + static_cast<long long>(r) * 2 * I;
   for (int c = threadIdx.x; c < I; c += blockDim.x)
     h[static_cast<long long>(r) * I + c] = g[c] / (1.0f + expf(-g[c])) * g[I + c];
+}
+
+// h[r, i] = max(u[r, i], 0)^2 of the rows in use (may be in place)
+__global__ void __launch_bounds__(256)
+    relu2_rows_f32_kernel(const float* u, float* h, int I, const int* num_valid_rows) {
+  const int r = blockIdx.x;
+  if (r >= *num_valid_rows) return;
+  for (int c = threadIdx.x; c < I; c += blockDim.x)
+    h[static_cast<long long>(r) * I + c] = relu2_f(u[static_cast<long long>(r) * I + c]);
 }
 
 // out[t] = (add ? add[t] : 0) + alpha * sum_s y[pos_of[t * k + s]]   (fp32 accumulation)
@@ -498,6 +522,25 @@ B200_API int b200_moe_permute(const void* x, long long ldx, void* out, long long
   return static_cast<int>(cudaGetLastError());
 }
 
+// x [T, ldx], H columns; out rows [cap, ldo] of Ho >= H columns (zeros behind H); dtype 0 bf16,
+// 2 fp32.
+B200_API int b200_moe_permute_any(const void* x, long long ldx, void* out, long long ldo,
+                                  const int* sorted_ids, const int* num_post_pad, int numel, int k,
+                                  int H, int Ho, int cap, int dtype, void* stream) {
+  if (cap <= 0) return 0;
+  if (Ho < H || ldo < Ho || k <= 0 || (dtype != 0 && dtype != 2)) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 0)
+    moe_permute_any_kernel<__nv_bfloat16><<<cap, 256, 0, s>>>(
+        static_cast<const __nv_bfloat16*>(x), ldx, static_cast<__nv_bfloat16*>(out), ldo,
+        sorted_ids, num_post_pad, numel, k, H, Ho);
+  else
+    moe_permute_any_kernel<float><<<cap, 256, 0, s>>>(
+        static_cast<const float*>(x), ldx, static_cast<float*>(out), ldo, sorted_ids, num_post_pad,
+        numel, k, H, Ho);
+  return static_cast<int>(cudaGetLastError());
+}
+
 // x fp32 [T, ldx], H columns; out bf16 (dtype 0) or fp32 (2) rows [cap, ldo] of Ho >= H columns
 // (zeros behind H); Ho and ldo are multiples of 4.
 B200_API int b200_moe_permute_weighted(const float* x, long long ldx, const float* topk_w,
@@ -536,6 +579,14 @@ B200_API int b200_silu_mul_rows_f32(const float* u, float* h, int rows, int I,
   if (rows <= 0 || I <= 0) return 0;
   silu_mul_rows_f32_kernel<<<rows, 256, 0, static_cast<cudaStream_t>(stream)>>>(u, h, I,
                                                                              num_valid_rows);
+  return static_cast<int>(cudaGetLastError());
+}
+
+B200_API int b200_relu2_rows_f32(const float* u, float* h, int rows, int I,
+                                 const int* num_valid_rows, void* stream) {
+  if (rows <= 0 || I <= 0) return 0;
+  relu2_rows_f32_kernel<<<rows, 256, 0, static_cast<cudaStream_t>(stream)>>>(u, h, I,
+                                                                          num_valid_rows);
   return static_cast<int>(cudaGetLastError());
 }
 

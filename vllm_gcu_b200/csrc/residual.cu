@@ -11,10 +11,14 @@
 //
 // and around one whose norms sit on the sublayers' outputs only:
 //
-//   start_rows      x = s * embedding row
-//   add_normed      x = x + norm(y) with a layer norm or an RMS norm (weight, optional bias);
-//                   optionally the final norm of the new row in the same pass
+//   start_rows      x = s * embedding row (+ a vector); optionally the norm in front of the first
+//                   sublayer in the same pass
+//   add_normed      x = x + norm(y) (+ a vector) with a layer norm or an RMS norm (weight, optional
+//                   bias); optionally the norm of the new row in the same pass (the final one, or
+//                   that in front of the next sublayer).  y is a dense row, or the weighted sum of
+//                   a token's routed-expert rows plus a shared expert's row times its gate
 //   silu_mul_rows   h = silu(g) * u of rows [g | u], any width
+//   relu2           h = max(u, 0)^2
 //   head_gate       o = o * sigmoid(z) * s from rows whose heads are padded
 //
 // The residual stream, the statistics and the averages are fp32; LO is the type of the rows that
@@ -249,30 +253,70 @@ __global__ void __launch_bounds__(256)
 }
 
 // ---------------------------------------------------------------------------
+struct StartArgs {
+  const void* e;         // [T, lde] embedding rows
+  const float* step;     // [H] vector added to every row, or null
+  const float* w;        // [H] weight of the norm of the new row, or null
+  float* x;              // [T, H]
+  void* lo;              // [T, H] copy of x, or its norm
+  long long lde;
+  int H;
+  float scale, eps;
+};
+
 template <typename T, int V>
-__global__ void __launch_bounds__(256)
-    start_rows_kernel(const T* e, long long lde, float scale, float* x, T* lo, int H) {
+__global__ void __launch_bounds__(512) start_rows_kernel(const StartArgs a) {
+  __shared__ float red[32];
   const long long t = blockIdx.x;
-  for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
+  const T* e = static_cast<const T*>(a.e) + t * a.lde;
+  float* x = a.x + t * a.H;
+  T* lo = static_cast<T*>(a.lo) + t * a.H;
+  float ss = 0.0f;
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
     float f[V];
-    ldv<V>(e + t * lde + c, f);
+    ldv<V>(e + c, f);
 #pragma unroll
-    for (int i = 0; i < V; ++i) f[i] *= scale;
-    stv<V>(x + t * H + c, f);
-    stv<V>(lo + t * H + c, f);
+    for (int i = 0; i < V; ++i) f[i] *= a.scale;
+    if (a.step != nullptr) {
+      float s[V];
+      ldv<V>(a.step + c, s);
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] += s[i];
+    }
+    stv<V>(x + c, f);
+    if (a.w == nullptr) stv<V>(lo + c, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += f[i] * f[i];
+  }
+  if (a.w == nullptr) return;
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / static_cast<float>(a.H) + a.eps);
+  for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {   // what this thread wrote
+    float f[V], w[V];
+    ldv<V>(x + c, f);
+    ldv<V>(a.w + c, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] *= inv * w[i];
+    stv<V>(lo + c, f);
   }
 }
 
 struct AddNormArgs {
   const float* x;        // [T, H] residual stream
-  const void* y;         // [T, ldy] sublayer output
+  const void* y;         // [T, ldy] sublayer output; routed: expert-sorted rows [cap, ldy]
+  const int* pos_of;     // routed: [T, k] row of every (token, slot) pair (-1: none), else null
+  const float* row_w;    // routed: [T, k] weights
+  const void* shared;    // routed: [T, ldsh] shared expert's rows, or null
+  const float* gate;     // routed: logit of the shared expert's gate, one per ldg (null: no gate)
+  const float* step;     // [H] vector added to the sum, or null
   const float* w;        // [H] norm weight
   const float* b;        // [H] norm bias, or null
   const float* fw;       // [H] final norm's weight, or null
   const float* fb;       // [H] final norm's bias, or null
   float* xo;             // [T, H] the sum (may be x), or null
   void* lo;              // [T, H] LO copy: of the sum, or of its final norm times fscale
-  long long ldy;
+  long long ldy, ldsh, ldg;
+  int k;
   int T, H, centred;     // centred: layer norm (mean taken off), else RMS norm
   float eps, fscale;
 };
@@ -293,17 +337,39 @@ __device__ __forceinline__ float row_stats(const float* z, float sum, int H, int
   return 1.0f / sqrtf(ss / static_cast<float>(H) + eps);
 }
 
-template <typename T, int V>
+template <typename T, int V, bool kRouted>
 __global__ void __launch_bounds__(512) add_normed_kernel(const AddNormArgs a) {
   extern __shared__ float z[];       // [H]; every thread reads back only what it wrote
   __shared__ float red[32];
   const long long t = blockIdx.x;
   const long long row = t * a.H;
-  const T* y = static_cast<const T*>(a.y) + t * a.ldy;
+  const T* y = static_cast<const T*>(a.y) + (kRouted ? 0 : t * a.ldy);
+  float gate = 1.0f;
+  if (kRouted && a.gate != nullptr) gate = 1.0f / (1.0f + expf(-a.gate[t * a.ldg]));
   float sum = 0.0f;
   for (int c = threadIdx.x * V; c < a.H; c += blockDim.x * V) {
     float f[V];
-    ldv<V>(y + c, f);
+    if constexpr (kRouted) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] = 0.0f;
+      for (int s = 0; s < a.k; ++s) {
+        const int p = a.pos_of[t * a.k + s];
+        if (p < 0) continue;
+        const float w = a.row_w[t * a.k + s];
+        float e[V];
+        ldv<V>(y + static_cast<long long>(p) * a.ldy + c, e);
+#pragma unroll
+        for (int i = 0; i < V; ++i) f[i] += w * e[i];
+      }
+      if (a.shared != nullptr) {
+        float e[V];
+        ldv<V>(static_cast<const T*>(a.shared) + t * a.ldsh + c, e);
+#pragma unroll
+        for (int i = 0; i < V; ++i) f[i] += gate * e[i];
+      }
+    } else {
+      ldv<V>(y + c, f);
+    }
 #pragma unroll
     for (int i = 0; i < V; ++i) sum += f[i];
     stv<V>(z + c, f);
@@ -326,8 +392,14 @@ __global__ void __launch_bounds__(512) add_normed_kernel(const AddNormArgs a) {
 #pragma unroll
     for (int i = 0; i < V; ++i) {
       x[i] += (f[i] - mean) * inv * w[i] + b[i];
-      sum += x[i];
     }
+    if (a.step != nullptr) {
+      ldv<V>(a.step + c, b);
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[i] += b[i];
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) sum += x[i];
     if (a.xo != nullptr) stv<V>(a.xo + row + c, x);
     if (a.fw == nullptr) stv<V>(lo + c, x);
     else stv<V>(z + c, x);
@@ -386,6 +458,24 @@ __global__ void __launch_bounds__(256)
   }
 }
 
+// out[t, c] = max(x[t, c], 0)^2; may run in place
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+    relu2_kernel(const T* x, long long ldx, T* out, long long ldo, long long rows, int D) {
+  const int nv = D / V;
+  const long long n = rows * nv;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long t = i / nv;
+    const int c = static_cast<int>(i - t * nv) * V;
+    float f[V];
+    ldv<V>(x + t * ldx + c, f);
+#pragma unroll
+    for (int k = 0; k < V; ++k) f[k] = relu2_f(f[k]);
+    stv<V>(out + t * ldo + c, f);
+  }
+}
+
 static int row_threads(int H, int V, int most) {
   int n = (H / V + 31) / 32 * 32;
   return n < 32 ? 32 : (n > most ? most : n);
@@ -407,19 +497,24 @@ static int launch_post_norm(const PostNormArgs& a, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-template <typename T, int V>
-static int launch_add_normed(const AddNormArgs& a, cudaStream_t s) {
+template <typename T, int V, bool kRouted>
+static int launch_add_normed_as(const AddNormArgs& a, cudaStream_t s) {
   const size_t smem = static_cast<size_t>(a.H) * sizeof(float);
   if (smem > 200 * 1024) return -2;
   if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(add_normed_kernel<T, V>,
+    cudaError_t e = cudaFuncSetAttribute(add_normed_kernel<T, V, kRouted>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   const int threads = row_threads(a.H, V, a.T < 2 * sm_count() ? 512 : 256);
-  add_normed_kernel<T, V><<<a.T, threads, smem, s>>>(a);
+  add_normed_kernel<T, V, kRouted><<<a.T, threads, smem, s>>>(a);
   return static_cast<int>(cudaGetLastError());
+}
+template <typename T, int V>
+static int launch_add_normed(const AddNormArgs& a, cudaStream_t s) {
+  return a.pos_of != nullptr ? launch_add_normed_as<T, V, true>(a, s)
+                             : launch_add_normed_as<T, V, false>(a, s);
 }
 
 static bool aligned(const void* p, int bytes) {
@@ -514,47 +609,83 @@ B200_API int b200_sigmoid_gate(const void* o, long long ldo, const void* z, long
   return static_cast<int>(cudaGetLastError());
 }
 
-// x = scale * e (fp32) and its copy `lo` in e's type; dtype (of e and lo): 0 bf16, 2 fp32.
-B200_API int b200_start_rows(const void* e, long long lde, float scale, float* x, void* lo, int T,
-                             int H, int dtype, void* stream) {
+// x = scale * e (+ step) in fp32; lo in e's type: a copy of x, or with w its RMS norm times w.
+// dtype (of e and lo): 0 bf16, 2 fp32.
+B200_API int b200_start_rows(const void* e, long long lde, float scale, const float* step,
+                             const float* w, float eps, float* x, void* lo, int T, int H, int dtype,
+                             void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || (dtype != 0 && dtype != 2)) return -2;
+  StartArgs a;
+  a.e = e; a.step = step; a.w = w; a.x = x; a.lo = lo; a.lde = lde; a.H = H; a.scale = scale;
+  a.eps = eps;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const bool v4 = (H % 4) == 0 && (lde % 4) == 0 && aligned(e, 16) && aligned(x, 16) &&
-                  aligned(lo, 16);
-  const int th = row_threads(H, v4 ? 4 : 1, 256);
+                  aligned(lo, 16) && aligned(step, 16) && aligned(w, 16);
+  const int th = row_threads(H, v4 ? 4 : 1, T < 2 * sm_count() ? 512 : 256);
   if (dtype == 0) {
-    const __nv_bfloat16* pe = static_cast<const __nv_bfloat16*>(e);
-    __nv_bfloat16* pl = static_cast<__nv_bfloat16*>(lo);
-    if (v4) start_rows_kernel<__nv_bfloat16, 4><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
-    else start_rows_kernel<__nv_bfloat16, 1><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
+    if (v4) start_rows_kernel<__nv_bfloat16, 4><<<T, th, 0, s>>>(a);
+    else start_rows_kernel<__nv_bfloat16, 1><<<T, th, 0, s>>>(a);
   } else {
-    const float* pe = static_cast<const float*>(e);
-    float* pl = static_cast<float*>(lo);
-    if (v4) start_rows_kernel<float, 4><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
-    else start_rows_kernel<float, 1><<<T, th, 0, s>>>(pe, lde, scale, x, pl, H);
+    if (v4) start_rows_kernel<float, 4><<<T, th, 0, s>>>(a);
+    else start_rows_kernel<float, 1><<<T, th, 0, s>>>(a);
   }
   return static_cast<int>(cudaGetLastError());
 }
 
-// xo = x + norm(y) * w + b; lo: the sum, or with fw (norm(sum) * fw + fb) * fscale.  centred 1:
-// layer norm, 0: RMS norm.  dtype (of y and lo): 0 bf16, 2 fp32.
-B200_API int b200_add_normed(const float* x, const void* y, long long ldy, const float* w,
+// xo = x + norm(y) * w + b (+ step); lo: the sum, or with fw (norm(sum) * fw + fb) * fscale.
+// centred 1: layer norm, 0: RMS norm.  With pos_of [T, k]: y holds expert-sorted rows, and the row
+// that is normalised is sum_s row_w[t, s] * y[pos_of[t, s]] + sigmoid(gate[t * ldg]) * shared[t].
+// dtype (of y, shared and lo): 0 bf16, 2 fp32.
+B200_API int b200_add_normed(const float* x, const void* y, long long ldy, const int* pos_of,
+                             const float* row_w, int k, const void* shared, long long ldsh,
+                             const float* gate, long long ldg, const float* step, const float* w,
                              const float* b, int centred, float eps, float* xo, const float* fw,
                              const float* fb, float fscale, void* lo, int T, int H, int dtype,
                              void* stream) {
   if (T <= 0) return 0;
-  if (H <= 0 || (dtype != 0 && dtype != 2) || lo == nullptr) return -2;
+  if (H <= 0 || (dtype != 0 && dtype != 2) || lo == nullptr ||
+      (pos_of != nullptr && (row_w == nullptr || k <= 0)))
+    return -2;
   AddNormArgs a;
   a.x = x; a.y = y; a.w = w; a.b = b; a.fw = fw; a.fb = fb; a.xo = xo; a.lo = lo; a.ldy = ldy;
-  a.T = T; a.H = H; a.centred = centred; a.eps = eps; a.fscale = fscale;
+  a.T = T; a.H = H; a.centred = centred; a.eps = eps; a.fscale = fscale; a.pos_of = pos_of;
+  a.row_w = row_w; a.k = k; a.shared = shared; a.ldsh = ldsh; a.gate = gate; a.ldg = ldg;
+  a.step = step;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool v4 = (H % 4) == 0 && (ldy % 4) == 0 && aligned(x, 16) && aligned(y, 16) &&
-                  aligned(w, 16) && aligned(b, 16) && aligned(fw, 16) && aligned(fb, 16) &&
-                  aligned(xo, 16) && aligned(lo, 16);
+  const bool v4 = (H % 4) == 0 && (ldy % 4) == 0 && (ldsh % 4) == 0 && aligned(x, 16) &&
+                  aligned(y, 16) && aligned(shared, 16) && aligned(step, 16) && aligned(w, 16) &&
+                  aligned(b, 16) && aligned(fw, 16) && aligned(fb, 16) && aligned(xo, 16) &&
+                  aligned(lo, 16);
   if (dtype == 0)
     return v4 ? launch_add_normed<__nv_bfloat16, 4>(a, s) : launch_add_normed<__nv_bfloat16, 1>(a, s);
   return v4 ? launch_add_normed<float, 4>(a, s) : launch_add_normed<float, 1>(a, s);
+}
+
+// out [T, D] = max(x, 0)^2, in place if the pointers are equal; dtype 0 bf16, 2 fp32.
+B200_API int b200_relu2(const void* x, long long ldx, void* out, long long ldo, int T, int D,
+                        int dtype, void* stream) {
+  if (T <= 0 || D <= 0) return 0;
+  if (dtype != 0 && dtype != 2) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const bool v4 = (D % 4) == 0 && (ldx % 4) == 0 && (ldo % 4) == 0 && aligned(x, 16) &&
+                  aligned(out, 16);
+  const long long items = static_cast<long long>(T) * (v4 ? D / 4 : D);
+  long long blocks = (items + 255) / 256;
+  const long long cap = static_cast<long long>(sm_count()) * 16;
+  const int g = static_cast<int>(blocks > cap ? cap : blocks);
+  if (dtype == 0) {
+    const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(x);
+    __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
+    if (v4) relu2_kernel<__nv_bfloat16, 4><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
+    else relu2_kernel<__nv_bfloat16, 1><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
+  } else {
+    const float* p = static_cast<const float*>(x);
+    float* o = static_cast<float*>(out);
+    if (v4) relu2_kernel<float, 4><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
+    else relu2_kernel<float, 1><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
+  }
+  return static_cast<int>(cudaGetLastError());
 }
 
 // o [T, N, DC] -> out [T, N * D]: times sigmoid(z) and scale.

@@ -291,6 +291,9 @@ class LLMEngine:
                 or getattr(self.model, "has_request_state", False):
             raise ValueError(f"{self.cfg.model.architecture} keeps recurrent state with its "
                              "requests, which the connector does not ship")
+        if "layer_shapes" in self.model.kv_cache_spec():
+            raise ValueError(f"the caches of {self.cfg.model.architecture} differ from layer to "
+                             "layer, which the connector does not ship")
         self.disagg = DisaggCoordinator(self, connector, recv_timeout_s)
         self.scheduler.on_free = self.disagg.before_free
         return self.disagg

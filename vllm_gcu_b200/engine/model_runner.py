@@ -222,8 +222,9 @@ class ModelRunner:
                 * torch.empty((), dtype=self.cfg.model.dtype).element_size() \
                 + 4 * sum(spec.get("block_state", ()))
         elif "layer_shapes" in spec:
-            bytes_per_block = max(1, 2 * self.block_size * sum(
-                h * d for h, d in (s for s in spec["layer_shapes"] if s is not None))
+            bytes_per_block = max(1, self.block_size * sum(
+                2 * s[0] * s[1] if len(s) == 2 else s[0]
+                for s in spec["layer_shapes"] if s is not None)
                 * torch.empty((), dtype=self.cfg.model.dtype).element_size())
         else:
             bytes_per_block = self.cfg.model.kv_bytes_per_token(
@@ -278,11 +279,14 @@ class ModelRunner:
             widths = spec.get("widths") or [spec["width"]] * spec["layers"]
             self.kv_caches = [torch.zeros(num_blocks, self.block_size, w, dtype=dt,
                                           device=self.device) for w in widths]
-        elif "layer_shapes" in spec:       # sizes per layer; layers without a cache hold nothing
-            if self.is_cuda and dt != mc.dtype:
+        elif "layer_shapes" in spec:
+            # sizes per layer: (key heads, head dimension), (row width) of a latent cache, None for
+            # a layer without one
+            if self.is_cuda and (dt != mc.dtype or kvd not in ("auto", "bfloat16", "float32")):
                 raise ValueError(f"{mc.architecture} has no 8-bit KV cache")
-            self.kv_caches = [torch.zeros(2, num_blocks if s else 0, self.block_size,
-                                          *(s or (1, 1)), dtype=dt, device=self.device)
+            new = lambda *s: torch.zeros(*s, dtype=dt, device=self.device)  # noqa: E731
+            self.kv_caches = [new(num_blocks, self.block_size, *s) if s and len(s) == 1 else
+                              new(2, num_blocks if s else 0, self.block_size, *(s or (1, 1)))
                               for s in spec["layer_shapes"]]
         else:
             self.kv_caches = [torch.zeros(2, num_blocks, self.block_size, spec["kv_heads"],
@@ -306,7 +310,7 @@ class ModelRunner:
                 self.drafter_caches = [torch.zeros(2, num_blocks, self.block_size, ds["kv_heads"],
                                                    ds["head_dim"], dtype=dt, device=self.device)
                                        for _ in range(ds["layers"])]
-        if self.is_cuda and spec["type"] == "gqa":
+        if self.is_cuda and spec["type"] in ("gqa", "layers"):
             Hq = spec.get("q_heads") or \
                 mc.num_attention_heads // self.cfg.parallel.tensor_parallel_size
             ns = 32
@@ -317,7 +321,7 @@ class ModelRunner:
                             device=self.device))
 
     def _decode_splits(self, batch: int, max_seq_len: int) -> int:
-        if not self.is_cuda or self.model.kv_cache_spec()["type"] != "gqa":
+        if not self.is_cuda or self.model.kv_cache_spec()["type"] not in ("gqa", "layers"):
             return 1
         from ..ops import cuda as C
         spec = self.model.kv_cache_spec()

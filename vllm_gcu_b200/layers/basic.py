@@ -68,6 +68,18 @@ class ScalarGain(nn.Module):
         self.gain.data.copy_(full.reshape(()))
 
 
+class RMSNormParams(nn.Module):
+    """fp32 weight of an RMS norm that is fused with a residual sum."""
+
+    def __init__(self, hidden_size: int, device=None):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=torch.float32, device=device),
+                                   requires_grad=False)
+
+    def load_weight(self, name: str, full: torch.Tensor, shard_id=None) -> None:
+        self.weight.data.copy_(full)
+
+
 class LayerNormParams(nn.Module):
     """fp32 weight and bias of a layer norm that is fused with a residual sum."""
 
@@ -97,11 +109,12 @@ def _yarn_mscale(scale: float, mscale: float = 1.0) -> float:
 
 
 def build_cos_sin_cache(rot_dim: int, max_pos: int, base: float,
-                        rope_scaling: Optional[dict]) -> torch.Tensor:
-    """fp32 ``[max_pos, rot_dim]`` = ``[cos | sin]``; handles plain, linear, llama3 and
+                        rope_scaling: Optional[dict] = None,
+                        dtype: torch.dtype = torch.float32) -> torch.Tensor:
+    """``[max_pos, rot_dim]`` = ``[cos | sin]``, computed in ``dtype``; handles plain, linear, llama3 and
     YaRN / deepseek_yarn scaling (the variants used by the reference's models,
     vllm_gcu/kernels/rotary_embedding.py:67-106, deepseek_v3.py:393-411)."""
-    inv_freq = 1.0 / (base ** (torch.arange(0, rot_dim, 2, dtype=torch.float32) / rot_dim))
+    inv_freq = 1.0 / (base ** (torch.arange(0, rot_dim, 2, dtype=dtype) / rot_dim))
     mscale = 1.0
     t_scale = 1.0
     if rope_scaling:
@@ -143,7 +156,7 @@ def build_cos_sin_cache(rot_dim: int, max_pos: int, base: float,
                           / _yarn_mscale(factor, float(ms_all or 0.0)))
             else:
                 mscale = _yarn_mscale(factor)
-    t = torch.arange(max_pos, dtype=torch.float32) / t_scale
+    t = torch.arange(max_pos, dtype=dtype) / t_scale
     freqs = torch.outer(t, inv_freq)
     return torch.cat([freqs.cos() * mscale, freqs.sin() * mscale], dim=-1)
 

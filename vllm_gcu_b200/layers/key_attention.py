@@ -1,8 +1,12 @@
-"""Attention whose queries and keys are normalised over the whole projection, with attention
-sinks and an output gate; the values are the projected keys themselves.
+"""Grouped attention over normalised queries and keys, as parts of a mixer.
 
-Paged cache ``[2, blocks, block_size, kv_heads, DC]`` as in ``PagedAttention``: rotated keys and
-raw keys (the values), heads padded to a width the tensor-core kernels take.  On the GPU one kernel
+* ``KeyAttention``: norm over the whole projection, rotary positions, attention sinks and an output
+  gate; the values are the projected keys themselves.
+* ``ChunkAttention``: norm over every head, no positions, soft capped scores, keys of the query's own
+  chunk of positions only; values of their own, of any width.
+
+Paged cache ``[2, blocks, block_size, kv_heads, DC]`` as in ``PagedAttention``: normalised (rotated)
+keys and values, heads padded to a width the tensor-core kernels take.  On the GPU one kernel
 normalises, rotates and writes the cache; decode rows run through the split-KV kernels, portions
 through the tcgen05 prefill kernel, everything else (32-bit models, wide heads, large groups)
 through the general kernel of csrc/attention_any.cu.
@@ -37,59 +41,60 @@ def cached_head_dim(head_dim: int, dtype: torch.dtype) -> int:
     return -(-head_dim // 4) * 4
 
 
-class KeyAttention(MixerPart):
-    def __init__(self, spec: AttentionSpec, eps: float, dtype, device, prefix: str,
-                 rotary: RotaryEmbedding):
+class CachedAttention(MixerPart):
+    """Heads, cache and attention kernels that the kinds of attention share."""
+
+    def __init__(self, spec: AttentionSpec, eps: float, dtype, prefix: str):
         super().__init__()
-        self.spec, self.eps, self.rotary = spec, eps, rotary
-        H, G, D = spec.num_heads, spec.num_kv_heads, spec.head_dim
+        self.spec, self.eps = spec, eps
+        H, G = spec.num_heads, spec.num_kv_heads
+        self.VD = spec.v_head_dim or spec.head_dim
+        widest = max(spec.head_dim, self.VD)
         tp = tp_size()
         if H % G:
             raise ValueError(f"{prefix}: {H} query heads over {G} key heads")
         if H % tp or G % tp:
             raise ValueError(f"{prefix}: {H} query and {G} key heads over {tp} ranks")
-        if D > MAX_HEAD_DIM:
-            raise ValueError(f"{prefix}: heads of {D} dimensions, at most {MAX_HEAD_DIM}")
-        if spec.rot_dims % 2 or not 0 <= spec.rot_dims <= D:
-            raise ValueError(f"{prefix}: {spec.rot_dims} rotated of {D} dimensions")
-        self.H, self.G, self.DC = H // tp, G // tp, cached_head_dim(D, dtype)
-        self.width = H * D
-        self.projections = [("q", H * D, True), ("k", G * D, True), ("g", H * D, True)]
-        self.q_norm = self.new(self.H * D, device=device)
-        self.k_norm = self.new(self.G * D, device=device)
-        self.sink = self.new(self.H, device=device)
+        if widest > MAX_HEAD_DIM:
+            raise ValueError(f"{prefix}: heads of {widest} dimensions, at most {MAX_HEAD_DIM}")
+        self.H, self.G, self.DC = H // tp, G // tp, cached_head_dim(widest, dtype)
+        self.width = H * self.VD
+        self.sink = None
 
     def cache_shape(self) -> tuple[int, int]:
         return self.G, self.DC
 
-    _OWN = {"q.norm": "q_norm", "k.norm": "k_norm", "sink": "sink"}
+    _OWN: dict = {}
 
     def own_tensors(self) -> set[str]:
         return set(self._OWN)
 
-    def load(self, name: str, full: torch.Tensor) -> bool:
-        if name not in self._OWN:
-            return False
-        getattr(self, self._OWN[name]).data.copy_(self.shard(full))
-        return True
-
-    def _attend(self, q: torch.Tensor, cache: torch.Tensor, md: AttentionMetadata) -> torch.Tensor:
+    def _attend(self, q: torch.Tensor, cache: torch.Tensor, md: AttentionMetadata,
+                out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``out``: rows ``[T, H, VD]`` (the row pitch is free) for the first VD columns of every
+        head's result; None: all DC columns."""
         s = self.spec
         kc, vc = cache[0], cache[1]
         nd, npf, nr = md.num_decode_tokens, md.num_prefills, md.num_decodes
+        od = self.DC if out is None else self.VD
+        rest = dict(scale=s.scale, sink=self.sink, softcap=s.softcap, chunk=s.chunk, out_dim=od)
         if not ops.use_native(q):
             return ref.any_attention(q, kc, vc, md.block_tables, md.seq_lens, nd, md.cu_q_prefill,
-                                     s.scale, self.sink)
-        rest = dict(scale=s.scale, sink=self.sink)
+                                     out=out, **rest)
         tensor_cores = q.dtype == torch.bfloat16 and self.DC in (64, 96, 128)
         if not tensor_cores:
             return C.any_attention(q, kc, vc, md.block_tables, md.seq_lens, nd, md.cu_q_prefill,
-                                   **rest)
-        out = torch.empty_like(q)
+                                   out=out, **rest)
+        if out is None:
+            out = torch.empty_like(q)
         if nd > 0:
             if self.H // self.G <= MAX_DECODE_GROUP:
+                splits = md.decode_splits
+                if s.chunk:          # no more keys than a chunk holds
+                    splits = min(splits, C.decode_num_splits(nd, self.G,
+                                                             min(s.chunk, max(md.max_seq_len, 1))))
                 C.paged_decode(q[:nd], kc, vc, md.block_tables[:nd], md.seq_lens[:nd], out=out[:nd],
-                               num_splits=md.decode_splits, workspace=md.decode_workspace, **rest)
+                               num_splits=splits, workspace=md.decode_workspace, **rest)
             else:
                 C.any_attention(q[:nd], kc, vc, md.block_tables[:nd], md.seq_lens[:nd], nd, None,
                                 out=out[:nd], **rest)
@@ -100,6 +105,28 @@ class KeyAttention(MixerPart):
             if done is None:
                 C.any_attention(q[nd:], kc, vc, bt, sl, 0, md.cu_q_prefill, out=out[nd:], **rest)
         return out
+
+
+class KeyAttention(CachedAttention):
+    def __init__(self, spec: AttentionSpec, eps: float, dtype, device, prefix: str,
+                 rotary: RotaryEmbedding):
+        super().__init__(spec, eps, dtype, prefix)
+        self.rotary = rotary
+        H, G, D = spec.num_heads, spec.num_kv_heads, spec.head_dim
+        if spec.rot_dims % 2 or not 0 <= spec.rot_dims <= D:
+            raise ValueError(f"{prefix}: {spec.rot_dims} rotated of {D} dimensions")
+        self.projections = [("q", H * D, True), ("k", G * D, True), ("g", H * D, True)]
+        self.q_norm = self.new(self.H * D, device=device)
+        self.k_norm = self.new(self.G * D, device=device)
+        self.sink = self.new(self.H, device=device)
+
+    _OWN = {"q.norm": "q_norm", "k.norm": "k_norm", "sink": "sink"}
+
+    def load(self, name: str, full: torch.Tensor) -> bool:
+        if name not in self._OWN:
+            return False
+        getattr(self, self._OWN[name]).data.copy_(self.shard(full))
+        return True
 
     def mix(self, h, y, f, fw, md: AttentionMetadata, cache: Optional[torch.Tensor],
             state: Optional[dict], scale: float, out: torch.Tensor) -> None:
@@ -117,3 +144,36 @@ class KeyAttention(MixerPart):
                                    self.rotary.cos_sin_cache, self.rotary.is_neox, md.positions,
                                    md.slot_mapping, cache[0], cache[1], D, sumsq, tp)
         o_.head_gate(self._attend(qn, cache, md), y["g"][:, :self.H * D], scale, D, out)
+
+
+class ChunkAttention(CachedAttention):
+    def __init__(self, spec: AttentionSpec, eps: float, dtype, device, prefix: str):
+        super().__init__(spec, eps, dtype, prefix)
+        H, G, D = spec.num_heads, spec.num_kv_heads, spec.head_dim
+        if spec.rot_dims or not spec.v_head_dim:
+            raise ValueError(f"{prefix}: chunked attention has no rotation and values of its own")
+        self.projections = [("q", H * D, True), ("k", G * D, True), ("v", G * self.VD, True)]
+        self.q_norm = self.new(D, device=device)
+        self.k_norm = self.new(D, device=device)
+
+    _OWN = {"q.norm": "q_norm", "k.norm": "k_norm"}
+
+    def load(self, name: str, full: torch.Tensor) -> bool:
+        if name not in self._OWN:
+            return False
+        getattr(self, self._OWN[name]).data.copy_(full)      # shared by the heads of all ranks
+        return True
+
+    def mix(self, h, y, f, fw, md: AttentionMetadata, cache: Optional[torch.Tensor],
+            state: Optional[dict], scale: float, out: torch.Tensor) -> None:
+        D = self.spec.head_dim
+        if cache is None or md.is_dummy:
+            out.zero_()
+            return
+        o_ = C if ops.use_native(out) else ref
+        qn = o_.head_norm_cache(y["q"][:, :self.H * D], y["k"][:, :self.G * D],
+                                y["v"][:, :self.G * self.VD], self.q_norm, self.k_norm, self.eps,
+                                md.slot_mapping, cache[0], cache[1], D)
+        self._attend(qn, cache, md, out.unflatten(1, (self.H, self.VD)))
+        if scale != 1.0:
+            out.mul_(scale)

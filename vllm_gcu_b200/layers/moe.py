@@ -39,7 +39,8 @@ from ..ops import ref
 from ..parallel.communicator import get_comm
 from ..parallel.state import (ep_rank, ep_size, exchange_dp_rows, get_state, tp_rank,
                               tp_size)
-from .linear import ReplicatedLinear
+from .linear import (ColumnParallelLinear, MixedParallelLinear, ReplicatedLinear,
+                     RowParallelLinear, linear_fp32)
 
 
 def select_experts(router_logits: torch.Tensor, cfg: ModelConfig,
@@ -59,25 +60,24 @@ def select_experts(router_logits: torch.Tensor, cfg: ModelConfig,
         w = torch.full((T, k), 1.0 / k, dtype=torch.float32, device=router_logits.device)
         return w, ids
     grouped = cfg.n_group > 1 or cfg.scoring_func == "sigmoid" or bias is not None
-    scale = cfg.routed_scaling_factor if grouped else 1.0
-    # plain softmax top-k with a scaling factor (DeepSeek-V2 "greedy" routing): the router
-    # paths below fold the factor in only for the grouped form
-    post = float(cfg.routed_scaling_factor) if not grouped else 1.0
+    scale = float(cfg.routed_scaling_factor)
     if ops.use_native(router_logits):
         w, ids = C.moe_topk(router_logits, k, cfg.norm_topk_prob, cfg.n_group, cfg.topk_group,
                             bias, cfg.scoring_func == "sigmoid", scale,
                             log2phy=eplb.log2phy if eplb is not None else None,
                             replica_count=eplb.replica_count if eplb is not None else None,
                             load=eplb.load if eplb is not None else None)
-        return (w * post if post != 1.0 else w), ids
+        return w, ids
     if grouped:
         w, ids = ref.grouped_topk(router_logits, k, cfg.norm_topk_prob, max(cfg.n_group, 1),
                                   max(cfg.topk_group, 1), bias, cfg.scoring_func, scale)
     else:
         w, ids = ref.topk_softmax(router_logits, k, cfg.norm_topk_prob)
+        # plain softmax top-k with a scaling factor (DeepSeek-V2 "greedy" routing)
+        w = w * scale if scale != 1.0 else w
     if eplb is not None:
         ids = ref.eplb_map_to_physical(ids, eplb.log2phy, eplb.replica_count, eplb.load)
-    return (w * post if post != 1.0 else w), ids
+    return w, ids
 
 
 class FusedMoE(nn.Module):
@@ -443,6 +443,128 @@ class InputWeightedMoE(FusedMoE):
                 ) -> tuple[torch.Tensor, torch.Tensor]:
         op = C.input_weighted_experts if ops.use_native(x) else ref.input_weighted_experts
         return op(x, self.w13, self.w2, topk_w, topk_ids)
+
+
+class SquaredReluMoE(FusedMoE):
+    """Routed experts without a gate: ``down_e(max(up_e(h), 0)^2)``.
+
+    ``forward`` returns the experts' unweighted output rows in sorted order and the row of every
+    (token, slot) pair, which the norm after the residual sum weights and adds up (this rank's slice
+    of the intermediate dimension under TP).  On the GPU the stacked weights are padded with zeros
+    to the tile sizes of the grouped GEMM, which leaves the result as it is."""
+
+    def __init__(self, num_experts: int, hidden: int, inter: int, dtype, device, prefix: str = ""):
+        tp = tp_size()
+        if inter % tp:
+            raise ValueError(f"{prefix}: experts of width {inter} over {tp} ranks")
+        self.hidden_full, self.inter_real = hidden, inter // tp
+        native = torch.device(device).type == "cuda" if device is not None else False
+        m = 64 if native and dtype == torch.bfloat16 else 1
+        up = lambda n: -(-n // m) * m  # noqa: E731
+        super().__init__(num_experts, up(hidden), up(self.inter_real) * tp, dtype, device, False,
+                         prefix)
+        E, I, H = self.local_experts, self.inter, self.hidden
+        del self.w13
+        self.w1 = nn.Parameter(torch.zeros(E, I, H, dtype=dtype, device=device),
+                               requires_grad=False)
+        self.w2.data.zero_()
+
+    def _load_one(self, expert_id: int, which: str, full: torch.Tensor) -> bool:
+        I, H, lo = self.inter_real, self.hidden_full, self.shard_index * self.inter_real
+        if not 0 <= expert_id < self.local_experts or which not in ("up", "down"):
+            return False
+        if which == "up":
+            self.w1.data[expert_id, :I, :H].copy_(full[lo:lo + I])
+        else:
+            self.w2.data[expert_id, :H, :I].copy_(full[:, lo:lo + I])
+        return True
+
+    def finalize(self) -> None:
+        """Clears the padding (after a random initialisation of the whole parameters)."""
+        for w in (self.w1.data, self.w2.data.transpose(1, 2)):
+            w[:, self.inter_real:] = 0
+            w[:, :, self.hidden_full:] = 0
+
+    def forward(self, x: torch.Tensor, topk_ids: torch.Tensor
+                ) -> tuple[torch.Tensor, torch.Tensor]:
+        op = C.squared_relu_experts if ops.use_native(x) else ref.squared_relu_experts
+        return op(x, self.w1, self.w2, topk_ids)
+
+
+class SquaredReluMLP(nn.Module):
+    """``down(max(up(x), 0)^2)``; the result is this rank's part of the sum."""
+
+    def __init__(self, hidden: int, inter: int, dtype, device, prefix: str):
+        super().__init__()
+        self.up_proj = ColumnParallelLinear(hidden, inter, dtype=dtype, device=device,
+                                            prefix=prefix + ".up_proj")
+        self.down_proj = RowParallelLinear(inter, hidden, reduce_results=False, dtype=dtype,
+                                           device=device, prefix=prefix + ".down_proj")
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        if ops.use_native(x) and x.dtype == torch.bfloat16:
+            return self.down_proj(C.gemm_bf16(x, self.up_proj.weight, epilogue=C.EPI_RELU2))
+        return self.down_proj((C if ops.use_native(x) else ref).relu2(self.up_proj(x)))
+
+
+class GatedSharedMoE(nn.Module):
+    """fp32 softmax router with renormalised weights, squared-ReLU experts and an optional shared
+    expert behind a gate of one number per token.
+
+    ``forward`` returns ``(y, operands)`` for ``ops.add_normed``, which weights and sums the rows.
+    Router and shared expert's gate are one narrow GEMM with fp32 results."""
+
+    def __init__(self, num_experts: int, top: int, scale: float, hidden: int, inter: int,
+                 shared_inter: int, dtype, device, prefix: str):
+        super().__init__()
+        self.route_cfg = ModelConfig(num_experts=num_experts, num_experts_per_tok=top,
+                                     routed_scaling_factor=scale, scoring_func="softmax",
+                                     norm_topk_prob=True)
+        self.router = MixedParallelLinear(hidden, [num_experts] + [1] * (shared_inter > 0),
+                                          [False] * (1 + (shared_inter > 0)), dtype=dtype,
+                                          device=device, prefix=prefix + ".router", align=8)
+        self.experts = SquaredReluMoE(num_experts, hidden, inter, dtype, device,
+                                      prefix + ".experts")
+        self.shared = SquaredReluMLP(hidden, shared_inter, dtype, device, prefix + ".shared") \
+            if shared_inter > 0 else None
+
+    def load(self, name: str, full: torch.Tensor) -> bool:
+        """False if there is no tensor of that name."""
+        if name == "router":
+            self.router.load_weight("weight", full, 0)
+        elif name.startswith("shared.") and self.shared is None:
+            return False
+        elif name == "shared.sg":
+            self.router.load_weight("weight", full, 1)
+        elif name in ("shared.up", "shared.down"):
+            getattr(self.shared, name[7:] + "_proj").load_weight("weight", full)
+        else:
+            e, _, which = name.partition(".")
+            return e[:1] == "e" and e[1:].isdigit() and \
+                self.experts.load_expert_weight(int(e[1:]), which, full)
+        return True
+
+    def tensor_names(self) -> set[str]:
+        names = {f"e{e}.{k}" for e in range(self.experts.local_experts) for k in ("up", "down")}
+        return names | {"router"} | ({"shared.up", "shared.down", "shared.sg"}
+                                     if self.shared is not None else set())
+
+    def forward(self, h: torch.Tensor) -> tuple[torch.Tensor, dict]:
+        z = self.router.split(linear_fp32(h, self.router.weight))
+        w, ids = select_experts(z[0], self.route_cfg)
+        y, pos_of = self.experts(h, ids)
+        rows = dict(pos_of=pos_of, row_w=w)
+        if self.shared is not None:
+            rows.update(shared=self.shared(h), gate=z[1][:, 0])
+        if tp_size() == 1:
+            return y, rows
+        # every rank has its slice of the intermediate dimensions: sum rows, then ranks
+        T, k = w.shape
+        p = pos_of.view(-1)[:T * k].view(T, k).long()
+        out = (y[p.clamp(min=0)].float() * (w * (p >= 0)).unsqueeze(-1)).sum(1)[:, :h.shape[1]]
+        if self.shared is not None:
+            out += torch.sigmoid(rows["gate"]).unsqueeze(-1) * rows["shared"].float()
+        return get_comm("tp").all_reduce(out.to(h.dtype).contiguous()), {}
 
 
 class EplbState:

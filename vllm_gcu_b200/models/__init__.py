@@ -52,6 +52,7 @@ _REGISTRY: dict[str, str] = {
     "DeepseekVLV2ForCausalLM": "vllm_gcu_b200.models.deepseek_vl2:DeepseekVLV2ForCausalLM",
     "SapapelForCausalLM": "vllm_gcu_b200.models.sapapel:SapapelForCausalLM",
     "FizunexForCausalLM": "vllm_gcu_b200.models.fizunex:FizunexForCausalLM",
+    "FepopelForCausalLM": "vllm_gcu_b200.models.fepopel:FepopelForCausalLM",
     "DeepSeekMTPModel": "vllm_gcu_b200.models.deepseek_mtp:DeepSeekMTP",
     # pooling models (no KV cache; built by build_pooling_model)
     "XLMRobertaForSequenceClassification":

@@ -14,7 +14,7 @@ import torch
 from . import _native as N
 from ._native import DTYPE_CODE, call, ptr, stream_ptr
 
-EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RESIDUAL, EPI_FP32 = 0, 1, 2, 3, 4
+EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RESIDUAL, EPI_FP32, EPI_RELU2 = 0, 1, 2, 3, 4, 9
 
 NORM_QMODES = {None: 0, "fp8_static": 1, "fp8_token": 2, "fp8_group128": 3,
                "int8_static": 4, "int8_token": 5}
@@ -141,6 +141,8 @@ def gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = No
         if bias is None and residual is None and epilogue == EPI_SILU_MUL:
             w4 = want.view(want.shape[0], -1, 2, ref.GATE_UP_BLOCK)
             want = (torch.nn.functional.silu(w4[:, :, 0]) * w4[:, :, 1]).reshape(want.shape[0], -1)
+        if epilogue == EPI_RELU2:
+            want = want.clamp(min=0).square()
         oracle_compare("gemm_bf16", res, want, 3e-2, 3e-2 * max(1.0, float(want.abs().mean())))
     return res
 
@@ -151,7 +153,7 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
     """``out[M,N] = a[M,K] @ b[N,K]^T`` on the tcgen05 path (bf16 in, fp32 accumulate).
 
     epilogue EPI_SILU_MUL expects ``b`` interleaved by ``ref.interleave_gate_up`` and
-    yields ``[M, N/2]``; EPI_FP32 writes fp32."""
+    yields ``[M, N/2]``; EPI_FP32 writes fp32; EPI_RELU2 yields ``max(out, 0)^2``."""
     assert a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16
     a = _rowmajor_2d(a)
     M, K = a.shape
@@ -176,10 +178,12 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
             y = y + bias
         if residual is not None:
             y = y + residual
+        if epilogue == EPI_RELU2:
+            y = relu2(y)
         out.copy_(y)
         return out
     if (USE_PAIR_GEMM and PAIR_MIN_M <= M < WIDE2_MIN_M and Nn % 256 == 0 and K % 64 == 0
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL)
+            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2)
             and -(-M // 256) * (Nn // 256) >= PAIR_MIN_TILES):
         # enough 256 x 256 tiles to occupy the SM pairs (gate_up, LM head at decode batch sizes;
         # graph-replay timing at 256 rows: gate_up 62.5 -> 57.9 us, LM head 266 -> 228 us)
@@ -206,7 +210,7 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
                 raise N.NativeError(f"b200_gemm_pair_split failed with code {rc}")
     silu_256 = epilogue != EPI_SILU_MUL or Nn % 256 == 0     # these two kernels: 256-wide tiles
     if M <= SKINNY_MAX_M and USE_SKINNY_GEMM and silu_256 \
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL):
+            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2):
         ws, ctr = _skinny_workspace(a.device)
         rc = N.lib().b200_gemm_skinny(
             ptr(a), a.stride(0), ptr(b), b.stride(0), ptr(out), out.stride(0), M, Nn, K,
@@ -219,7 +223,7 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
         if rc != -20:
             raise N.NativeError(f"b200_gemm_skinny failed with code {rc}")
     if (USE_PAIR_GEMM and M >= WIDE2_MIN_M and Nn % 256 == 0 and K % 64 == 0
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL) and _wide2_pays(M, Nn)):
+            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2) and _wide2_pays(M, Nn)):
         # one 256 x 256 tile per pair of CTAs (gemm_pair.cu); -20 = shape or device not covered
         rc = N.lib().b200_gemm_pair(ptr(a), a.stride(0), ptr(b), b.stride(0), ptr(out),
                                     out.stride(0), M, Nn, K, ptr(bias), epilogue, stream_ptr())
@@ -449,11 +453,13 @@ def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                  workspace: Optional[tuple[torch.Tensor, torch.Tensor]] = None,
                  max_seq_len: int = 0, kv_quant: Optional[tuple] = None,
                  alibi_slopes: Optional[torch.Tensor] = None,
-                 sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 sink: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
+                 out_dim: int = 0) -> torch.Tensor:
     res = _paged_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, out, num_splits,
-                        workspace, max_seq_len, kv_quant, alibi_slopes, sink)
+                        workspace, max_seq_len, kv_quant, alibi_slopes, sink, softcap, chunk,
+                        out_dim)
     if (oracle_enabled("paged_decode") and k_cache.element_size() > 1 and alibi_slopes is None
-            and sink is None
+            and sink is None and not softcap and not chunk and not out_dim
             and not torch.cuda.is_current_stream_capturing()):
         from . import ref
         live = seq_lens > 0
@@ -469,16 +475,21 @@ def _paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                   workspace: Optional[tuple[torch.Tensor, torch.Tensor]] = None,
                   max_seq_len: int = 0, kv_quant: Optional[tuple] = None,
                   alibi_slopes: Optional[torch.Tensor] = None,
-                  sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  sink: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
+                  out_dim: int = 0) -> torch.Tensor:
     """q ``[B, Hq, D]`` (row stride free), caches ``[blocks, bs, Hkv, D]``.  For fp8 / int8
     caches ``kv_quant = (k_scale, v_scale, k_zero_point, v_zero_point)`` (floats).
     ``alibi_slopes`` fp32 ``[Hq]`` adds slope * (key position - query position) to the scores
-    (bf16 / fp16 caches).  ``sink`` fp32 ``[Hq]``: exp(sink) joins the softmax denominator."""
+    (bf16 / fp16 caches).  ``sink`` fp32 ``[Hq]``: exp(sink) joins the softmax denominator.
+    ``softcap``: scores become softcap * tanh(score / softcap).  ``chunk``: only the keys of the
+    query's own chunk of positions.  ``out_dim``: only the first columns of every head's output."""
     B, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
+    od = out_dim or D
     assert q.stride(2) == 1 and q.stride(1) == D
     if out is None:
-        out = torch.empty((B, Hq, D), device=q.device, dtype=q.dtype)
+        out = torch.empty((B, Hq, od), device=q.device, dtype=q.dtype)
+    assert out.stride(2) == 1 and out.stride(1) == od
     if num_splits <= 0:
         num_splits = decode_num_splits(B, Hkv, max_seq_len or block_tables.shape[1] * bs)
     tmp_out = tmp_lse = None
@@ -500,11 +511,11 @@ def _paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
         assert alibi_slopes.dtype == torch.float32 and alibi_slopes.numel() == Hq
         call("b200_paged_decode_alibi", *args[:-1], ptr(alibi_slopes), stream_ptr())
         return out
-    if sink is not None:
+    if sink is not None or softcap or chunk or od != D:
         if k_cache.element_size() == 1:
-            raise NotImplementedError("attention sinks over an 8-bit KV cache")
-        assert sink.dtype == torch.float32 and sink.numel() == Hq
-        tail = (ptr(sink), stream_ptr())
+            raise NotImplementedError("attention sinks, caps and chunks over an 8-bit KV cache")
+        assert sink is None or (sink.dtype == torch.float32 and sink.numel() == Hq)
+        tail = (ptr(sink), float(softcap), int(chunk), od, stream_ptr())
         if USE_TMA_DECODE and D == 128 and bs % 16 == 0 and k_cache.stride(2) == 128 \
                 and k_cache.stride(1) == Hkv * 128:
             rc = N.lib().b200_paged_decode_tma_sink(*args[:-1], *tail)
@@ -611,19 +622,24 @@ def _varlen_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
 def fmha_prefill_sink(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       block_tables: torch.Tensor, cu_q: torch.Tensor, seq_lens: torch.Tensor,
                       scale: float, num_q_tiles_128: int, sink: Optional[torch.Tensor],
-                      out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """Causal tcgen05 prefill attention for head dimensions 64, 96 and 128 with optional sinks
-    (see ``paged_decode``); None when the layout is not covered (then use ``any_attention``)."""
+                      out: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
+                      out_dim: int = 0) -> Optional[torch.Tensor]:
+    """Causal tcgen05 prefill attention for head dimensions 64, 96 and 128 with optional sinks, soft
+    cap, chunks and output columns (see ``paged_decode``); None when the layout is not covered (then
+    use ``any_attention``)."""
     T, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
+    od = out_dim or D
     assert q.stride(2) == 1 and q.stride(1) == D
     if out is None:
-        out = torch.empty((T, Hq, D), device=q.device, dtype=q.dtype)
+        out = torch.empty((T, Hq, od), device=q.device, dtype=q.dtype)
+    assert out.stride(2) == 1 and out.stride(1) == od
     rc = N.lib().b200_fmha_prefill_sink(
         ptr(q), q.stride(0), ptr(out), out.stride(0), None, ptr(cu_q), ptr(seq_lens), ptr(k_cache),
         ptr(v_cache), k_cache.stride(1), k_cache.stride(2), nb * bs, ptr(block_tables),
         block_tables.stride(0), bs, block_tables.shape[0], T, num_q_tiles_128, Hq, Hkv, D,
-        float(scale), 1, 0, DTYPE_CODE[q.dtype], ptr(sink), stream_ptr())
+        float(scale), 1, 0, DTYPE_CODE[q.dtype], ptr(sink), float(softcap), int(chunk), od,
+        stream_ptr())
     N.launch_count += 1
     if rc == -20:
         return None
@@ -635,20 +651,45 @@ def fmha_prefill_sink(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
 def any_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                   block_tables: torch.Tensor, seq_lens: torch.Tensor, num_decodes: int,
                   cu_q: Optional[torch.Tensor], scale: float, sink: Optional[torch.Tensor] = None,
-                  out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  out: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
+                  out_dim: int = 0) -> torch.Tensor:
     """Causal paged attention for any head dimension (<= 512) and group size, fp32 or bf16
     (csrc/attention_any.cu): q ``[T, Hq, D]``, the first ``num_decodes`` tokens one per request,
-    the rest by ``cu_q``."""
+    the rest by ``cu_q``.  ``softcap``, ``chunk``, ``out_dim``: see ``paged_decode``."""
     T, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
+    od = out_dim or D
     assert q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()
     assert k_cache.dtype == q.dtype and k_cache.shape[3] == D
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty((T, Hq, od), dtype=q.dtype, device=q.device)
+    assert out.stride(2) == 1 and out.stride(1) == od
     call("b200_any_attention", ptr(q), ptr(k_cache), ptr(v_cache), nb * bs, ptr(out),
-         ptr(block_tables), block_tables.stride(0), bs, ptr(seq_lens), ptr(cu_q), ptr(sink), T, Hq,
-         Hkv, D, num_decodes, cu_q.shape[0] - 1 if cu_q is not None else 0, float(scale),
-         DTYPE_CODE[q.dtype], stream_ptr())
+         out.stride(0), od, ptr(block_tables), block_tables.stride(0), bs, ptr(seq_lens), ptr(cu_q),
+         ptr(sink), T, Hq, Hkv, D, num_decodes, cu_q.shape[0] - 1 if cu_q is not None else 0,
+         float(scale), float(softcap), int(chunk), DTYPE_CODE[q.dtype], stream_ptr())
+    return out
+
+
+def head_norm_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_weight: torch.Tensor,
+                    k_weight: torch.Tensor, eps: float, slot_mapping: torch.Tensor,
+                    k_cache: torch.Tensor, v_cache: torch.Tensor, head_dim: int) -> torch.Tensor:
+    """RMS norm of every query and key head over its ``head_dim`` columns (weights ``[head_dim]``
+    fp32, shared by all heads); keys and values into the paged caches ``[blocks, bs, Hkv, DC]`` with
+    zeros behind their columns.  q ``[T, Hq * D]``, k ``[T, Hkv * D]``, v ``[T, Hkv * VD]``
+    (row-strided views are fine).  Returns the queries ``[T, Hq, DC]``."""
+    T = q.shape[0]
+    nb, bs, Hkv, DC = k_cache.shape
+    D = head_dim
+    Hq = q.shape[1] // D
+    assert q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == q.dtype
+    assert q_weight.dtype == torch.float32 and k_weight.dtype == torch.float32
+    out = torch.empty((T, Hq, DC), dtype=q.dtype, device=q.device)
+    call("b200_head_norm_cache", ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v), v.stride(0),
+         ptr(q_weight), ptr(k_weight), float(eps), ptr(slot_mapping), ptr(out), ptr(k_cache),
+         ptr(v_cache), nb * bs, T, Hq, Hkv, D, v.shape[1] // Hkv, DC, DTYPE_CODE[q.dtype],
+         stream_ptr())
     return out
 
 
@@ -718,12 +759,15 @@ def mla_attention_supported(q: torch.Tensor, cache: torch.Tensor, L: int) -> boo
 def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
                   seq_lens: torch.Tensor, cu_q: Optional[torch.Tensor], num_tiles: int,
                   max_seq_len: int, scale: float, out: Optional[torch.Tensor] = None,
-                  splits: Optional[int] = None, L: int = 512) -> torch.Tensor:
+                  splits: Optional[int] = None, L: int = 512,
+                  sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None
+                  ) -> torch.Tensor:
     """Latent-absorbed multi-head latent attention (attention_mla.cu).  q ``[T, N, W]``,
     cache ``[blocks, block_size, W]`` whose first ``L`` columns are the value, returns
     ``[T, N, L]``.  ``cu_q`` None: one query token per request (decode).  ``num_tiles`` >= sum
     over requests of ceil(q_len / (128 // N)).  Causal inside each request over absolute
-    positions."""
+    positions.  ``sink`` fp32 ``[N]``: exp(sink) joins the softmax denominator.  ``gate`` bf16
+    ``[T, N]`` (row-strided view): head h's output is multiplied by sigmoid(gate[t, h])."""
     T, Nh, W = q.shape
     assert q.is_contiguous() and cache.is_contiguous()
     nb, bs, _ = cache.shape
@@ -743,7 +787,8 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tens
     rc = N.lib().b200_mla_attention(
         ptr(q), ptr(out), ptr(cache), nb * bs, ptr(cu_q), ptr(seq_lens), ptr(block_tables),
         block_tables.stride(0), bs, B, T, Nh, W, L, int(num_tiles), int(splits), ptr(ws),
-        float(scale), stream_ptr())
+        float(scale), ptr(sink), ptr(gate), gate.stride(0) if gate is not None else 0,
+        stream_ptr())
     N.launch_count += 1
     if rc != 0:
         raise N.NativeError(f"b200_mla_attention failed with code {rc}")
@@ -753,24 +798,45 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tens
 def latent_cache(kv: torch.Tensor, weight: torch.Tensor, eps: float, cache: torch.Tensor,
                  slot_mapping: torch.Tensor, x: Optional[torch.Tensor] = None,
                  state: Optional[torch.Tensor] = None, num_decodes: int = 0,
-                 cu_q: Optional[torch.Tensor] = None) -> None:
+                 cu_q: Optional[torch.Tensor] = None, cos_sin: Optional[torch.Tensor] = None,
+                 positions: Optional[torch.Tensor] = None, q: Optional[torch.Tensor] = None,
+                 q_lat: Optional[torch.Tensor] = None) -> None:
     """RMSNorm of the latent projection ``kv [T, L]`` (a row-strided view) into the rows of
     ``cache [blocks, block_size, W >= L]`` (zeros behind L).  With ``state [blocks, H]`` fp32 the
-    row of ``x [T, H]`` fp32 of the last token that the step writes into a block is kept there."""
-    T, L = kv.shape
+    row of ``x [T, H]`` fp32 of the last token that the step writes into a block is kept there.
+
+    With a rotary table ``cos_sin [max_pos, R]`` fp32, ``kv [T, L + R]`` brings the key's rotated part
+    behind the latent: neighbours are turned by the angle of their position and land behind the
+    latent in the cache row.  The last R columns of every head of ``q [T, N * (dim + R)]`` are turned
+    into columns ``L .. L + R`` of ``q_lat [T, N, W]``."""
+    T = kv.shape[0]
+    L = weight.shape[0]
     nb, bs, W = cache.shape
+    R = Nh = dim = 0
+    if cos_sin is not None:
+        R, Nh = cos_sin.shape[1], q_lat.shape[1]
+        dim = q.shape[1] // Nh - R
+        assert q.stride(1) == 1 and q_lat.is_contiguous() and q_lat.shape[2] == W
+        assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous()
+    assert kv.shape[1] == L + R
     assert kv.stride(1) == 1 and cache.is_contiguous() and cache.dtype == kv.dtype
     call("b200_latent_cache", ptr(kv), kv.stride(0), ptr(weight), float(eps), ptr(cache), nb * bs,
          W, ptr(slot_mapping), ptr(x), ptr(state), ptr(cu_q), T, L,
          x.shape[1] if x is not None else 0, num_decodes,
-         cu_q.shape[0] - 1 if cu_q is not None else 0, bs, DTYPE_CODE[kv.dtype], stream_ptr())
+         cu_q.shape[0] - 1 if cu_q is not None else 0, bs, R, Nh, dim,
+         ptr(q) if R else None, q.stride(0) if R else 0, ptr(q_lat) if R else None, ptr(cos_sin),
+         cos_sin.shape[0] if R else 0, ptr(positions) if R else None, DTYPE_CODE[kv.dtype],
+         stream_ptr())
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
                      seq_lens: torch.Tensor, num_decodes: int, cu_q: Optional[torch.Tensor],
-                     scale: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     scale: float, out: Optional[torch.Tensor] = None,
+                     sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None
+                     ) -> torch.Tensor:
     """Latent attention for any width and head count, fp32 or bf16 (csrc/latent.cu): q
-    ``[T, N, W]``, the first ``num_decodes`` tokens one per request, the rest by ``cu_q``."""
+    ``[T, N, W]``, the first ``num_decodes`` tokens one per request, the rest by ``cu_q``.
+    ``sink`` and ``gate`` (in q's type): see ``mla_attention``."""
     T, Nh, W = q.shape
     nb, bs, _ = cache.shape
     assert q.is_contiguous() and cache.is_contiguous() and cache.dtype == q.dtype
@@ -778,8 +844,8 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
         out = torch.empty_like(q)
     call("b200_latent_attention", ptr(q), ptr(cache), nb * bs, ptr(out), ptr(block_tables),
          block_tables.stride(0), bs, ptr(seq_lens), ptr(cu_q), T, Nh, W, num_decodes,
-         cu_q.shape[0] - 1 if cu_q is not None else 0, float(scale), DTYPE_CODE[q.dtype],
-         stream_ptr())
+         cu_q.shape[0] - 1 if cu_q is not None else 0, float(scale), ptr(sink), ptr(gate),
+         gate.stride(0) if gate is not None else 0, DTYPE_CODE[q.dtype], stream_ptr())
     return out
 
 
@@ -830,13 +896,16 @@ def sigmoid_gate(o: torch.Tensor, z: torch.Tensor, out: Optional[torch.Tensor] =
     return out
 
 
-def start_rows(e: torch.Tensor, scale: float) -> tuple[torch.Tensor, torch.Tensor]:
-    """``(scale * e`` in fp32, the same in ``e``'s type)."""
+def start_rows(e: torch.Tensor, scale: float, step: Optional[torch.Tensor] = None,
+               weight: Optional[torch.Tensor] = None, eps: float = 0.0
+               ) -> tuple[torch.Tensor, torch.Tensor]:
+    """``(x, lo)``: ``x = scale * e (+ step)`` in fp32, ``lo`` the same in ``e``'s type, or with
+    ``weight`` its RMS norm.  step, weight fp32 ``[H]``."""
     T, H = e.shape
     x = torch.empty((T, H), dtype=torch.float32, device=e.device)
     lo = torch.empty((T, H), dtype=e.dtype, device=e.device)
-    call("b200_start_rows", ptr(e), e.stride(0), float(scale), ptr(x), ptr(lo), T, H,
-         DTYPE_CODE[e.dtype], stream_ptr())
+    call("b200_start_rows", ptr(e), e.stride(0), float(scale), ptr(step), ptr(weight), float(eps),
+         ptr(x), ptr(lo), T, H, DTYPE_CODE[e.dtype], stream_ptr())
     return x, lo
 
 
@@ -844,14 +913,23 @@ def add_normed(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor,
                bias: Optional[torch.Tensor], eps: float, lo: torch.Tensor,
                out: Optional[torch.Tensor] = None, layer_norm: bool = True,
                final_weight: Optional[torch.Tensor] = None,
-               final_bias: Optional[torch.Tensor] = None, final_scale: float = 1.0) -> None:
-    """``s = x + norm(y) * weight + bias`` over fp32 rows ``x [T, H]`` (layer norm or RMS norm);
-    ``out`` takes s (may be ``x``), ``lo`` takes s in ``y``'s type, or with ``final_weight`` its
-    norm ``(norm(s) * final_weight + final_bias) * final_scale``."""
+               final_bias: Optional[torch.Tensor] = None, final_scale: float = 1.0,
+               step: Optional[torch.Tensor] = None, pos_of: Optional[torch.Tensor] = None,
+               row_w: Optional[torch.Tensor] = None, shared: Optional[torch.Tensor] = None,
+               gate: Optional[torch.Tensor] = None) -> None:
+    """``s = x + norm(y) * weight + bias (+ step)`` over fp32 rows ``x [T, H]`` (layer norm or RMS
+    norm); ``out`` takes s (may be ``x``), ``lo`` takes s in ``y``'s type, or with ``final_weight``
+    its norm ``(norm(s) * final_weight + final_bias) * final_scale``.
+
+    With ``pos_of [T * k]`` the row that is normalised is the sum of the token's expert-sorted rows
+    ``y[pos_of]`` times ``row_w [T, k]`` plus ``shared [T, H]`` times sigmoid(``gate [T]``, fp32)."""
     T, H = x.shape
-    call("b200_add_normed", ptr(x), ptr(y), y.stride(0), ptr(weight), ptr(bias), int(layer_norm),
-         float(eps), ptr(out), ptr(final_weight), ptr(final_bias), float(final_scale), ptr(lo), T, H,
-         DTYPE_CODE[y.dtype], stream_ptr())
+    call("b200_add_normed", ptr(x), ptr(y), y.stride(0), ptr(pos_of), ptr(row_w),
+         row_w.shape[1] if row_w is not None else 0, ptr(shared),
+         shared.stride(0) if shared is not None else 0, ptr(gate),
+         gate.stride(0) if gate is not None else 0, ptr(step), ptr(weight), ptr(bias),
+         int(layer_norm), float(eps), ptr(out), ptr(final_weight), ptr(final_bias),
+         float(final_scale), ptr(lo), T, H, DTYPE_CODE[y.dtype], stream_ptr())
 
 
 def head_gate(o: torch.Tensor, z: torch.Tensor, scale: float, head_dim: int, out: torch.Tensor
@@ -877,6 +955,14 @@ def silu_mul_rows(x: torch.Tensor) -> torch.Tensor:
     call("b200_silu_mul_rows", ptr(x2), x2.stride(0), ptr(out), D, T, D, DTYPE_CODE[x.dtype],
          stream_ptr())
     return out.view(*shape[:-1], D)
+
+
+def relu2(x: torch.Tensor) -> torch.Tensor:
+    """``max(x, 0)^2`` in place, bf16 or fp32."""
+    x2 = x if x.dim() == 2 else x.view(-1, x.shape[-1])
+    call("b200_relu2", ptr(x2), x2.stride(0), ptr(x2), x2.stride(0), x2.shape[0], x2.shape[1],
+         DTYPE_CODE[x.dtype], stream_ptr())
+    return x
 
 
 # ---------------------------------------------------------------------------
@@ -1101,7 +1187,7 @@ def moe_align(topk_ids: torch.Tensor, num_local_experts: int, cap: Optional[int]
 def gemm_bf16_grouped(a: torch.Tensor, w: torch.Tensor, expert_ids: torch.Tensor,
                       num_valid_rows: torch.Tensor, silu_mul: bool = False,
                       row_scale: Optional[torch.Tensor] = None,
-                      out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      out: Optional[torch.Tensor] = None, relu2: bool = False) -> torch.Tensor:
     """a ``[M_cap, K]`` expert-sorted rows, w ``[E, N, K]``."""
     M_cap, K = a.shape
     E, Nn, _ = w.shape
@@ -1111,7 +1197,7 @@ def gemm_bf16_grouped(a: torch.Tensor, w: torch.Tensor, expert_ids: torch.Tensor
         out = torch.empty((M_cap, out_cols), device=a.device, dtype=torch.bfloat16)
     call("b200_gemm_bf16_grouped", ptr(a), a.stride(0), ptr(w), K, ptr(out), out.stride(0), M_cap,
          Nn, K, E, ptr(expert_ids), ptr(num_valid_rows), ptr(row_scale),
-         EPI_SILU_MUL if silu_mul else EPI_NONE, stream_ptr())
+         EPI_SILU_MUL if silu_mul else EPI_RELU2 if relu2 else EPI_NONE, stream_ptr())
     return out
 
 
@@ -1171,6 +1257,38 @@ def input_weighted_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor,
          ptr(expert_ids), ptr(npp), stream_ptr())
     h = torch.empty((cap, I), device=x.device, dtype=torch.float32)
     call("b200_silu_mul_rows_f32", ptr(u), ptr(h), cap, I, ptr(npp), stream_ptr())
+    y = torch.empty((cap, Hp), device=x.device, dtype=torch.float32)
+    call("b200_grouped_gemm_f32", ptr(h), I, ptr(w2), ptr(y), Hp, cap, Hp, I, E, ptr(expert_ids),
+         ptr(npp), stream_ptr())
+    return y, pos_of
+
+
+def squared_relu_experts(x: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor,
+                         topk_ids: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """Routed experts without a gate, ``down(max(up(x), 0)^2)``: align -> permute rows ``x [T, H]`` ->
+    grouped GEMM1 with the activation in its epilogue -> grouped GEMM2.  ``w1 [E, I, Hp]``, ``w2
+    [E, Hp, I]`` with Hp >= H padded by zeros.  Returns the expert-sorted outputs ``[cap, Hp]``, not
+    weighted, and ``pos_of [T * k]``; ``add_normed`` weights and sums them."""
+    T, H = x.shape
+    k = topk_ids.shape[1]
+    E, I, Hp = w1.shape
+    numel = T * k
+    cap = moe_align_cap(numel, E)
+    sorted_ids, expert_ids, npp, pos_of = moe_align(topk_ids, E, cap)
+    a_sorted = torch.empty((cap, Hp), device=x.device, dtype=x.dtype)
+    if x.dtype == torch.bfloat16 and H == Hp and H % 8 == 0:
+        call("b200_moe_permute", ptr(x), x.stride(0), ptr(a_sorted), Hp, ptr(sorted_ids), ptr(npp),
+             numel, k, H, cap, DTYPE_CODE[x.dtype], stream_ptr())
+    else:
+        call("b200_moe_permute_any", ptr(x), x.stride(0), ptr(a_sorted), Hp, ptr(sorted_ids),
+             ptr(npp), numel, k, H, Hp, cap, DTYPE_CODE[x.dtype], stream_ptr())
+    if x.dtype == torch.bfloat16:
+        h = gemm_bf16_grouped(a_sorted, w1, expert_ids, npp, relu2=True)
+        return gemm_bf16_grouped(h, w2, expert_ids, npp), pos_of
+    h = torch.empty((cap, I), device=x.device, dtype=torch.float32)
+    call("b200_grouped_gemm_f32", ptr(a_sorted), Hp, ptr(w1), ptr(h), I, cap, I, Hp, E,
+         ptr(expert_ids), ptr(npp), stream_ptr())
+    call("b200_relu2_rows_f32", ptr(h), ptr(h), cap, I, ptr(npp), stream_ptr())
     y = torch.empty((cap, Hp), device=x.device, dtype=torch.float32)
     call("b200_grouped_gemm_f32", ptr(h), I, ptr(w2), ptr(y), Hp, cap, Hp, I, E, ptr(expert_ids),
          ptr(npp), stream_ptr())

@@ -579,11 +579,12 @@ def advance_step(num_seqs: int, num_queries: int, block_size: int, input_tokens:
 # latent attention, fp32 residual stream
 # ---------------------------------------------------------------------------
 def latent_attention(q_full: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor,
-                     q_lens: list[int], seq_lens: list[int], scale: float, L: int
+                     q_lens: list[int], seq_lens: list[int], scale: float, L: int,
+                     sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None
                      ) -> torch.Tensor:
     """q_full ``[T, N, W]`` (latent query, then the rotated rope part if there is one); cache
     ``[blocks, bs, W]``.  Returns the latent-space output ``[T, N, L]``.  Causal inside each
-    request."""
+    request.  ``sink [N]``, ``gate [T, N]``: see ``ops.cuda.mla_attention``."""
     T, N, W = q_full.shape
     nb, bs, _ = cache.shape
     flat = cache.view(nb * bs, W)
@@ -600,8 +601,13 @@ def latent_attention(q_full: torch.Tensor, cache: torch.Tensor, block_tables: to
         s = torch.einsum("qhw,nw->hqn", q, kv) * scale
         qpos = torch.arange(n - ql, n, device=cache.device)[:, None]
         s = s.masked_fill((pos[None, :] > qpos)[None], float("-inf"))
-        p = torch.softmax(s, dim=-1)
-        out[t0:t0 + ql] = torch.einsum("hqn,nl->qhl", p, kv[:, :L]).to(out.dtype)
+        if sink is not None:
+            s = torch.cat([s, sink.float()[:, None, None].expand(-1, ql, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :n]
+        o = torch.einsum("hqn,nl->qhl", p, kv[:, :L])
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t0:t0 + ql].float())[..., None]
+        out[t0:t0 + ql] = o.to(out.dtype)
         t0 += ql
     return out
 
@@ -616,11 +622,18 @@ def _portions(T: int, num_decodes: int, cu_q: Optional[torch.Tensor]) -> list[tu
 
 
 def latent_cache(kv, weight, eps, cache, slot_mapping, x=None, state=None, num_decodes=0,
-                 cu_q=None) -> None:
+                 cu_q=None, cos_sin=None, positions=None, q=None, q_lat=None) -> None:
     """See ``ops.cuda.latent_cache``."""
-    L = kv.shape[1]
+    L = weight.shape[0]
     nb, bs, W = cache.shape
-    c = rms_norm(kv, weight, eps)
+    c = rms_norm(kv[:, :L], weight, eps)
+    if cos_sin is not None:
+        R, N = cos_sin.shape[1], q_lat.shape[1]
+        heads = q.unflatten(1, (N, -1))[..., -R:].flatten(1)
+        qr, kr = rotary_embedding(positions, heads, kv[:, L:], R, cos_sin, False)
+        q_lat[..., L:L + R] = qr.view(-1, N, R)
+        c = torch.cat([c, kr.to(c.dtype)], dim=1)
+        L += R
     ok = slot_mapping >= 0
     rows = torch.zeros(int(ok.sum()), W, dtype=cache.dtype, device=cache.device)
     rows[:, :L] = c[ok].to(cache.dtype)
@@ -676,15 +689,28 @@ def sigmoid_gate(o: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
     return (o.float() * torch.sigmoid(z.float())).to(o.dtype)
 
 
-def start_rows(e: torch.Tensor, scale: float) -> tuple[torch.Tensor, torch.Tensor]:
+def start_rows(e: torch.Tensor, scale: float, step=None, weight=None, eps=0.0
+               ) -> tuple[torch.Tensor, torch.Tensor]:
     """See ``ops.cuda.start_rows``."""
     x = e.float() * scale
-    return x, x.to(e.dtype)
+    if step is not None:
+        x = x + step
+    return x, (x if weight is None else rms_norm(x, weight, eps)).to(e.dtype)
 
 
 def add_normed(x, y, weight, bias, eps, lo, out=None, layer_norm=True, final_weight=None,
-               final_bias=None, final_scale=1.0) -> None:
+               final_bias=None, final_scale=1.0, step=None, pos_of=None, row_w=None, shared=None,
+               gate=None) -> None:
     """See ``ops.cuda.add_normed``."""
+    if pos_of is not None:
+        T, k = row_w.shape
+        pos = pos_of.view(-1)[:T * k].view(T, k).long()
+        w = (row_w * (pos >= 0)).unsqueeze(-1)
+        y = (y[pos.clamp(min=0)].float() * w).sum(1)[:, :x.shape[1]]
+        if shared is not None:
+            g = 1.0 if gate is None else torch.sigmoid(gate.float()).unsqueeze(-1)
+            y = y + g * shared.float()
+
     def norm(r, w, b):
         if layer_norm:
             r = r - r.mean(-1, keepdim=True)
@@ -692,6 +718,8 @@ def add_normed(x, y, weight, bias, eps, lo, out=None, layer_norm=True, final_wei
         return r if b is None else r + b
 
     s = x + norm(y.float(), weight, bias)
+    if step is not None:
+        s = s + step
     if out is not None:
         out.copy_(s)
     lo.copy_(s if final_weight is None else norm(s, final_weight, final_bias) * final_scale)
@@ -701,6 +729,26 @@ def head_gate(o, z, scale, head_dim, out) -> torch.Tensor:
     """See ``ops.cuda.head_gate``."""
     out.copy_(o[..., :head_dim].flatten(1).float() * torch.sigmoid(z.float()) * scale)
     return out
+
+
+def relu2(x: torch.Tensor) -> torch.Tensor:
+    """See ``ops.cuda.relu2``."""
+    return x.clamp_(min=0).square_()
+
+
+def head_norm_cache(q, k, v, q_weight, k_weight, eps, slot_mapping, k_cache, v_cache, head_dim
+                    ) -> torch.Tensor:
+    """See ``ops.cuda.head_norm_cache``."""
+    nb, bs, Hkv, DC = k_cache.shape
+    heads = lambda x, d: x.unflatten(1, (-1, d))  # noqa: E731
+    pad = lambda x: torch.nn.functional.pad(x, (0, DC - x.shape[-1]))  # noqa: E731
+    qn = rms_norm(heads(q, head_dim), q_weight, eps)
+    kn = rms_norm(heads(k, head_dim), k_weight, eps)
+    ok = slot_mapping >= 0
+    at = slot_mapping[ok].long()
+    k_cache.view(nb * bs, Hkv, DC)[at] = pad(kn)[ok].to(k_cache.dtype)
+    v_cache.view(nb * bs, Hkv, DC)[at] = pad(heads(v, v.shape[1] // Hkv))[ok].to(v_cache.dtype)
+    return pad(qn).to(q.dtype)
 
 
 def qk_norm_rope_cache(q, k, v, q_weight, k_weight, eps, cos_sin, is_neox, positions, slot_mapping,
@@ -726,10 +774,11 @@ def qk_norm_rope_cache(q, k, v, q_weight, k_weight, eps, cos_sin, is_neox, posit
 
 
 def any_attention(q, k_cache, v_cache, block_tables, seq_lens, num_decodes, cu_q, scale, sink=None,
-                  out=None) -> torch.Tensor:
+                  out=None, softcap=0.0, chunk=0, out_dim=0) -> torch.Tensor:
     """See ``ops.cuda.any_attention``."""
     T, Hq, D = q.shape
-    out = torch.zeros_like(q) if out is None else out
+    od = out_dim or D
+    out = q.new_zeros(T, Hq, od) if out is None else out
     for r, (lo, hi) in enumerate(_portions(T, num_decodes, cu_q)):
         n = int(seq_lens[r])
         if n == 0 or hi == lo:
@@ -738,12 +787,18 @@ def any_attention(q, k_cache, v_cache, block_tables, seq_lens, num_decodes, cu_q
         G = Hq // k.shape[1]
         k, v = k.repeat_interleave(G, dim=1), v.repeat_interleave(G, dim=1)
         s = torch.einsum("qhd,nhd->hqn", q[lo:hi].float(), k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         qpos = torch.arange(n - (hi - lo), n, device=q.device)[:, None]
-        s = s.masked_fill((torch.arange(n, device=q.device)[None, :] > qpos)[None], float("-inf"))
+        kpos = torch.arange(n, device=q.device)[None, :]
+        hidden = kpos > qpos
+        if chunk:
+            hidden = hidden | (kpos // chunk != qpos // chunk)
+        s = s.masked_fill(hidden[None], float("-inf"))
         if sink is not None:
             s = torch.cat([s, sink.float()[:, None, None].expand(-1, hi - lo, 1)], dim=-1)
         p = torch.softmax(s, dim=-1)[..., :n]
-        out[lo:hi] = torch.einsum("hqn,nhd->qhd", p, v).to(out.dtype)
+        out[lo:hi] = torch.einsum("hqn,nhd->qhd", p, v)[..., :od].to(out.dtype)
     return out
 
 
@@ -856,6 +911,22 @@ def input_weighted_experts(x, w13, w2, topk_w, topk_ids) -> tuple[torch.Tensor, 
         if rows.numel():
             h = silu_and_mul(a[rows] @ w13[e].t())
             y[rows] = h @ w2[e].t()
+    return y, torch.arange(T * k, dtype=torch.int32, device=x.device)
+
+
+def squared_relu_experts(x, w1, w2, topk_ids) -> tuple[torch.Tensor, torch.Tensor]:
+    """See ``ops.cuda.squared_relu_experts``; one output row per (token, slot) pair, so ``pos_of``
+    is the identity."""
+    T, H = x.shape
+    k = topk_ids.shape[1]
+    Hp = w1.shape[2]
+    y = torch.zeros(T * k, Hp, dtype=w1.dtype, device=x.device)
+    a = torch.nn.functional.pad(x, (0, Hp - H))
+    flat = topk_ids.reshape(-1)
+    for e in range(w1.shape[0]):
+        rows = (flat == e).nonzero(as_tuple=True)[0]
+        if rows.numel():
+            y[rows] = relu2(a[rows // k] @ w1[e].t()) @ w2[e].t()
     return y, torch.arange(T * k, dtype=torch.int32, device=x.device)
 
 
