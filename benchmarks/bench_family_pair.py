@@ -7,6 +7,10 @@ sizes, both through ``LLM.generate`` with random weights.
 * Fizunex beside Llama (grouped-query attention, dense feed-forward): same width, heads, head
   dimension, feed-forward, layers and vocabulary.  Half of Fizunex's layers are gated delta layers
   (full query / key heads), the others run attention with Llama's heads and a matrix memory.
+* Fepopel beside DeepSeek: same width, heads, head and rotary dimensions, latent rank, experts,
+  experts per token, expert width (routed and shared) and vocabulary; as many layer runs as DeepSeek
+  has layers, two of them a second pass of a loop.  Every second layer of Fepopel has chunked grouped
+  attention in place of latent attention; its experts have two matrices, DeepSeek's three.
 
 Timed on the device: the CUDA events that bracket every engine step.  Prefill: ``prompts x
 input_len`` tokens in steps of 8192, one output token.  Decode: the steps of ``batch`` requests
@@ -38,8 +42,16 @@ SIZES = {"sapapel": {
                layers=8),
     8192: dict(heads=64, kv_heads=8, dim=128, mem_heads=16, mem_dim=128, mem_vdim=256, ff=28672,
                layers=4),
+}, "fepopel": {
+    2048: dict(heads=16, kv_heads=4, dim=128, rank=512, chunk=512, experts=64, top=6, ff=1408,
+               layers=8),
+    4096: dict(heads=32, kv_heads=8, dim=128, rank=512, chunk=512, experts=32, top=4, ff=1536,
+               layers=6),
+    7168: dict(heads=128, kv_heads=8, dim=128, rank=512, chunk=512, experts=64, top=8, ff=2048,
+               layers=4),
 }}
-PAIRS = {"sapapel": ("sapapel", "deepseek"), "fizunex": ("fizunex", "llama")}
+PAIRS = {"sapapel": ("sapapel", "deepseek"), "fizunex": ("fizunex", "llama"),
+         "fepopel": ("fepopel", "deepseek")}
 VOCAB = 32768
 
 
@@ -58,6 +70,13 @@ def model_config(pair: str, family: str, width: int):
             intermediate_size=s["ff"], num_hidden_layers=s["layers"],
             num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"],
             head_dim=s["dim"], tie_word_embeddings=True, dtype="bfloat16")
+    if family == "fepopel":
+        from vllm_gcu_b200.config import _fepopel_preset
+        n = s["layers"] - 2                # the loop runs two layers once more
+        return ModelConfig.from_hf_dict(_fepopel_preset(
+            " ".join(("le", "ce")[i % 2] for i in range(n)), (0, 2, 2), VOCAB, width, s["heads"],
+            s["dim"], 64, s["rank"], s["kv_heads"], s["chunk"], 0, s["experts"], s["top"], s["ff"],
+            s["ff"]), dtype="bfloat16")
     if family == "sapapel":
         layer = {"type": "latent_attention",
                  "mixer": {"heads": s["heads"], "dim": s["dim"], "vdim": s["dim"],
@@ -67,14 +86,16 @@ def model_config(pair: str, family: str, width: int):
         return ModelConfig.from_hf_dict(
             {"architecture": "Sapapel", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
              "postln_alpha": 2.0, "layers": [layer] * s["layers"]}, dtype="bfloat16")
+    shared = pair == "fepopel"
     return ModelConfig(
         architecture="DeepseekV2ForCausalLM", vocab_size=VOCAB, hidden_size=width,
         intermediate_size=s["ff"], num_hidden_layers=s["layers"],
         num_attention_heads=s["heads"], num_key_value_heads=s["heads"], q_lora_rank=0,
         kv_lora_rank=s["rank"], qk_nope_head_dim=s["dim"], qk_rope_head_dim=64,
         v_head_dim=s["dim"], head_dim=s["dim"] + 64, num_experts=s["experts"],
-        num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"], num_shared_experts=0,
-        first_k_dense_replace=0, scoring_func="sigmoid", norm_topk_prob=False,
+        num_experts_per_tok=s["top"], moe_intermediate_size=s["ff"],
+        num_shared_experts=int(shared), first_k_dense_replace=0,
+        scoring_func="softmax" if shared else "sigmoid", norm_topk_prob=shared,
         rope_is_neox=False, dtype="bfloat16")
 
 

@@ -100,6 +100,24 @@ def greedy(config: dict, weights: dict, prompt, n: int) -> list:
     return out
 
 
+def clear_choices(config: dict, weights: dict, tokens, gap: float = 0.2) -> torch.Tensor:
+    """Rows at which no router's choice is close: the last chosen expert's logit is ``gap`` above the
+    next one's."""
+    real, rows = O.route, torch.ones(len(tokens), dtype=torch.bool)
+
+    def route(h, router, top, scale):
+        z = (h @ router.T).sort(dim=-1, descending=True).values
+        if top < z.shape[1]:
+            rows.logical_and_(z[:, top - 1] - z[:, top] > gap)
+        return real(h, router, top, scale)
+    O.route = route
+    try:
+        O.forward(config, weights, tokens)
+    finally:
+        O.route = real
+    return rows
+
+
 def chunk_edges(n: int, size: int) -> list[int]:
     """Positions just in front of and behind the edges of chunks, pages and tiles below ``n``."""
     at = {0, 1, n - 1}
