@@ -179,6 +179,8 @@ def main() -> None:
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--width", type=int, default=4096)
     ap.add_argument("--chunk", type=int, default=512)
+    ap.add_argument("--experts", type=int, nargs=3, default=[32, 4, 1536],
+                    help="experts, experts per token, expert width")
     ap.add_argument("--only", default="")
     a = ap.parse_args()
     path = os.path.join(ROOT, "MEASURED_PEAKS.json")
@@ -186,7 +188,7 @@ def main() -> None:
         PEAKS.update(json.load(open(path)))
     flush = torch.empty(512 << 20, dtype=torch.uint8, device="cuda")
     sizes = dict(H=a.width, N=a.width // 128, G=max(1, a.width // 512), D=128, L=512, R=64,
-                 chunk=a.chunk, E=32, k=4, F=1536)
+                 chunk=a.chunk, **dict(zip("EkF", a.experts)))
     for kind, lens in (("prefill", [a.input_len] * a.prompts), ("decode", [1] * a.batch)):
         rows, fracs = [], {}
         for name, like, fn, nbytes, flops in cases(lens, a.input_len, kind == "decode", **sizes):

@@ -102,11 +102,10 @@ struct Args {
   unsigned int* status;
 };
 
-__device__ __forceinline__ float head_gate(const __nv_bfloat16* gate, long long ldg, long long row,
-                                           int N) {
+__device__ __forceinline__ float head_gate(const __nv_bfloat16* gate, long long ldg, long long t,
+                                           int head) {
   if (gate == nullptr) return 1.0f;
-  const long long t = row / N;
-  return 1.0f / (1.0f + __expf(-__bfloat162float(gate[t * ldg + (row - t * N)])));
+  return 1.0f / (1.0f + __expf(-__bfloat162float(gate[t * ldg + head])));
 }
 
 // kResident CTAs share an SM: two where shared and tensor memory allow it (narrow latents, whose
@@ -361,6 +360,12 @@ __global__ void __launch_bounds__(kThreads, kResident)
     const int hi = row_ok ? min(pos0 + r / a.N, seq_len - 1) : -1;   // last visible key
     const int hi_first = min(pos0, seq_len - 1);
     const float sl2 = a.scale * 1.4426950408889634f;
+    float sink2 = 0.0f, gate = 1.0f;             // read while the first tiles are on their way
+    if (a.splits == 1 && row_ok) {
+      const int tok = r / a.N, head = r - tok * a.N;
+      if (a.sink != nullptr) sink2 = a.sink[head] * 1.4426950408889634f;
+      gate = head_gate(a.gate, a.ldg, static_cast<long long>(q_start) + tok0 + tok, head);
+    }
     float m_used = -INFINITY, l = 0.0f;
     float* xch = reinterpret_cast<float*>(smem + kOffX);    // [2][128]
     bool ok = true;
@@ -461,9 +466,9 @@ __global__ void __launch_bounds__(kThreads, kResident)
       const long long grow = row0 + r;
       float inv = l > 0.0f ? 1.0f / l : 0.0f;
       if (a.splits == 1 && row_ok && l > 0.0f) {
-        if (a.sink != nullptr)       // relative to the running maximum, like the row sum
-          inv = 1.0f / (l + exp2f(fmaf(-m_used, sl2, a.sink[r % a.N] * 1.4426950408889634f)));
-        inv *= head_gate(a.gate, a.ldg, grow, a.N);
+        // relative to the running maximum, like the row sum
+        if (a.sink != nullptr) inv = 1.0f / (l + exp2f(fmaf(-m_used, sl2, sink2)));
+        inv *= gate;
       }
       const int col0 = c0 * 64 + g * nc * 32;
 #pragma unroll 1
@@ -525,7 +530,7 @@ __global__ void __launch_bounds__(128)
   const int c = threadIdx.x * 4;
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
   if (den > 0.0f) {
-    const float g = head_gate(gate, ldg, row, N) / den;
+    const float g = head_gate(gate, ldg, row / N, static_cast<int>(row % N)) / den;
     for (int z = 0; z < splits; ++z) {
       const float v = ws_lse[z * rows_total + row];
       if (v == -INFINITY) continue;

@@ -31,9 +31,12 @@ namespace residual {
 
 template <int V>
 __device__ __forceinline__ void ldv(const float* p, float (&f)[V]) {
-  if constexpr (V == 4) {
-    const float4 u = *reinterpret_cast<const float4*>(p);
-    f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
+  if constexpr (V >= 4) {
+#pragma unroll
+    for (int i = 0; i < V; i += 4) {
+      const float4 u = *reinterpret_cast<const float4*>(p + i);
+      f[i] = u.x; f[i + 1] = u.y; f[i + 2] = u.z; f[i + 3] = u.w;
+    }
   } else {
     f[0] = p[0];
   }
@@ -52,8 +55,10 @@ __device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&f)[V]) {
 }
 template <int V>
 __device__ __forceinline__ void stv(float* p, const float (&f)[V]) {
-  if constexpr (V == 4) {
-    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  if constexpr (V >= 4) {
+#pragma unroll
+    for (int i = 0; i < V; i += 4)
+      *reinterpret_cast<float4*>(p + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
   } else {
     p[0] = f[0];
   }
@@ -422,6 +427,129 @@ __global__ void __launch_bounds__(512) add_normed_kernel(const AddNormArgs a) {
   }
 }
 
+// The same for rows of whole vectors that fit the threads' registers, NI vectors each: the residual
+// row is on its way while the sublayer's is summed, two expert rows are in flight at a time,
+// and little but the sums goes through shared memory.
+constexpr int kMaxSlots = 32;      // expert rows per token
+
+template <typename T, int V, int NI, bool kRouted>
+__global__ void __launch_bounds__(NI == 1 ? 1024 : 512) add_normed_reg_kernel(const AddNormArgs a) {
+  __shared__ float red[32];
+  __shared__ int s_pos[kMaxSlots];
+  __shared__ float s_w[kMaxSlots];
+  const long long t = blockIdx.x;
+  const long long row = t * a.H;
+  const int c0 = threadIdx.x * V, pitch = blockDim.x * V;
+  const T* y = static_cast<const T*>(a.y) + (kRouted ? 0 : t * a.ldy);
+  if (kRouted && threadIdx.x < a.k) {
+    s_pos[threadIdx.x] = a.pos_of[t * a.k + threadIdx.x];
+    s_w[threadIdx.x] = a.row_w[t * a.k + threadIdx.x];
+  }
+  float f[NI][V], x[NI][V];
+#pragma unroll
+  for (int n = 0; n < NI; ++n) {
+    const int c = c0 + n * pitch;
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[n][i] = x[n][i] = 0.0f;
+    if (c >= a.H) continue;
+    if constexpr (!kRouted) ldv<V>(y + c, f[n]);
+    ldv<V>(a.x + row + c, x[n]);
+  }
+  if constexpr (kRouted) {
+    // rows 0 .. k - 1 of the experts, row k the shared one
+    const int rows = a.k + (a.shared != nullptr ? 1 : 0);
+    const float gate = a.gate != nullptr ? 1.0f / (1.0f + expf(-a.gate[t * a.ldg])) : 1.0f;
+    __syncthreads();
+    auto place = [&](int s, const T*& e, float& w) {
+      e = nullptr;
+      w = 0.0f;
+      if (s < a.k) {
+        if (s_pos[s] >= 0) e = y + static_cast<long long>(s_pos[s]) * a.ldy;
+        w = s_w[s];
+      } else if (s < rows) {
+        e = static_cast<const T*>(a.shared) + t * a.ldsh;
+        w = gate;
+      }
+    };
+    for (int s = 0; s < rows; s += 2) {
+      const T *e0, *e1;
+      float w0, w1;
+      place(s, e0, w0);
+      place(s + 1, e1, w1);
+      float g0[NI][V], g1[NI][V];
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        const int c = c0 + n * pitch;
+#pragma unroll
+        for (int i = 0; i < V; ++i) g0[n][i] = g1[n][i] = 0.0f;
+        if (c < a.H && e0 != nullptr) ldv<V>(e0 + c, g0[n]);
+        if (c < a.H && e1 != nullptr) ldv<V>(e1 + c, g1[n]);
+      }
+#pragma unroll
+      for (int n = 0; n < NI; ++n)
+#pragma unroll
+        for (int i = 0; i < V; ++i) f[n][i] += w0 * g0[n][i] + w1 * g1[n][i];
+    }
+  }
+  // mean (layer norm) and 1 / root of the mean square of the row in v
+  auto stats = [&](const float (&v)[NI][V], float& mean) {
+    mean = 0.0f;
+    if (a.centred) {
+      float sum = 0.0f;
+#pragma unroll
+      for (int n = 0; n < NI; ++n)
+#pragma unroll
+        for (int i = 0; i < V; ++i) sum += v[n][i];
+      mean = block_sum(sum, red) / static_cast<float>(a.H);
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      if (c0 + n * pitch >= a.H) continue;
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += (v[n][i] - mean) * (v[n][i] - mean);
+    }
+    return 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(a.H) + a.eps);
+  };
+  float mean;
+  const float inv = stats(f, mean);
+  T* lo = static_cast<T*>(a.lo) + row;
+#pragma unroll
+  for (int n = 0; n < NI; ++n) {
+    const int c = c0 + n * pitch;
+    if (c >= a.H) continue;
+    float w[V], b[V];
+    ldv<V>(a.w + c, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) x[n][i] += (f[n][i] - mean) * inv * w[i];
+    if (a.b != nullptr) {
+      ldv<V>(a.b + c, b);
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[n][i] += b[i];
+    }
+    if (a.step != nullptr) {
+      ldv<V>(a.step + c, b);
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[n][i] += b[i];
+    }
+    if (a.xo != nullptr) stv<V>(a.xo + row + c, x[n]);
+    if (a.fw == nullptr) stv<V>(lo + c, x[n]);
+  }
+  if (a.fw == nullptr) return;
+  const float inv2 = stats(x, mean);
+#pragma unroll
+  for (int n = 0; n < NI; ++n) {
+    const int c = c0 + n * pitch;
+    if (c >= a.H) continue;
+    float o[V], w[V], b[V] = {};
+    ldv<V>(a.fw + c, w);
+    if (a.fb != nullptr) ldv<V>(a.fb + c, b);
+#pragma unroll
+    for (int i = 0; i < V; ++i) o[i] = ((x[n][i] - mean) * inv2 * w[i] + b[i]) * a.fscale;
+    stv<V>(lo + c, o);
+  }
+}
+
 // out[t, h * D + c] = o[t, h * DC + c] * sigmoid(z[t, h * D + c]) * scale
 template <typename T, int V>
 __global__ void __launch_bounds__(512)
@@ -499,6 +627,21 @@ static int launch_post_norm(const PostNormArgs& a, cudaStream_t s) {
 
 template <typename T, int V, bool kRouted>
 static int launch_add_normed_as(const AddNormArgs& a, cudaStream_t s) {
+  // few rows: more threads per row, so that a row's loads are in flight together
+  const bool few = a.T < 2 * sm_count();
+  const int most = few ? 512 : 256;
+  // 16-byte loads of the experts' 16-bit rows, of the fp32 row otherwise
+  constexpr int R = kRouted ? 8 : 4;
+  const int nvec = a.H / R;
+  if (V == 4 && (a.H % R) == 0 && nvec <= 2048 && a.k <= kMaxSlots && a.ldy % R == 0 &&
+      a.ldsh % R == 0) {
+    const int ni = few && nvec <= 1024 ? 1 : (nvec <= 1024 ? 2 : 4);
+    const int th = row_threads((nvec + ni - 1) / ni, 1, 1024);
+    if (ni == 1) add_normed_reg_kernel<T, R, 1, kRouted><<<a.T, th, 0, s>>>(a);
+    else if (ni == 2) add_normed_reg_kernel<T, R, 2, kRouted><<<a.T, th, 0, s>>>(a);
+    else add_normed_reg_kernel<T, R, 4, kRouted><<<a.T, th, 0, s>>>(a);
+    return static_cast<int>(cudaGetLastError());
+  }
   const size_t smem = static_cast<size_t>(a.H) * sizeof(float);
   if (smem > 200 * 1024) return -2;
   if (smem > 48 * 1024) {
@@ -507,7 +650,7 @@ static int launch_add_normed_as(const AddNormArgs& a, cudaStream_t s) {
                                          static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  const int threads = row_threads(a.H, V, a.T < 2 * sm_count() ? 512 : 256);
+  const int threads = row_threads(a.H, V, most);
   add_normed_kernel<T, V, kRouted><<<a.T, threads, smem, s>>>(a);
   return static_cast<int>(cudaGetLastError());
 }
