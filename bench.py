@@ -23,8 +23,8 @@ Launch: ``python bench.py`` (1 GPU) or
 ``--impl reference`` reports why the reference cannot run on this hardware;
 ``--impl vllm-stock`` runs the same workload through stock vLLM on the CUDA platform (the
 stand-in baseline, benchmarks/baseline_vllm_stock.py).
-``--workload fepopel`` / ``fizunex`` / ``sapapel`` runs another measurement instead: one model family beside
-another.
+``--workload fepopel`` / ``fizunex`` / ``sapapel`` runs another measurement instead: one model
+family beside another.
 """
 from __future__ import annotations
 

@@ -9,9 +9,9 @@ import pytest
 import torch
 
 import fepopel_oracle as O
-from fepopel_cases import (CONFIGS, build, chunked, clear_choices, dense, errors, greedy, latent, mixed_steps,
-                           model_config, moe, oracle, paged_batch, peaked_model, portions, replayer,
-                           run, spread, tokens_for)
+from fepopel_cases import (CONFIGS, build, chunked, clear_choices, dense, errors, greedy,
+                           latent, mixed_steps, model_config, moe, oracle, paged_batch,
+                           peaked_model, portions, replayer, run, spread, tokens_for)
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -89,6 +89,18 @@ def test_gemm_with_squared_relu(M, N, K):
     _status()
     want = (a.cuda().float() @ b.cuda().float().t()).clamp(min=0).square().cpu()
     _close(got, want, BF16)
+
+
+@pytest.mark.parametrize("M,N,K", [(64, 72, 7168), (1, 40, 2048), (128, 264, 4096), (100, 8, 8192),
+                                   (3, 24, 256), (129, 72, 4096), (5, 1024, 5120)])
+def test_gemm_with_fp32_results(M, N, K):
+    from vllm_gcu_b200.ops import cuda as C
+    g = torch.Generator().manual_seed(N)
+    a, b = torch.randn(M, K, generator=g).to(BF16), (torch.randn(N, K, generator=g) * K ** -0.5).to(BF16)
+    got = C.gemm_bf16(a.cuda(), b.cuda(), epilogue=C.EPI_FP32)
+    _status()
+    assert got.dtype == F32
+    _close(got, (a.cuda().double() @ b.cuda().double().t()).float().cpu(), F32)
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])

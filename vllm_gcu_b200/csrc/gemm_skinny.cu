@@ -17,7 +17,7 @@
 //     workspace, meet at a counter (bounded wait), and each reduces a row slice of the tile
 //     in a fixed order (bitwise reproducible), applying the epilogue;
 //   * epilogues: none, + bias, max(x, 0)^2, SiLU(gate) * up (gate / up interleaved in blocks of 32
-//     rows).
+//     rows), fp32 results (two-kernel K split only).
 //
 // Replaces the vendor matmul behind the decode path of every unquantised linear layer of the
 // reference (vllm_gcu/kernels/linear.py; SiluAndMul of vllm_gcu/kernels/activation.py:20-32
@@ -35,7 +35,7 @@ constexpr int BK = 64;
 constexpr int UMMA_K = 16;
 constexpr int kThreads = 192;
 
-enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kRelu2 = 9 };
+enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kFp32 = 4, kRelu2 = 9 };
 
 struct Args {
   __nv_bfloat16* C;
@@ -608,7 +608,7 @@ struct Plan {
 // C = sum over K slices of the partial sums a split launch left in ws (+ bias): the slices of
 // a column tile lie one after the other, [tile][slice][R x bn]; fixed summation order.
 __global__ void __launch_bounds__(256)
-    skinny_reduce_kernel(const float* ws, __nv_bfloat16* C, long long ldc,
+    skinny_reduce_kernel(const float* ws, __nv_bfloat16* C, float* C32, long long ldc,
                          const __nv_bfloat16* bias, int relu2, int M, int N, int bn, int R,
                          int splits) {
   const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
@@ -633,6 +633,10 @@ __global__ void __launch_bounds__(256)
     acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y);
     acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w);
   }
+  if (C32 != nullptr) {
+    *reinterpret_cast<float4*>(C32 + static_cast<long long>(row) * ldc + col) = acc;
+    return;
+  }
   uint2 o;
   o.x = pack_bf16x2(acc.x, acc.y);
   o.y = pack_bf16x2(acc.z, acc.w);
@@ -653,8 +657,8 @@ inline Plan make_plan2(int M, int N, int K, int epi, int sms) {
   for (int ci = 0; ci < 3; ++ci) {
     const int bn = cands[ci];
     if (epi == kSiluMul && bn != 256) continue;
-    if (N % bn != 0) continue;
-    const int tiles = N / bn;
+    if (N % bn != 0 && (epi != kFp32 || bn > 128)) continue;   // narrow fp32 results: a partial tile
+    const int tiles = (N + bn - 1) / bn;
     for (int sl = 1; sl <= 16; ++sl) {
       if (sl > 1 && (epi == kSiluMul || tiles * sl > sms || num_kb / sl < 8)) break;
       const double units = static_cast<double>(tiles) * sl;
@@ -712,7 +716,8 @@ B200_API int b200_gemm_skinny_workspace(int N, long long* ws_bytes, int* ctr_wor
 }
 
 // C[M,N] (bf16) = A[M,K] * B[N,K]^T for M <= 256 with epilogue epi: 0 none, 1 + bias[N],
-// 2 SiLU(gate)*up (B rows interleaved gate/up in blocks of 32; C is [M, N/2]), 9 max(x, 0)^2.
+// 2 SiLU(gate)*up (B rows interleaved gate/up in blocks of 32; C is [M, N/2]), 9 max(x, 0)^2; 4: C
+// is fp32, only where a two-kernel K split (allow_split = 2) pays.
 // Row pitches in elements; K, lda, ldb, N, ldc multiples of 8; 16-byte aligned pointers.
 // ws / ctr: see b200_gemm_skinny_workspace (ctr must be zero before the first call; the kernel
 // leaves it zero).  Launches on one stream may share the workspace; concurrent streams need
@@ -734,9 +739,10 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
     return -3;
   if (epi == kSiluMul && (N % 256) != 0) return -4;
   if (epi == kBias && bias == nullptr) return -5;
-  if (epi != kRelu2 && (epi < 0 || epi > 2)) return -20;
+  if (epi != kRelu2 && epi != kFp32 && (epi < 0 || epi > 2)) return -20;
   const int sms = sm_count();
   Plan pl = allow_split == 2 ? make_plan2(M, N, K, epi, sms) : make_plan(M, N, K, epi, sms);
+  if (epi == kFp32 && (allow_split != 2 || pl.splits == 1)) return -20;
   if (allow_split == 2 && pl.splits == 1) {
     // without a split this kernel only takes what it took before: one wave of 256-wide tiles
     const int tiles = (N + 255) / 256;
@@ -782,6 +788,7 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
   switch (epi) {                                                                    \
     case kNone: rc = launch<BN_, MT_, ST_, kNone>(tmA, tmB, a, units, s); break;    \
     case kBias: rc = launch<BN_, MT_, ST_, kBias>(tmA, tmB, a, units, s); break;    \
+    case kFp32: rc = launch<BN_, MT_, ST_, kNone>(tmA, tmB, a, units, s); break;    \
     case kRelu2:                                                                    \
       rc = a.splits > 1 && a.ctr == nullptr                                         \
                ? launch<BN_, MT_, ST_, kNone>(tmA, tmB, a, units, s)                \
@@ -805,7 +812,8 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
   // two-kernel K split: add the partial sums
   const long long work = static_cast<long long>(M) * (N / 4);
   skinny_reduce_kernel<<<static_cast<unsigned>((work + 255) / 256), 256, 0, s>>>(
-      a.ws, a.C, a.ldc, epi == kBias ? a.bias : nullptr, epi == kRelu2, M, N, pl.bn, mt * BM, a.splits);
+      a.ws, a.C, epi == kFp32 ? static_cast<float*>(C) : nullptr, a.ldc,
+      epi == kBias ? a.bias : nullptr, epi == kRelu2, M, N, pl.bn, mt * BM, a.splits);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -210,7 +210,8 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
                 raise N.NativeError(f"b200_gemm_pair_split failed with code {rc}")
     silu_256 = epilogue != EPI_SILU_MUL or Nn % 256 == 0     # these two kernels: 256-wide tiles
     if M <= SKINNY_MAX_M and USE_SKINNY_GEMM and silu_256 \
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2):
+            and (epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2)
+                 or epilogue == EPI_FP32 and M <= SKINNY_SPLIT2_MAX_M):
         ws, ctr = _skinny_workspace(a.device)
         rc = N.lib().b200_gemm_skinny(
             ptr(a), a.stride(0), ptr(b), b.stride(0), ptr(out), out.stride(0), M, Nn, K,
