@@ -87,7 +87,7 @@ def cases(lens: list[int], ctx: int, decode: bool, H: int, N: int, G: int, D: in
     a_s, h_s = rnd(cap, H).to(bf), rnd(cap, F).to(bf)
     w13 = (rnd(E, 2 * F, H) * 0.02).to(bf)
     out.append(("grouped up + squared ReLU", "grouped gate_up + SiLU-mul", lambda: C.gemm_bf16_grouped(
-        a_s, m.experts.w1, eid, npp, relu2=True), touched * F * H * 2 + T * k * (H + F) * 2,
+        a_s, m.experts.w1, eid, npp, act="relu2"), touched * F * H * 2 + T * k * (H + F) * 2,
         2 * T * k * F * H))
     out.append(("grouped gate_up + SiLU-mul", None, lambda: C.gemm_bf16_grouped(
         a_s, w13, eid, npp, silu_mul=True), touched * F * H * 4 + T * k * (H + F) * 2,

@@ -74,7 +74,7 @@ def test_residual_kernels(T, H, dtype):
             _close(gx, out, F32)
             _close(glo, lo, dtype)
     u = torch.randn(T, H, generator=g).to(dtype)
-    _close(C.relu2(u.cuda()), u.float().clamp(min=0).square(), dtype)
+    _close(C.ungated_act(u.cuda(), "relu2"), u.float().clamp(min=0).square(), dtype)
 
 
 # -- squared-ReLU products --------------------------------------------------------------

@@ -62,7 +62,7 @@ def test_residual_kernels(T, H, dtype):
         _close(gout, out, F32)
         _close(glo, lo, dtype)
     u = torch.randn(T, 2 * (H // 2) + 2 * (H % 2), generator=g).to(dtype)
-    _close(C.silu_mul_rows(u.cuda()), ref.silu_and_mul(u.float()), dtype)
+    _close(C.act_mul_rows(u.cuda()), ref.silu_and_mul(u.float()), dtype)
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])

@@ -38,6 +38,19 @@ class AttentionSpec:
     v_head_dim: int = 0                    # 0: the keys are their own values
     softcap: float = 0.0                   # scores become softcap * tanh(score / softcap); 0: none
     chunk: int = 0                         # keys of the query's own chunk of positions; 0: all
+    window: int = 0                        # the last keys up to the query; 0: all
+    # what follows is read by GroupedAttention
+    rot_halves: bool = False               # dimension i turns with i + rot_dims / 2, not neighbours
+    # YaRN: factor, original length, turns of the fast and of the slow end of the ramp
+    rot_scaling: tuple[float, ...] = ()
+    qk_norm: bool = False                  # norms over the whole query and key projections
+    v_norm: bool = False                   # values divided by their root mean square, per head
+    v_mix: bool = False                    # values mixed with those of the first such layer
+    sink: str = ""                         # "learnt" score per head, "zero" (1 joins the sum), none
+    distance_bias: bool = False            # a slope per head times the distance comes off the score
+    # queries times 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) at position p
+    temp_coef: float = 0.0
+    temp_every: int = 1
 
     @property
     def cached_per_token(self) -> int:
@@ -66,6 +79,15 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
+class TimeMixSpec:
+    """Linear recurrence with one decay per head and key channel and a bonus for the current token
+    (layers/recurrent.py)."""
+    num_heads: int
+    head_dim: int                          # keys and values
+    decay_rank: int                        # inner width of the decay's two-step projection
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One layer of a design whose layers differ: mixer type and sizes, feed-forward sizes."""
     mixer: str                             # "latent_attention", or with ``parts`` any name
@@ -80,6 +102,8 @@ class LayerSpec:
     intermediate_size: int = 0             # dense feed-forward
     shared_intermediate_size: int = 0      # shared expert beside the routed ones
     router_scale: float = 1.0              # factor of the routing weights
+    router_groups: int = 1                 # groups of neighbouring experts
+    router_keep: int = 1                   # groups a token's experts come from
     rot_dim: int = 0                       # latent attention: rotated query / key dimensions
     rot_base: float = 10000.0
     sink: bool = False                     # latent attention: learnt term in the denominator
@@ -150,6 +174,9 @@ class ModelConfig:
     # designs described layer by layer (None: every layer has the sizes above)
     layer_specs: Optional[tuple[LayerSpec, ...]] = None
     residual_alpha: float = 1.0            # norm after the sum: norm(alpha * x + sublayer(x))
+    residual_mult: float = 1.0             # norm in front: x + residual_mult * sublayer(norm(x))
+    norm_groups: int = 1                   # parts of a row that are normalised each for itself
+    conv_taps: int = 0                     # causal convolution in front of every mixer; 0: none
     embed_scale: float = 1.0
     logit_scale: float = 1.0
     # (start, stop, times): layers start .. stop - 1 run that often in a row, same weights
@@ -260,6 +287,9 @@ class ModelConfig:
         if d.get("architecture") == "Fepopel" or "FepopelForCausalLM" in (
                 d.get("architectures") or ()):
             return cls._from_looped_list(d, **overrides)
+        if d.get("architecture") == "Vadelix" or "VadelixForCausalLM" in (
+                d.get("architectures") or ()):
+            return cls._from_prenorm_list(d, **overrides)
         archs = d.get("architectures") or ["LlamaForCausalLM"]
         for nested in ("text_config", "language_config", "llm_config"):
             if isinstance(d.get(nested), dict):
@@ -514,10 +544,89 @@ class ModelConfig:
         return cls(**kw)
 
     @classmethod
+    def _from_prenorm_list(cls, d: dict, **overrides) -> "ModelConfig":
+        """Vadelix's ``config.json``: ``vocab``, ``width``, ``norm`` (eps, groups),
+        ``residual_mult``, ``canon.taps`` and one entry of ``layers`` per layer.  The inner width of
+        a decay's two-step projection is no number of the file: a checkpoint's tensors give it
+        (``tensor_shapes``), else ``decay_rank`` of the mixer, else its ``dim``."""
+        shapes = overrides.pop("tensor_shapes", None) or {}
+        specs = []
+        for i, layer in enumerate(d["layers"]):
+            m, f, where = layer["mixer"], layer.get("mlp"), f"layer {i}"
+            kw: dict[str, Any] = {}
+            if f is not None and f.get("kind", "dense") == "dense":
+                kw["intermediate_size"] = int(f["ff"])
+            elif f is not None and f["kind"] == "moe":
+                r, shared = f["router"], f.get("shared")
+                groups = r.get("groups") or {"count": 1, "keep": 1}
+                kw.update(num_experts=int(r["experts"]), num_experts_per_tok=int(r["top"]),
+                          router_groups=int(groups["count"]), router_keep=int(groups["keep"]),
+                          moe_intermediate_size=int(f["expert"]["ff"]),
+                          shared_intermediate_size=int(shared["ff"]) if shared else 0)
+                E, count, keep = kw["num_experts"], kw["router_groups"], kw["router_keep"]
+                if E % count or not 0 < keep <= count:
+                    raise ValueError(f"{where}: {keep} of {count} groups of {E} experts")
+                if not 0 < kw["num_experts_per_tok"] <= E // count * keep:
+                    raise ValueError(f"{where}: {kw['num_experts_per_tok']} of "
+                                     f"{E // count * keep} experts per token")
+            elif f is not None:
+                raise ValueError(f"{where}: unknown feed-forward {f['kind']!r}")
+            if layer["type"] == "wkv":
+                rank = shapes.get(f"l{i}.mix.w1")
+                spec: Any = TimeMixSpec(int(m["heads"]), int(m["dim"]), int(
+                    rank[0] if rank is not None else m.get("decay_rank") or m["dim"]))
+            elif layer["type"] in ("attention", "attention_2"):
+                size = dict(num_heads=int(m["heads"]), num_kv_heads=int(m["kv_heads"]),
+                            head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
+                            scale=float(m["scale"]), v_mix=bool(m.get("v_mix")))
+                if layer["type"] == "attention":
+                    rot, y = m["rot"], m["rot"].get("scaling")
+                    spec = AttentionSpec(
+                        rot_dims=int(rot["dims"]), rot_base=float(rot["base"]), rot_halves=True,
+                        rot_scaling=tuple(float(y[k]) for k in ("factor", "original", "fast",
+                                                                "slow")) if y else (),
+                        qk_norm=True, v_norm=True, sink="learnt", **size)
+                else:
+                    t = m.get("q_temp") or {"coef": 0.0, "every": 1}
+                    spec = AttentionSpec(
+                        window=int((m.get("mask") or {}).get("size") or 0), distance_bias=True,
+                        sink="zero", temp_coef=float(t["coef"]), temp_every=int(t["every"]), **size)
+            else:
+                raise ValueError(f"{where}: unknown mixer {layer['type']!r}")
+            specs.append(LayerSpec(layer["type"], parts=(("", 1.0, spec),), **kw))
+        if not specs:
+            raise ValueError("the configuration lists no layers")
+        H, groups = int(d["width"]), int(d["norm"].get("groups", 1))
+        if H % groups:
+            raise ValueError(f"a norm of {groups} groups over {H} coordinates")
+        attn = [s for sp in specs for _, _, s in sp.parts if isinstance(s, AttentionSpec)]
+        kw = dict(
+            architecture="VadelixForCausalLM", vocab_size=int(d["vocab"]), hidden_size=H,
+            num_hidden_layers=len(specs), layer_specs=tuple(specs),
+            rms_norm_eps=float(d["norm"]["eps"]), norm_groups=groups,
+            residual_mult=float(d.get("residual_mult", 1.0)),
+            conv_taps=int(d["canon"]["taps"]), hidden_act="gelu_tanh",
+            # the largest layer stands for the model where one number is asked for
+            intermediate_size=max(s.intermediate_size for s in specs),
+            num_attention_heads=max((s.num_heads for s in attn), default=1),
+            num_key_value_heads=max((s.num_kv_heads for s in attn), default=1),
+            head_dim=max((max(s.head_dim, s.v_head_dim) for s in attn), default=1),
+            num_experts=max(s.num_experts for s in specs),
+            num_experts_per_tok=max(s.num_experts_per_tok for s in specs),
+            moe_intermediate_size=max(s.moe_intermediate_size for s in specs),
+            # no limit of the design's own: bounds the rotary and block tables only
+            max_position_embeddings=int(d.get("max_position_embeddings", 131072)),
+            extra={k: v for k, v in d.items() if k not in (
+                "layers", "vocab", "width", "norm", "canon", "residual_mult", "architecture",
+                "architectures", "max_position_embeddings")})
+        kw.update(overrides)
+        return cls(**kw)
+
+    @classmethod
     def from_pretrained(cls, path: str, **overrides) -> "ModelConfig":
         p = Path(path)
         d = json.loads((p / "config.json").read_text())
-        if d.get("architecture") == "Fizunex":
+        if d.get("architecture") in ("Fizunex", "Vadelix"):
             from .utils.weights import tensor_shapes
             overrides = {"tensor_shapes": tensor_shapes(path), **overrides}
         cfg = cls.from_hf_dict(d, **overrides)
@@ -650,6 +759,30 @@ def _fepopel_preset(pattern: str, loop: tuple[int, int, int], vocab: int, width:
                        for p in pattern.split()]}
 
 
+def _vadelix_preset(pattern: str, vocab: int, width: int, heads: int, kv_heads: int, dim: int,
+                    window: int, wkv_heads: int, wkv_dim: int, ff: int, experts: int, top: int,
+                    groups: tuple[int, int], expert_ff: int, shared_ff: int, rank: int) -> dict:
+    """``pattern``: two letters per layer, r for rotary attention, b for windowed attention with
+    distance biases or w for time mixing, then d for a dense feed-forward or e for experts."""
+    size = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+            "v_mix": True}
+    mixers = {
+        "r": ("attention", {**size, "rot": {
+            "dims": dim // 2, "base": 500000.0,
+            "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}),
+        "b": ("attention_2", {**size, "mask": {"size": window},
+                              "q_temp": {"coef": 0.1, "every": 8192}}),
+        "w": ("wkv", {"heads": wkv_heads, "dim": wkv_dim, "decay_rank": rank})}
+    mlps = {"d": {"kind": "dense", "ff": ff},
+            "e": {"kind": "moe", "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff},
+                  "router": {"experts": experts, "top": top,
+                             "groups": {"count": groups[0], "keep": groups[1]}}}}
+    return {"architecture": "Vadelix", "vocab": vocab, "width": width, "residual_mult": 0.5,
+            "norm": {"eps": 1e-5, "groups": 8}, "canon": {"taps": 4},
+            "layers": [{"type": mixers[p[0]][0], "mixer": mixers[p[0]][1], "mlp": mlps[p[1]]}
+                       for p in pattern.split()]}
+
+
 #: configurations of designs that are described layer by layer
 _LAYER_LIST_PRESETS: dict[str, dict] = {
     "tiny-sapapel": _sapapel_preset(3, 1024, 128, 4, 24, 40, 48, 6, 2, 48),
@@ -660,6 +793,11 @@ _LAYER_LIST_PRESETS: dict[str, dict] = {
     # layers of the size of DeepSeek-V2-Lite's
     "fepopel-16b": _fepopel_preset("ld" + " le ce le" * 8 + " le", (1, 4, 2), 102400, 2048, 16, 128,
                                    64, 512, 4, 1024, 10944, 64, 6, 1408, 2816),
+    "tiny-vadelix": _vadelix_preset("rd we be rd", 1024, 128, 4, 2, 24, 32, 4, 24, 192, 8, 2, (4, 2),
+                                    48, 40, 12),
+    # layers of the size of Llama-3-8B's, experts of the size of DeepSeek-V2-Lite's
+    "vadelix-12b": _vadelix_preset("rd we be we" + " rd we be we" * 7, 128256, 4096, 32, 8, 128,
+                                   1024, 64, 64, 14336, 32, 4, (4, 2), 1536, 3072, 64),
     "tiny-fizunex": _fizunex_preset("dpd", 1024, 128, 192, *_fizunex_mixers(4, 2, 32, 2, 24, 40)),
     # layers of the size of Llama-3-8B's
     "fizunex-8b": _fizunex_preset("dddp" * 8, 128256, 4096, 14336,

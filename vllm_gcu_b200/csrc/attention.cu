@@ -158,6 +158,7 @@ struct DecodeArgs {
   // kShaped kernels only
   float softcap;        // > 0: scores become softcap * tanh(score / softcap)
   int chunk;            // > 0: keys of the query's own chunk of that many positions
+  int window;           // > 0: the last keys up to the query
   int OD;               // output columns per head (the first of the HD)
 };
 
@@ -170,7 +171,7 @@ __device__ __forceinline__ float sink_share(float M, float L, float sink) {
   return keys / (keys + exp2f(s2 - top));
 }
 
-// kShaped: soft cap, chunk and output columns of DecodeArgs are in force
+// kShaped: soft cap, chunk, window and output columns of DecodeArgs are in force
 template <typename T, int HD, bool kShaped = false>
 __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs a) {
   constexpr int kStride = HD + kPad;
@@ -188,7 +189,8 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
   const int seq_len = a.seq_lens[b];
   const int OD = kShaped ? a.OD : HD;
   // first key the query sees
-  const int first = kShaped && a.chunk > 0 && seq_len > 0 ? (seq_len - 1) / a.chunk * a.chunk : 0;
+  int first = kShaped && a.chunk > 0 && seq_len > 0 ? (seq_len - 1) / a.chunk * a.chunk : 0;
+  if (kShaped && a.window > 0) first = max(first, seq_len - a.window);
   const int per_split = (seq_len - first + a.num_splits - 1) / a.num_splits;
   const int chunk = ((per_split + kTile - 1) / kTile) * kTile;
   const int start = first + split * chunk;
@@ -279,7 +281,9 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(const DecodeArgs
           float v = (tok < end)
                         ? s[j][e] * sl2 + al[e >> 1] * static_cast<float>(tok - (seq_len - 1))
                         : -INFINITY;
-          if (kShaped && capped && tok < end) v = cap2 * tanh_fast(s[j][e] * in2);
+          if (kShaped && capped && tok < end)
+            v = cap2 * tanh_fast(s[j][e] * in2) +
+                al[e >> 1] * static_cast<float>(tok - (seq_len - 1));
           s[j][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -704,7 +708,7 @@ static int paged_decode_impl(const void* q, long long ldq, void* out, long long 
                              int dtype, int qmode, float k_scale, float v_scale, float k_zp,
                              float v_zp, void* stream, const float* alibi = nullptr,
                              const float* sink = nullptr, float softcap = 0.0f, int chunk = 0,
-                             int OD = 0) {
+                             int OD = 0, int window = 0) {
   if (B <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16) return -2;
   if (num_splits < 1) return -2;
@@ -720,9 +724,9 @@ static int paged_decode_impl(const void* q, long long ldq, void* out, long long 
   a.scale = scale;
   a.alibi = alibi;
   a.sink = sink;
-  a.softcap = softcap; a.chunk = chunk; a.OD = OD > 0 ? OD : HD;
+  a.softcap = softcap; a.chunk = chunk; a.window = window; a.OD = OD > 0 ? OD : HD;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (softcap > 0.0f || chunk > 0 || a.OD != HD) {
+  if (softcap > 0.0f || chunk > 0 || window > 0 || a.OD != HD) {
     if (dtype == 0 && HD == 128) return launch_decode<__nv_bfloat16, 128, true>(a, s);
     if (dtype == 0 && HD == 64) return launch_decode<__nv_bfloat16, 64, true>(a, s);
     if (dtype == 0 && HD == 96) return launch_decode<__nv_bfloat16, 96, true>(a, s);
@@ -776,8 +780,9 @@ B200_API int b200_paged_decode_alibi(const void* q, long long ldq, void* out, lo
 
 // Decode attention with, each optional: one learnt sink per query head (exp(sink) is added to the
 // softmax denominator; it has no key and no value and is not scaled); a soft cap of the scores; only
-// the keys of the query's own chunk of positions, counted from 0; only the first OD columns of a
-// head's output stored, heads side by side.  The last three: bf16, HD 64, 96 or 128.
+// the keys of the query's own chunk of positions, counted from 0; only the last `window` keys up to
+// the query; ALiBi slopes (see b200_paged_decode_alibi); only the first OD columns of a head's output
+// stored, heads side by side.  Caps, chunks, windows and columns: bf16, HD 64, 96 or 128.
 B200_API int b200_paged_decode_sink(const void* q, long long ldq, void* out, long long ldo,
                                     const void* k_cache, const void* v_cache,
                                     long long slot_stride, long long head_stride,
@@ -785,12 +790,13 @@ B200_API int b200_paged_decode_sink(const void* q, long long ldq, void* out, lon
                                     int block_size, const int* seq_lens, float* tmp_out,
                                     float* tmp_lse, int num_splits, int B, int Hq, int Hkv,
                                     int HD, float scale, int dtype, const float* sink,
-                                    float softcap, int chunk, int OD, void* stream) {
-  if (OD < 0 || OD > HD || chunk < 0) return -2;
+                                    float softcap, int chunk, int window, const float* alibi,
+                                    int OD, void* stream) {
+  if (OD < 0 || OD > HD || chunk < 0 || window < 0) return -2;
   return paged_decode_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride, num_slots,
                            block_tables, max_blocks, block_size, seq_lens, tmp_out, tmp_lse,
                            num_splits, B, Hq, Hkv, HD, scale, dtype, 0, 1.0f, 1.0f, 0.0f, 0.0f,
-                           stream, nullptr, sink, softcap, chunk, OD);
+                           stream, alibi, sink, softcap, chunk, OD, window);
 }
 
 // Decode attention over an 8-bit KV cache (same layout, one byte per element; slot_stride and

@@ -67,22 +67,25 @@ struct Args {
   long long ldo;
   int B, T, Hq, Hkv, max_blocks, block_size, causal, window;
   float scale;
-  // kShaped kernels only
+  // shaped and biased kernels only
   float softcap;           // > 0: scores become softcap * tanh(score / softcap)
   int chunk;               // > 0: keys of the query's own chunk of that many positions
   int OD;                  // output columns per head (the first of the HD)
+  const float* slopes;     // biased kernels: [Hq], slope * (key - query position) joins the score
   unsigned int* status;
 };
 
 // HD below 128 uses the same tiles: the second 64-column half then carries columns of the next
 // head (or zeros) behind HD, which no contraction step and no store touches.
-// kShaped: soft cap, chunk and output columns of Args are in force.  The soft cap is monotonic, so
-// row maxima are taken over uncapped scores.
-template <int HD, bool kShaped>
+// MODE 1 (shaped): soft cap, chunk and output columns of Args are in force.  The soft cap is
+// monotonic, so row maxima are taken over uncapped scores.  MODE 2 (biased): slopes and output columns;
+// row maxima are those of the biased scores, in the log2 domain.
+template <int HD, int MODE>
 __global__ void __launch_bounds__(kThreads, 1)
     fmha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ,
                         const __grid_constant__ CUtensorMap tmK,
                         const __grid_constant__ CUtensorMap tmV, const Args a) {
+  constexpr bool kShaped = MODE == 1, kBiased = MODE == 2;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>(
       (reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -288,7 +291,14 @@ __global__ void __launch_bounds__(kThreads, 1)
     const float cap2 = capped ? a.softcap * 1.4426950408889634f : 0.0f;
     const float in2 = capped ? a.scale / a.softcap : 0.0f;
     // log2-domain value of a score
-    auto l2 = [&](float raw) { return capped ? cap2 * tanh_fast(raw * in2) : raw * sl2; };
+    auto l2 = [&](float raw) {
+      return kBiased ? raw : capped ? cap2 * tanh_fast(raw * in2) : raw * sl2;
+    };
+    const float slope2 = kBiased ? a.slopes[head] * 1.4426950408889634f : 0.0f;
+    // biased score of element i of 32, `base` the bias of the first
+    auto biased = [&](uint32_t raw, int i, float base) {
+      return fmaf(__uint_as_float(raw), sl2, fmaf(slope2, static_cast<float>(i), base));
+    };
     float m_used = -INFINITY, l = 0.0f;
     uint8_t* sp = smem + kOffP + g * kSub;      // this group's 64-key sub-tile of P
     float* xch = reinterpret_cast<float*>(smem + kOffX);   // [2][128]
@@ -315,6 +325,11 @@ __global__ void __launch_bounds__(kThreads, 1)
           uint32_t v[32];
           tmem_ld_32x32(s_addr + c * 32, v);
           tmem_ld_wait();
+          if constexpr (kBiased) {
+            const float base = slope2 * static_cast<float>(key0 + c * 32 - pos);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(biased(v[i], i, base));
+          }
           if (need_mask) {
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
@@ -341,7 +356,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       float alpha = 1.0f;
       float m_new = m_used;
       float mb;
-      if constexpr (kShaped) {
+      if constexpr (MODE != 0) {
         if (mt > m_used && (m_used == -INFINITY || l2(mt) - l2(m_used) > 8.0f)) {
           m_new = mt;
           alpha = m_used == -INFINITY ? 0.0f : ex2_approx(l2(m_used) - l2(m_new));
@@ -355,7 +370,8 @@ __global__ void __launch_bounds__(kThreads, 1)
         mb = (m_new == -INFINITY ? 0.0f : m_new) * sl2;
       }
       // exponential of a score relative to the running maximum
-      auto prob = [&](uint32_t raw) {
+      auto prob = [&](uint32_t raw, int i, float base) {
+        if constexpr (kBiased) return ex2_approx(biased(raw, i, base));
         const float x = __uint_as_float(raw);
         if constexpr (kShaped) {
           if (capped) return ex2_approx(fmaf(cap2, tanh_fast(x * in2), -mb));
@@ -371,12 +387,14 @@ __global__ void __launch_bounds__(kThreads, 1)
           uint32_t v[32];
           tmem_ld_32x32(s_addr + c * 32, v);
           tmem_ld_wait();
+          const float base =
+              kBiased ? fmaf(slope2, static_cast<float>(key0 + c * 32 - pos), -mb) : 0.0f;
           if (need_mask) {
 #pragma unroll
             for (int i = 0; i < 32; i += 2) {
               const int key = key0 + c * 32 + i;
-              float p0 = prob(v[i]);
-              float p1 = prob(v[i + 1]);
+              float p0 = prob(v[i], i, base);
+              float p1 = prob(v[i + 1], i + 1, base);
               if (key > hi || key < lo) p0 = 0.0f;
               if (key + 1 > hi || key + 1 < lo) p1 = 0.0f;
               rs0 += p0;
@@ -386,8 +404,8 @@ __global__ void __launch_bounds__(kThreads, 1)
           } else {
 #pragma unroll
             for (int i = 0; i < 32; i += 2) {
-              const float p0 = prob(v[i]);
-              const float p1 = prob(v[i + 1]);
+              const float p0 = prob(v[i], i, base);
+              const float p1 = prob(v[i + 1], i + 1, base);
               rs0 += p0;
               rs1 += p1;
               pk[c * 16 + (i >> 1)] = pack_bf16x2(p0, p1);
@@ -441,7 +459,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         den += exp2f(fmaf(a.sink[head], 1.4426950408889634f, -l2(m_used)));
       const float inv = l > 0.0f ? 1.0f / den : 0.0f;
       const bool row_ok = r < rows;
-      const int OD = kShaped ? a.OD : HD;
+      const int OD = MODE != 0 ? a.OD : HD;
       __nv_bfloat16* orow =
           a.out + static_cast<long long>(q_start + q0 + r) * a.ldo + head * OD + g * 64;
 #pragma unroll 1
@@ -457,7 +475,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             u.y = pack_bf16x2(__uint_as_float(v[i * 8 + 2]) * inv, __uint_as_float(v[i * 8 + 3]) * inv);
             u.z = pack_bf16x2(__uint_as_float(v[i * 8 + 4]) * inv, __uint_as_float(v[i * 8 + 5]) * inv);
             u.w = pack_bf16x2(__uint_as_float(v[i * 8 + 6]) * inv, __uint_as_float(v[i * 8 + 7]) * inv);
-            if constexpr (kShaped) {
+            if constexpr (MODE != 0) {
               const int col = g * 64 + c * 32 + i * 8;
               if ((OD & 7) != 0) {
 #pragma unroll
@@ -529,20 +547,20 @@ static int get_map(const void* base, unsigned long long rows, unsigned long long
 namespace b200 {
 namespace fmha {
 
-template <int HD, bool kShaped>
+template <int HD, int MODE>
 static int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                   const Args& a, int num_q_tiles, cudaStream_t s) {
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel<HD, kShaped>,
+    cudaError_t e = cudaFuncSetAttribute(fmha_prefill_kernel<HD, MODE>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev] = true;
   }
   dim3 grid(num_q_tiles, a.Hq);
-  fmha_prefill_kernel<HD, kShaped><<<grid, kThreads, kSmemBytes, s>>>(tmQ, tmK, tmV, a);
+  fmha_prefill_kernel<HD, MODE><<<grid, kThreads, kSmemBytes, s>>>(tmQ, tmK, tmV, a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -551,8 +569,10 @@ static int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensor
 
 // Same contract as b200_varlen_prefill for bf16, head_dim 64, 96 or 128, caches laid out as
 // [num_slots, Hkv * HD] rows and a block size that is a multiple of 16; num_q_tiles must be
-// >= sum_b ceil(q_len_b / 128).  sink, softcap, chunk and OD: optional, see b200_paged_decode_sink
-// (OD that is no multiple of 8 is stored element by element).  Returns -20 when the layout does not qualify (callers use another kernel).
+// >= sum_b ceil(q_len_b / 128).  sink, softcap, chunk, slopes and OD: optional, see
+// b200_paged_decode_sink (OD that is no multiple of 8 is stored element by element; slopes do not go
+// with a soft cap or chunks).  Returns -20 when the layout does not qualify (callers use another
+// kernel).
 B200_API int b200_fmha_prefill_sink(const void* q, long long ldq, void* out, long long ldo,
                                     float* lse, const int* cu_q, const int* seq_lens,
                                     const void* k_cache, const void* v_cache,
@@ -560,13 +580,14 @@ B200_API int b200_fmha_prefill_sink(const void* q, long long ldq, void* out, lon
                                     long long num_slots, const int* block_tables, int max_blocks,
                                     int block_size, int B, int T, int num_q_tiles, int Hq, int Hkv,
                                     int HD, float scale, int causal, int window, int dtype,
-                                    const float* sink, float softcap, int chunk, int OD,
-                                    void* stream) {
+                                    const float* sink, float softcap, int chunk,
+                                    const float* slopes, int OD, void* stream) {
   using namespace b200;
   using namespace b200::fmha;
   if (B <= 0 || T <= 0 || num_q_tiles <= 0) return 0;
   if (OD <= 0) OD = HD;
   if (OD > HD || chunk < 0) return -2;
+  if (slopes != nullptr && (softcap > 0.0f || chunk > 0)) return -20;
   if (dtype != 0 || (HD != 64 && HD != 96 && HD != 128) || (block_size % kPage) != 0 ||
       head_stride != HD || slot_stride != static_cast<long long>(Hkv) * HD || Hkv <= 0 ||
       Hq % Hkv != 0 || (ldq % 8) != 0 || ((OD % 8) == 0 && (ldo % 8) != 0) ||
@@ -588,17 +609,19 @@ B200_API int b200_fmha_prefill_sink(const void* q, long long ldq, void* out, lon
   a.lse = lse; a.sink = sink; a.cu_q = cu_q; a.seq_lens = seq_lens; a.block_tables = block_tables;
   a.ldo = ldo; a.B = B; a.T = T; a.Hq = Hq; a.Hkv = Hkv; a.max_blocks = max_blocks;
   a.block_size = block_size; a.causal = causal; a.window = window; a.scale = scale;
-  a.softcap = softcap; a.chunk = chunk; a.OD = OD;
+  a.softcap = softcap; a.chunk = chunk; a.OD = OD; a.slopes = slopes;
   a.status = status_ptr();
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (softcap > 0.0f || chunk > 0 || OD != HD) {
-    if (HD == 64) return launch<64, true>(tmQ, tmK, tmV, a, num_q_tiles, s);
-    if (HD == 96) return launch<96, true>(tmQ, tmK, tmV, a, num_q_tiles, s);
-    return launch<128, true>(tmQ, tmK, tmV, a, num_q_tiles, s);
-  }
-  if (HD == 64) return launch<64, false>(tmQ, tmK, tmV, a, num_q_tiles, s);
-  if (HD == 96) return launch<96, false>(tmQ, tmK, tmV, a, num_q_tiles, s);
-  return launch<128, false>(tmQ, tmK, tmV, a, num_q_tiles, s);
+#define B200_FMHA(MODE)                                                        \
+  do {                                                                         \
+    if (HD == 64) return launch<64, MODE>(tmQ, tmK, tmV, a, num_q_tiles, s);   \
+    if (HD == 96) return launch<96, MODE>(tmQ, tmK, tmV, a, num_q_tiles, s);   \
+    return launch<128, MODE>(tmQ, tmK, tmV, a, num_q_tiles, s);                \
+  } while (0)
+  if (slopes != nullptr) B200_FMHA(2);
+  if (softcap > 0.0f || chunk > 0 || OD != HD) B200_FMHA(1);
+  B200_FMHA(0);
+#undef B200_FMHA
 }
 
 B200_API int b200_fmha_prefill(const void* q, long long ldq, void* out, long long ldo, float* lse,
@@ -611,5 +634,5 @@ B200_API int b200_fmha_prefill(const void* q, long long ldq, void* out, long lon
   return b200_fmha_prefill_sink(q, ldq, out, ldo, lse, cu_q, seq_lens, k_cache, v_cache,
                                 slot_stride, head_stride, num_slots, block_tables, max_blocks,
                                 block_size, B, T, num_q_tiles, Hq, Hkv, HD, scale, causal, window,
-                                dtype, nullptr, 0.0f, 0, 0, stream);
+                                dtype, nullptr, 0.0f, 0, nullptr, 0, stream);
 }

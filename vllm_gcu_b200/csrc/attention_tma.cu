@@ -81,11 +81,12 @@ struct Args {
   float scale;
   const float* sink;     // optional [Hq], see b200_paged_decode_sink
   float softcap;         // kShaped kernels: see b200_paged_decode_sink
-  int chunk, OD;
+  int chunk, window, OD;
+  const float* alibi;    // kShaped kernels: [Hq] slopes or null
   unsigned int* status;
 };
 
-// kShaped: soft cap, chunk and output columns are in force
+// kShaped: soft cap, chunk, window, slopes and output columns are in force
 template <typename T, bool kShaped>
 __global__ void __launch_bounds__(kThreads)
     paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK,
@@ -103,7 +104,8 @@ __global__ void __launch_bounds__(kThreads)
   const int seq_len = a.seq_lens[b];
   const int OD = kShaped ? a.OD : HD;
   // first key the query sees; copies start at whole boxes, the keys in front of it are masked
-  const int lo = kShaped && a.chunk > 0 && seq_len > 0 ? (seq_len - 1) / a.chunk * a.chunk : 0;
+  int lo = kShaped && a.chunk > 0 && seq_len > 0 ? (seq_len - 1) / a.chunk * a.chunk : 0;
+  if (kShaped && a.window > 0) lo = max(lo, seq_len - a.window);
   const int first = lo / kChunk * kChunk;
   const int per_split = (seq_len - first + a.num_splits - 1) / a.num_splits;
   const int chunk = ((per_split + kTile - 1) / kTile) * kTile;
@@ -192,6 +194,11 @@ __global__ void __launch_bounds__(kThreads)
   const bool capped = kShaped && a.softcap > 0.0f;
   const float cap2 = capped ? a.softcap * kLog2e : 0.0f, in2 = capped ? a.scale / a.softcap : 0.0f;
   const uint32_t smem_base = smem_u32(smem);
+  float al[2] = {0.0f, 0.0f};
+  if (kShaped && a.alibi != nullptr) {
+    if (g < G) al[0] = a.alibi[kvh * G + g] * kLog2e;
+    if (g + 8 < G) al[1] = a.alibi[kvh * G + g + 8] * kLog2e;
+  }
 
   int stage = 0;
   uint32_t phase = 0;
@@ -228,6 +235,7 @@ __global__ void __launch_bounds__(kThreads)
           const int tok = tok0 + j * 8 + 2 * tig + (e & 1);
           float v = s[j][e] * sl2;
           if (kShaped && capped) v = cap2 * tanh_fast(s[j][e] * in2);
+          if (kShaped) v += al[e >> 1] * static_cast<float>(tok - (seq_len - 1));
           if (tok >= end || (kShaped && tok < lo)) v = -INFINITY;
           s[j][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -389,8 +397,8 @@ static int paged_decode_tma_impl(const void* q, long long ldq, void* out, long l
                                  const int* block_tables, int max_blocks, int block_size,
                                  const int* seq_lens, float* tmp_out, float* tmp_lse,
                                  int num_splits, int B, int Hq, int Hkv, int HD, float scale,
-                                 int dtype, const float* sink, float softcap, int chunk, int OD,
-                                 void* stream) {
+                                 int dtype, const float* sink, float softcap, int chunk,
+                                 int window, const float* alibi, int OD, void* stream) {
   using namespace b200;
   using namespace b200::attn_tma;
   if (B <= 0) return 0;
@@ -412,8 +420,9 @@ static int paged_decode_tma_impl(const void* q, long long ldq, void* out, long l
   a.block_tables = block_tables; a.ldq = ldq; a.ldo = ldo; a.B = B; a.Hq = Hq; a.Hkv = Hkv;
   a.num_splits = num_splits; a.max_blocks = max_blocks; a.block_size = block_size;
   a.scale = scale; a.sink = sink; a.softcap = softcap; a.chunk = chunk; a.OD = OD > 0 ? OD : HD;
+  a.window = window; a.alibi = alibi;
   a.status = status_ptr();
-  const bool shaped = softcap > 0.0f || chunk > 0 || a.OD != HD;
+  const bool shaped = softcap > 0.0f || chunk > 0 || window > 0 || alibi != nullptr || a.OD != HD;
   if (shaped && dtype != 0) return -20;
   constexpr int smem = kStages * kStageBytes + 256 + 1024;
   static_assert(kStages * kStageBytes >= (128 + 4 * 16 * b200::attn_tma::HD) * 4,
@@ -464,10 +473,10 @@ B200_API int b200_paged_decode_tma(const void* q, long long ldq, void* out, long
   return paged_decode_tma_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride,
                                num_slots, block_tables, max_blocks, block_size, seq_lens, tmp_out,
                                tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, nullptr, 0.0f, 0, 0,
-                               stream);
+                               nullptr, 0, stream);
 }
 
-// The same with sinks, soft cap, chunk and output columns (see b200_paged_decode_sink).
+// The same with sinks, soft cap, chunk, window, slopes and output columns (see b200_paged_decode_sink).
 B200_API int b200_paged_decode_tma_sink(const void* q, long long ldq, void* out, long long ldo,
                                         const void* k_cache, const void* v_cache,
                                         long long slot_stride, long long head_stride,
@@ -475,11 +484,11 @@ B200_API int b200_paged_decode_tma_sink(const void* q, long long ldq, void* out,
                                         int max_blocks, int block_size, const int* seq_lens,
                                         float* tmp_out, float* tmp_lse, int num_splits, int B,
                                         int Hq, int Hkv, int HD, float scale, int dtype,
-                                        const float* sink, float softcap, int chunk, int OD,
-                                        void* stream) {
-  if (OD < 0 || OD > HD || chunk < 0) return -2;
+                                        const float* sink, float softcap, int chunk, int window,
+                                        const float* alibi, int OD, void* stream) {
+  if (OD < 0 || OD > HD || chunk < 0 || window < 0) return -2;
   return paged_decode_tma_impl(q, ldq, out, ldo, k_cache, v_cache, slot_stride, head_stride,
                                num_slots, block_tables, max_blocks, block_size, seq_lens, tmp_out,
-                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, sink, softcap, chunk, OD,
-                               stream);
+                               tmp_lse, num_splits, B, Hq, Hkv, HD, scale, dtype, sink, softcap, chunk,
+                               window, alibi, OD, stream);
 }

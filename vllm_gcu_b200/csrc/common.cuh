@@ -357,6 +357,20 @@ __device__ __forceinline__ float relu2_f(float x) {
   return r * r;
 }
 
+// x times the normal distribution function, and its tanh form
+__device__ __forceinline__ float gelu_f(float x) {
+  return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
+}
+__device__ __forceinline__ float gelu_tanh_f(float x) {
+  return 0.5f * x * (1.0f + tanh_fast(0.79788456080286536f * fmaf(0.044715f * x * x, x, x)));
+}
+// gated activation of a GEMM's epilogue
+template <bool GELU>
+__device__ __forceinline__ float gated_f(float gate, float up) {
+  if constexpr (GELU) return gelu_tanh_f(gate) * up;
+  else return silu_f(gate) * up;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -38,7 +38,11 @@ enum Epilogue : int {
   kEpiGatherA = 7,    // A rows are gathered from the peers' shards by extra warps of this kernel
   kEpiReduceNorm = 8, // row-parallel partial -> row owners reduce (+ residual, RMSNorm) and broadcast
   kEpiRelu2 = 9,      // max(x, 0)^2
+  kEpiGelu = 10,      // GELU through the error function
+  kEpiGeluMul = 11,   // GELU (tanh form) of the gate times up, laid out as for kEpiSiluMul
 };
+template <int EPI>
+constexpr bool kGatedEpi = EPI == kEpiSiluMul || EPI == kEpiGeluMul;
 
 template <int EPI>
 constexpr int kThreadsFor =
@@ -1164,9 +1168,9 @@ __global__ void __launch_bounds__(kThreadsFor<EPI>, 1)
       const uint32_t taddr =
           tmem_base + (static_cast<uint32_t>(q * 32) << 16) + static_cast<uint32_t>(acc * BN);
 
-      if constexpr (EPI == kEpiSiluMul) {
+      if constexpr (kGatedEpi<EPI>) {
         // every 64-column group of the tile = 32 gate columns, then the 32 matching up columns
-        static_assert(EPI != kEpiSiluMul || BN % 64 == 0, "SiLU-mul epilogue: 64-column groups");
+        static_assert(!kGatedEpi<EPI> || BN % 64 == 0, "gated epilogue: 64-column groups");
         const int out_n0 = (n0 >> 1);
         const int out_n = p.N >> 1;
         __nv_bfloat16* crow =
@@ -1180,7 +1184,7 @@ __global__ void __launch_bounds__(kThreadsFor<EPI>, 1)
           float v[32];
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            v[i] = silu_f(__uint_as_float(g[i])) * __uint_as_float(u[i]);
+            v[i] = gated_f<EPI == kEpiGeluMul>(__uint_as_float(g[i]), __uint_as_float(u[i]));
           const int col = out_n0 + c * 32;
           if (row_ok && col < out_n) store_row_bf16(crow + col, v, min(32, out_n - col));
         }
@@ -1327,6 +1331,10 @@ __global__ void __launch_bounds__(kThreadsFor<EPI>, 1)
 #pragma unroll
             for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
           }
+          if constexpr (EPI == kEpiGelu) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[i] = gelu_f(v[i]);
+          }
           if (p.row_scale != nullptr) {
             const float rs = p.row_scale[row];
 #pragma unroll
@@ -1441,7 +1449,8 @@ B200_API int b200_gemm_bf16(const void* A, long long lda, const void* B, long lo
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B) |
        reinterpret_cast<uintptr_t>(C)) & 15)
     return -3;
-  if (epi == kEpiSiluMul && (N % 64) != 0) return -4;
+  const bool gated = epi == kEpiSiluMul || epi == kEpiGeluMul;
+  if (gated && (N % 64) != 0) return -4;
   if (epi == kEpiBias && bias == nullptr) return -5;
   if (epi == kEpiResidual && residual == nullptr) return -5;
 
@@ -1456,8 +1465,8 @@ B200_API int b200_gemm_bf16(const void* A, long long lda, const void* B, long lo
     for (int i = 0; i < 4; ++i) {
       const int c = cands[i];
       if (c == 256 && (N % 256) != 0) continue;
-      // the SiLU-mul epilogue pairs 32 + 32 columns: whole 64-column groups per tile
-      if (epi == kEpiSiluMul && ((c % 64) != 0 || (N % c) != 0)) continue;
+      // the gated epilogues pair 32 + 32 columns: whole 64-column groups per tile
+      if (gated && ((c % 64) != 0 || (N % c) != 0)) continue;
       const long long tiles = static_cast<long long>(tiles_m) * ((N + c - 1) / c);
       const long long waves = (tiles + sm_count() - 1) / sm_count();
       const long long cost = waves * (c + 32);
@@ -1512,6 +1521,11 @@ B200_API int b200_gemm_bf16(const void* A, long long lda, const void* B, long lo
     B200_GEMM_CASE(kEpiResidual)
     B200_GEMM_CASE(kEpiFp32)
     B200_GEMM_CASE(kEpiRelu2)
+    B200_GEMM_CASE(kEpiGelu)
+    case kEpiGeluMul:
+      if (bn == 64) return launch<64, 8, kEpiGeluMul>(tmA, tmB, a, s);
+      if (bn == 128) return launch<128, 6, kEpiGeluMul>(tmA, tmB, a, s);
+      return launch<256, 4, kEpiGeluMul>(tmA, tmB, a, s);
     case kEpiSiluMul:
       if (bn == 64) return launch<64, 8, kEpiSiluMul>(tmA, tmB, a, s);
       if (bn == 128) return launch<128, 6, kEpiSiluMul>(tmA, tmB, a, s);
@@ -1845,7 +1859,7 @@ B200_API int b200_gemm_bf16_gather_a(void* const* shard, long long lds, const in
 // tiles at or past *num_valid_rows are skipped, so M_cap may be a static upper bound).
 // epi 0: C[M_cap, N] = A * B_e^T (optionally scaled per row by row_scale);
 // epi 2: SiLU(gate) * up with the gate / up rows of every expert interleaved in blocks of
-// 32 (C is [M_cap, N / 2]); epi 9: max(x, 0)^2.  N must be a multiple of the tile width (256 for
+// 32 (C is [M_cap, N / 2]); epi 9: max(x, 0)^2; epi 10: GELU (error function).  N must be a multiple of the tile width (256 for
 // epi 2, else 128 or 64).
 B200_API int b200_gemm_bf16_grouped(const void* A, long long lda, const void* B, long long ldb,
                                     void* C, long long ldc, int M_cap, int N, int K, int E,
@@ -1861,8 +1875,8 @@ B200_API int b200_gemm_bf16_grouped(const void* A, long long lda, const void* B,
   if (epi == kEpiSiluMul) {
     if ((N % 256) != 0) return -4;
     bn = 256;
-  } else if (epi == kEpiNone || epi == kEpiRelu2) {
-    bn = epi == kEpiRelu2 && (N % 256) == 0 ? 256 : (N % 128) == 0 ? 128 : 64;
+  } else if (epi == kEpiNone || epi == kEpiRelu2 || epi == kEpiGelu) {
+    bn = epi != kEpiNone && (N % 256) == 0 ? 256 : (N % 128) == 0 ? 128 : 64;
     if ((N % bn) != 0) return -4;
   } else {
     return -7;
@@ -1899,6 +1913,11 @@ B200_API int b200_gemm_bf16_grouped(const void* A, long long lda, const void* B,
     if (bn == 256) return launch<256, 4, kEpiRelu2>(tmA, tmB, a, s);
     if (bn == 128) return launch<128, 6, kEpiRelu2>(tmA, tmB, a, s);
     return launch<64, 8, kEpiRelu2>(tmA, tmB, a, s);
+  }
+  if (epi == kEpiGelu) {
+    if (bn == 256) return launch<256, 4, kEpiGelu>(tmA, tmB, a, s);
+    if (bn == 128) return launch<128, 6, kEpiGelu>(tmA, tmB, a, s);
+    return launch<64, 8, kEpiGelu>(tmA, tmB, a, s);
   }
   if (bn == 128) return launch<128, 6, kEpiNone>(tmA, tmB, a, s);
   return launch<64, 8, kEpiNone>(tmA, tmB, a, s);

@@ -49,7 +49,9 @@ constexpr int BK = 64;
 constexpr int UMMA_K = 16;
 constexpr int kThreads = 192;
 
-enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kRelu2 = 9 };
+enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kRelu2 = 9, kGelu = 10, kGeluMul = 11 };
+template <int EPI>
+constexpr bool kGated = EPI == kSiluMul || EPI == kGeluMul;
 
 struct Args {
   __nv_bfloat16* C;
@@ -318,7 +320,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const uint32_t taddr =
             tmem_base + (static_cast<uint32_t>(q * 32) << 16) +
             static_cast<uint32_t>((mt + b) * BN);
-        if constexpr (EPI == kSiluMul) {
+        if constexpr (kGated<EPI>) {
           __nv_bfloat16* crow = p.C + static_cast<long long>(row) * p.ldc + (n0 >> 1);
 #pragma unroll 1
           for (int c = 0; c < BN / 64; ++c) {
@@ -330,7 +332,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              v[i] = silu_f(__uint_as_float(g[i])) * __uint_as_float(u[i]);
+              v[i] = gated_f<EPI == kGeluMul>(__uint_as_float(g[i]), __uint_as_float(u[i]));
             if (row_ok) {
 #pragma unroll
               for (int i = 0; i < 4; ++i) store8_bf16(crow + c * 32 + i * 8, v + i * 8);
@@ -350,6 +352,10 @@ __global__ void __launch_bounds__(kThreads, 1)
             if constexpr (EPI == kRelu2) {
 #pragma unroll
               for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
+            }
+            if constexpr (EPI == kGelu) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) v[i] = gelu_f(v[i]);
             }
             if constexpr (EPI == kBias) {
 #pragma unroll
@@ -530,7 +536,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const int r0 = static_cast<int>(static_cast<long long>(idx) * rows_used / members);
         const int r1 = static_cast<int>(static_cast<long long>(idx + 1) * rows_used / members);
         const float* base = p.ws + static_cast<long long>(tile) * p.splits * (R * BN);
-        if constexpr (EPI == kSiluMul) {
+        if constexpr (kGated<EPI>) {
           constexpr int kV = 128 / 4;                       // float4 groups of the gate half
           for (int e = te; e < (r1 - r0) * kV; e += 128) {
             const int rw = r0 + e / kV, c4 = (e % kV) * 4;
@@ -546,8 +552,9 @@ __global__ void __launch_bounds__(kThreads, 1)
               u.x += b.x; u.y += b.y; u.z += b.z; u.w += b.w;
             }
             uint2 o;
-            o.x = pack_bf16x2(silu_f(g.x) * u.x, silu_f(g.y) * u.y);
-            o.y = pack_bf16x2(silu_f(g.z) * u.z, silu_f(g.w) * u.w);
+            constexpr bool kG = EPI == kGeluMul;
+            o.x = pack_bf16x2(gated_f<kG>(g.x, u.x), gated_f<kG>(g.y, u.y));
+            o.y = pack_bf16x2(gated_f<kG>(g.z, u.z), gated_f<kG>(g.w, u.w));
             *reinterpret_cast<uint2*>(p.C + static_cast<long long>(m0 + rw) * p.ldc + (n0 >> 1) +
                                       c4) = o;
           }
@@ -711,7 +718,9 @@ B200_API int b200_gemm_pair(const void* A, long long lda, const void* B, long lo
   using namespace b200;
   using namespace b200::pair;
   if (M <= 0 || N <= 0) return 0;
-  if ((N % 256) != 0 || (K % BK) != 0 || K <= 0 || (epi != kRelu2 && (epi < 0 || epi > 2))) return -20;
+  if ((N % 256) != 0 || (K % BK) != 0 || K <= 0 ||
+      (epi < kRelu2 && (epi < 0 || epi > 2)) || epi > kGeluMul)
+    return -20;
   if ((lda % 8) != 0 || (ldb % 8) != 0 || (ldc % 8) != 0) return -2;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B) |
        reinterpret_cast<uintptr_t>(C)) & 15)
@@ -731,7 +740,8 @@ B200_API int b200_gemm_pair(const void* A, long long lda, const void* B, long lo
   a.ldc = ldc;
   a.bias = static_cast<const __nv_bfloat16*>(bias);
   a.M = M; a.N = N; a.K = K;
-  const int mt = getenv("VLLM_B200_PAIR_MT") != nullptr && atoi(getenv("VLLM_B200_PAIR_MT")) == 2
+  const int mt = epi < kGelu && getenv("VLLM_B200_PAIR_MT") != nullptr &&
+                         atoi(getenv("VLLM_B200_PAIR_MT")) == 2
                      ? 2 : 1;
   a.tiles_m = (M + 256 * mt - 1) / (256 * mt);
   a.tiles_n = N / 256;
@@ -750,6 +760,8 @@ B200_API int b200_gemm_pair(const void* A, long long lda, const void* B, long lo
     if (epi == kSiluMul) return launch<kSiluMul, 1>(tmA, tmB, a, s);
     if (epi == kBias) return launch<kBias, 1>(tmA, tmB, a, s);
     if (epi == kRelu2) return launch<kRelu2, 1>(tmA, tmB, a, s);
+    if (epi == kGelu) return launch<kGelu, 1>(tmA, tmB, a, s);
+    if (epi == kGeluMul) return launch<kGeluMul, 1>(tmA, tmB, a, s);
     return launch<kNone, 1>(tmA, tmB, a, s);
   }
   if (epi == kSiluMul) return launch<kSiluMul, 2>(tmA, tmB, a, s);
@@ -778,7 +790,8 @@ B200_API int b200_gemm_pair_split(const void* A, long long lda, const void* B, l
   using namespace b200;
   using namespace b200::pair;
   if (M <= 0 || N <= 0) return 0;
-  if ((N % 256) != 0 || (K % BK) != 0 || K <= 0 || epi < 0 || epi > 2 || M > 512 ||
+  if ((N % 256) != 0 || (K % BK) != 0 || K <= 0 || epi < 0 ||
+      (epi > 2 && epi != kGeluMul) || M > 512 ||
       ws == nullptr || ctr == nullptr)
     return -20;
   if ((lda % 8) != 0 || (ldb % 8) != 0 || (ldc % 8) != 0) return -2;
@@ -818,6 +831,7 @@ B200_API int b200_gemm_pair_split(const void* A, long long lda, const void* B, l
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int units = tiles * splits;
   if (epi == kSiluMul) return launch_split<kSiluMul>(tmA, tmB, a, units, s);
+  if (epi == kGeluMul) return launch_split<kGeluMul>(tmA, tmB, a, units, s);
   if (epi == kBias) return launch_split<kBias>(tmA, tmB, a, units, s);
   return launch_split<kNone>(tmA, tmB, a, units, s);
 }

@@ -35,7 +35,8 @@ constexpr int BK = 64;
 constexpr int UMMA_K = 16;
 constexpr int kThreads = 192;
 
-enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kFp32 = 4, kRelu2 = 9 };
+enum Epi : int { kNone = 0, kBias = 1, kSiluMul = 2, kFp32 = 4, kRelu2 = 9, kGelu = 10, kGeluMul = 11 };
+__host__ __device__ constexpr bool gated(int epi) { return epi == kSiluMul || epi == kGeluMul; }
 
 struct Args {
   __nv_bfloat16* C;
@@ -75,7 +76,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   constexpr uint32_t kAccCols = MT * BN;
   constexpr uint32_t kTmemCols = kAccCols <= 32 ? 32 : (kAccCols <= 64 ? 64 : (kAccCols <= 128 ? 128 : (kAccCols <= 256 ? 256 : 512)));
   constexpr uint32_t kIdesc = make_idesc(BM, BN, 1, 1);
-  static_assert(EPI != kSiluMul || BN == 256, "SiLU-mul epilogue needs BN = 256");
+  static_assert(!gated(EPI) || BN == 256, "gated epilogues need BN = 256");
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>(
@@ -183,7 +184,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const bool row_ok = row < p.M;
         const uint32_t taddr =
             tmem_base + (static_cast<uint32_t>(q * 32) << 16) + static_cast<uint32_t>(mt * BN);
-        if constexpr (EPI == kSiluMul) {
+        if constexpr (gated(EPI)) {
           __nv_bfloat16* crow = p.C + static_cast<long long>(row) * p.ldc + (n0 >> 1);
           const int out_n = p.N >> 1;
 #pragma unroll 1
@@ -196,7 +197,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              v[i] = silu_f(__uint_as_float(g[i])) * __uint_as_float(u[i]);
+              v[i] = gated_f<EPI == kGeluMul>(__uint_as_float(g[i]), __uint_as_float(u[i]));
             if (row_ok && (n0 >> 1) + c * 32 < out_n) {
 #pragma unroll
               for (int i = 0; i < 4; ++i) store8_bf16(crow + c * 32 + i * 8, v + i * 8);
@@ -216,6 +217,10 @@ __global__ void __launch_bounds__(kThreads, 1)
             if constexpr (EPI == kRelu2) {
 #pragma unroll
               for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
+            }
+            if constexpr (EPI == kGelu) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) v[i] = gelu_f(v[i]);
             }
             __nv_bfloat16* crow = p.C + static_cast<long long>(row) * p.ldc + col;
             if (col + 32 <= p.N) {
@@ -283,7 +288,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const int r0 = static_cast<int>(static_cast<long long>(split) * rows_used / p.splits);
         const int r1 = static_cast<int>(static_cast<long long>(split + 1) * rows_used / p.splits);
         const float* base = p.ws + static_cast<long long>(tile) * p.splits * (R * BN);
-        if constexpr (EPI == kSiluMul) {
+        if constexpr (gated(EPI)) {
           constexpr int kV = 128 / 4;   // float4 groups of the gate half
           const int out_n = p.N >> 1;
           for (int e = te; e < (r1 - r0) * kV; e += 128) {
@@ -302,8 +307,9 @@ __global__ void __launch_bounds__(kThreads, 1)
             const int col = (n0 >> 1) + c4;
             if (col < out_n) {
               uint2 o;
-              o.x = pack_bf16x2(silu_f(g.x) * u.x, silu_f(g.y) * u.y);
-              o.y = pack_bf16x2(silu_f(g.z) * u.z, silu_f(g.w) * u.w);
+              constexpr bool kG = EPI == kGeluMul;
+              o.x = pack_bf16x2(gated_f<kG>(g.x, u.x), gated_f<kG>(g.y, u.y));
+              o.y = pack_bf16x2(gated_f<kG>(g.z, u.z), gated_f<kG>(g.w, u.w));
               *reinterpret_cast<uint2*>(p.C + static_cast<long long>(row) * p.ldc + col) = o;
             }
           }
@@ -322,6 +328,10 @@ __global__ void __launch_bounds__(kThreads, 1)
             if constexpr (EPI == kRelu2) {
               acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y);
               acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w);
+            }
+            if constexpr (EPI == kGelu) {
+              acc.x = gelu_f(acc.x); acc.y = gelu_f(acc.y);
+              acc.z = gelu_f(acc.z); acc.w = gelu_f(acc.w);
             }
             if constexpr (EPI == kBias) {
               acc.x += __bfloat162float(p.bias[col]);
@@ -527,7 +537,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const bool row_ok = row < p.M;
         const uint32_t taddr =
             tmem_base + (static_cast<uint32_t>(q * 32) << 16) + static_cast<uint32_t>(mt * BN);
-        if constexpr (EPI == kSiluMul) {
+        if constexpr (gated(EPI)) {
           __nv_bfloat16* crow = p.C + static_cast<long long>(row) * p.ldc + (n0 >> 1);
           const int out_n = p.N >> 1;
 #pragma unroll 1
@@ -540,7 +550,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              v[i] = silu_f(__uint_as_float(g[i])) * __uint_as_float(u[i]);
+              v[i] = gated_f<EPI == kGeluMul>(__uint_as_float(g[i]), __uint_as_float(u[i]));
             if (row_ok && (n0 >> 1) + c * 32 < out_n) {
 #pragma unroll
               for (int i = 0; i < 4; ++i) store8_bf16(crow + c * 32 + i * 8, v + i * 8);
@@ -609,7 +619,7 @@ struct Plan {
 // a column tile lie one after the other, [tile][slice][R x bn]; fixed summation order.
 __global__ void __launch_bounds__(256)
     skinny_reduce_kernel(const float* ws, __nv_bfloat16* C, float* C32, long long ldc,
-                         const __nv_bfloat16* bias, int relu2, int M, int N, int bn, int R,
+                         const __nv_bfloat16* bias, int epi, int M, int N, int bn, int R,
                          int splits) {
   const long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   const int n4 = N >> 2;
@@ -629,9 +639,12 @@ __global__ void __launch_bounds__(256)
     acc.z += __bfloat162float(bias[col + 2]);
     acc.w += __bfloat162float(bias[col + 3]);
   }
-  if (relu2) {
+  if (epi == kRelu2) {
     acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y);
     acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w);
+  } else if (epi == kGelu) {
+    acc.x = gelu_f(acc.x); acc.y = gelu_f(acc.y);
+    acc.z = gelu_f(acc.z); acc.w = gelu_f(acc.w);
   }
   if (C32 != nullptr) {
     *reinterpret_cast<float4*>(C32 + static_cast<long long>(row) * ldc + col) = acc;
@@ -656,11 +669,11 @@ inline Plan make_plan2(int M, int N, int K, int epi, int sms) {
   const int cands[3] = {256, 128, 64};
   for (int ci = 0; ci < 3; ++ci) {
     const int bn = cands[ci];
-    if (epi == kSiluMul && bn != 256) continue;
+    if (gated(epi) && bn != 256) continue;
     if (N % bn != 0 && (epi != kFp32 || bn > 128)) continue;   // narrow fp32 results: a partial tile
     const int tiles = (N + bn - 1) / bn;
     for (int sl = 1; sl <= 16; ++sl) {
-      if (sl > 1 && (epi == kSiluMul || tiles * sl > sms || num_kb / sl < 8)) break;
+      if (sl > 1 && (gated(epi) || tiles * sl > sms || num_kb / sl < 8)) break;
       const double units = static_cast<double>(tiles) * sl;
       const double waves = units <= sms ? 1.0 : units / sms;
       const double unit_bytes = (mt * 128.0 + bn) * (static_cast<double>(K) / sl) * 2.0;
@@ -684,7 +697,7 @@ inline Plan make_plan(int M, int N, int K, int epi, int sms) {
   const int cands[3] = {256, 128, 64};
   for (int ci = 0; ci < 3; ++ci) {
     const int bn = cands[ci];
-    if (epi == kSiluMul && bn != 256) continue;
+    if (gated(epi) && bn != 256) continue;
     if (bn > 64 && N < bn) continue;
     const int tiles = (N + bn - 1) / bn;
     for (int s = 1; s <= 16; ++s) {
@@ -716,7 +729,7 @@ B200_API int b200_gemm_skinny_workspace(int N, long long* ws_bytes, int* ctr_wor
 }
 
 // C[M,N] (bf16) = A[M,K] * B[N,K]^T for M <= 256 with epilogue epi: 0 none, 1 + bias[N],
-// 2 SiLU(gate)*up (B rows interleaved gate/up in blocks of 32; C is [M, N/2]), 9 max(x, 0)^2; 4: C
+// 2 SiLU(gate)*up (B rows interleaved gate/up in blocks of 32; C is [M, N/2]), 9 max(x, 0)^2, 10 GELU, 11 GELU(gate)*up; 4: C
 // is fp32, only where a two-kernel K split (allow_split = 2) pays.
 // Row pitches in elements; K, lda, ldb, N, ldc multiples of 8; 16-byte aligned pointers.
 // ws / ctr: see b200_gemm_skinny_workspace (ctr must be zero before the first call; the kernel
@@ -737,9 +750,9 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B) |
        reinterpret_cast<uintptr_t>(C)) & 15)
     return -3;
-  if (epi == kSiluMul && (N % 256) != 0) return -4;
+  if (gated(epi) && (N % 256) != 0) return -4;
   if (epi == kBias && bias == nullptr) return -5;
-  if (epi != kRelu2 && epi != kFp32 && (epi < 0 || epi > 2)) return -20;
+  if (epi != kFp32 && (epi < kRelu2 || epi > kGeluMul) && (epi < 0 || epi > 2)) return -20;
   const int sms = sm_count();
   Plan pl = allow_split == 2 ? make_plan2(M, N, K, epi, sms) : make_plan(M, N, K, epi, sms);
   if (epi == kFp32 && (allow_split != 2 || pl.splits == 1)) return -20;
@@ -794,11 +807,20 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
                ? launch<BN_, MT_, ST_, kNone>(tmA, tmB, a, units, s)                \
                : launch<BN_, MT_, ST_, kRelu2>(tmA, tmB, a, units, s);              \
       break;                                                                        \
+    case kGelu:                                                                     \
+      rc = a.splits > 1 && a.ctr == nullptr                                         \
+               ? launch<BN_, MT_, ST_, kNone>(tmA, tmB, a, units, s)                \
+               : launch<BN_, MT_, ST_, kGelu>(tmA, tmB, a, units, s);               \
+      break;                                                                        \
     default: break;                                                                 \
   }
   if (epi == kSiluMul) {
     if (mt == 2) return launch<256, 2, 3, kSiluMul>(tmA, tmB, a, units, s);
     return launch<256, 1, 4, kSiluMul>(tmA, tmB, a, units, s);
+  }
+  if (epi == kGeluMul) {
+    if (mt == 2) return launch<256, 2, 3, kGeluMul>(tmA, tmB, a, units, s);
+    return launch<256, 1, 4, kGeluMul>(tmA, tmB, a, units, s);
   }
   if (pl.bn == 256) {
     if (mt == 2) { B200_SK(256, 2, 3) } else { B200_SK(256, 1, 4) }
@@ -813,7 +835,7 @@ B200_API int b200_gemm_skinny(const void* A, long long lda, const void* B, long 
   const long long work = static_cast<long long>(M) * (N / 4);
   skinny_reduce_kernel<<<static_cast<unsigned>((work + 255) / 256), 256, 0, s>>>(
       a.ws, a.C, epi == kFp32 ? static_cast<float*>(C) : nullptr, a.ldc,
-      epi == kBias ? a.bias : nullptr, epi == kRelu2, M, N, pl.bn, mt * BM, a.splits);
+      epi == kBias ? a.bias : nullptr, epi, M, N, pl.bn, mt * BM, a.splits);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -835,7 +857,7 @@ B200_API int b200_gemm_wide2(const void* A, long long lda, const void* B, long l
   using namespace b200;
   using namespace b200::skinny;
   if (M <= 0 || N <= 0) return 0;
-  if ((N % 256) != 0 || M < 512 || epi < 0 || epi > 2) return -20;
+  if ((N % 256) != 0 || M < 512 || epi < 0 || (epi > 2 && epi != kGeluMul)) return -20;
   if (K <= 0 || (K % 8) != 0 || (lda % 8) != 0 || (ldb % 8) != 0 || (ldc % 8) != 0) return -2;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B) |
        reinterpret_cast<uintptr_t>(C)) & 15)
@@ -868,6 +890,7 @@ B200_API int b200_gemm_wide2(const void* A, long long lda, const void* B, long l
   }
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (epi == kSiluMul) return launch_wide2<kSiluMul>(tmA, tmB, a, s);
+  if (epi == kGeluMul) return launch_wide2<kGeluMul>(tmA, tmB, a, s);
   if (epi == kBias) return launch_wide2<kBias>(tmA, tmB, a, s);
   return launch_wide2<kNone>(tmA, tmB, a, s);
 }

@@ -370,13 +370,16 @@ __global__ void __launch_bounds__(256)
     h[static_cast<long long>(r) * I + c] = g[c] / (1.0f + expf(-g[c])) * g[I + c];
 }
 
-// h[r, i] = max(u[r, i], 0)^2 of the rows in use (may be in place)
+// h[r, i] = max(u[r, i], 0)^2 or GELU of the rows in use (may be in place)
+template <bool GELU>
 __global__ void __launch_bounds__(256)
-    relu2_rows_f32_kernel(const float* u, float* h, int I, const int* num_valid_rows) {
+    ungated_rows_f32_kernel(const float* u, float* h, int I, const int* num_valid_rows) {
   const int r = blockIdx.x;
   if (r >= *num_valid_rows) return;
-  for (int c = threadIdx.x; c < I; c += blockDim.x)
-    h[static_cast<long long>(r) * I + c] = relu2_f(u[static_cast<long long>(r) * I + c]);
+  for (int c = threadIdx.x; c < I; c += blockDim.x) {
+    const float x = u[static_cast<long long>(r) * I + c];
+    h[static_cast<long long>(r) * I + c] = GELU ? gelu_f(x) : relu2_f(x);
+  }
 }
 
 // out[t] = (add ? add[t] : 0) + alpha * sum_s y[pos_of[t * k + s]]   (fp32 accumulation)
@@ -582,11 +585,14 @@ B200_API int b200_silu_mul_rows_f32(const float* u, float* h, int rows, int I,
   return static_cast<int>(cudaGetLastError());
 }
 
-B200_API int b200_relu2_rows_f32(const float* u, float* h, int rows, int I,
-                                 const int* num_valid_rows, void* stream) {
+// act 9: max(x, 0)^2, 10: GELU
+B200_API int b200_ungated_rows_f32(const float* u, float* h, int rows, int I,
+                                   const int* num_valid_rows, int act, void* stream) {
   if (rows <= 0 || I <= 0) return 0;
-  relu2_rows_f32_kernel<<<rows, 256, 0, static_cast<cudaStream_t>(stream)>>>(u, h, I,
-                                                                          num_valid_rows);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (act == 9) ungated_rows_f32_kernel<false><<<rows, 256, 0, s>>>(u, h, I, num_valid_rows);
+  else if (act == 10) ungated_rows_f32_kernel<true><<<rows, 256, 0, s>>>(u, h, I, num_valid_rows);
+  else return -2;
   return static_cast<int>(cudaGetLastError());
 }
 

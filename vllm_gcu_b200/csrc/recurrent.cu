@@ -1,10 +1,13 @@
 // Linear recurrences with a matrix state per head (sm_100a): gated delta rule with one decay per
-// key channel, and the matrix memory with exponential gates (mLSTM).
+// key channel, the matrix memory with exponential gates (mLSTM), and time mixing of the RWKV kind
+// (one decay per key channel, a bonus for the current token):
+//   o_t = S^T r_t + (r_t . (u k_t)) v_t,  then  S = diag(w_t) S + k_t v_t^T
 //
 //   delta_inputs    short causal convolution + SiLU of q, k, v, unit vectors, decays, step sizes
 //   memory_inputs   q (scaled), k, v in fp32, log gates of the matrix memory
+//   wkv_inputs      r, k, v in fp32, decays and the bonus' products r . (u k)
 //   recurrent_scan  the recurrence over portions of prompts
-//   head_norm_gate  o / rms(o) per head, times the norm weight, a sigmoid gate and a factor
+//   head_norm_gate  o / rms(o) per head, times the norm weight, a sigmoid or SiLU gate and a factor
 //   recurrent_step  all of these (and the narrow projections in front of them) for requests that
 //                   bring a single token: one CTA per request and head
 //
@@ -29,7 +32,7 @@
 namespace b200 {
 namespace recurrent {
 
-constexpr int kDelta = 0, kMemory = 1;
+constexpr int kDelta = 0, kMemory = 1, kWkv = 2;
 
 // fp32 pairs: two multiply-adds per instruction
 struct __align__(16) Quad {
@@ -391,13 +394,72 @@ __global__ void __launch_bounds__(256) memory_inputs_kernel(const MemoryIn a) {
 }
 
 // ---------------------------------------------------------------------------
+struct WkvIn {
+  const void *r, *k, *v;     // [T, N * D] views, row pitch ld
+  const float* z;            // [T, N * D] decay projection
+  const float *base, *bonus; // [N * D]
+  float *ro, *ko, *go;       // out: [T, N, DP]
+  float* vo;                 // out: [T, N, VP]
+  float* now;                // out: [T, N] r . (bonus k)
+  long long ld, ldz;
+  int T, N, D, DP, VP;
+};
+
+// LPH lanes per token and head, W neighbouring channels each.
+template <typename T, int W, int LPH>
+__global__ void __launch_bounds__(256) wkv_inputs_kernel(const WkvIn a) {
+  const long long job = (blockIdx.x * 256ll + threadIdx.x) / LPH;
+  if (job >= static_cast<long long>(a.T) * a.N) return;      // (whole groups of lanes leave)
+  const int l = threadIdx.x & (LPH - 1);
+  const long long t = job / a.N;
+  const int h = static_cast<int>(job - t * a.N), at = h * a.D;
+  const long long row = t * a.ld + at;
+  float sum = 0.0f;
+  for (int d = l * W; d < a.DP; d += LPH * W) {
+    float r[W], k[W], v[W], g[W];
+#pragma unroll
+    for (int i = 0; i < W; ++i) r[i] = k[i] = v[i] = g[i] = 0.0f;
+    if (d < a.D) {
+      float b[W], u[W];
+      load_n<T, W>(static_cast<const T*>(a.r) + row + d, r);
+      load_n<T, W>(static_cast<const T*>(a.k) + row + d, k);
+      load_n<T, W>(static_cast<const T*>(a.v) + row + d, v);
+      load_n<float, W>(a.z + t * a.ldz + at + d, g);
+      load_n<float, W>(a.base + at + d, b);
+      load_n<float, W>(a.bonus + at + d, u);
+#pragma unroll
+      for (int i = 0; i < W; ++i) {
+        g[i] = exp_t<T>(-exp_t<T>(g[i] + b[i]));
+        sum += r[i] * u[i] * k[i];
+      }
+    }
+    store_n<W>(a.ro + job * a.DP + d, r);
+    store_n<W>(a.ko + job * a.DP + d, k);
+    store_n<W>(a.go + job * a.DP + d, g);
+    if (d < a.VP) store_n<W>(a.vo + job * a.VP + d, v);
+  }
+  const unsigned int mask = LPH == 32 ? 0xffffffffu
+                                      : ((1u << (LPH & 31)) - 1u) << (threadIdx.x & (32 - LPH));
+#pragma unroll
+  for (int o = 1; o < LPH; o <<= 1) sum += __shfl_xor_sync(mask, sum, o);
+  if (l == 0) a.now[job] = sum;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_rows_kernel(const float* x, T* out, long long n) {
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i < n) out[i] = from_f32<T>(tanhf(x[i]));
+}
+
+// ---------------------------------------------------------------------------
 constexpr int kChunk = 16;       // tokens staged at a time
 
 struct ScanArgs {
   const float *q, *k;        // [T, G, DP]
-  const float* g;            // delta: decays [T, N, DP]
+  const float* g;            // delta, wkv: decays [T, N, DP]
   const float* v;            // [T, N, VP]
-  const float *s0, *s1;      // delta: step sizes | memory: log input gate, log forget gate [T, N]
+  const float *s0, *s1;      // delta: step sizes | memory: log input gate, log forget gate |
+                             // wkv: products of the bonus [T, N]
   float* out;                // [T, N, V] (memory: not yet divided)
   float *nq, *low;           // memory: [T, N] normaliser . q, exp(-m)
   const float* m0;           // memory: [requests, N] m in front of the portion
@@ -438,13 +500,13 @@ __device__ void keep_taps(const ScanArgs& a, const Portion& po, int slot, int h)
 
 template <int MODE, int DP>
 __host__ __device__ constexpr int stage_floats(int cols) {
-  return kChunk * ((MODE == kDelta ? 3 : 2) * DP + cols + 4);
+  return kChunk * ((MODE == kMemory ? 2 : 3) * DP + cols + 4);
 }
 
 template <int MODE, int LPC, int RPL, int CPT>
 __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
   constexpr int DP = LPC * RPL, P = RPL / 2;     // P: row pairs per lane
-  constexpr int kRows = MODE == kDelta ? 3 : 2;  // staged rows of DP floats per token
+  constexpr int kRows = MODE == kMemory ? 2 : 3; // staged rows of DP floats per token
   constexpr int kGroups = 32 / LPC;              // columns groups of a warp
   extern __shared__ float4 smem4[];
   float* smem = reinterpret_cast<float*>(smem4);
@@ -482,7 +544,7 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
   const long long v_step = static_cast<long long>(a.N) * a.VP;
   const float* q_src = a.q + po.first * qk_step + kvh * DP + lane * 4;
   const float* k_src = a.k + po.first * qk_step + kvh * DP + lane * 4;
-  const float* g_src = MODE == kDelta ? a.g + po.first * g_step + h * DP + lane * 4 : nullptr;
+  const float* g_src = MODE != kMemory ? a.g + po.first * g_step + h * DP + lane * 4 : nullptr;
   const float* v_src = a.v + po.first * v_step + static_cast<long long>(h) * a.VP + z * a.cols + lane * 4;
   auto fetch = [&](int i0, int b) {
     const int n = min(kChunk, po.count - i0);
@@ -496,7 +558,7 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
         if (kVec % 32 != 0 && lane + c >= kVec) break;
         copy16(dst + i * DP + c * 4, q_src + t * qk_step + c * 4);
         copy16(dst + (kChunk + i) * DP + c * 4, k_src + t * qk_step + c * 4);
-        if (MODE == kDelta) copy16(dst + (2 * kChunk + i) * DP + c * 4, g_src + t * g_step + c * 4);
+        if (MODE != kMemory) copy16(dst + (2 * kChunk + i) * DP + c * 4, g_src + t * g_step + c * 4);
       }
       float* dv = dst + kRows * kChunk * DP + i * a.cols;
       for (int c = lane * 4; c < a.cols; c += 128) {
@@ -545,7 +607,7 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
     const int n = min(kChunk, po.count - i0);
     const float* sq = smem + b * stage + 4 * l;
     const float* sk = sq + kChunk * DP;
-    const float* sg = sk + kChunk * DP;                         // delta only
+    const float* sg = sk + kChunk * DP;                         // not memory
     const float* sv = smem + b * stage + kRows * kChunk * DP;
     const float* ss = sv + kChunk * a.cols;
 
@@ -653,6 +715,32 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
 #pragma unroll
           for (int u = 0; u < P; ++u) S[j][u] = fma2(kk[u], u2, S[j][u]);
         }
+      } else if (MODE == kWkv) {
+        // the read-out is of the state before this token; only it needs the reduction, the state's
+        // own chain is one multiply-add per token
+#pragma unroll
+        for (int u = 0; u < P / 2; ++u) {
+          const Quad g = *reinterpret_cast<const Quad*>(sg + i * DP + 4 * LPC * u);
+          const Quad q = *reinterpret_cast<const Quad*>(sq + i * DP + 4 * LPC * u);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            e0[j] = fma2(S[j][2 * u], q.x, e0[j]);
+            e1[j] = fma2(S[j][2 * u + 1], q.y, e1[j]);
+            const float2 v2 = both(v[j]);
+            S[j][2 * u] = fma2(kk[2 * u], v2, mul2(S[j][2 * u], g.x));
+            S[j][2 * u + 1] = fma2(kk[2 * u + 1], v2, mul2(S[j][2 * u + 1], g.y));
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) o[j] = halves_sum(e0[j]) + halves_sum(e1[j]);
+#pragma unroll
+        for (int w = 1; w < LPC; w <<= 1) {
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) o[j] += __shfl_xor_sync(0xffffffffu, o[j], w);
+        }
+        const float now = ss[i];
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) o[j] += now * v[j];
       } else {
         const float2 a2 = both(__shfl_sync(0xffffffffu, keep, i));
         const float b1 = __shfl_sync(0xffffffffu, add, i);
@@ -704,7 +792,7 @@ __global__ void __launch_bounds__(128) recurrent_scan_kernel(const ScanArgs a) {
   }
   if (MODE == kMemory) {
     if (z == 0 && threadIdx.x == 0) a.scalar[head_at] = m;
-  } else if (z == 0 && a.ntaps > 1) {
+  } else if (MODE == kDelta && z == 0 && a.ntaps > 1) {
     if (a.elt == 2) keep_taps<uint16_t>(a, po, slot, h);
     else keep_taps<uint32_t>(a, po, slot, h);
   }
@@ -767,7 +855,7 @@ struct HeadNormArgs {
   const void* z;             // [T, N * V] gate projection, row pitch ldz
   void* out;                 // [T, N * V], row pitch ldo
   long long ldz, ldo;
-  int T, N, V, per_head;
+  int T, N, V, per_head, silu;
   float eps, scale;
 };
 
@@ -822,7 +910,7 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormArgs 
     float b[W];
     load_n<float, W>(w + c, b);
 #pragma unroll
-    for (int j = 0; j < W; ++j) x[j] = x[j] * inv * b[j] * sigmoid_t<T>(gate[j]);
+    for (int j = 0; j < W; ++j) x[j] = x[j] * inv * b[j] * (a.silu ? silu<T>(gate[j]) : sigmoid_t<T>(gate[j]));
     store_t<T, W>(out + c, x);
   };
 #pragma unroll
@@ -846,8 +934,10 @@ struct StepArgs {
   const void* x[3];          // q, k, v projections, row pitch ld
   const void* gate;          // [nd, N V] output gate projection, row pitch ldg
   const float* z;            // delta: decay projection [nd, N D], row pitch ldz
+                             // wkv: inner row of the decay's projection [nd, H]
   const void *w0, *w1;       // rows [N, H]: delta step size, - ; memory input gate, forget gate
-  const float *b0, *b1;      // memory: their biases [N]
+                             // wkv: second step of the decay's projection [N D, H], -
+  const float *b0, *b1;      // memory: their biases [N]; wkv: decay base, bonus [N D]
   const float* taps_w[3];    // delta: convolution weights
   const float *dt_bias, *a_log;
   const float* norm;         // [V], or [N V] with per_head
@@ -892,8 +982,9 @@ __device__ __forceinline__ float dot_share(const T* x, const T* w, int n, bool v
   return s;
 }
 
-__host__ __device__ inline int step_floats(int DP, int V) {
-  return 3 * DP + 3 * ((V + 3) / 4 * 4) + 64;
+// inner: wkv's decay rank
+__host__ __device__ inline int step_floats(int DP, int V, int inner) {
+  return 3 * DP + 3 * ((V + 3) / 4 * 4) + 64 + inner;
 }
 
 template <typename T, int MODE, int RPL, int CPT>
@@ -941,19 +1032,24 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
   };
   load_state(0);                                  // in flight while the inputs are computed
 
-  const T* hr = static_cast<const T*>(a.hrow) + static_cast<long long>(r) * a.ldh;
+  const T* hr = MODE == kWkv ? nullptr
+                             : static_cast<const T*>(a.hrow) + static_cast<long long>(r) * a.ldh;
   const bool vec = (a.H % 8) == 0 && ((reinterpret_cast<uintptr_t>(hr) |
                                        reinterpret_cast<uintptr_t>(a.w0) |
                                        reinterpret_cast<uintptr_t>(a.w1)) & 15) == 0;
   const long long xrow = static_cast<long long>(r) * a.ld;
-  const float d0 = dot_share<T>(hr, static_cast<const T*>(a.w0) + static_cast<long long>(h) * a.H,
-                                a.H, vec);
+  float d0 = 0.0f;
+  if (MODE != kWkv)
+    d0 = dot_share<T>(hr, static_cast<const T*>(a.w0) + static_cast<long long>(h) * a.H, a.H, vec);
   float d1 = 0.0f;
   if (MODE == kMemory)
     d1 = dot_share<T>(hr, static_cast<const T*>(a.w1) + static_cast<long long>(h) * a.H, a.H, vec);
 
   const T* gz = static_cast<const T*>(a.gate) + static_cast<long long>(r) * a.ldg + h * a.V;
-  for (int c = tid; c < a.V; c += blockDim.x) sz[c] = sigmoid_t<T>(to_f32<T>(gz[c]));
+  for (int c = tid; c < a.V; c += blockDim.x) {
+    const float g = to_f32<T>(gz[c]);
+    sz[c] = MODE == kWkv ? silu<T>(g) : sigmoid_t<T>(g);
+  }
   if (MODE == kDelta) {
     const int C = 2 * a.G * a.D + a.N * a.V;
     const T* ring = static_cast<const T*>(a.taps) + static_cast<long long>(slot) * a.ntaps * C;
@@ -989,10 +1085,14 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
     for (int c = tid; c < a.V; c += blockDim.x)
       sv[c] = to_f32<T>(static_cast<const T*>(a.x[2])[xrow + h * a.V + c]);
   }
+  if (MODE == kWkv) {                             // inner row of the decay's projection
+    float* st = red + 64;
+    for (int c = tid; c < a.H; c += blockDim.x) st[c] = tanhf(a.z[r * a.ldz + c]);
+  }
   const float z0 = block_sum(d0, red);            // (synchronises: the shared rows are complete)
   const float z1 = MODE == kMemory ? block_sum(d1, red) : 0.0f;
 
-  float beta = 0.0f, keep = 0.0f, add = 0.0f, den = 1.0f;
+  float beta = 0.0f, keep = 0.0f, add = 0.0f, den = 1.0f, now = 0.0f;
   if (MODE == kDelta) {
     beta = sigmoid(z0);
     if (warp < 2) {                               // unit vectors
@@ -1015,6 +1115,29 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
       }
     }
     __syncthreads();
+  } else if (MODE == kWkv) {
+    const float* st = red + 64;
+    float part = 0.0f;
+    for (int d = tid; d < a.D; d += blockDim.x) part += sq[d] * sk[d] * a.b1[h * a.D + d];
+    // decays: four threads a channel, 8 inner columns at a time
+    for (int base = 0; base < DP; base += 64) {
+      const int d = base + (tid >> 2);
+      float s = 0.0f;
+      if (d < a.D) {
+        const T* w = static_cast<const T*>(a.w0) + (static_cast<long long>(h) * a.D + d) * a.H;
+        for (int c = (tid & 3) * 8; c < a.H; c += 32) {
+          float f[8];
+          load8<T>(w + c, f);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) s += f[i] * st[c + i];
+        }
+      }
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      if ((tid & 3) == 0 && d < DP)
+        sg[d] = d < a.D ? exp_t<T>(-exp_t<T>(s + a.b0[h * a.D + d])) : 0.0f;
+    }
+    now = block_sum(part, red);                   // (synchronises: the decays are complete)
   } else {
     const float li = soft_cap(z0 + a.b0[h], a.cap);
     const float lf = -softplus(-soft_cap(z1 + a.b1[h], a.cap));
@@ -1064,11 +1187,21 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
     }
 #pragma unroll
     for (int j = 0; j < CPT; ++j) {
-      const float2 u2 = both(MODE == kDelta ? beta * (v[j] - d[j]) : add * v[j]);
+      const float2 u2 = both(MODE == kDelta ? beta * (v[j] - d[j]) : MODE == kWkv ? v[j] : add * v[j]);
       const float2 a2 = both(keep);
       float2 e0 = both(0.0f), e1 = both(0.0f);
 #pragma unroll
       for (int u = 0; u < P / 2; ++u) {
+        if (MODE == kWkv) {                       // the read-out is of the state before this token
+          const Quad g = *reinterpret_cast<const Quad*>(sg + 4 * l + 32 * u);
+          const Quad k = *reinterpret_cast<const Quad*>(sk + 4 * l + 32 * u);
+          const Quad q = *reinterpret_cast<const Quad*>(sq + 4 * l + 32 * u);
+          e0 = fma2(S[j][2 * u], q.x, e0);
+          e1 = fma2(S[j][2 * u + 1], q.y, e1);
+          S[j][2 * u] = fma2(k.x, u2, mul2(S[j][2 * u], g.x));
+          S[j][2 * u + 1] = fma2(k.y, u2, mul2(S[j][2 * u + 1], g.y));
+          continue;
+        }
         const Quad k = *reinterpret_cast<const Quad*>(sk + 4 * l + 32 * u);
         const Quad q = *reinterpret_cast<const Quad*>(sq + 4 * l + 32 * u);
         if (MODE == kMemory) {
@@ -1098,7 +1231,7 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
 #pragma unroll
       for (int j = 0; j < CPT; ++j) {
         if (c0 + j >= a.V) continue;
-        o[j] *= den;
+        o[j] = o[j] * den + now * v[j];
         so[c0 + j] = o[j];
         ss += o[j] * o[j];
       }
@@ -1113,7 +1246,7 @@ __global__ void __launch_bounds__(256, RPL < 32 ? 2 : 1) recurrent_step_kernel(c
 
 template <typename T, int MODE, int RPL, int CPT>
 static int launch_step(const StepArgs& a, int requests, cudaStream_t s) {
-  const int smem = step_floats(8 * RPL, a.V) * static_cast<int>(sizeof(float));
+  const int smem = step_floats(8 * RPL, a.V, MODE == kWkv ? a.H : 0) * static_cast<int>(sizeof(float));
   if (smem > 48 * 1024) return -20;
   recurrent_step_kernel<T, MODE, RPL, CPT><<<dim3(requests, a.N), 256, smem, s>>>(a);
   return static_cast<int>(cudaGetLastError());
@@ -1262,16 +1395,17 @@ B200_API int b200_memory_scan(const float* q, const float* k, const float* v, co
   return dispatch_scan<kMemory>(a, DP, nd + np, static_cast<cudaStream_t>(stream));
 }
 
-// out = o' / rms(o') per head * w * sigmoid(z) * scale with o' = o, or with nq and low
-// o / (max(|nq|, low) + 1e-6).  per_head: w is [N * V], else [V].  dtype (of z and out): 0 bf16,
+// out = o' / rms(o') per head * w * sigmoid(z) (silu 1: SiLU(z)) * scale with o' = o, or with nq and
+// low o / (max(|nq|, low) + 1e-6).  per_head: w is [N * V], else [V].  dtype (of z and out): 0 bf16,
 // 2 fp32.
 B200_API int b200_head_norm_gate(const float* o, const float* nq, const float* low, const float* w,
                                  int per_head, const void* z, long long ldz, void* out,
                                  long long ldo, float eps, float scale, int T, int N, int V,
-                                 int dtype, void* stream) {
+                                 int silu, int dtype, void* stream) {
   if (T <= 0) return 0;
   if (N <= 0 || V <= 0 || (dtype != 0 && dtype != 2)) return -2;
   HeadNormArgs a;
+  a.silu = silu;
   a.o = o; a.nq = nq; a.low = low; a.w = w; a.z = z; a.out = out; a.ldz = ldz; a.ldo = ldo;
   a.T = T; a.N = N; a.V = V; a.per_head = per_head; a.eps = eps; a.scale = scale;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -1337,4 +1471,92 @@ B200_API int b200_memory_step(const void* h, long long ldh, int H, const void* x
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   return dtype == 0 ? dispatch_step<__nv_bfloat16, kMemory>(a, DP, nd, s)
                     : dispatch_step<float, kMemory>(a, DP, nd, s);
+}
+
+// fp32 inputs of time mixing: ro, ko, go [T, N, DP], vo [T, N, VP], now [T, N]; z [T, N * D] is the
+// decay's projection, decays are exp(-exp(z + base)).  dtype (of r, k, v): 0 bf16, 2 fp32.
+B200_API int b200_wkv_inputs(const void* r, const void* k, const void* v, long long ld,
+                             const float* z, long long ldz, const float* base, const float* bonus,
+                             float* ro, float* ko, float* go, float* vo, float* now, int T, int N,
+                             int D, int DP, int VP, int dtype, void* stream) {
+  if (T <= 0) return 0;
+  if (N <= 0 || D <= 0 || D > DP || DP > 256 || VP < D || VP > DP || (VP % 4) != 0 ||
+      (dtype != 0 && dtype != 2))
+    return -2;
+  WkvIn a;
+  a.r = r; a.k = k; a.v = v; a.z = z; a.base = base; a.bonus = bonus; a.ro = ro; a.ko = ko;
+  a.go = go; a.vo = vo; a.now = now; a.ld = ld; a.ldz = ldz; a.T = T; a.N = N; a.D = D; a.DP = DP;
+  a.VP = VP;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const uintptr_t x = reinterpret_cast<uintptr_t>(r) | reinterpret_cast<uintptr_t>(k) |
+                      reinterpret_cast<uintptr_t>(v);
+  const uintptr_t f = reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(base) |
+                      reinterpret_cast<uintptr_t>(bonus);
+  const bool v4 = (D % 4) == 0 && (ld % 4) == 0 && (ldz % 4) == 0 &&
+                  (x % (dtype == 0 ? 8 : 16)) == 0 && (f % 16) == 0;
+  const auto blocks = [&](int lanes) {
+    return static_cast<unsigned int>((static_cast<long long>(T) * N * lanes + 255) / 256);
+  };
+#define B200_WI(TT)                                                            \
+  do {                                                                         \
+    if (!v4) wkv_inputs_kernel<TT, 1, 32><<<blocks(32), 256, 0, s>>>(a);       \
+    else if (DP <= 32) wkv_inputs_kernel<TT, 4, 8><<<blocks(8), 256, 0, s>>>(a);   \
+    else if (DP <= 64) wkv_inputs_kernel<TT, 4, 16><<<blocks(16), 256, 0, s>>>(a); \
+    else wkv_inputs_kernel<TT, 4, 32><<<blocks(32), 256, 0, s>>>(a);           \
+  } while (0)
+  if (dtype == 0) B200_WI(__nv_bfloat16);
+  else B200_WI(float);
+#undef B200_WI
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Time mixing over the portions of a step (nd single tokens, then np portions by cu_q).
+B200_API int b200_wkv_scan(const float* r, const float* k, const float* g, const float* v,
+                           const float* now, float* out, float* matrix, const long long* positions,
+                           const int* slots, int num_slots, const int* cu_q, int N, int D, int DP,
+                           int VP, int nd, int np, void* stream) {
+  if (nd + np <= 0) return 0;
+  if (N <= 0 || D <= 0 || D > VP || (VP % 4) != 0) return -2;
+  ScanArgs a{};
+  a.q = r; a.k = k; a.g = g; a.v = v; a.s0 = now; a.out = out; a.matrix = matrix;
+  a.positions = positions; a.slots = slots; a.num_slots = num_slots; a.cu_q = cu_q; a.G = N;
+  a.N = N; a.D = D; a.V = D; a.VP = VP; a.nd = nd; a.np = np; a.ntaps = 1;
+  return dispatch_scan<kWkv>(a, DP, nd + np, static_cast<cudaStream_t>(stream));
+}
+
+// out = tanh(x), n elements; dtype (of out): 0 bf16, 2 fp32.
+B200_API int b200_tanh_rows(const float* x, void* out, long long n, int dtype, void* stream) {
+  if (n <= 0) return 0;
+  if (dtype != 0 && dtype != 2) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const unsigned int blocks = static_cast<unsigned int>((n + 255) / 256);
+  if (dtype == 0)
+    tanh_rows_kernel<__nv_bfloat16><<<blocks, 256, 0, s>>>(x, static_cast<__nv_bfloat16*>(out), n);
+  else
+    tanh_rows_kernel<float><<<blocks, 256, 0, s>>>(x, static_cast<float*>(out), n);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// One token of `nd` requests through time mixing, from the projections to the gated output: inner
+// [nd, R] is the first step of the decay's projection (before its tanh), w2 [N D, R] the second's
+// weights (R a multiple of 8, rows 16-byte aligned), gate the output gate's projection.  dtype: 0
+// bf16, 2 fp32.  -20: not covered (very wide heads or ranks).
+B200_API int b200_wkv_step(const void* r, const void* k, const void* v, const void* gate,
+                           long long ld, const float* inner, long long ldi, int R, const void* w2,
+                           const float* base, const float* bonus, const float* norm, float* matrix,
+                           const long long* positions, const int* slots, int num_slots, void* out,
+                           long long ldo, float eps, int nd, int N, int D, int DP, int dtype,
+                           void* stream) {
+  if (nd <= 0) return 0;
+  if (N <= 0 || D <= 0 || D > DP || R <= 0 || (R % 8) != 0 ||
+      (reinterpret_cast<uintptr_t>(w2) & 15) != 0 || (dtype != 0 && dtype != 2))
+    return -2;
+  StepArgs a{};
+  a.H = R; a.x[0] = r; a.x[1] = k; a.x[2] = v; a.gate = gate; a.ldg = ld; a.ld = ld; a.z = inner;
+  a.ldz = ldi; a.w0 = w2; a.b0 = base; a.b1 = bonus; a.qscale = 1.0f; a.norm = norm; a.per_head = 1;
+  a.matrix = matrix; a.positions = positions; a.slots = slots; a.num_slots = num_slots; a.out = out;
+  a.ldo = ldo; a.eps = eps; a.scale = 1.0f; a.G = N; a.N = N; a.D = D; a.V = D;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return dtype == 0 ? dispatch_step<__nv_bfloat16, kWkv>(a, DP, nd, s)
+                    : dispatch_step<float, kWkv>(a, DP, nd, s);
 }

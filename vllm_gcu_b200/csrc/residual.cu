@@ -17,62 +17,17 @@
 //                   bias); optionally the norm of the new row in the same pass (the final one, or
 //                   that in front of the next sublayer).  y is a dense row, or the weighted sum of
 //                   a token's routed-expert rows plus a shared expert's row times its gate
-//   silu_mul_rows   h = silu(g) * u of rows [g | u], any width
-//   relu2           h = max(u, 0)^2
+//   act_mul_rows    h = act(g) * u of rows [g | u], any width
+//   ungated_act     h = max(u, 0)^2 or GELU
 //   head_gate       o = o * sigmoid(z) * s from rows whose heads are padded
 //
 // The residual stream, the statistics and the averages are fp32; LO is the type of the rows that
 // feed matrix products (bf16, or fp32 when the whole model runs in 32-bit).  One CTA per row,
 // vectors of V elements (4 where every row is 4-aligned, else 1).
-#include "common.cuh"
+#include "rows.cuh"
 
 namespace b200 {
 namespace residual {
-
-template <int V>
-__device__ __forceinline__ void ldv(const float* p, float (&f)[V]) {
-  if constexpr (V >= 4) {
-#pragma unroll
-    for (int i = 0; i < V; i += 4) {
-      const float4 u = *reinterpret_cast<const float4*>(p + i);
-      f[i] = u.x; f[i + 1] = u.y; f[i + 2] = u.z; f[i + 3] = u.w;
-    }
-  } else {
-    f[0] = p[0];
-  }
-}
-template <int V>
-__device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&f)[V]) {
-  if constexpr (V == 8) {
-    vec8_load<__nv_bfloat16>(p, f);
-  } else if constexpr (V == 4) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
-    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
-  } else {
-    f[0] = __bfloat162float(p[0]);
-  }
-}
-template <int V>
-__device__ __forceinline__ void stv(float* p, const float (&f)[V]) {
-  if constexpr (V >= 4) {
-#pragma unroll
-    for (int i = 0; i < V; i += 4)
-      *reinterpret_cast<float4*>(p + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
-  } else {
-    p[0] = f[0];
-  }
-}
-template <int V>
-__device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&f)[V]) {
-  if constexpr (V == 8) {
-    vec8_store<__nv_bfloat16>(p, f);
-  } else if constexpr (V == 4) {
-    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
-  } else {
-    p[0] = __float2bfloat16(f[0]);
-  }
-}
 
 // ---------------------------------------------------------------------------
 struct ShiftArgs {
@@ -572,24 +527,35 @@ __global__ void __launch_bounds__(512)
   }
 }
 
-template <typename T, int V>
+// activations by the codes of the GEMM epilogues (2 SiLU and 11 GELU-tanh, gated; 9 squared ReLU and
+// 10 GELU); 32-bit models take the exact tanh
+template <typename T, int ACT>
+__device__ __forceinline__ float act_of(float x) {
+  if constexpr (ACT == 2) return x / (1.0f + expf(-x));
+  else if constexpr (ACT == 9) return relu2_f(x);
+  else if constexpr (ACT == 10) return gelu_f(x);
+  else if constexpr (sizeof(T) == 2) return gelu_tanh_f(x);
+  else return 0.5f * x * (1.0f + tanhf(0.79788456080286536f * fmaf(0.044715f * x * x, x, x)));
+}
+
+template <typename T, int V, int ACT>
 __global__ void __launch_bounds__(256)
-    silu_mul_rows_kernel(const T* x, long long ldx, T* out, long long ldo, int D) {
+    act_mul_rows_kernel(const T* x, long long ldx, T* out, long long ldo, int D) {
   const T* g = x + blockIdx.x * ldx;
   for (int c = threadIdx.x * V; c < D; c += blockDim.x * V) {
     float a[V], b[V];
     ldv<V>(g + c, a);
     ldv<V>(g + D + c, b);
 #pragma unroll
-    for (int i = 0; i < V; ++i) a[i] = a[i] / (1.0f + expf(-a[i])) * b[i];
+    for (int i = 0; i < V; ++i) a[i] = act_of<T, ACT>(a[i]) * b[i];
     stv<V>(out + blockIdx.x * ldo + c, a);
   }
 }
 
-// out[t, c] = max(x[t, c], 0)^2; may run in place
-template <typename T, int V>
+// out[t, c] = act(x[t, c]); may run in place
+template <typename T, int V, int ACT>
 __global__ void __launch_bounds__(256)
-    relu2_kernel(const T* x, long long ldx, T* out, long long ldo, long long rows, int D) {
+    ungated_act_kernel(const T* x, long long ldx, T* out, long long ldo, long long rows, int D) {
   const int nv = D / V;
   const long long n = rows * nv;
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
@@ -599,14 +565,9 @@ __global__ void __launch_bounds__(256)
     float f[V];
     ldv<V>(x + t * ldx + c, f);
 #pragma unroll
-    for (int k = 0; k < V; ++k) f[k] = relu2_f(f[k]);
+    for (int k = 0; k < V; ++k) f[k] = act_of<T, ACT>(f[k]);
     stv<V>(out + t * ldo + c, f);
   }
-}
-
-static int row_threads(int H, int V, int most) {
-  int n = (H / V + 31) / 32 * 32;
-  return n < 32 ? 32 : (n > most ? most : n);
 }
 
 template <typename Y, typename LO, int V>
@@ -658,10 +619,6 @@ template <typename T, int V>
 static int launch_add_normed(const AddNormArgs& a, cudaStream_t s) {
   return a.pos_of != nullptr ? launch_add_normed_as<T, V, true>(a, s)
                              : launch_add_normed_as<T, V, false>(a, s);
-}
-
-static bool aligned(const void* p, int bytes) {
-  return (reinterpret_cast<uintptr_t>(p) % bytes) == 0;
 }
 
 }  // namespace residual
@@ -805,11 +762,12 @@ B200_API int b200_add_normed(const float* x, const void* y, long long ldy, const
   return v4 ? launch_add_normed<float, 4>(a, s) : launch_add_normed<float, 1>(a, s);
 }
 
-// out [T, D] = max(x, 0)^2, in place if the pointers are equal; dtype 0 bf16, 2 fp32.
-B200_API int b200_relu2(const void* x, long long ldx, void* out, long long ldo, int T, int D,
-                        int dtype, void* stream) {
+// out [T, D] = act(x), in place if the pointers are equal; act 9: max(x, 0)^2, 10: GELU; dtype 0 bf16,
+// 2 fp32.
+B200_API int b200_ungated_act(const void* x, long long ldx, void* out, long long ldo, int T, int D,
+                              int act, int dtype, void* stream) {
   if (T <= 0 || D <= 0) return 0;
-  if (dtype != 0 && dtype != 2) return -2;
+  if ((dtype != 0 && dtype != 2) || (act != 9 && act != 10)) return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const bool v4 = (D % 4) == 0 && (ldx % 4) == 0 && (ldo % 4) == 0 && aligned(x, 16) &&
                   aligned(out, 16);
@@ -817,17 +775,20 @@ B200_API int b200_relu2(const void* x, long long ldx, void* out, long long ldo, 
   long long blocks = (items + 255) / 256;
   const long long cap = static_cast<long long>(sm_count()) * 16;
   const int g = static_cast<int>(blocks > cap ? cap : blocks);
-  if (dtype == 0) {
-    const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(x);
-    __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
-    if (v4) relu2_kernel<__nv_bfloat16, 4><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
-    else relu2_kernel<__nv_bfloat16, 1><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
-  } else {
-    const float* p = static_cast<const float*>(x);
-    float* o = static_cast<float*>(out);
-    if (v4) relu2_kernel<float, 4><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
-    else relu2_kernel<float, 1><<<g, 256, 0, s>>>(p, ldx, o, ldo, T, D);
-  }
+#define B200_UA(TT, W, A)                                                                     \
+  ungated_act_kernel<TT, W, A><<<g, 256, 0, s>>>(static_cast<const TT*>(x), ldx,             \
+                                                 static_cast<TT*>(out), ldo, T, D)
+#define B200_UA2(TT)                      \
+  do {                                    \
+    if (v4 && act == 9) B200_UA(TT, 4, 9); \
+    else if (v4) B200_UA(TT, 4, 10);      \
+    else if (act == 9) B200_UA(TT, 1, 9); \
+    else B200_UA(TT, 1, 10);              \
+  } while (0)
+  if (dtype == 0) B200_UA2(__nv_bfloat16);
+  else B200_UA2(float);
+#undef B200_UA2
+#undef B200_UA
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -861,25 +822,28 @@ B200_API int b200_head_gate(const void* o, int DC, const void* z, long long ldz,
   return static_cast<int>(cudaGetLastError());
 }
 
-// out [T, D] = silu(x[:, :D]) * x[:, D:]; dtype 0 bf16, 2 fp32.
-B200_API int b200_silu_mul_rows(const void* x, long long ldx, void* out, long long ldo, int T, int D,
-                                int dtype, void* stream) {
+// out [T, D] = act(x[:, :D]) * x[:, D:]; act 2: SiLU, 11: GELU (tanh form); dtype 0 bf16, 2 fp32.
+B200_API int b200_act_mul_rows(const void* x, long long ldx, void* out, long long ldo, int T, int D,
+                               int act, int dtype, void* stream) {
   if (T <= 0 || D <= 0) return 0;
-  if (dtype != 0 && dtype != 2) return -2;
+  if ((dtype != 0 && dtype != 2) || (act != 2 && act != 11)) return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const bool v4 = (D % 4) == 0 && (ldx % 4) == 0 && (ldo % 4) == 0 && aligned(x, 16) &&
                   aligned(out, 16);
   const int th = row_threads(D, v4 ? 4 : 1, 256);
-  if (dtype == 0) {
-    const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(x);
-    __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out);
-    if (v4) silu_mul_rows_kernel<__nv_bfloat16, 4><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
-    else silu_mul_rows_kernel<__nv_bfloat16, 1><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
-  } else {
-    const float* p = static_cast<const float*>(x);
-    float* o = static_cast<float*>(out);
-    if (v4) silu_mul_rows_kernel<float, 4><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
-    else silu_mul_rows_kernel<float, 1><<<T, th, 0, s>>>(p, ldx, o, ldo, D);
-  }
+#define B200_AM(TT, W, A)                                                                 \
+  act_mul_rows_kernel<TT, W, A><<<T, th, 0, s>>>(static_cast<const TT*>(x), ldx,          \
+                                                 static_cast<TT*>(out), ldo, D)
+#define B200_AM2(TT)                      \
+  do {                                    \
+    if (v4 && act == 2) B200_AM(TT, 4, 2); \
+    else if (v4) B200_AM(TT, 4, 11);      \
+    else if (act == 2) B200_AM(TT, 1, 2); \
+    else B200_AM(TT, 1, 11);              \
+  } while (0)
+  if (dtype == 0) B200_AM2(__nv_bfloat16);
+  else B200_AM2(float);
+#undef B200_AM2
+#undef B200_AM
   return static_cast<int>(cudaGetLastError());
 }

@@ -63,6 +63,8 @@ class AttentionMetadata:
     # ``has_request_state``, and the slot of every request of the step ``[B]`` int32 (-1: padding)
     request_state: Optional[list] = None
     state_slots: Optional[torch.Tensor] = None
+    # value cache of the layer whose values later layers mix into theirs
+    first_values: Optional[torch.Tensor] = None
     cu_q_all: Optional[torch.Tensor] = None
 
 

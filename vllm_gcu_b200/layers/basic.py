@@ -139,7 +139,7 @@ def build_cos_sin_cache(rot_dim: int, max_pos: int, base: float,
             low = max(math.floor(_yarn_find_correction_dim(beta_fast, rot_dim, base, orig)), 0)
             high = min(math.ceil(_yarn_find_correction_dim(beta_slow, rot_dim, base, orig)),
                        rot_dim - 1)
-            ramp = ((torch.arange(rot_dim // 2, dtype=torch.float32) - low)
+            ramp = ((torch.arange(rot_dim // 2, dtype=dtype) - low)
                     / max(high - low, 1e-3)).clamp(0, 1)
             mask = 1.0 - ramp
             inv_freq = inv_freq / factor * (1 - mask) + inv_freq * mask

@@ -74,8 +74,9 @@ class UnquantizedLinearMethod(LinearMethod):
         if ops.use_native(x) and x.dtype == torch.bfloat16:
             shape = x.shape
             x2 = x.reshape(-1, shape[-1])
+            act = getattr(layer, "fused_act", "silu")
             if getattr(layer, "_interleaved", False):
-                y = C.gemm_bf16(x2, w, epilogue=C.EPI_SILU_MUL)
+                y = C.gemm_bf16(x2, w, epilogue=C.GATED_EPI[act])
             else:
                 if bias is not None and residual is not None:
                     y = C.gemm_bf16(x2, w, bias=bias)
@@ -83,14 +84,15 @@ class UnquantizedLinearMethod(LinearMethod):
                 else:
                     y = C.gemm_bf16(x2, w, bias=bias, residual=residual)
                 if getattr(layer, "fuse_silu", False):
-                    y = C.activation(y, "silu") if y.shape[-1] % 16 == 0 else C.silu_mul_rows(y)
+                    y = C.activation(y, act) if y.shape[-1] % 16 == 0 else C.act_mul_rows(y, act)
             return y.view(*shape[:-1], y.shape[-1])
         y = F.linear(x, w, bias)
         if residual is not None:
             y = y + residual
         if getattr(layer, "fuse_silu", False):
-            y = C.silu_mul_rows(y) if y.dtype == torch.float32 and ops.use_native(y) \
-                else ref.silu_and_mul(y)
+            act = getattr(layer, "fused_act", "silu")
+            y = C.act_mul_rows(y, act) if y.dtype == torch.float32 and ops.use_native(y) \
+                else ref.act_and_mul(y, act)
         return y
 
 
@@ -240,9 +242,14 @@ def linear_fp32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 
 class MergedColumnParallelLinear(LinearBase):
+    """``fuse_silu``: the result is the gated activation ``fused_act`` ("silu" or "gelu_tanh") of the
+    two halves."""
+
     def __init__(self, in_features, output_sizes: Sequence[int], bias=False, fuse_silu=False,
-                 dtype=torch.bfloat16, device=None, quant_method=None, prefix=""):
+                 dtype=torch.bfloat16, device=None, quant_method=None, prefix="",
+                 fused_act: str = "silu"):
         tp = tp_size()
+        self.fused_act = fused_act
         self.output_sizes = list(output_sizes)
         assert all(s % tp == 0 for s in output_sizes)
         self.fuse_silu = fuse_silu

@@ -24,10 +24,13 @@ from .linear import MixedParallelLinear, MixedRowParallelLinear, linear_fp32
 Projection = tuple[str, int, bool]      # name, output features, sharded over TP
 
 
-def linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+def linear(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None
+           ) -> torch.Tensor:
+    """``out``: where the rows go (a row-strided view is fine)."""
     if ops.use_native(x) and x.dtype == torch.bfloat16:
-        return C.gemm_bf16(x, weight)
-    return F.linear(x, weight)
+        return C.gemm_bf16(x, weight, out=out)
+    y = F.linear(x, weight)
+    return y if out is None else out.copy_(y)
 
 
 class MixerPart(nn.Module):
@@ -39,7 +42,7 @@ class MixerPart(nn.Module):
     width: int
 
     def new(self, *shape, dtype=torch.float32, device=None) -> nn.Parameter:
-        return nn.Parameter(torch.zeros(*shape, dtype=dtype, device=device), requires_grad=False)
+        return nn.Parameter(torch.zeros(shape, dtype=dtype, device=device), requires_grad=False)
 
     @staticmethod
     def shard(full: torch.Tensor, dim: int = 0) -> torch.Tensor:

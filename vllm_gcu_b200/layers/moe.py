@@ -445,16 +445,19 @@ class InputWeightedMoE(FusedMoE):
         return op(x, self.w13, self.w2, topk_w, topk_ids)
 
 
-class SquaredReluMoE(FusedMoE):
-    """Routed experts without a gate: ``down_e(max(up_e(h), 0)^2)``.
+class UngatedMoE(FusedMoE):
+    """Routed experts without a gate: ``down_e(act(up_e(h)))``; ``act``: "relu2" (squared ReLU) or
+    "gelu" (through the error function).
 
     ``forward`` returns the experts' unweighted output rows in sorted order and the row of every
     (token, slot) pair, which the norm after the residual sum weights and adds up (this rank's slice
     of the intermediate dimension under TP).  On the GPU the stacked weights are padded with zeros
     to the tile sizes of the grouped GEMM, which leaves the result as it is."""
 
-    def __init__(self, num_experts: int, hidden: int, inter: int, dtype, device, prefix: str = ""):
+    def __init__(self, num_experts: int, hidden: int, inter: int, dtype, device, prefix: str = "",
+                 act: str = "relu2"):
         tp = tp_size()
+        self.ungated_act = act
         if inter % tp:
             raise ValueError(f"{prefix}: experts of width {inter} over {tp} ranks")
         self.hidden_full, self.inter_real = hidden, inter // tp
@@ -487,15 +490,17 @@ class SquaredReluMoE(FusedMoE):
 
     def forward(self, x: torch.Tensor, topk_ids: torch.Tensor
                 ) -> tuple[torch.Tensor, torch.Tensor]:
-        op = C.squared_relu_experts if ops.use_native(x) else ref.squared_relu_experts
-        return op(x, self.w1, self.w2, topk_ids)
+        op = C.ungated_experts if ops.use_native(x) else ref.ungated_experts
+        return op(x, self.w1, self.w2, topk_ids, self.ungated_act)
 
 
-class SquaredReluMLP(nn.Module):
-    """``down(max(up(x), 0)^2)``; the result is this rank's part of the sum."""
+class UngatedMLP(nn.Module):
+    """``down(act(up(x)))``, ``act`` as in ``UngatedMoE``; the result is this rank's part of the
+    sum."""
 
-    def __init__(self, hidden: int, inter: int, dtype, device, prefix: str):
+    def __init__(self, hidden: int, inter: int, dtype, device, prefix: str, act: str = "relu2"):
         super().__init__()
+        self.act = act
         self.up_proj = ColumnParallelLinear(hidden, inter, dtype=dtype, device=device,
                                             prefix=prefix + ".up_proj")
         self.down_proj = RowParallelLinear(inter, hidden, reduce_results=False, dtype=dtype,
@@ -503,29 +508,35 @@ class SquaredReluMLP(nn.Module):
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         if ops.use_native(x) and x.dtype == torch.bfloat16:
-            return self.down_proj(C.gemm_bf16(x, self.up_proj.weight, epilogue=C.EPI_RELU2))
-        return self.down_proj((C if ops.use_native(x) else ref).relu2(self.up_proj(x)))
+            return self.down_proj(C.gemm_bf16(x, self.up_proj.weight,
+                                              epilogue=C.UNGATED_EPI[self.act]))
+        return self.down_proj((C if ops.use_native(x) else ref).ungated_act(self.up_proj(x),
+                                                                            self.act))
 
 
 class GatedSharedMoE(nn.Module):
-    """fp32 softmax router with renormalised weights, squared-ReLU experts and an optional shared
-    expert behind a gate of one number per token.
+    """fp32 softmax router with renormalised weights, experts without gates (``act``: see
+    ``UngatedMoE``) and an optional shared expert, behind a gate of one number per token if
+    ``shared_gate``.  ``groups = (count, keep)``: a token's experts come from the ``keep`` best of
+    ``count`` groups of neighbours.
 
     ``forward`` returns ``(y, operands)`` for ``ops.add_normed``, which weights and sums the rows.
     Router and shared expert's gate are one narrow GEMM with fp32 results."""
 
     def __init__(self, num_experts: int, top: int, scale: float, hidden: int, inter: int,
-                 shared_inter: int, dtype, device, prefix: str):
+                 shared_inter: int, dtype, device, prefix: str, act: str = "relu2",
+                 groups: tuple[int, int] = (1, 1), shared_gate: bool = True):
         super().__init__()
         self.route_cfg = ModelConfig(num_experts=num_experts, num_experts_per_tok=top,
                                      routed_scaling_factor=scale, scoring_func="softmax",
-                                     norm_topk_prob=True)
-        self.router = MixedParallelLinear(hidden, [num_experts] + [1] * (shared_inter > 0),
-                                          [False] * (1 + (shared_inter > 0)), dtype=dtype,
+                                     norm_topk_prob=True, n_group=groups[0], topk_group=groups[1])
+        self.shared_gate = shared_gate and shared_inter > 0
+        self.router = MixedParallelLinear(hidden, [num_experts] + [1] * self.shared_gate,
+                                          [False] * (1 + self.shared_gate), dtype=dtype,
                                           device=device, prefix=prefix + ".router", align=8)
-        self.experts = SquaredReluMoE(num_experts, hidden, inter, dtype, device,
-                                      prefix + ".experts")
-        self.shared = SquaredReluMLP(hidden, shared_inter, dtype, device, prefix + ".shared") \
+        self.experts = UngatedMoE(num_experts, hidden, inter, dtype, device, prefix + ".experts",
+                                  act)
+        self.shared = UngatedMLP(hidden, shared_inter, dtype, device, prefix + ".shared", act) \
             if shared_inter > 0 else None
 
     def load(self, name: str, full: torch.Tensor) -> bool:
@@ -535,6 +546,8 @@ class GatedSharedMoE(nn.Module):
         elif name.startswith("shared.") and self.shared is None:
             return False
         elif name == "shared.sg":
+            if not self.shared_gate:
+                return False
             self.router.load_weight("weight", full, 1)
         elif name in ("shared.up", "shared.down"):
             getattr(self.shared, name[7:] + "_proj").load_weight("weight", full)
@@ -546,8 +559,8 @@ class GatedSharedMoE(nn.Module):
 
     def tensor_names(self) -> set[str]:
         names = {f"e{e}.{k}" for e in range(self.experts.local_experts) for k in ("up", "down")}
-        return names | {"router"} | ({"shared.up", "shared.down", "shared.sg"}
-                                     if self.shared is not None else set())
+        return names | {"router"} | ({"shared.up", "shared.down"} if self.shared is not None
+                                     else set()) | ({"shared.sg"} if self.shared_gate else set())
 
     def forward(self, h: torch.Tensor) -> tuple[torch.Tensor, dict]:
         z = self.router.split(linear_fp32(h, self.router.weight))
@@ -555,7 +568,7 @@ class GatedSharedMoE(nn.Module):
         y, pos_of = self.experts(h, ids)
         rows = dict(pos_of=pos_of, row_w=w)
         if self.shared is not None:
-            rows.update(shared=self.shared(h), gate=z[1][:, 0])
+            rows.update(shared=self.shared(h), gate=z[1][:, 0] if self.shared_gate else None)
         if tp_size() == 1:
             return y, rows
         # every rank has its slice of the intermediate dimensions: sum rows, then ranks
@@ -563,7 +576,8 @@ class GatedSharedMoE(nn.Module):
         p = pos_of.view(-1)[:T * k].view(T, k).long()
         out = (y[p.clamp(min=0)].float() * (w * (p >= 0)).unsqueeze(-1)).sum(1)[:, :h.shape[1]]
         if self.shared is not None:
-            out += torch.sigmoid(rows["gate"]).unsqueeze(-1) * rows["shared"].float()
+            gate = 1.0 if rows["gate"] is None else torch.sigmoid(rows["gate"]).unsqueeze(-1)
+            out += gate * rows["shared"].float()
         return get_comm("tp").all_reduce(out.to(h.dtype).contiguous()), {}
 
 

@@ -1,4 +1,4 @@
-"""Mixer parts with a matrix state per head: gated delta rule and matrix memory.
+"""Mixer parts with a matrix state per head: gated delta rule, matrix memory and time mixing.
 
 Their state belongs to a request, not to its cache blocks: it lives in the request's state slot
 (``AttentionMetadata.state_slots``) in fp32 and is updated in place by every step.  A portion at
@@ -11,14 +11,15 @@ from dataclasses import dataclass
 from typing import Optional
 
 import torch
+import torch.nn as nn
 
 from .. import ops
-from ..config import DeltaSpec, MemorySpec
+from ..config import DeltaSpec, MemorySpec, TimeMixSpec
 from ..ops import cuda as C
 from ..ops import ref
 from ..parallel.state import tp_size
 from .attention import AttentionMetadata
-from .linear import linear_fp32
+from .linear import MixedParallelLinear, ReplicatedLinear, RowParallelLinear, linear_fp32
 from .mixer import MixerPart, fused_tokens, linear
 
 #: padded key dimensions of the scan kernel
@@ -181,3 +182,90 @@ class MatrixMemory(MixerPart):
                                       self.f_bias, s.gate_cap, *sizes, Place.behind(md, n1),
                                       None if md.is_dummy else state)
         o_.head_norm_gate(o, self.norm, g[n1:], self.eps, scale, out[n1:], nq, low)
+
+
+class TimeMix(nn.Module):
+    """Linear recurrence of the RWKV kind: a matrix per head that decays per key channel, and a bonus
+    for the current token.
+
+    A mixer of its own (not a part of a ``MixerBlock``): its five projections (r, k, v, the output
+    gate g, the decay's first step w) read five different mixtures of a token's row with the row of
+    the token before it, which come from the input convolution's kernel as ``h [5, T, H]``, in the
+    order of ``MIXES`` (``layers/input_conv.py``)."""
+
+    MIXES = ("r", "k", "v", "g", "w")
+
+    def __init__(self, spec: TimeMixSpec, hidden: int, eps: float, dtype, device, prefix: str):
+        super().__init__()
+        self.spec, self.eps, self.dtype = spec, eps, dtype
+        N, D, R = spec.num_heads, spec.head_dim, spec.decay_rank
+        self.N = _local_heads(N, prefix)
+        self.rows = state_rows(D, prefix)
+        new = lambda *s, dt=torch.float32: nn.Parameter(  # noqa: E731
+            torch.zeros(*s, dtype=dt, device=device), requires_grad=False)
+        self.mu = new(len(self.MIXES), hidden)
+        self.in_proj = MixedParallelLinear(hidden, [N * D] * 4, [True] * 4, dtype=dtype,
+                                           device=device, prefix=prefix + ".in_proj", align=8)
+        pad = -(-R // 8) * 8
+        self.w1 = ReplicatedLinear(hidden, pad, dtype=dtype, device=device, prefix=prefix + ".w1")
+        self.w2 = new(self.N * D, pad, dt=dtype)           # columns behind the rank stay zero
+        self.w0, self.bonus = new(self.N * D), new(self.N * D)
+        self.norm = new(self.N * D)
+        self.o_proj = RowParallelLinear(N * D, hidden, dtype=dtype, device=device,
+                                        prefix=prefix + ".o_proj")
+
+    def cache_shape(self) -> None:
+        return None
+
+    def state_shapes(self) -> dict:
+        """Recurrent state per request: name -> (shape, dtype)."""
+        return {"matrix": ((self.N, self.spec.head_dim, self.rows), torch.float32)}
+
+    _OWN = {"w0": "w0", "u": "bonus", "norm": "norm"}
+
+    def tensor_names(self) -> set[str]:
+        return {"mu." + c for c in self.MIXES} | {"r", "k", "v", "g", "w1", "w2", "o"} | set(self._OWN)
+
+    def load(self, name: str, full: torch.Tensor) -> bool:
+        """False if there is no tensor of that name."""
+        if name not in self.tensor_names():
+            return False
+        if name.startswith("mu."):
+            self.mu.data[self.MIXES.index(name[3:])].copy_(full)
+        elif name == "w1":
+            self.w1.weight.data[:self.spec.decay_rank].copy_(full)
+        elif name == "w2":
+            self.w2.data[:, :self.spec.decay_rank].copy_(MixerPart.shard(full))
+        elif name == "o":
+            self.o_proj.load_weight("weight", full)
+        elif name in self._OWN:
+            getattr(self, self._OWN[name]).data.copy_(MixerPart.shard(full.reshape(-1)))
+        else:
+            self.in_proj.load_weight("weight", full, self.MIXES.index(name))
+        return True
+
+    def finalize(self) -> None:
+        self.w1.weight.data[self.spec.decay_rank:] = 0
+        self.w2.data[:, self.spec.decay_rank:] = 0
+
+    def forward(self, h: torch.Tensor, md: AttentionMetadata, state: Optional[dict]) -> torch.Tensor:
+        T, D, n = h.shape[1], self.spec.head_dim, self.N * self.spec.head_dim
+        pad = self.in_proj.padded_sizes[0]
+        y = torch.empty(T, 4 * pad, dtype=h.dtype, device=h.device)
+        for i in range(4):
+            linear(h[i], self.in_proj.weight[i * pad:(i + 1) * pad], out=y[:, i * pad:(i + 1) * pad])
+        r, k, v, g = (y[:, i * pad:i * pad + n] for i in range(4))
+        a = linear_fp32(h[4], self.w1.weight)              # the decay's inner row, unrounded
+        out = torch.empty(T, n, dtype=h.dtype, device=h.device)
+        S = state["matrix"] if state is not None and not md.is_dummy else None
+        n1 = fused_tokens(h, md)
+        if n1:
+            C.wkv_step(r[:n1], k[:n1], v[:n1], g[:n1], a[:n1], self.w2, self.w0, self.bonus,
+                       self.norm, D, self.rows, md.positions, md.state_slots, S, self.eps, out[:n1])
+        if n1 < T:
+            o_ = C if ops.use_native(out) else ref
+            z = linear_fp32(o_.tanh_rows(a[n1:], self.dtype), self.w2)
+            o = o_.wkv(r[n1:], k[n1:], v[n1:], z, self.w0, self.bonus, D, self.rows,
+                       Place.behind(md, n1), S)
+            o_.head_norm_gate(o, self.norm, g[n1:], self.eps, 1.0, out[n1:], act="silu")
+        return self.o_proj(out)

@@ -52,8 +52,8 @@ class LoRALinear(nn.Module):
             max_loras, n, max_rank, dtype=dt, device=dev), requires_grad=False)
             for n in self.slices])
         self.scaling = torch.ones(max_loras)
-        for attr in ("fuse_silu", "_interleaved", "num_heads", "num_kv_heads", "head_dim",
-                     "q_size", "kv_size", "output_sizes"):
+        for attr in ("fuse_silu", "fused_act", "_interleaved", "num_heads", "num_kv_heads",
+                     "head_dim", "q_size", "kv_size", "output_sizes"):
             if hasattr(base, attr):
                 object.__setattr__(self, attr, getattr(base, attr))
 
@@ -98,7 +98,7 @@ class LoRALinear(nn.Module):
             y = torch.nn.functional.linear(x, w, base.bias)
             self.punica.add_lora_linear(y, x, list(self.lora_a), list(self.lora_b), 1.0,
                                         self.slices)
-            return act_and_mul(y, "silu")
+            return act_and_mul(y, getattr(base, "fused_act", "silu"))
         if isinstance(base, RowParallelLinear) and tp_size() > 1:
             # the delta is a partial sum over the sharded input like the base output
             y = base.quant_method.apply(base, x, skip_bias=True)

@@ -53,6 +53,7 @@ _REGISTRY: dict[str, str] = {
     "SapapelForCausalLM": "vllm_gcu_b200.models.sapapel:SapapelForCausalLM",
     "FizunexForCausalLM": "vllm_gcu_b200.models.fizunex:FizunexForCausalLM",
     "FepopelForCausalLM": "vllm_gcu_b200.models.fepopel:FepopelForCausalLM",
+    "VadelixForCausalLM": "vllm_gcu_b200.models.vadelix:VadelixForCausalLM",
     "DeepSeekMTPModel": "vllm_gcu_b200.models.deepseek_mtp:DeepSeekMTP",
     # pooling models (no KV cache; built by build_pooling_model)
     "XLMRobertaForSequenceClassification":

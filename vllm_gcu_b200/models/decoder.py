@@ -53,10 +53,12 @@ def fused_input_quant(linear, x: torch.Tensor, width: Optional[int] = None):
 
 class DenseMLP(nn.Module):
     def __init__(self, cfg: ModelConfig, hidden: int, inter: int, device, prefix: str,
-                 reduce_results: bool = True):
+                 reduce_results: bool = True, fused_act: str = "silu"):
+        """``fused_act``: the activation that the first GEMM applies if it is the model's."""
         super().__init__()
         self.gate_up_proj = MergedColumnParallelLinear(
-            hidden, [inter, inter], bias=cfg.mlp_bias, fuse_silu=(cfg.hidden_act == "silu"),
+            hidden, [inter, inter], bias=cfg.mlp_bias, fuse_silu=(cfg.hidden_act == fused_act),
+            fused_act=fused_act,
             dtype=cfg.dtype, device=device,
             quant_method=get_linear_method(cfg, prefix + ".gate_up_proj"),
             prefix=prefix + ".gate_up_proj")

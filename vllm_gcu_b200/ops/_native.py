@@ -130,21 +130,27 @@ class _Sigs:
     b200_token_shift = [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P]
     b200_post_norm = [P, P, L, P, I, P, F, F, P, P, L, I, P, P, P, P, I, I, I, P]
     b200_sigmoid_gate = [P, L, P, L, P, L, I, I, I, P]
-    b200_silu_mul_rows = [P, L, P, L, I, I, I, P]
+    b200_act_mul_rows = [P, L, P, L, I, I, I, I, P]
     b200_start_rows = [P, L, F, P, P, F, P, P, I, I, I, P]
     b200_add_normed = [P, P, L, P, P, I, P, L, P, L, P, P, P, I, F, P, P, P, F, P, I, I, I, P]
-    b200_relu2 = [P, L, P, L, I, I, I, P]
+    b200_ungated_act = [P, L, P, L, I, I, I, I, P]
     b200_head_gate = [P, I, P, L, F, P, L, I, I, I, I, P]
     b200_qk_norm_rope_cache = [P, L, P, L, P, L, P, P, P, I, I, F, P, I, L, I, P, P, P, P, P, L, I,
                                I, I, I, I, I, P]
     b200_head_norm_cache = [P, L, P, L, P, L, P, P, F, P, P, P, P, L, I, I, I, I, I, I, I, P]
-    b200_any_attention = [P, P, P, L, P, L, I, P, I, I, P, P, P, I, I, I, I, I, I, F, F, I, I, P]
+    b200_qkv_cache = [P, L, P, L, P, L, P, P, P, I, I, F, P, I, L, F, I, I, P, P, L, I, I, P, P, P,
+                      P, P, L, I, I, I, I, I, I, I, P]
+    b200_any_attention = [P, P, P, L, P, L, I, P, I, I, P, P, P, I, I, I, I, I, I, F, F, I, I, P, I,
+                          P]
+    b200_add_group_norm = [P, P, L, P, L, F, P, P, I, P, L, P, L, P, I, F, P, P, P, I, P, I, P, I, P,
+                           P, P, L, L, I, I, I, I, P]
+    b200_input_conv = [P, P, I, P, I, P, I, P, P, P, P, L, L, I, I, I, I, I, P]
     b200_paged_decode_sink = [P, L, P, L, P, P, L, L, L, P, I, I, P, P, P, I, I, I, I, I, F, I, P,
-                              F, I, I, P]
+                              F, I, I, P, I, P]
     b200_paged_decode_tma_sink = [P, L, P, L, P, P, L, L, L, P, I, I, P, P, P, I, I, I, I, I, F, I,
-                                  P, F, I, I, P]
+                                  P, F, I, I, P, I, P]
     b200_fmha_prefill_sink = [P, L, P, L, P, P, P, P, P, L, L, L, P, I, I, I, I, I, I, I, I, F,
-                              I, I, I, P, F, I, I, P]
+                              I, I, I, P, F, I, P, I, P]
     b200_recurrent_rows = [I]
     b200_delta_inputs = [P, P, P, L, P, P, P, I, P, I, P, L, P, L, P, P, P, P, P, P, P, P, P, P,
                          I, I, I, I, I, I, I, I, I, I, P]
@@ -153,7 +159,11 @@ class _Sigs:
     b200_delta_scan = [P, P, P, P, P, P, P, P, P, P, L, P, I, P, P, I, P, I, I, I, I, I, I, I, I,
                        I, P]
     b200_memory_scan = [P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, P]
-    b200_head_norm_gate = [P, P, P, P, I, P, L, P, L, F, F, I, I, I, I, P]
+    b200_head_norm_gate = [P, P, P, P, I, P, L, P, L, F, F, I, I, I, I, I, P]
+    b200_wkv_inputs = [P, P, P, L, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P]
+    b200_wkv_scan = [P, P, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, P]
+    b200_tanh_rows = [P, P, L, I, P]
+    b200_wkv_step = [P, P, P, P, L, P, L, I, P, P, P, P, P, P, P, I, P, L, F, I, I, I, I, I, P]
     b200_delta_step = [P, L, I, P, P, P, L, P, L, P, L, P, P, P, P, I, P, P, P, P, P, P, P, I, P, L,
                        F, F, I, I, I, I, I, I, I, P]
     b200_memory_step = [P, L, I, P, P, P, P, L, P, P, P, P, F, F, P, P, P, P, P, P, I, P, L, F, F,
@@ -172,7 +182,7 @@ class _Sigs:
     b200_moe_permute_weighted = [P, L, P, P, L, P, P, I, I, I, I, I, I, P]
     b200_grouped_gemm_f32 = [P, L, P, P, L, I, I, I, I, P, P, P]
     b200_silu_mul_rows_f32 = [P, P, I, I, P, P]
-    b200_relu2_rows_f32 = [P, P, I, I, P, P]
+    b200_ungated_rows_f32 = [P, P, I, I, P, I, P]
     b200_moe_row_weights = [P, P, P, P, I, I, P]
     b200_moe_unpermute_sum = [P, L, P, P, L, P, L, P, I, I, I, F, I, P]
     b200_get_ep_indices = [P, I, I, I, I, P, P, P, P]

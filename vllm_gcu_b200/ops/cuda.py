@@ -15,6 +15,13 @@ from . import _native as N
 from ._native import DTYPE_CODE, call, ptr, stream_ptr
 
 EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RESIDUAL, EPI_FP32, EPI_RELU2 = 0, 1, 2, 3, 4, 9
+EPI_GELU, EPI_GELU_MUL = 10, 11
+#: epilogues of gated and of plain activations
+GATED_EPI = {"silu": EPI_SILU_MUL, "gelu_tanh": EPI_GELU_MUL}
+UNGATED_EPI = {"relu2": EPI_RELU2, "gelu": EPI_GELU}
+_GATED = tuple(GATED_EPI.values())
+_WIDE_EPI = (EPI_NONE, EPI_BIAS, *_GATED)
+_PAIR_EPI = (*_WIDE_EPI, EPI_RELU2, EPI_GELU)
 
 NORM_QMODES = {None: 0, "fp8_static": 1, "fp8_token": 2, "fp8_group128": 3,
                "int8_static": 4, "int8_token": 5}
@@ -138,11 +145,12 @@ def gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = No
         from . import ref
         a2 = a.reshape(-1, a.shape[-1])
         want = ref.gemm(a2, b, bias=bias, residual=residual, out_dtype=torch.float32)
-        if bias is None and residual is None and epilogue == EPI_SILU_MUL:
+        if bias is None and residual is None and epilogue in _GATED:
             w4 = want.view(want.shape[0], -1, 2, ref.GATE_UP_BLOCK)
-            want = (torch.nn.functional.silu(w4[:, :, 0]) * w4[:, :, 1]).reshape(want.shape[0], -1)
-        if epilogue == EPI_RELU2:
-            want = want.clamp(min=0).square()
+            act = "silu" if epilogue == EPI_SILU_MUL else "gelu_tanh"
+            want = (ref._act(act, w4[:, :, 0]) * w4[:, :, 1]).reshape(want.shape[0], -1)
+        if epilogue in (EPI_RELU2, EPI_GELU):
+            want = ref.ungated_act(want, "relu2" if epilogue == EPI_RELU2 else "gelu")
         oracle_compare("gemm_bf16", res, want, 3e-2, 3e-2 * max(1.0, float(want.abs().mean())))
     return res
 
@@ -153,7 +161,8 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
     """``out[M,N] = a[M,K] @ b[N,K]^T`` on the tcgen05 path (bf16 in, fp32 accumulate).
 
     epilogue EPI_SILU_MUL expects ``b`` interleaved by ``ref.interleave_gate_up`` and
-    yields ``[M, N/2]``; EPI_FP32 writes fp32; EPI_RELU2 yields ``max(out, 0)^2``."""
+    yields ``[M, N/2]``, EPI_GELU_MUL the same with the tanh form of GELU; EPI_FP32 writes fp32;
+    EPI_RELU2 yields ``max(out, 0)^2``, EPI_GELU the GELU of the result."""
     assert a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16
     a = _rowmajor_2d(a)
     M, K = a.shape
@@ -163,13 +172,13 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
         epilogue = EPI_BIAS
     if residual is not None:
         epilogue = EPI_RESIDUAL
-    out_cols = Nn // 2 if epilogue == EPI_SILU_MUL else Nn
+    out_cols = Nn // 2 if epilogue in _GATED else Nn
     if out is None:
         out = torch.empty((M, out_cols), device=a.device,
                           dtype=torch.float32 if epilogue == EPI_FP32 else torch.bfloat16)
     assert out.stride(-1) == 1 and out.shape[-1] == out_cols
     if (K % 8 or Nn % 8 or a.stride(0) % 8 or b.stride(0) % 8 or out.stride(0) % 8) \
-            and epilogue != EPI_SILU_MUL:
+            and epilogue not in _GATED:
         # rows that are not a multiple of 16 bytes cannot be described to TMA (a router over
         # four experts, an odd head count): the library GEMM takes these rare, tiny shapes
         y = torch.matmul(a.float() if epilogue == EPI_FP32 else a,
@@ -178,12 +187,12 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
             y = y + bias
         if residual is not None:
             y = y + residual
-        if epilogue == EPI_RELU2:
-            y = relu2(y)
+        if epilogue in (EPI_RELU2, EPI_GELU):
+            y = ungated_act(y, "relu2" if epilogue == EPI_RELU2 else "gelu")
         out.copy_(y)
         return out
     if (USE_PAIR_GEMM and PAIR_MIN_M <= M < WIDE2_MIN_M and Nn % 256 == 0 and K % 64 == 0
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2)
+            and epilogue in _PAIR_EPI
             and -(-M // 256) * (Nn // 256) >= PAIR_MIN_TILES):
         # enough 256 x 256 tiles to occupy the SM pairs (gate_up, LM head at decode batch sizes;
         # graph-replay timing at 256 rows: gate_up 62.5 -> 57.9 us, LM head 266 -> 228 us)
@@ -195,7 +204,7 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
         if rc != -20:
             raise N.NativeError(f"b200_gemm_pair failed with code {rc}")
     if (USE_PAIR_SPLIT and PAIR_MIN_M <= M <= 512 and Nn % 256 == 0 and K % 64 == 0
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL)
+            and epilogue in _WIDE_EPI
             and -(-M // 256) * (Nn // 256) < PAIR_MIN_TILES):
         # few 256 x 256 tiles (qkv, o_proj, down_proj at decode batch sizes): K split over pairs
         wsp = _pair_split_workspace(a.device)
@@ -208,9 +217,9 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
                 return out
             if rc != -20:
                 raise N.NativeError(f"b200_gemm_pair_split failed with code {rc}")
-    silu_256 = epilogue != EPI_SILU_MUL or Nn % 256 == 0     # these two kernels: 256-wide tiles
-    if M <= SKINNY_MAX_M and USE_SKINNY_GEMM and silu_256 \
-            and (epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2)
+    gated_256 = epilogue not in _GATED or Nn % 256 == 0      # these two kernels: 256-wide tiles
+    if M <= SKINNY_MAX_M and USE_SKINNY_GEMM and gated_256 \
+            and (epilogue in _PAIR_EPI
                  or epilogue == EPI_FP32 and M <= SKINNY_SPLIT2_MAX_M):
         ws, ctr = _skinny_workspace(a.device)
         rc = N.lib().b200_gemm_skinny(
@@ -224,7 +233,7 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
         if rc != -20:
             raise N.NativeError(f"b200_gemm_skinny failed with code {rc}")
     if (USE_PAIR_GEMM and M >= WIDE2_MIN_M and Nn % 256 == 0 and K % 64 == 0
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL, EPI_RELU2) and _wide2_pays(M, Nn)):
+            and epilogue in _PAIR_EPI and _wide2_pays(M, Nn)):
         # one 256 x 256 tile per pair of CTAs (gemm_pair.cu); -20 = shape or device not covered
         rc = N.lib().b200_gemm_pair(ptr(a), a.stride(0), ptr(b), b.stride(0), ptr(out),
                                     out.stride(0), M, Nn, K, ptr(bias), epilogue, stream_ptr())
@@ -234,7 +243,7 @@ def _gemm_bf16(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = N
         if rc != -20:
             raise N.NativeError(f"b200_gemm_pair failed with code {rc}")
     if (USE_WIDE2_GEMM and M >= WIDE2_MIN_M and Nn % 256 == 0
-            and epilogue in (EPI_NONE, EPI_BIAS, EPI_SILU_MUL) and _wide2_pays(M, Nn)):
+            and epilogue in _WIDE_EPI and _wide2_pays(M, Nn)):
         rc = N.lib().b200_gemm_wide2(ptr(a), a.stride(0), ptr(b), b.stride(0), ptr(out),
                                      out.stride(0), M, Nn, K, ptr(bias), epilogue, stream_ptr())
         N.launch_count += 1
@@ -455,12 +464,13 @@ def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                  max_seq_len: int = 0, kv_quant: Optional[tuple] = None,
                  alibi_slopes: Optional[torch.Tensor] = None,
                  sink: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
-                 out_dim: int = 0) -> torch.Tensor:
+                 out_dim: int = 0, window: int = 0, slopes: Optional[torch.Tensor] = None
+                 ) -> torch.Tensor:
     res = _paged_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, out, num_splits,
                         workspace, max_seq_len, kv_quant, alibi_slopes, sink, softcap, chunk,
-                        out_dim)
+                        out_dim, window, slopes)
     if (oracle_enabled("paged_decode") and k_cache.element_size() > 1 and alibi_slopes is None
-            and sink is None and not softcap and not chunk and not out_dim
+            and sink is None and not (softcap or chunk or out_dim or window) and slopes is None
             and not torch.cuda.is_current_stream_capturing()):
         from . import ref
         live = seq_lens > 0
@@ -477,13 +487,16 @@ def _paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                   max_seq_len: int = 0, kv_quant: Optional[tuple] = None,
                   alibi_slopes: Optional[torch.Tensor] = None,
                   sink: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
-                  out_dim: int = 0) -> torch.Tensor:
+                  out_dim: int = 0, window: int = 0, slopes: Optional[torch.Tensor] = None
+                  ) -> torch.Tensor:
     """q ``[B, Hq, D]`` (row stride free), caches ``[blocks, bs, Hkv, D]``.  For fp8 / int8
     caches ``kv_quant = (k_scale, v_scale, k_zero_point, v_zero_point)`` (floats).
     ``alibi_slopes`` fp32 ``[Hq]`` adds slope * (key position - query position) to the scores
     (bf16 / fp16 caches).  ``sink`` fp32 ``[Hq]``: exp(sink) joins the softmax denominator.
     ``softcap``: scores become softcap * tanh(score / softcap).  ``chunk``: only the keys of the
-    query's own chunk of positions.  ``out_dim``: only the first columns of every head's output."""
+    query's own chunk of positions.  ``out_dim``: only the first columns of every head's output.
+    ``window``: only the last keys up to the query.  ``slopes``: ``alibi_slopes`` together with any of
+    these."""
     B, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
     od = out_dim or D
@@ -512,11 +525,11 @@ def _paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
         assert alibi_slopes.dtype == torch.float32 and alibi_slopes.numel() == Hq
         call("b200_paged_decode_alibi", *args[:-1], ptr(alibi_slopes), stream_ptr())
         return out
-    if sink is not None or softcap or chunk or od != D:
+    if sink is not None or softcap or chunk or window or slopes is not None or od != D:
         if k_cache.element_size() == 1:
             raise NotImplementedError("attention sinks, caps and chunks over an 8-bit KV cache")
         assert sink is None or (sink.dtype == torch.float32 and sink.numel() == Hq)
-        tail = (ptr(sink), float(softcap), int(chunk), od, stream_ptr())
+        tail = (ptr(sink), float(softcap), int(chunk), int(window), ptr(slopes), od, stream_ptr())
         if USE_TMA_DECODE and D == 128 and bs % 16 == 0 and k_cache.stride(2) == 128 \
                 and k_cache.stride(1) == Hkv * 128:
             rc = N.lib().b200_paged_decode_tma_sink(*args[:-1], *tail)
@@ -624,9 +637,10 @@ def fmha_prefill_sink(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                       block_tables: torch.Tensor, cu_q: torch.Tensor, seq_lens: torch.Tensor,
                       scale: float, num_q_tiles_128: int, sink: Optional[torch.Tensor],
                       out: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
-                      out_dim: int = 0) -> Optional[torch.Tensor]:
+                      out_dim: int = 0, window: int = 0, slopes: Optional[torch.Tensor] = None
+                      ) -> Optional[torch.Tensor]:
     """Causal tcgen05 prefill attention for head dimensions 64, 96 and 128 with optional sinks, soft
-    cap, chunks and output columns (see ``paged_decode``); None when the layout is not covered (then
+    cap, chunks, window, slopes and output columns (see ``paged_decode``); None when the layout is not covered (then
     use ``any_attention``)."""
     T, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
@@ -639,8 +653,8 @@ def fmha_prefill_sink(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         ptr(q), q.stride(0), ptr(out), out.stride(0), None, ptr(cu_q), ptr(seq_lens), ptr(k_cache),
         ptr(v_cache), k_cache.stride(1), k_cache.stride(2), nb * bs, ptr(block_tables),
         block_tables.stride(0), bs, block_tables.shape[0], T, num_q_tiles_128, Hq, Hkv, D,
-        float(scale), 1, 0, DTYPE_CODE[q.dtype], ptr(sink), float(softcap), int(chunk), od,
-        stream_ptr())
+        float(scale), 1, int(window), DTYPE_CODE[q.dtype], ptr(sink), float(softcap), int(chunk),
+        ptr(slopes), od, stream_ptr())
     N.launch_count += 1
     if rc == -20:
         return None
@@ -653,10 +667,12 @@ def any_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                   block_tables: torch.Tensor, seq_lens: torch.Tensor, num_decodes: int,
                   cu_q: Optional[torch.Tensor], scale: float, sink: Optional[torch.Tensor] = None,
                   out: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0,
-                  out_dim: int = 0) -> torch.Tensor:
+                  out_dim: int = 0, window: int = 0, slopes: Optional[torch.Tensor] = None
+                  ) -> torch.Tensor:
     """Causal paged attention for any head dimension (<= 512) and group size, fp32 or bf16
     (csrc/attention_any.cu): q ``[T, Hq, D]``, the first ``num_decodes`` tokens one per request,
-    the rest by ``cu_q``.  ``softcap``, ``chunk``, ``out_dim``: see ``paged_decode``."""
+    the rest by ``cu_q``.  ``softcap``, ``chunk``, ``out_dim``, ``window``, ``slopes``: see
+    ``paged_decode``."""
     T, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
     od = out_dim or D
@@ -668,7 +684,42 @@ def any_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
     call("b200_any_attention", ptr(q), ptr(k_cache), ptr(v_cache), nb * bs, ptr(out),
          out.stride(0), od, ptr(block_tables), block_tables.stride(0), bs, ptr(seq_lens), ptr(cu_q),
          ptr(sink), T, Hq, Hkv, D, num_decodes, cu_q.shape[0] - 1 if cu_q is not None else 0,
-         float(scale), float(softcap), int(chunk), DTYPE_CODE[q.dtype], stream_ptr())
+         float(scale), float(softcap), int(chunk), int(window), ptr(slopes), DTYPE_CODE[q.dtype],
+         stream_ptr())
+    return out
+
+
+def qkv_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_weight: Optional[torch.Tensor],
+              k_weight: Optional[torch.Tensor], eps: float, cos_sin: Optional[torch.Tensor],
+              positions: torch.Tensor, slot_mapping: torch.Tensor, k_cache: torch.Tensor,
+              v_cache: torch.Tensor, head_dim: int, v_dim: int, v_norm: bool = False,
+              temp: tuple[float, int] = (0.0, 1), sumsq: Optional[torch.Tensor] = None,
+              ranks: int = 1, share: Optional[torch.Tensor] = None,
+              first: Optional[torch.Tensor] = None, first_dim: int = 0) -> torch.Tensor:
+    """What grouped attention needs of its projections ``q [T, Hq * D]``, ``k [T, Hkv * D]``, ``v [T,
+    Hkv * VD]`` (row-strided views are fine), in one pass; each optional: RMS norm of the whole query
+    and key rows (``q_weight`` / ``k_weight``; ``sumsq [T, 2]`` and ``ranks`` as in
+    :func:`qk_norm_rope_cache`), rotation of the first ``cos_sin.shape[1]`` dimensions of every head
+    (i with i + half), queries times ``1 + temp[0] * ln(floor((p + 1) / temp[1]) + 1)``, values of
+    every head divided by their root mean square, values mixed as ``(1 - share) * v + share * first``
+    with what the cache ``first [blocks, bs, heads, DC']`` holds for the token in the first
+    ``first_dim`` columns of its heads.  Keys and values go into the paged caches with zeros behind
+    their columns.  Returns the queries ``[T, Hq, DC]``."""
+    T = q.shape[0]
+    nb, bs, Hkv, DC = k_cache.shape
+    Hq = q.shape[1] // head_dim
+    assert q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == q.dtype
+    assert first is None or (first.is_contiguous() and first.dtype == q.dtype)
+    out = torch.empty((T, Hq, DC), dtype=q.dtype, device=q.device)
+    call("b200_qkv_cache", ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v), v.stride(0),
+         ptr(q_weight), ptr(k_weight), ptr(sumsq), Hq * head_dim * ranks, Hkv * head_dim * ranks,
+         float(eps), ptr(cos_sin), cos_sin.shape[1] if cos_sin is not None else 0,
+         cos_sin.shape[0] if cos_sin is not None else 0, float(temp[0]), int(temp[1]), int(v_norm),
+         ptr(share), ptr(first), first.stride(1) if first is not None else 0, first_dim,
+         first.shape[3] if first is not None else 0, ptr(positions), ptr(slot_mapping), ptr(out),
+         ptr(k_cache), ptr(v_cache), nb * bs, T, Hq, Hkv, head_dim, v_dim, DC, DTYPE_CODE[q.dtype],
+         stream_ptr())
     return out
 
 
@@ -933,6 +984,52 @@ def add_normed(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor,
          float(final_scale), ptr(lo), T, H, DTYPE_CODE[y.dtype], stream_ptr())
 
 
+def add_group_norm(x: torch.Tensor, y: Optional[torch.Tensor], mult: float, weight: torch.Tensor,
+                   groups: int, eps: float, lo: torch.Tensor, out: Optional[torch.Tensor] = None,
+                   pos_of: Optional[torch.Tensor] = None, row_w: Optional[torch.Tensor] = None,
+                   shared: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                   conv: Optional[tuple] = None) -> None:
+    """``s = x + mult * y`` with ``x [T, H]`` fp32, or rows of the model's type (y may be None);
+    ``out`` takes s (may be ``x``), ``lo`` takes s with each of ``groups`` consecutive parts of a row
+    divided by its root mean square, times ``weight``.  ``pos_of`` / ``row_w`` / ``shared`` /
+    ``gate``: y as the sum of expert rows, see :func:`add_normed`.
+
+    ``conv = (weight, mu, positions, slots, ring, rows, n)``: the first n rows (single tokens) go on
+    through the convolution of :func:`input_conv` into ``rows``, not into ``lo``."""
+    T, H = x.shape
+    f32 = x.dtype == torch.float32 and lo.dtype != torch.float32 or y is not None
+    w, mu, pos, slots, ring, rows, n1 = conv if conv is not None else (None,) * 6 + (0,)
+    call("b200_add_group_norm", ptr(x) if f32 else None, None if f32 else ptr(x),
+         x.stride(0), ptr(y), y.stride(0) if y is not None else 0, float(mult), ptr(pos_of),
+         ptr(row_w), row_w.shape[1] if row_w is not None else 0, ptr(shared),
+         shared.stride(0) if shared is not None else 0, ptr(gate),
+         gate.stride(0) if gate is not None else 0, ptr(weight), groups, float(eps), ptr(out),
+         ptr(lo), ptr(w), w.shape[0] if w is not None else 0, ptr(mu),
+         mu.shape[0] if mu is not None else 0, ptr(ring), ring.shape[0] if ring is not None else 0,
+         ptr(pos), ptr(slots), ptr(rows), rows.stride(0) if mu is not None else 0,
+         rows.stride(-2) if rows is not None else 0, n1, T, H, DTYPE_CODE[lo.dtype], stream_ptr())
+
+
+def input_conv(h: torch.Tensor, weight: torch.Tensor, mu: Optional[torch.Tensor], md,
+               ring: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """``c = h + sum_j weight[j] * (h of taps - 1 - j tokens ago)`` over the portions of a step, ``h [T,
+    H]``, ``weight [taps, H]`` fp32; with ``mu [M, H]`` the mixtures ``c + (c' - c) * mu_m`` with the
+    row c' of the token before take c's place.  ``ring [slots, taps - 1 (with mu: taps), H]`` holds a
+    request's last rows by position, addressed by ``md.state_slots`` (None: zeros in front of the
+    portions); ``md`` also gives ``positions``, ``num_decode_tokens`` and ``cu_q_prefill``.  ``out``:
+    ``[T, H]`` or ``[M, T, H]`` (row-strided views are fine)."""
+    T, H = h.shape
+    nd, npf, cu = _scan_place(md)
+    if nd + npf == 0 or md.state_slots is None:
+        out.zero_()
+        return
+    call("b200_input_conv", ptr(h), ptr(weight), weight.shape[0], ptr(mu),
+         mu.shape[0] if mu is not None else 0, ptr(ring), ring.shape[0] if ring is not None else 0,
+         ptr(md.positions), ptr(md.state_slots), ptr(cu), ptr(out),
+         out.stride(0) if mu is not None else 0, out.stride(-2), T, H, nd, npf,
+         DTYPE_CODE[h.dtype], stream_ptr())
+
+
 def head_gate(o: torch.Tensor, z: torch.Tensor, scale: float, head_dim: int, out: torch.Tensor
               ) -> torch.Tensor:
     """``out = o * sigmoid(z) * scale`` with ``o [T, N, DC >= head_dim]`` and ``z``, ``out``
@@ -947,22 +1044,23 @@ def head_gate(o: torch.Tensor, z: torch.Tensor, scale: float, head_dim: int, out
 # ---------------------------------------------------------------------------
 # gated activation of any width
 # ---------------------------------------------------------------------------
-def silu_mul_rows(x: torch.Tensor) -> torch.Tensor:
-    """``silu(x[:, :D]) * x[:, D:]`` for rows of any width, bf16 or fp32."""
+def act_mul_rows(x: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """``act(x[:, :D]) * x[:, D:]`` ("silu" or "gelu_tanh") for rows of any width, bf16 or fp32."""
     shape = x.shape
     x2 = _rowmajor_2d(x)
     T, D = x2.shape[0], x2.shape[1] // 2
     out = torch.empty((T, D), dtype=x.dtype, device=x.device)
-    call("b200_silu_mul_rows", ptr(x2), x2.stride(0), ptr(out), D, T, D, DTYPE_CODE[x.dtype],
-         stream_ptr())
+    call("b200_act_mul_rows", ptr(x2), x2.stride(0), ptr(out), D, T, D, GATED_EPI[act],
+         DTYPE_CODE[x.dtype], stream_ptr())
     return out.view(*shape[:-1], D)
 
 
-def relu2(x: torch.Tensor) -> torch.Tensor:
-    """``max(x, 0)^2`` in place, bf16 or fp32."""
+def ungated_act(x: torch.Tensor, act: str) -> torch.Tensor:
+    """``max(x, 0)^2`` ("relu2") or GELU through the error function ("gelu") in place, bf16 or
+    fp32."""
     x2 = x if x.dim() == 2 else x.view(-1, x.shape[-1])
-    call("b200_relu2", ptr(x2), x2.stride(0), ptr(x2), x2.stride(0), x2.shape[0], x2.shape[1],
-         DTYPE_CODE[x.dtype], stream_ptr())
+    call("b200_ungated_act", ptr(x2), x2.stride(0), ptr(x2), x2.stride(0), x2.shape[0],
+         x2.shape[1], UNGATED_EPI[act], DTYPE_CODE[x.dtype], stream_ptr())
     return x
 
 
@@ -1041,15 +1139,70 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, zi: torch.T
 
 def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, z: torch.Tensor, eps: float,
                    scale: float, out: torch.Tensor, nq: Optional[torch.Tensor] = None,
-                   low: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``out = o / rms(o) * weight * sigmoid(z) * scale`` with ``o [T, N, V]`` fp32 normalised per
+                   low: Optional[torch.Tensor] = None, act: str = "sigmoid") -> torch.Tensor:
+    """``out = o / rms(o) * weight * act(z) * scale`` ("sigmoid" or "silu") with ``o [T, N, V]`` fp32 normalised per
     head, ``weight`` ``[V]`` or ``[N * V]``, ``z`` and ``out`` ``[T, N * V]`` (views are fine).  With
     ``nq`` and ``low`` (:func:`matrix_memory`) o is divided first."""
     T, Nh, V = o.shape
     assert z.stride(1) == 1 and out.stride(1) == 1 and z.dtype == out.dtype
     call("b200_head_norm_gate", ptr(o), ptr(nq), ptr(low), ptr(weight), int(weight.numel() != V),
          ptr(z), z.stride(0), ptr(out), out.stride(0), float(eps), float(scale), T, Nh, V,
-         DTYPE_CODE[out.dtype], stream_ptr())
+         int(act == "silu"), DTYPE_CODE[out.dtype], stream_ptr())
+    return out
+
+
+def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, base: torch.Tensor,
+        bonus: torch.Tensor, head_dim: int, rows: int, md, state: Optional[torch.Tensor]
+        ) -> torch.Tensor:
+    """Time mixing over the portions of a step: r, k, v projections ``[T, N * head_dim]`` (views of one
+    row), ``z`` fp32 the decay's, decays ``exp(-exp(z + base))``; per head ``o = S^T r + (r . (bonus k))
+    v``, then ``S = decay S + k v^T``.  ``state [slots, N, head_dim, rows]`` fp32, addressed by
+    ``md.state_slots``.  Returns fp32 ``[T, N, head_dim]``."""
+    T, D = r.shape[0], head_dim
+    Nh = r.shape[1] // D
+    VP = -(-D // 4) * 4
+    assert r.stride(0) == k.stride(0) == v.stride(0) and z.dtype == torch.float32
+    new = lambda *s: torch.empty(s, dtype=torch.float32, device=r.device)  # noqa: E731
+    out = new(T, Nh, D)
+    if state is None:
+        return out.zero_()
+    ro, ko, go, vo, now = new(T, Nh, rows), new(T, Nh, rows), new(T, Nh, rows), new(T, Nh, VP), \
+        new(T, Nh)
+    nd, npf, cu = _scan_place(md)
+    call("b200_wkv_inputs", ptr(r), ptr(k), ptr(v), r.stride(0), ptr(z), z.stride(0), ptr(base),
+         ptr(bonus), ptr(ro), ptr(ko), ptr(go), ptr(vo), ptr(now), T, Nh, D, rows, VP,
+         DTYPE_CODE[r.dtype], stream_ptr())
+    call("b200_wkv_scan", ptr(ro), ptr(ko), ptr(go), ptr(vo), ptr(now), ptr(out), ptr(state),
+         ptr(md.positions), ptr(md.state_slots), state.shape[0], ptr(cu), Nh, D, rows, VP, nd, npf,
+         stream_ptr())
+    return out
+
+
+def tanh_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """tanh of contiguous fp32 rows, in ``dtype``."""
+    assert x.is_contiguous() and x.dtype == torch.float32
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+    call("b200_tanh_rows", ptr(x), ptr(out), x.numel(), DTYPE_CODE[dtype], stream_ptr())
+    return out
+
+
+def wkv_step(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor,
+             inner: torch.Tensor, w2: torch.Tensor, base: torch.Tensor, bonus: torch.Tensor,
+             norm: torch.Tensor, head_dim: int, rows: int, positions: torch.Tensor,
+             slots: torch.Tensor, state: torch.Tensor, eps: float, out: torch.Tensor
+             ) -> torch.Tensor:
+    """One token of every request through time mixing in one kernel: :func:`wkv` and
+    :func:`head_norm_gate` (SiLU gate), with the second step of the decay's projection included:
+    ``z = tanh(inner) @ w2^T``, ``inner [nd, R]`` fp32."""
+    nd, D = r.shape[0], head_dim
+    Nh = r.shape[1] // D
+    ld = r.stride(0)
+    assert all(t.stride(0) == ld and t.stride(1) == 1 for t in (k, v, gate))
+    assert w2.is_contiguous() and w2.dtype == r.dtype and inner.dtype == torch.float32
+    call("b200_wkv_step", ptr(r), ptr(k), ptr(v), ptr(gate), ld, ptr(inner), inner.stride(0),
+         w2.shape[1], ptr(w2), ptr(base), ptr(bonus), ptr(norm), ptr(state), ptr(positions),
+         ptr(slots), state.shape[0], ptr(out), out.stride(0), float(eps), nd, Nh, D, rows,
+         DTYPE_CODE[r.dtype], stream_ptr())
     return out
 
 
@@ -1188,8 +1341,8 @@ def moe_align(topk_ids: torch.Tensor, num_local_experts: int, cap: Optional[int]
 def gemm_bf16_grouped(a: torch.Tensor, w: torch.Tensor, expert_ids: torch.Tensor,
                       num_valid_rows: torch.Tensor, silu_mul: bool = False,
                       row_scale: Optional[torch.Tensor] = None,
-                      out: Optional[torch.Tensor] = None, relu2: bool = False) -> torch.Tensor:
-    """a ``[M_cap, K]`` expert-sorted rows, w ``[E, N, K]``."""
+                      out: Optional[torch.Tensor] = None, act: str = "") -> torch.Tensor:
+    """a ``[M_cap, K]`` expert-sorted rows, w ``[E, N, K]``; ``act``: see :func:`ungated_act`."""
     M_cap, K = a.shape
     E, Nn, _ = w.shape
     assert w.is_contiguous() and a.stride(1) == 1
@@ -1198,7 +1351,7 @@ def gemm_bf16_grouped(a: torch.Tensor, w: torch.Tensor, expert_ids: torch.Tensor
         out = torch.empty((M_cap, out_cols), device=a.device, dtype=torch.bfloat16)
     call("b200_gemm_bf16_grouped", ptr(a), a.stride(0), ptr(w), K, ptr(out), out.stride(0), M_cap,
          Nn, K, E, ptr(expert_ids), ptr(num_valid_rows), ptr(row_scale),
-         EPI_SILU_MUL if silu_mul else EPI_RELU2 if relu2 else EPI_NONE, stream_ptr())
+         EPI_SILU_MUL if silu_mul else UNGATED_EPI.get(act, EPI_NONE), stream_ptr())
     return out
 
 
@@ -1264,9 +1417,9 @@ def input_weighted_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor,
     return y, pos_of
 
 
-def squared_relu_experts(x: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor,
-                         topk_ids: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
-    """Routed experts without a gate, ``down(max(up(x), 0)^2)``: align -> permute rows ``x [T, H]`` ->
+def ungated_experts(x: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor, topk_ids: torch.Tensor,
+                    act: str = "relu2") -> tuple[torch.Tensor, torch.Tensor]:
+    """Routed experts without a gate, ``down(act(up(x)))``: align -> permute rows ``x [T, H]`` ->
     grouped GEMM1 with the activation in its epilogue -> grouped GEMM2.  ``w1 [E, I, Hp]``, ``w2
     [E, Hp, I]`` with Hp >= H padded by zeros.  Returns the expert-sorted outputs ``[cap, Hp]``, not
     weighted, and ``pos_of [T * k]``; ``add_normed`` weights and sums them."""
@@ -1284,12 +1437,12 @@ def squared_relu_experts(x: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor,
         call("b200_moe_permute_any", ptr(x), x.stride(0), ptr(a_sorted), Hp, ptr(sorted_ids),
              ptr(npp), numel, k, H, Hp, cap, DTYPE_CODE[x.dtype], stream_ptr())
     if x.dtype == torch.bfloat16:
-        h = gemm_bf16_grouped(a_sorted, w1, expert_ids, npp, relu2=True)
+        h = gemm_bf16_grouped(a_sorted, w1, expert_ids, npp, act=act)
         return gemm_bf16_grouped(h, w2, expert_ids, npp), pos_of
     h = torch.empty((cap, I), device=x.device, dtype=torch.float32)
     call("b200_grouped_gemm_f32", ptr(a_sorted), Hp, ptr(w1), ptr(h), I, cap, I, Hp, E,
          ptr(expert_ids), ptr(npp), stream_ptr())
-    call("b200_relu2_rows_f32", ptr(h), ptr(h), cap, I, ptr(npp), stream_ptr())
+    call("b200_ungated_rows_f32", ptr(h), ptr(h), cap, I, ptr(npp), UNGATED_EPI[act], stream_ptr())
     y = torch.empty((cap, Hp), device=x.device, dtype=torch.float32)
     call("b200_grouped_gemm_f32", ptr(h), I, ptr(w2), ptr(y), Hp, cap, Hp, I, E, ptr(expert_ids),
          ptr(npp), stream_ptr())

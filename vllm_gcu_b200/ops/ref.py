@@ -703,13 +703,7 @@ def add_normed(x, y, weight, bias, eps, lo, out=None, layer_norm=True, final_wei
                gate=None) -> None:
     """See ``ops.cuda.add_normed``."""
     if pos_of is not None:
-        T, k = row_w.shape
-        pos = pos_of.view(-1)[:T * k].view(T, k).long()
-        w = (row_w * (pos >= 0)).unsqueeze(-1)
-        y = (y[pos.clamp(min=0)].float() * w).sum(1)[:, :x.shape[1]]
-        if shared is not None:
-            g = 1.0 if gate is None else torch.sigmoid(gate.float()).unsqueeze(-1)
-            y = y + g * shared.float()
+        y = _routed_rows(y, x.shape[1], pos_of, row_w, shared, gate)
 
     def norm(r, w, b):
         if layer_norm:
@@ -725,15 +719,63 @@ def add_normed(x, y, weight, bias, eps, lo, out=None, layer_norm=True, final_wei
     lo.copy_(s if final_weight is None else norm(s, final_weight, final_bias) * final_scale)
 
 
+def _routed_rows(y, width, pos_of, row_w, shared, gate) -> torch.Tensor:
+    """fp32 sum of every token's weighted expert rows and its shared row."""
+    T, k = row_w.shape
+    pos = pos_of.view(-1)[:T * k].view(T, k).long()
+    w = (row_w * (pos >= 0)).unsqueeze(-1)
+    y = (y[pos.clamp(min=0)].float() * w).sum(1)[:, :width]
+    if shared is not None:
+        g = 1.0 if gate is None else torch.sigmoid(gate.float()).unsqueeze(-1)
+        y = y + g * shared.float()
+    return y
+
+
+def add_group_norm(x, y, mult, weight, groups, eps, lo, out=None, pos_of=None, row_w=None,
+                   shared=None, gate=None, conv=None) -> None:
+    """See ``ops.cuda.add_group_norm`` (every row goes to ``lo``: no fused convolution here)."""
+    s = x.float()
+    if y is not None:
+        if pos_of is not None:
+            y = _routed_rows(y, x.shape[1], pos_of, row_w, shared, gate)
+        s = s + mult * y.float()
+    if out is not None:
+        out.copy_(s)
+    p = s.unflatten(1, (groups, -1))
+    lo.copy_((p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) * weight)
+
+
+def input_conv(h, weight, mu, md, state, out) -> None:
+    """See ``ops.cuda.input_conv``."""
+    n = weight.shape[0]
+    back = n - (mu is None)                   # earlier rows that a row's result depends on
+    out.zero_()
+    for lo, hi, slot, fresh in _recurrent_portions(h.shape[0], md) if state is not None or \
+            back == 0 else ():
+        p0 = int(md.positions[lo])
+        ring = state[slot] if back else None
+        past = [ring[p % back].float() if p >= 0 else torch.zeros(h.shape[1])
+                for p in range(p0 - back, p0)]
+        seq = torch.cat([torch.stack(past), h[lo:hi].float()]) if past else h[lo:hi].float()
+        c = seq[n - 1:] + sum(weight[j] * seq[j:seq.shape[0] - n + 1 + j] for j in range(n))
+        if mu is None:
+            out[lo:hi] = c.to(out.dtype)
+        else:
+            now, before = c[1:], c[:-1]
+            out[:, lo:hi] = (now + (before - now) * mu[:, None]).to(out.dtype)
+        for t in range(max(lo, hi - back), hi):
+            ring[(p0 + t - lo) % back] = h[t]
+
+
 def head_gate(o, z, scale, head_dim, out) -> torch.Tensor:
     """See ``ops.cuda.head_gate``."""
     out.copy_(o[..., :head_dim].flatten(1).float() * torch.sigmoid(z.float()) * scale)
     return out
 
 
-def relu2(x: torch.Tensor) -> torch.Tensor:
-    """See ``ops.cuda.relu2``."""
-    return x.clamp_(min=0).square_()
+def ungated_act(x: torch.Tensor, act: str) -> torch.Tensor:
+    """See ``ops.cuda.ungated_act``."""
+    return x.clamp_(min=0).square_() if act == "relu2" else _act(act, x.float()).to(x.dtype)
 
 
 def head_norm_cache(q, k, v, q_weight, k_weight, eps, slot_mapping, k_cache, v_cache, head_dim
@@ -773,8 +815,44 @@ def qk_norm_rope_cache(q, k, v, q_weight, k_weight, eps, cos_sin, is_neox, posit
     return pad(qn).to(q.dtype)
 
 
+def qkv_cache(q, k, v, q_weight, k_weight, eps, cos_sin, positions, slot_mapping, k_cache, v_cache,
+              head_dim, v_dim, v_norm=False, temp=(0.0, 1), sumsq=None, ranks=1, share=None,
+              first=None, first_dim=0) -> torch.Tensor:
+    """See ``ops.cuda.qkv_cache``."""
+    T, D, VD = q.shape[0], head_dim, v_dim
+    nb, bs, Hkv, DC = k_cache.shape
+
+    def norm(x, w, i):
+        f = x.float()
+        if w is None:
+            return f
+        ss = f.pow(2).sum(-1) if sumsq is None else sumsq[:, i]
+        return f * torch.rsqrt(ss[:, None] / (x.shape[1] * ranks) + eps) * w
+
+    qn, kn = norm(q, q_weight, 0), norm(k, k_weight, 1)
+    if cos_sin is not None:
+        qn, kn = rotary_embedding(positions, qn, kn, D, cos_sin, True)
+    if temp[0]:
+        qn = qn * (1.0 + temp[0] * torch.log(
+            torch.div(positions + 1, temp[1], rounding_mode="floor").float() + 1.0))[:, None]
+    vf = v.float().view(T, Hkv, VD)
+    if v_norm:
+        vf = vf * torch.rsqrt(vf.pow(2).mean(-1, keepdim=True) + eps)
+    pad = lambda x: torch.nn.functional.pad(x, (0, DC - x.shape[-1]))  # noqa: E731
+    ok = slot_mapping >= 0
+    at = slot_mapping[ok].long()
+    vf = vf[ok]
+    if first is not None:
+        f = first.reshape(nb * bs, first.shape[2], first.shape[3])[at][..., :first_dim].float()
+        vf = (1.0 - share) * vf + share * f.reshape(vf.shape)
+    k_cache.view(nb * bs, Hkv, DC)[at] = pad(kn.view(T, Hkv, D))[ok].to(k_cache.dtype)
+    v_cache.view(nb * bs, Hkv, DC)[at] = pad(vf).to(v_cache.dtype)
+    return pad(qn.view(T, -1, D)).to(q.dtype)
+
+
 def any_attention(q, k_cache, v_cache, block_tables, seq_lens, num_decodes, cu_q, scale, sink=None,
-                  out=None, softcap=0.0, chunk=0, out_dim=0) -> torch.Tensor:
+                  out=None, softcap=0.0, chunk=0, out_dim=0, window=0, slopes=None
+                  ) -> torch.Tensor:
     """See ``ops.cuda.any_attention``."""
     T, Hq, D = q.shape
     od = out_dim or D
@@ -789,11 +867,17 @@ def any_attention(q, k_cache, v_cache, block_tables, seq_lens, num_decodes, cu_q
         s = torch.einsum("qhd,nhd->hqn", q[lo:hi].float(), k) * scale
         if softcap:
             s = softcap * torch.tanh(s / softcap)
+        if slopes is not None:
+            back = torch.arange(n - (hi - lo), n, device=q.device)[:, None] - \
+                torch.arange(n, device=q.device)[None, :]
+            s = s - slopes[:, None, None] * back
         qpos = torch.arange(n - (hi - lo), n, device=q.device)[:, None]
         kpos = torch.arange(n, device=q.device)[None, :]
         hidden = kpos > qpos
         if chunk:
             hidden = hidden | (kpos // chunk != qpos // chunk)
+        if window:
+            hidden = hidden | (kpos <= qpos - window)
         s = s.masked_fill(hidden[None], float("-inf"))
         if sink is not None:
             s = torch.cat([s, sink.float()[:, None, None].expand(-1, hi - lo, 1)], dim=-1)
@@ -885,14 +969,41 @@ def matrix_memory(q, k, v, zi, zf, i_bias, f_bias, cap, head_dim, v_dim, rows, m
     return out, nqs, low
 
 
-def head_norm_gate(o, weight, z, eps, scale, out, nq=None, low=None) -> torch.Tensor:
+def wkv(r, k, v, z, base, bonus, head_dim, rows, md, state) -> torch.Tensor:
+    """See ``ops.cuda.wkv``."""
+    T, D = r.shape[0], head_dim
+    Nh = r.shape[1] // D
+    out = torch.zeros(T, Nh, D, dtype=torch.float32, device=r.device)
+    if state is None:
+        return out
+    decay = torch.exp(-torch.exp(z + base)).view(T, Nh, D)
+    rf, kf, vf = (t.float().reshape(T, Nh, D) for t in (r, k, v))
+    now = (rf * bonus.view(Nh, D) * kf).sum(-1)
+    for lo, hi, slot, fresh in _recurrent_portions(T, md):
+        S = state[slot, :, :, :D]                              # [N, values, keys], a view
+        S = torch.zeros_like(S) if fresh else S.clone()
+        for t in range(lo, hi):
+            out[t] = (S * rf[t][:, None, :]).sum(-1) + now[t][:, None] * vf[t]
+            S = S * decay[t][:, None, :] + vf[t][:, :, None] * kf[t][:, None, :]
+        state[slot, :, :, :D] = S
+    return out
+
+
+def tanh_rows(x, dtype) -> torch.Tensor:
+    """See ``ops.cuda.tanh_rows``."""
+    return torch.tanh(x).to(dtype)
+
+
+def head_norm_gate(o, weight, z, eps, scale, out, nq=None, low=None, act="sigmoid"
+                   ) -> torch.Tensor:
     """See ``ops.cuda.head_norm_gate``."""
     T, Nh, V = o.shape
     if nq is not None:
         o = o / (torch.maximum(nq.abs(), low) + 1e-6).unsqueeze(-1)
     r = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
     r = r * (weight.view(Nh, V) if weight.numel() != V else weight)
-    out.copy_(r.flatten(1) * torch.sigmoid(z.float()) * scale)
+    g = torch.sigmoid(z.float())
+    out.copy_(r.flatten(1) * (g * z.float() if act == "silu" else g) * scale)
     return out
 
 
@@ -914,8 +1025,8 @@ def input_weighted_experts(x, w13, w2, topk_w, topk_ids) -> tuple[torch.Tensor, 
     return y, torch.arange(T * k, dtype=torch.int32, device=x.device)
 
 
-def squared_relu_experts(x, w1, w2, topk_ids) -> tuple[torch.Tensor, torch.Tensor]:
-    """See ``ops.cuda.squared_relu_experts``; one output row per (token, slot) pair, so ``pos_of``
+def ungated_experts(x, w1, w2, topk_ids, act="relu2") -> tuple[torch.Tensor, torch.Tensor]:
+    """See ``ops.cuda.ungated_experts``; one output row per (token, slot) pair, so ``pos_of``
     is the identity."""
     T, H = x.shape
     k = topk_ids.shape[1]
@@ -926,7 +1037,7 @@ def squared_relu_experts(x, w1, w2, topk_ids) -> tuple[torch.Tensor, torch.Tenso
     for e in range(w1.shape[0]):
         rows = (flat == e).nonzero(as_tuple=True)[0]
         if rows.numel():
-            y[rows] = relu2(a[rows // k] @ w1[e].t()) @ w2[e].t()
+            y[rows] = ungated_act(a[rows // k] @ w1[e].t(), act) @ w2[e].t()
     return y, torch.arange(T * k, dtype=torch.int32, device=x.device)
 
 
