@@ -246,3 +246,73 @@ def forward(config: dict, weights: dict, tokens, dtype=torch.float64) -> torch.T
     n = config["norm"]
     return group_norm(x, weights["final.norm"].to(dtype), n["groups"], n["eps"]) @ \
         weights["head"].to(dtype).T
+
+
+def tensor_shapes(config: dict, ranks=5) -> dict:
+    """Names and shapes of all tensors; ``ranks``: inner width of the decays' two-step projections (no
+    number of the configuration)."""
+    H = config["width"]
+    s = {"embed": (config["vocab"], H), "final.norm": (H,), "head": (config["vocab"], H)}
+    for i, layer in enumerate(config["layers"]):
+        p, m, f = f"l{i}.", layer["mixer"], layer["mlp"]
+        s.update({p + "norm1": (H,), p + "canon1": (H, config["canon"]["taps"])})
+        x = p + "mix."
+        if layer["type"] == "wkv":
+            n = m["heads"] * m["dim"]
+            s.update({x + "mu." + c: (H,) for c in "rkvgw"})
+            s.update({x + c: (n, H) for c in "rkvg"})
+            s.update({x + "w1": (ranks, H), x + "w2": (n, ranks), x + "w0": (n,), x + "norm": (n,),
+                      x + "u": (m["heads"], m["dim"]), x + "o": (H, n)})
+        else:
+            q, k, v = (m[a] * m[b] for a, b in (("heads", "dim"), ("kv_heads", "dim"),
+                                                ("kv_heads", "vdim")))
+            s.update({x + "q": (q, H), x + "k": (k, H), x + "v": (v, H),
+                      x + "o": (H, m["heads"] * m["vdim"])})
+            if m.get("v_mix"):
+                s[x + "vmix"] = ()
+            if layer["type"] == "attention":
+                s.update({x + "q.norm": (q,), x + "k.norm": (k,), x + "sink": (m["heads"],)})
+        if f is None:
+            continue
+        s[p + "norm2"] = (H,)
+        x = p + "mlp."
+        if f["kind"] == "dense":
+            s.update({x + "gate": (f["ff"], H), x + "up": (f["ff"], H), x + "down": (H, f["ff"])})
+            continue
+        s[x + "router"] = (f["router"]["experts"], H)
+        names = [(f"e{e}", f["expert"]["ff"]) for e in range(f["router"]["experts"])]
+        for n, ff in names + ([("shared", f["shared"]["ff"])] if f.get("shared") else []):
+            s.update({f"{x}{n}.up": (ff, H), f"{x}{n}.down": (H, ff)})
+    return s
+
+
+def random_model(config: dict, seed: int, ranks=5) -> dict:
+    """Random bf16 weights under which every part has a say: decays that reach from a few tokens to the
+    whole sequence, sinks of the size of the scores, mixed values, norm weights away from one, routers
+    with clear choices."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(config, ranks).items():
+        r = torch.randn(*shape, generator=g) if shape else torch.randn((), generator=g)
+        if name.endswith(("norm", "norm1", "norm2")):
+            t = 1.0 + 0.3 * r
+        elif name.endswith(".sink"):
+            t = 1.0 + r
+        elif name.endswith(".vmix"):
+            t = 0.5 + 0.3 * r
+        elif name.endswith(".canon1"):
+            t = 0.5 * r
+        elif ".mu." in name:
+            t = torch.rand(*shape, generator=g)
+        elif name.endswith(".w0"):
+            t = -2.5 + 1.5 * r
+        elif name.endswith(".u"):
+            t = r
+        elif name.endswith(".router"):
+            t = 4.0 * r * shape[-1] ** -0.5
+        elif name == "embed":
+            t = r
+        else:
+            t = r * shape[-1] ** -0.5
+        out[name] = t.to(torch.bfloat16)
+    return out
