@@ -23,8 +23,8 @@ Launch: ``python bench.py`` (1 GPU) or
 ``--impl reference`` reports why the reference cannot run on this hardware;
 ``--impl vllm-stock`` runs the same workload through stock vLLM on the CUDA platform (the
 stand-in baseline, benchmarks/baseline_vllm_stock.py).
-``--workload fepopel`` / ``fizunex`` / ``sapapel`` runs another measurement instead: one model
-family beside another.
+``--workload vadelix`` / ``vadelix-experts`` / ``fepopel`` / ``fizunex`` / ``sapapel`` runs another
+measurement instead: one model family beside another.
 """
 from __future__ import annotations
 
@@ -120,9 +120,11 @@ def main() -> None:
     ap.add_argument("--no-async", action="store_true")
     ap.add_argument("--eager", action="store_true")
     ap.add_argument("--layers", type=int, default=0, help="debug only: truncate the model")
-    ap.add_argument("--workload", default="default", choices=["default", "sapapel", "fizunex", "fepopel"],
-                    help="prefill / decode throughput of Fizunex layers beside Llama's or of "
-                         "Sapapel or Fepopel layers beside DeepSeek's at equal sizes "
+    ap.add_argument("--workload", default="default", choices=["default", "sapapel", "fizunex", "fepopel",
+                                                               "vadelix", "vadelix-experts"],
+                    help="prefill / decode throughput of Fizunex layers beside Llama's, of "
+                         "Sapapel or Fepopel layers beside DeepSeek's, or of Vadelix layers "
+                         "beside Fizunex's (with experts: Fepopel's) at equal sizes "
                          "(benchmarks/bench_family_pair.py), one line per size")
     args = ap.parse_args()
     if args.workload != "default":

@@ -11,6 +11,11 @@ sizes, both through ``LLM.generate`` with random weights.
   experts per token, expert width (routed and shared) and vocabulary; as many layer runs as DeepSeek
   has layers, two of them a second pass of a loop.  Every second layer of Fepopel has chunked grouped
   attention in place of latent attention; its experts have two matrices, DeepSeek's three.
+* Vadelix beside Fizunex: same width, heads, key heads, head dimension, feed-forward, layers and
+  vocabulary.  Half of the layers of both are recurrent; the others of Vadelix run attention alone, in
+  turn over all keys and over a window.  Vadelix with experts beside Fepopel: same width, heads, key
+  heads, experts, experts per token and expert width (routed and shared), as many layers as Fepopel has
+  layer runs.
 
 Timed on the device: the CUDA events that bracket every engine step.  Prefill: ``prompts x
 input_len`` tokens in steps of 8192, one output token.  Decode: the steps of ``batch`` requests
@@ -49,9 +54,22 @@ SIZES = {"sapapel": {
                layers=6),
     7168: dict(heads=128, kv_heads=8, dim=128, rank=512, chunk=512, experts=64, top=8, ff=2048,
                layers=4),
+}, "vadelix": {
+    2048: dict(heads=16, kv_heads=4, dim=128, window=512, rank=64, mem_heads=4, mem_dim=128,
+               mem_vdim=256, ff=8192, layers=8),
+    4096: dict(heads=32, kv_heads=8, dim=128, window=512, rank=64, mem_heads=8, mem_dim=128,
+               mem_vdim=256, ff=14336, layers=8),
+    8192: dict(heads=64, kv_heads=8, dim=128, window=512, rank=64, mem_heads=16, mem_dim=128,
+               mem_vdim=256, ff=28672, layers=4),
+}, "vadelix-experts": {
+    2048: dict(heads=16, kv_heads=4, dim=128, window=512, rank=512, chunk=512, experts=64, top=6,
+               ff=1408, layers=8),
+    4096: dict(heads=32, kv_heads=8, dim=128, window=512, rank=512, chunk=512, experts=32, top=4,
+               ff=1536, layers=8),
 }}
 PAIRS = {"sapapel": ("sapapel", "deepseek"), "fizunex": ("fizunex", "llama"),
-         "fepopel": ("fepopel", "deepseek")}
+         "fepopel": ("fepopel", "deepseek"), "vadelix": ("vadelix", "fizunex"),
+         "vadelix-experts": ("vadelix", "fepopel")}
 VOCAB = 32768
 
 
@@ -64,6 +82,14 @@ def model_config(pair: str, family: str, width: int):
                                  s["mem_dim"], s["mem_vdim"])
         return ModelConfig.from_hf_dict(_fizunex_preset(
             ("dp" * s["layers"])[:s["layers"]], VOCAB, width, s["ff"], *mixers), dtype="bfloat16")
+    if family == "vadelix":
+        from vllm_gcu_b200.config import _vadelix_preset
+        e = "experts" in s
+        kinds = ("we", "re", "we", "be") if e else ("wd", "rd", "wd", "bd")
+        return ModelConfig.from_hf_dict(_vadelix_preset(
+            " ".join((kinds * s["layers"])[:s["layers"]]), VOCAB, width, s["heads"], s["kv_heads"],
+            s["dim"], s["window"], s["heads"], s["dim"], s["ff"], s.get("experts", 0),
+            s.get("top", 0), (4, 2), s["ff"], s["ff"], 64), dtype="bfloat16")
     if family == "llama":
         return ModelConfig(
             architecture="LlamaForCausalLM", vocab_size=VOCAB, hidden_size=width,

@@ -99,7 +99,7 @@ def test_input_convolution(H, taps, mixes, dtype):
     ref.add_group_norm(x, None, 1.0, nw, 1, 1e-4, h)
     h = h.to(dtype)
     want = torch.empty((T, H) if not mixes else (mixes, T, H))
-    state = None if ring is None else ring.float()
+    state = None if ring is None else ring.float().clone()
     ref.input_conv(h.float(), w, mu, step, state, want)
     dev, dmu, dring = step.to("cuda"), _cuda(mu), _cuda(ring)
     pitch = torch.zeros(*want.shape[:-1], H + 8, dtype=dtype, device="cuda")

@@ -70,7 +70,7 @@ CONFIGS = {
         rotary(3, 1, 7, 5, 6, 77.0, 0.6, None, moe(5, 3, 11, 13)),
         wkv(3, 5, dense(23)),
         biased(5, 5, 5, 1, 13, 0.5, 0.7, 11, moe(7, 2, 5)),
-        biased(3, 3, 11, 9, 19, 0.4, 0.0, 5, None, False)], 8, 1, 1.3, 1e-4),
+        biased(3, 3, 11, 9, 19, 0.4, 0.0, 5, None, False)], 8, 1, 0.5, 1e-4),
     # wider than one tile everywhere, groups of eight heads, a window over several pages and tiles,
     # a norm group for every vector of 8
     "wide": model_config(300, 192, [

@@ -580,7 +580,8 @@ class ModelConfig:
                             head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
                             scale=float(m["scale"]), v_mix=bool(m.get("v_mix")))
                 if layer["type"] == "attention":
-                    rot, y = m["rot"], m["rot"].get("scaling")
+                    rot = m.get("rot") or {"dims": 0, "base": 1.0}
+                    y = rot.get("scaling")
                     spec = AttentionSpec(
                         rot_dims=int(rot["dims"]), rot_base=float(rot["base"]), rot_halves=True,
                         rot_scaling=tuple(float(y[k]) for k in ("factor", "original", "fast",

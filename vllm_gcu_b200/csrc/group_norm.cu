@@ -233,9 +233,44 @@ struct PortionArgs {
   ConvArgs c;
 };
 
+// V neighbouring elements as they lie in memory
+template <typename T, int V>
+struct RawRow {
+  T e[V];
+};
+template <>
+struct __align__(16) RawRow<__nv_bfloat16, 8> {
+  uint4 u;
+};
+template <>
+struct __align__(16) RawRow<float, 4> {
+  float4 u;
+};
+template <typename T, int V>
+__device__ __forceinline__ RawRow<T, V> load_raw(const T* p) {
+  return *reinterpret_cast<const RawRow<T, V>*>(p);
+}
+template <typename T, int V>
+__device__ __forceinline__ void unpack_raw(const RawRow<T, V>& r, float (&f)[V]) {
+  if constexpr (V == 8) {
+    const uint32_t w[4] = {r.u.x, r.u.y, r.u.z, r.u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 p = unpack_bf16x2(w[i]);
+      f[2 * i] = p.x;
+      f[2 * i + 1] = p.y;
+    }
+  } else if constexpr (V == 4) {
+    f[0] = r.u.x; f[1] = r.u.y; f[2] = r.u.z; f[3] = r.u.w;
+  } else {
+    f[0] = to_f32<T>(r.e[0]);
+  }
+}
+
 // grid.x: at least the strips of all requests; grid.y: slabs of blockDim.x * V channels.
-template <typename T, int V, int NT>
-__global__ void __launch_bounds__(256) input_conv_kernel(const PortionArgs a) {
+template <typename T, int V, int NT, bool kMixed>
+__global__ void __launch_bounds__(256, NT <= 4 ? 2 : 1) input_conv_kernel(const PortionArgs a) {
+  constexpr int kBatch = kMixed ? 4 : 8;     // rows in flight
   __shared__ int s_req, s_strip;
   if (threadIdx.x < 32) {
     const int lane = threadIdx.x, want = blockIdx.x;
@@ -290,63 +325,69 @@ __global__ void __launch_bounds__(256) input_conv_kernel(const PortionArgs a) {
     for (int i = 0; i < V; ++i) w[o][i] = 0.0f;
     if (o < cv.taps) ldv<V>(cv.w + static_cast<long long>(cv.taps - 1 - o) * a.H + c, w[o]);
   }
-  float past[NT][V], before[V];              // [o]: row of o + 1 tokens ago; convolved row before
+  RawRow<T, V> past[NT];                     // [o]: row of o + 1 tokens ago, as it lies in memory
 #pragma unroll
   for (int o = 0; o < NT; ++o) {
-#pragma unroll
-    for (int i = 0; i < V; ++i) past[o][i] = 0.0f;
+    past[o] = RawRow<T, V>{};
     if (o >= cv.back) continue;
     const int i = i0 - 1 - o;
-    if (i >= 0) ldv<V>(h + static_cast<long long>(i) * a.H, past[o]);
+    if (i >= 0) past[o] = load_raw<T, V>(h + static_cast<long long>(i) * a.H);
     else if (ring != nullptr && p0 + i >= 0)
-      ldv<V>(ring + static_cast<long long>((p0 + i) % cv.back) * a.H, past[o]);
+      past[o] = load_raw<T, V>(ring + static_cast<long long>((p0 + i) % cv.back) * a.H);
   }
+  // now[1 ..]: convolved rows of the batch; now[0]: the one in front of it
+  float now[kBatch + 1][V];
+  if (kMixed) {
 #pragma unroll
-  for (int i = 0; i < V; ++i) before[i] = past[0][i];
+    for (int o = 0; o < NT; ++o) {
+      float f[V];
+      unpack_raw<T, V>(past[o], f);
 #pragma unroll
-  for (int o = 0; o < NT; ++o) {
-#pragma unroll
-    for (int i = 0; i < V; ++i) before[i] += w[o][i] * past[o][i];
+      for (int i = 0; i < V; ++i) now[kBatch][i] = (o == 0 ? f[i] : now[kBatch][i]) + w[o][i] * f[i];
+    }
   }
   T* out = static_cast<T*>(cv.out) + static_cast<long long>(first) * cv.ldo + c;
-  constexpr int kBatch = 8;                  // rows in flight
 #pragma unroll 1
   for (int b = i0; b < i1; b += kBatch) {
-    float rows[kBatch][V];
-#pragma unroll
-    for (int u = 0; u < kBatch; ++u)
-      if (b + u < i1) ldv<V>(h + static_cast<long long>(b + u) * a.H, rows[u]);
+    RawRow<T, V> rows[kBatch];               // all rows of the batch in flight at once
 #pragma unroll
     for (int u = 0; u < kBatch; ++u) {
-      if (b + u >= i1) break;
-      float now[V];
+      rows[u] = RawRow<T, V>{};
+      if (b + u < i1) rows[u] = load_raw<T, V>(h + static_cast<long long>(b + u) * a.H);
+    }
+    if (kMixed) {
 #pragma unroll
-      for (int i = 0; i < V; ++i) now[i] = rows[u][i] + w[0][i] * rows[u][i];
+      for (int i = 0; i < V; ++i) now[0][i] = now[kBatch][i];
+    }
+#pragma unroll
+    for (int u = 0; u < kBatch; ++u) {
+      float* n = now[u + 1];
+      float f[V];
+      unpack_raw<T, V>(rows[u], f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) n[i] = f[i] + w[0][i] * f[i];
 #pragma unroll
       for (int o = 1; o < NT; ++o) {
+        unpack_raw<T, V>(past[o - 1], f);
 #pragma unroll
-        for (int i = 0; i < V; ++i) now[i] += w[o][i] * past[o - 1][i];
+        for (int i = 0; i < V; ++i) n[i] += w[o][i] * f[i];
       }
 #pragma unroll
-      for (int o = NT - 1; o > 0; --o) {
+      for (int o = NT - 1; o > 0; --o) past[o] = past[o - 1];
+      past[0] = rows[u];
+      if (!kMixed && b + u < i1) stv<V>(out + static_cast<long long>(b + u) * cv.ldo, now[u + 1]);
+    }
+    if (!kMixed) continue;
+    for (int m = 0; m < cv.mixes; ++m) {
+      float k[V];
+      ldv<V>(cv.mu + static_cast<long long>(m) * a.H + c, k);
 #pragma unroll
-        for (int i = 0; i < V; ++i) past[o][i] = past[o - 1][i];
-      }
+      for (int u = 0; u < kBatch; ++u) {
+        if (b + u >= i1) break;
+        float o[V];
 #pragma unroll
-      for (int i = 0; i < V; ++i) past[0][i] = rows[u][i];
-      T* dst = out + static_cast<long long>(b + u) * cv.ldo;
-      if (cv.mu == nullptr) {
-        stv<V>(dst, now);
-      } else {
-        for (int m = 0; m < cv.mixes; ++m) {
-          float k[V], o[V];
-          ldv<V>(cv.mu + static_cast<long long>(m) * a.H + c, k);
-#pragma unroll
-          for (int i = 0; i < V; ++i) o[i] = now[i] + (before[i] - now[i]) * k[i];
-          stv<V>(dst + m * cv.mix_stride, o);
-        }
-#pragma unroll
-        for (int i = 0; i < V; ++i) before[i] = now[i];
+        for (int i = 0; i < V; ++i) o[i] = now[u + 1][i] + (now[u][i] - now[u + 1][i]) * k[i];
+        stv<V>(out + static_cast<long long>(b + u) * cv.ldo + m * cv.mix_stride, o);
       }
     }
   }
@@ -473,8 +514,14 @@ B200_API int b200_input_conv(const void* h, const float* w, int taps, const floa
   const dim3 grid(T / kStrip + nd + np, (lanes + th - 1) / th);
 #define B200_IC(TT, W)                                                    \
   do {                                                                    \
-    if (taps <= 4) input_conv_kernel<TT, W, 4><<<grid, th, 0, s>>>(a);    \
-    else input_conv_kernel<TT, W, 8><<<grid, th, 0, s>>>(a);              \
+    if (taps <= 4 && mu == nullptr)                                       \
+      input_conv_kernel<TT, W, 4, false><<<grid, th, 0, s>>>(a);          \
+    else if (taps <= 4)                                                   \
+      input_conv_kernel<TT, W, 4, true><<<grid, th, 0, s>>>(a);           \
+    else if (mu == nullptr)                                               \
+      input_conv_kernel<TT, W, 8, false><<<grid, th, 0, s>>>(a);          \
+    else                                                                  \
+      input_conv_kernel<TT, W, 8, true><<<grid, th, 0, s>>>(a);           \
   } while (0)
   if (dtype == 0) {
     if (vec) B200_IC(__nv_bfloat16, 8);
