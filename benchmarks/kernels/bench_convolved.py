@@ -121,7 +121,14 @@ def cases(lens: list[int], ctx: int, decode: bool, H: int, N: int, G: int, D: in
     mixed, wp = rnd(4, T, H).to(bf), rnd(4 * N * D, H).to(bf)
     proj = torch.empty(T, 4 * N * D, device=dev, dtype=bf)
 
+    tiles4 = torch.arange(4, device=dev, dtype=torch.int32)
+    rows4 = torch.tensor([4 * C.GROUP_ROWS], device=dev, dtype=torch.int32)
+    padded = rnd(4 * C.GROUP_ROWS, H).to(bf)
+
     def projections():
+        if T <= C.GROUP_ROWS:
+            C.gemm_bf16_grouped(padded, wp.view(4, N * D, H), tiles4, rows4)
+            return
         for i in range(4):
             at = slice(i * N * D, (i + 1) * N * D)
             C.gemm_bf16(mixed[i], wp[at], out=proj[:, at])

@@ -53,7 +53,11 @@ class InputConv(nn.Module):
         ``rows [T, H]`` in the model's type."""
         T = rows.shape[0]
         new = lambda *s: torch.empty(*s, dtype=self.dtype, device=rows.device)  # noqa: E731
-        out = new(T, self.hidden) if self.mu is None else new(self.mu.shape[0], T, self.hidden)
+        if self.mu is None:
+            out = new(T, self.hidden)
+        else:       # few rows: every mixture in a tile of rows of its own, as grouped products take it
+            out = new(self.mu.shape[0], max(T, C.GROUP_ROWS) if rows.is_cuda else T,
+                      self.hidden)[:, :T]
         ring = state["inputs"] if state is not None and self.back and not md.is_dummy else None
         n1 = fused_tokens(rows, md)
         lo = new(T, self.hidden)

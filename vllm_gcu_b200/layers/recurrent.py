@@ -213,6 +213,12 @@ class TimeMix(nn.Module):
         self.norm = new(self.N * D)
         self.o_proj = RowParallelLinear(N * D, hidden, dtype=dtype, device=device,
                                         prefix=prefix + ".o_proj")
+        # few rows: the four projections as one grouped product, a tile of rows each
+        self.tiles = self.tile_rows = None
+        if self.in_proj.weight.is_cuda and dtype == torch.bfloat16 and hidden % 8 == 0 \
+                and self.in_proj.padded_sizes[0] % 64 == 0:
+            self.tiles = torch.arange(4, dtype=torch.int32, device=device)
+            self.tile_rows = torch.tensor([4 * C.GROUP_ROWS], dtype=torch.int32, device=device)
 
     def cache_shape(self) -> None:
         return None
@@ -248,13 +254,22 @@ class TimeMix(nn.Module):
         self.w1.weight.data[self.spec.decay_rank:] = 0
         self.w2.data[:, self.spec.decay_rank:] = 0
 
-    def forward(self, h: torch.Tensor, md: AttentionMetadata, state: Optional[dict]) -> torch.Tensor:
-        T, D, n = h.shape[1], self.spec.head_dim, self.N * self.spec.head_dim
-        pad = self.in_proj.padded_sizes[0]
+    def _project(self, h: torch.Tensor, n: int) -> list[torch.Tensor]:
+        """r, k, v and the gate ``[T, n]``, views of equal row pitch."""
+        T, pad, w = h.shape[1], self.in_proj.padded_sizes[0], self.in_proj.weight
+        if self.tiles is not None and T <= C.GROUP_ROWS \
+                and h.stride(0) == C.GROUP_ROWS * h.shape[2]:
+            y = C.gemm_bf16_grouped(h.as_strided((4 * C.GROUP_ROWS, h.shape[2]), (h.stride(1), 1)),
+                                    w.view(4, pad, -1), self.tiles, self.tile_rows)
+            return [y[i * C.GROUP_ROWS:i * C.GROUP_ROWS + T, :n] for i in range(4)]
         y = torch.empty(T, 4 * pad, dtype=h.dtype, device=h.device)
         for i in range(4):
-            linear(h[i], self.in_proj.weight[i * pad:(i + 1) * pad], out=y[:, i * pad:(i + 1) * pad])
-        r, k, v, g = (y[:, i * pad:i * pad + n] for i in range(4))
+            linear(h[i], w[i * pad:(i + 1) * pad], out=y[:, i * pad:(i + 1) * pad])
+        return [y[:, i * pad:i * pad + n] for i in range(4)]
+
+    def forward(self, h: torch.Tensor, md: AttentionMetadata, state: Optional[dict]) -> torch.Tensor:
+        T, D, n = h.shape[1], self.spec.head_dim, self.N * self.spec.head_dim
+        r, k, v, g = self._project(h, n)
         a = linear_fp32(h[4], self.w1.weight)              # the decay's inner row, unrounded
         out = torch.empty(T, n, dtype=h.dtype, device=h.device)
         S = state["matrix"] if state is not None and not md.is_dummy else None

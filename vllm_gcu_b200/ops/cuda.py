@@ -1317,6 +1317,9 @@ def moe_topk(gating: torch.Tensor, k: int, renormalize: bool, n_group: int = 1,
     return w, ids
 
 
+GROUP_ROWS = 128        # rows of a tile of the grouped GEMM: one expert each
+
+
 def moe_align_cap(num_pairs: int, num_local_experts: int) -> int:
     return -(-(num_pairs + num_local_experts * 127) // 128) * 128
 
