@@ -6,7 +6,7 @@ import pytest
 import torch
 
 import vadelix_oracle as O
-from vadelix_cases import (CONFIGS, Step, biased, build, dense, errors, greedy, mixed_steps,
+from vadelix_cases import (CONFIGS, Step, biased, build, errors, greedy, mixed_steps,
                            model_config, moe, oracle, peaked_model, portions, replayer, rotary, run,
                            spread, tokens_for, wkv, write_checkpoint)
 
